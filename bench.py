@@ -693,6 +693,74 @@ def hybrid_moe_width():
     return replace(cfg, name="hybrid-mamba2-w1024")
 
 
+def sozurax_cfg(width, n_layers, vocab, h_heads, h_dim, h_vdim, a_heads, a_dim, a_rot, a_vdim, kv_rank, q_rank, window,
+                experts, top, ff, shared, dense_ff, taps):
+    """HGRN2 and latent-attention layers in turn; the attention layers in groups of three, of which the
+    second and third read the first one's cache rows; a PolyNorm dense feed-forward in the first layer,
+    gated experts with a plain always-on one in the others; `taps` taps on what every sublayer reads."""
+    layers, own = [], -1
+    for l in range(n_layers):
+        if l % 2 == 0:
+            kw = dict(mixer=C.MIXER_HGRN2, heads=h_heads, dim=h_dim, vdim=h_vdim)
+        else:
+            src = own if (l // 2) % 3 else -1
+            own = own if src >= 0 else l
+            kw = dict(mixer=C.MIXER_LATENT_ATTENTION, heads=a_heads, dim=a_dim, rot_dim=a_rot, vdim=a_vdim, kv_rank=kv_rank,
+                      q_rank=q_rank, rot_base=20000.0, rot_dims=a_rot, rot_pairs=1, scale=float((a_dim + a_rot) ** -0.5),
+                      window=window, kv_from=src)
+        if l == 0:
+            kw.update(mlp=C.MLP_DENSE, act=C.FFN_POLYNORM, ff=dense_ff)
+        else:
+            kw.update(mlp=C.MLP_MOE, act=C.FFN_SWIGLU, ff=ff, experts=experts, top=top, route_norm=1, route_bias=1, shared_ff=shared)
+        layers.append(C.LayerSpec(**kw))
+    return C.ListedModelConfig("sozurax", vocab, width, tuple(layers), 1e-5, embedding_scale=float(width ** 0.5),
+                               arch=C.ARCH_SOZURAX, block_style=C.LBLOCK_SEQUENTIAL_PRENORM, layer_norm=True, mixer_conv=taps,
+                               ffn_conv=taps)
+
+
+def sozurax_device_weights(cfg, device, seed=1234):
+    import torch
+    g = torch.Generator(device=f"cuda:{device}")
+    for i, (name, shape) in enumerate(cfg.tensor_shapes().items()):
+        g.manual_seed(seed * 1000003 + i)
+        t = torch.empty(shape, dtype=torch.float32, device=f"cuda:{device}")
+        if name.endswith(".lower"):
+            t.uniform_(0.0, 0.9, generator=g)
+        elif name.endswith(".f.b"):
+            t.uniform_(0.0, 3.0, generator=g)
+        elif name.endswith(".b"):
+            t.normal_(0.0, 0.1, generator=g)        # additive terms of the norms, router biases
+        elif name.endswith(".act"):
+            t.fill_(0.5)
+        elif len(shape) == 1:
+            t.normal_(1.0, 0.02, generator=g)
+        elif name.endswith((".canon1", ".canon2")):
+            t.normal_(0.0, shape[1] ** -0.5, generator=g)
+        else:
+            t.normal_(0.0, 0.02 if name == "embed" else shape[1] ** -0.5, generator=g)
+        yield name, t.to(torch.bfloat16).view(torch.int16).cpu().numpy().view(np.uint16)
+        del t
+
+
+# width 1024, 24 layers like Granite-MoE-1B: 12 HGRN2 layers (8 heads of 64 x 128 state, as the gated linear
+# attention of lz-1b) and 12 latent-attention layers (16 heads of 64 + 32 entries, values of 64, rank 128, window
+# 1024; 4 own caches); 32 gated experts of 512, 8 per token (Granite's), beside an always-on expert of 1024.
+def _so():
+    return sozurax_cfg(1024, 24, 49155, 8, 64, 128, 16, 64, 32, 64, 128, 384, 1024, 32, 8, 512, 1024, 4096, 4)
+
+
+SOZURAX_SIZES = {
+    "so-1b": (_so, "granite-moe-1b", 128, 128, 128),
+    "so-1b-long": (_so, "granite-moe-1b", 16, 4096, 64),
+    "so-1b-batch": (_so, "granite-moe-1b", 64, 512, 128),
+}
+
+
+def dugopel_moe_width():
+    """The other latent-attention design at the width, depth, expert and attention sizes of the sizes above."""
+    return dugopel_cfg(1024, 24, 16, 64, 32, 64, 128, 384, 512, 49155, moe=(32, 8, 8, 4))
+
+
 DESIGN_SIZES = {
     # name: (layer-listed config, closest uniform preset, batch, prompt, decode steps)
     "dense-1b": (lambda: dugopel_cfg(2048, 16, 32, 64, 32, 64, 128, 768, 8192, 128256), "llama-3.2-1b", 64, 512, 128),
@@ -715,29 +783,30 @@ def design_bench(args):
     peaks = load_peaks()
     R = nvllm_pkg.sub("runner")
     design = args.design
-    sizes = {"zozonex": ZOZONEX_SIZES, "lazovik": LAZOVIK_SIZES, "sutuvik": SUTUVIK_SIZES}.get(design, DESIGN_SIZES)
+    sizes = {"zozonex": ZOZONEX_SIZES, "lazovik": LAZOVIK_SIZES, "sutuvik": SUTUVIK_SIZES, "sozurax": SOZURAX_SIZES}.get(design, DESIGN_SIZES)
     gen = {"zozonex": zozonex_device_weights, "lazovik": lazovik_device_weights,
-           "sutuvik": sutuvik_device_weights}.get(design, dugopel_device_weights)
+           "sutuvik": sutuvik_device_weights, "sozurax": sozurax_device_weights}.get(design, dugopel_device_weights)
+    # further baselines: uniform models (configuration) and layer-listed ones (configuration, weights)
+    uniform = {"hybrid-mamba2-1b": hybrid_1b, "hybrid-mamba2-w1024": hybrid_moe_width}
+    listed = {"zozonex-1b": (zozonex_moe_width, zozonex_device_weights), "lazovik-w1024": (_lz(24), lazovik_device_weights),
+              "dugopel-w1024": (dugopel_moe_width, dugopel_device_weights)}
+    second = {"zozonex": ("hybrid-mamba2-1b",), "lazovik": ("zozonex-1b",), "sutuvik": ("hybrid-mamba2-w1024",),
+              "sozurax": ("lazovik-w1024", "dugopel-w1024")}.get(design, ())
     out = {"design": design, "dtype": "bf16", "data": "synthetic (random-init weights, random prompts)",
            "steps": args.steps, "warmup": args.warmup, "peaks": peaks, "sizes": {}}
     names = [n for n in sizes if args.design_size in (None, n)]
     for name in names:
         mk, base_name, batch, P, D = sizes[name]
         entry = {"batch": batch, "prompt_len": P, "decode_steps": D}
-        others = (base_name, "hybrid-mamba2-1b") if design == "zozonex" and not args.no_hybrid else (base_name,)
-        if design == "lazovik" and not args.no_hybrid:
-            others = (base_name, "zozonex-1b")
-        if design == "sutuvik" and not args.no_hybrid:
-            others = (base_name, "hybrid-mamba2-w1024")
+        others = (base_name,) + (() if args.no_hybrid else second)
         for which in (design,) + others:
-            cfg = mk() if which == design else hybrid_1b() if which == "hybrid-mamba2-1b" else \
-                hybrid_moe_width() if which == "hybrid-mamba2-w1024" else zozonex_moe_width() if which == "zozonex-1b" else C.PRESETS[base_name]()
+            cfg = mk() if which == design else listed[which][0]() if which in listed else uniform.get(which, C.PRESETS.get(which))()
             if which != design and hasattr(cfg, "max_seq_len") and cfg.max_seq_len < P + D + 1:
                 from dataclasses import replace
                 cfg = replace(cfg, max_seq_len=P + D + 32)
             job = Job(cfg, batch, P, D, 4321)
-            if which == design or which == "zozonex-1b":
-                wgen = gen if which == design else zozonex_device_weights
+            if which == design or which in listed:
+                wgen = gen if which == design else listed[which][1]
                 run = R.CudaModelRunner(cfg, wgen(cfg, device), precision=C.PREC_BF16,
                                         num_kv_blocks=job.num_blocks, device=device, max_num_seqs=job.n,
                                         max_batched_tokens=batch * P, sampling=None, num_state_slots=job.n)
@@ -823,12 +892,14 @@ def main():
     ap.add_argument("--no-profile", action="store_true")
     ap.add_argument("--no-tp", action="store_true",
                     help="skip the Falcon-7B tensor-parallel leg (configs[3] at tp = --gpus)")
-    ap.add_argument("--design", default=None, choices=["dugopel", "zozonex", "lazovik", "sutuvik"],
+    ap.add_argument("--design", default=None, choices=["dugopel", "zozonex", "lazovik", "sutuvik", "sozurax"],
                     help="instead of the default workload: the layer-listed design beside the closest "
                          "uniform model at equal size (prefill and decode, per-kernel roofline)")
     ap.add_argument("--no-hybrid", action="store_true",
-                    help="--design zozonex / lazovik / sutuvik: skip the second baseline (Mamba2 hybrid / Zozonex at equal width)")
-    ap.add_argument("--design-size", default=None, choices=sorted(DESIGN_SIZES) + sorted(ZOZONEX_SIZES) + sorted(LAZOVIK_SIZES) + sorted(SUTUVIK_SIZES))
+                    help="--design zozonex / lazovik / sutuvik / sozurax: only the closest uniform model as a baseline (no Mamba2 "
+                         "hybrid / other layer-listed design at equal width)")
+    ap.add_argument("--design-size", default=None, choices=sorted(DESIGN_SIZES) + sorted(ZOZONEX_SIZES) + sorted(LAZOVIK_SIZES) + sorted(SUTUVIK_SIZES) +
+                    sorted(SOZURAX_SIZES))
     args = ap.parse_args()
     if args.design:
         return design_bench(args)

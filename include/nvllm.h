@@ -190,9 +190,10 @@ int nvllm_create(const nvllm_config* cfg, const uint8_t* tp_id, nvllm_handle** o
  *                                   the sublayers read x itself, the norm sits on their output (Zozonex)
  *   NVLLM_LBLOCK_SEQUENTIAL_PRENORM   x += mixer(RMSNorm(x)), then x += feed_forward(RMSNorm(x)); a run of
  *                                   layers may repeat with the same weights (loop_*), every pass with caches and
- *                                   state of its own and a learned vector added to x at its start (Lazovik, Sutuvik)
+ *                                   state of its own and a learned vector added to x at its start (Lazovik, Sutuvik);
+ *                                   with layer_norm = 1 LayerNorm (weight and additive term) instead (Sozurax)
  * Tensors are handed in by checkpoint name (nvllm_set_named_weight, or nvllm_load_safetensors
- * with NVLLM_ARCH_DUGOPEL / NVLLM_ARCH_ZOZONEX / NVLLM_ARCH_LAZOVIK / NVLLM_ARCH_SUTUVIK). */
+ * with NVLLM_ARCH_DUGOPEL / NVLLM_ARCH_ZOZONEX / NVLLM_ARCH_LAZOVIK / NVLLM_ARCH_SUTUVIK / NVLLM_ARCH_SOZURAX). */
 enum nvllm_mixer_kind {
   NVLLM_MIXER_LATENT_ATTENTION = 1,
   NVLLM_MIXER_WINDOW_ATTENTION = 2, /* grouped-query attention over a sliding window of the paged K / V cache */
@@ -206,14 +207,19 @@ enum nvllm_mixer_kind {
                                        piecewise frequency scaling, a query multiplier that grows with the position, a
                                        multiplier per head, score cap, a bias linear in the distance, a sink of score 0 or a
                                        learned one per head, values mixed with an earlier layer's, a gate per head */
-  NVLLM_MIXER_MAMBA2 = 7            /* Mamba-2: per head S <- exp(-exp(A_log) dt) S + dt B x^T (state x vdim), y = S^T C + D x,
+  NVLLM_MIXER_MAMBA2 = 7,           /* Mamba-2: per head S <- exp(-exp(A_log) dt) S + dt B x^T (state x vdim), y = S^T C + D x,
                                        gated by silu(z) and then normed in groups; state and convolution tail per state slot */
+  NVLLM_MIXER_HGRN2 = 8             /* per head S <- diag(f) S + (1 - f) v^T (dim x vdim), o = S^T silu(q), f = l + (1 - l)
+                                       sigmoid(W_f h + b) per key entry with a lower bound l; read-outs RMS-normed per
+                                       head; state per slot */
 };
 enum nvllm_mlp_kind { NVLLM_MLP_NONE = 0, NVLLM_MLP_DENSE = 1, NVLLM_MLP_MOE = 2 };
 enum nvllm_ffn_act {
   NVLLM_FFN_GLU_CLAMPED = 0, /* W_down (g sigmoid(1.702 g) (u + 1)), g / u clamped by `limit` */
   NVLLM_FFN_RELU2 = 1,       /* W_down relu(W_up h)^2 */
-  NVLLM_FFN_SWIGLU = 2       /* W_down (silu(W_gate h) * (W_up h)) */
+  NVLLM_FFN_SWIGLU = 2,      /* W_down (silu(W_gate h) * (W_up h)) */
+  NVLLM_FFN_POLYNORM = 3     /* W_down (a N(z) + b N(z^2) + c N(z^3) + e), z = W_up h, powers element by element, N divides
+                                the row by its root mean square; {a, b, c, e} = tensor "mlp.act" */
 };
 enum nvllm_layered_block {
   NVLLM_LBLOCK_PARALLEL_PRENORM = 0,
@@ -227,7 +233,9 @@ typedef struct nvllm_layer_spec {
   /* latent attention: queries through a q_rank latent; keys / values through a kv_rank latent
    * plus one rotated key part of rot_dim shared by the heads.  Per head: dim unrotated and
    * rot_dim rotated query / key entries, vdim value entries.
-   * window attention / delta rule: heads, dim (query / key entries per head), vdim. */
+   * window attention / delta rule: heads, dim (query / key entries per head), vdim.
+   * In sequential pre-norm blocks latent attention also takes window, rot_pairs and head_gate (parallel
+   * blocks: no window, halves rotated, gates always). */
   int32_t heads, dim, rot_dim, vdim, kv_rank, q_rank;
   int32_t rot_dims;     /* leading entries of the rotated part that are rotated (<= rot_dim, even) */
   int32_t kv_from;      /* -1: own key/value projection and cache; j: reads layer j's cache */
@@ -264,7 +272,8 @@ typedef struct nvllm_layer_spec {
   /* mixture of experts with act = NVLLM_FFN_RELU2 */
   int32_t route_sigmoid;   /* 1: scores are sigmoid(logits) instead of a softmax over the experts */
   int32_t weight_on_input; /* 1: the routing weight multiplies the expert's input instead of its output */
-  int32_t shared_ff;       /* > 0: one more expert of this inner size runs for every token, times sigmoid(W_sg h) */
+  int32_t shared_ff;       /* > 0: one more expert of this inner size runs for every token (act = NVLLM_FFN_RELU2: times
+                              sigmoid(W_sg h); NVLLM_FFN_SWIGLU: as it is) */
   /* NVLLM_MIXER_ATTENTION (uses heads, kv_heads, dim, vdim, scale, softcap, sink, qk_norm, rot_base, rot_dims and
    * rot_factor / rot_original / rot_fast / rot_slow) */
   int32_t rot_pairs;       /* 1: entry 2i rotates with entry 2i + 1 (interleaved) instead of i with i + rot_dims / 2 */
@@ -288,6 +297,7 @@ typedef struct nvllm_layer_spec {
   int32_t route_correction; /* 1: tensor "mlp.correction" [experts] is added to the scores for the CHOICE only */
   int32_t group_top2;       /* 1: a group of experts scores as the sum of its two best choice scores (else its best) */
   int32_t route_norm;       /* 1 (with route_sigmoid): the weights are the chosen scores divided by their sum (+ 1e-20) */
+  int32_t route_bias;       /* 1: tensor "mlp.router.b" [experts] is added to the logits */
 } nvllm_layer_spec;
 
 typedef struct nvllm_layered_config {
@@ -311,12 +321,15 @@ typedef struct nvllm_layered_config {
   int32_t norm_groups;     /* > 1: every norm of the residual stream splits the row into this many equal parts, each
                               divided by its own root mean square */
   int32_t embed_norm;      /* 1: x = norm(embed[token]) with tensor "embed.norm" */
-  int32_t mixer_conv;      /* taps > 1: what a mixer reads is h + conv(h), a causal convolution over time per channel
+  int32_t mixer_conv;      /* taps >= 1: what a mixer reads is h + conv(h), a causal convolution over time per channel
                               (tensor "l<i>.canon1" [width, taps], last column = the current token); the last taps - 1
                               rows of h are part of the sequence's state slot */
   int32_t side_dim;        /* > 0: after a layer's feed-forward x += rmsnorm(W_proj (gelu_tanh(W_gate x) * e)) * w with
                               e = "side.embed"[token][layer * side_dim, (layer + 1) * side_dim) */
   float logit_scale;       /* != 0: logits are multiplied by it */
+  int32_t ffn_conv;        /* taps >= 1: the same on what a feed-forward reads (tensor "l<i>.canon2"; the router reads it too) */
+  int32_t layer_norm;      /* 1: the norms of the stream are LayerNorms with weight and additive term (tensors "<norm>",
+                              "<norm>.b") */
 } nvllm_layered_config;
 
 int nvllm_create_layered(const nvllm_layered_config* cfg, const nvllm_layer_spec* layers,
@@ -362,7 +375,8 @@ enum nvllm_arch {
   NVLLM_ARCH_DUGOPEL = 4,     /* layered handle: every tensor of the file by its own name */
   NVLLM_ARCH_ZOZONEX = 5,     /* layered handle, likewise */
   NVLLM_ARCH_LAZOVIK = 6,     /* layered handle, likewise */
-  NVLLM_ARCH_SUTUVIK = 7      /* layered handle, likewise */
+  NVLLM_ARCH_SUTUVIK = 7,     /* layered handle, likewise */
+  NVLLM_ARCH_SOZURAX = 8      /* layered handle, likewise */
 };
 
 /* Load every weight of the model straight from `model_dir` — model.safetensors, or the shards

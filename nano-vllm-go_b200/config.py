@@ -27,10 +27,11 @@ BLOCK_SEQUENTIAL, BLOCK_PARALLEL = 0, 1
 PREC_FP32, PREC_BF16 = 0, 1
 # enum nvllm_arch (checkpoint families of generic_loader.go:60-182)
 ARCH_GPT2, ARCH_FALCON, ARCH_LLAMA, ARCH_GRANITE_MOE, ARCH_DUGOPEL, ARCH_ZOZONEX, ARCH_LAZOVIK, ARCH_SUTUVIK = 0, 1, 2, 3, 4, 5, 6, 7
+ARCH_SOZURAX = 8
 MIXER_LATENT_ATTENTION, MIXER_WINDOW_ATTENTION, MIXER_DELTA, MIXER_GLA, MIXER_ATTN_TMIX = 1, 2, 3, 4, 5
-MIXER_ATTENTION, MIXER_MAMBA2 = 6, 7
+MIXER_ATTENTION, MIXER_MAMBA2, MIXER_HGRN2 = 6, 7, 8
 MLP_NONE, MLP_DENSE, MLP_MOE = 0, 1, 2
-FFN_GLU_CLAMPED, FFN_RELU2, FFN_SWIGLU = 0, 1, 2
+FFN_GLU_CLAMPED, FFN_RELU2, FFN_SWIGLU, FFN_POLYNORM = 0, 1, 2, 3
 LBLOCK_PARALLEL_PRENORM, LBLOCK_SEQUENTIAL_POSTNORM, LBLOCK_SEQUENTIAL_PRENORM = 0, 1, 2
 LPOS_NONE, LPOS_SINUSOIDAL = 0, 1
 DT_F32, DT_BF16, DT_F16 = 0, 1, 2
@@ -316,6 +317,7 @@ class CLayerSpec(ctypes.Structure):
         ("head_gate", ctypes.c_int32),
         ("state", ctypes.c_int32), ("ssm_groups", ctypes.c_int32), ("norm_groups", ctypes.c_int32),
         ("route_correction", ctypes.c_int32), ("group_top2", ctypes.c_int32), ("route_norm", ctypes.c_int32),
+        ("route_bias", ctypes.c_int32),
     ]
 
 
@@ -334,6 +336,7 @@ class CLayeredConfig(ctypes.Structure):
         ("loop_start", ctypes.c_int32), ("loop_stop", ctypes.c_int32), ("loop_times", ctypes.c_int32),
         ("norm_groups", ctypes.c_int32), ("embed_norm", ctypes.c_int32), ("mixer_conv", ctypes.c_int32),
         ("side_dim", ctypes.c_int32), ("logit_scale", ctypes.c_float),
+        ("ffn_conv", ctypes.c_int32), ("layer_norm", ctypes.c_int32),
     ]
 
 
@@ -398,6 +401,7 @@ class LayerSpec:
     route_correction: int = 0
     group_top2: int = 0
     route_norm: int = 0
+    route_bias: int = 0
 
     def to_c(self) -> CLayerSpec:
         c = CLayerSpec()
@@ -405,12 +409,13 @@ class LayerSpec:
             setattr(c, name, getattr(self, name))
         return c
 
-    def tensor_shapes(self, layer: int, width: int) -> dict:
-        """Checkpoint names and shapes of this layer's tensors (linears [out, in])."""
+    def tensor_shapes(self, layer: int, width: int, prenorm: bool = False) -> dict:
+        """Checkpoint names and shapes of this layer's tensors (linears [out, in]); prenorm: the layer
+        belongs to sequential pre-norm blocks (latent attention exists in two block styles)."""
         p = f"l{layer}."
         if self.mixer in (MIXER_GLA, MIXER_ATTN_TMIX):
             return self._prenorm_shapes(p, width)
-        if self.mixer in (MIXER_ATTENTION, MIXER_MAMBA2):
+        if self.mixer in (MIXER_ATTENTION, MIXER_MAMBA2, MIXER_HGRN2) or (self.mixer == MIXER_LATENT_ATTENTION and prenorm):
             return self._prenorm2_shapes(p, width)
         if self.mixer == MIXER_WINDOW_ATTENTION:
             d = {p + "norm1": (width,), p + "mix.q": (self.heads * self.dim, width),
@@ -488,7 +493,8 @@ LayerSpec._prenorm_shapes = _prenorm_shapes
 
 
 def _prenorm2_shapes(self, p: str, width: int) -> dict:
-    """Attention with its options / Mamba-2, and the mixture of gated experts."""
+    """Attention with its options / Mamba-2 / HGRN2 / latent attention, and the mixture of gated
+    experts or the PolyNorm dense layer."""
     d = {p + "norm1": (width,)}
     m = p + "mix."
     if self.mixer == MIXER_ATTENTION:
@@ -505,14 +511,34 @@ def _prenorm2_shapes(self, p: str, width: int) -> dict:
             d[m + "temp"] = (self.heads,)
         if self.head_gate:
             d[m + "g"] = (self.heads, width)
+    elif self.mixer == MIXER_HGRN2:
+        hd, hv = self.heads * self.dim, self.heads * self.vdim
+        d.update({m + "q": (hd, width), m + "f": (hd, width), m + "f.b": (hd,), m + "lower": (hd,), m + "v": (hv, width),
+                  m + "norm": (self.vdim,), m + "o": (width, hv)})
+    elif self.mixer == MIXER_LATENT_ATTENTION:
+        d.update({m + "dq": (self.q_rank, width), m + "dq.norm": (self.q_rank,),
+                  m + "uq": (self.heads * (self.dim + self.rot_dim), self.q_rank),
+                  m + "uk": (self.heads * self.dim, self.kv_rank), m + "uv": (self.heads * self.vdim, self.kv_rank),
+                  m + "o": (width, self.heads * self.vdim)})
+        if self.kv_from < 0:
+            d.update({m + "dkv": (self.kv_rank + self.rot_dim, width), m + "dkv.norm": (self.kv_rank,)})
+        if self.head_gate:
+            d[m + "g"] = (self.heads, width)
     else:
         inner, gn = self.heads * self.vdim, self.ssm_groups * self.state
         d.update({m + "in": (2 * inner + 2 * gn + self.heads, width), m + "conv": (inner + 2 * gn, self.conv),
                   m + "conv.b": (inner + 2 * gn,), m + "dt_bias": (self.heads,), m + "A_log": (self.heads,),
                   m + "D": (self.heads,), m + "norm": (inner,), m + "o": (width, inner)})
+    if self.mlp == MLP_DENSE:
+        d.update({p + "norm2": (width,), p + "mlp.up": (self.ff, width), p + "mlp.down": (width, self.ff), p + "mlp.act": (4,)})
     if self.mlp == MLP_MOE:
         d[p + "norm2"] = (width,)
         d[p + "mlp.router"] = (self.experts, width)
+        if self.route_bias:
+            d[p + "mlp.router.b"] = (self.experts,)
+        if self.shared_ff > 0:
+            d.update({p + "mlp.shared.gate": (self.shared_ff, width), p + "mlp.shared.up": (self.shared_ff, width),
+                      p + "mlp.shared.down": (width, self.shared_ff)})
         if self.route_correction:
             d[p + "mlp.correction"] = (self.experts,)
         for e in range(self.experts):
@@ -526,7 +552,7 @@ LayerSpec._prenorm2_shapes = _prenorm2_shapes
 
 @dataclass(frozen=True)
 class ListedModelConfig:
-    """A model whose config.json lists its layers (architectures "Dugopel", "Zozonex", "Lazovik", "Sutuvik")."""
+    """A model whose config.json lists its layers (architectures "Dugopel", "Zozonex", "Lazovik", "Sutuvik", "Sozurax")."""
     name: str
     vocab_size: int
     hidden: int
@@ -548,6 +574,8 @@ class ListedModelConfig:
     mixer_conv: int = 0   # taps of the causal convolution added to what every mixer reads
     side_dim: int = 0     # entries of the per-layer token input
     logit_scale: float = 0.0
+    ffn_conv: int = 0     # taps of the causal convolution added to what every feed-forward reads
+    layer_norm: bool = False  # the stream's norms are LayerNorms with weight and additive term
 
     @property
     def has_loop(self) -> bool:
@@ -568,9 +596,10 @@ class ListedModelConfig:
 
     @property
     def needs_state_slots(self) -> bool:
-        """True when some layer keeps recurrent state per sequence (delta rule)."""
-        return self.mixer_conv > 1 or any(l.mixer in (MIXER_DELTA, MIXER_GLA, MIXER_ATTN_TMIX, MIXER_MAMBA2)
-                                          for l in self.layers)
+        """True when some layer keeps state per sequence: a recurrence, the tail of a short convolution."""
+        return self.mixer_conv > 1 or any(
+            l.mixer in (MIXER_DELTA, MIXER_GLA, MIXER_ATTN_TMIX, MIXER_MAMBA2, MIXER_HGRN2) or
+            (self.ffn_conv > 1 and l.mlp != MLP_NONE) for l in self.layers)
 
     def tensor_shapes(self) -> dict:
         d = {"embed": (self.vocab_size, self.hidden), "final.norm": (self.hidden,)}
@@ -578,14 +607,21 @@ class ListedModelConfig:
             d["head"] = (self.vocab_size, self.hidden)
         if self.has_loop:
             d["loop.step"] = (self.loop_times, self.hidden)
+        if self.layer_norm:
+            d["final.norm.b"] = (self.hidden,)
         if self.embed_norm:
             d["embed.norm"] = (self.hidden,)
         if self.side_dim > 0:
             d["side.embed"] = (self.vocab_size, len(self.layers) * self.side_dim)
         for i, l in enumerate(self.layers):
-            d.update(l.tensor_shapes(i, self.hidden))
-            if self.mixer_conv > 1:
+            d.update(l.tensor_shapes(i, self.hidden, self.block_style == LBLOCK_SEQUENTIAL_PRENORM))
+            ffn = l.mlp != MLP_NONE
+            if self.mixer_conv > 0:
                 d[f"l{i}.canon1"] = (self.hidden, self.mixer_conv)
+            if self.ffn_conv > 0 and ffn:
+                d[f"l{i}.canon2"] = (self.hidden, self.ffn_conv)
+            if self.layer_norm:
+                d.update({f"l{i}.norm{k}.b": (self.hidden,) for k in ((1, 2) if ffn else (1,))})
             if self.side_dim > 0:
                 d.update({f"l{i}.side.gate": (self.side_dim, self.hidden), f"l{i}.side.proj": (self.hidden, self.side_dim),
                           f"l{i}.side.norm": (self.hidden,)})
@@ -594,7 +630,7 @@ class ListedModelConfig:
     def matmul_params(self) -> int:
         shapes = self.tensor_shapes()
         n = sum(s[0] * s[1] for k, s in shapes.items()
-                if len(s) == 2 and not k.endswith(".conv") and not k.endswith(".canon1") and k != "side.embed")
+                if len(s) == 2 and not k.endswith((".conv", ".canon1", ".canon2")) and k != "side.embed")
         return n - (0 if self.tied_head else self.vocab_size * self.hidden)
 
     def cache_bytes_per_token(self, bytes_per_el: int = 2) -> int:
@@ -609,11 +645,11 @@ class ListedModelConfig:
         return n
 
     def state_bytes_per_sequence(self) -> int:
-        """fp32 recurrent state + convolution tail of the delta-rule layers."""
+        """fp32 recurrent states + convolution tails of all layers."""
         n = sum(4 * (l.heads * l.dim * l.vdim + (l.conv - 1) * (2 * l.kv_heads * l.dim + l.heads * l.vdim))
                 for l in self.layers if l.mixer == MIXER_DELTA)
         for l in (self.layers[i] for i in self.runs):
-            if l.mixer == MIXER_GLA:
+            if l.mixer in (MIXER_GLA, MIXER_HGRN2):
                 n += 4 * l.heads * l.dim * l.vdim
             elif l.mixer == MIXER_ATTN_TMIX:
                 n += 4 * (l.heads2 * l.dim2 * l.dim2 + self.hidden +
@@ -622,6 +658,8 @@ class ListedModelConfig:
                 n += 4 * (l.heads * l.state * l.vdim + (l.conv - 1) * (l.heads * l.vdim + 2 * l.ssm_groups * l.state))
             if self.mixer_conv > 1:
                 n += 4 * (self.mixer_conv - 1) * self.hidden
+            if self.ffn_conv > 1 and l.mlp != MLP_NONE:
+                n += 4 * (self.ffn_conv - 1) * self.hidden
         return n
 
     def to_c(self, precision: int, num_kv_blocks: int = -1, max_num_seqs: int = 512,
@@ -637,6 +675,7 @@ class ListedModelConfig:
         c.loop_start, c.loop_stop, c.loop_times = self.loop_start, self.loop_stop, self.loop_times
         c.norm_groups, c.embed_norm, c.mixer_conv = self.norm_groups, int(self.embed_norm), self.mixer_conv
         c.side_dim, c.logit_scale = self.side_dim, self.logit_scale
+        c.ffn_conv, c.layer_norm = self.ffn_conv, int(self.layer_norm)
         specs = (CLayerSpec * len(self.layers))(*[l.to_c() for l in self.layers])
         return c, specs
 
@@ -821,6 +860,46 @@ def sutuvik_from_json(j: dict) -> ListedModelConfig:
         logit_scale=float(j.get("logit_scale") or 0.0))
 
 
+def _sozurax_layer(i: int, lc: dict) -> LayerSpec:
+    m = lc["mixer"]
+    kind = lc.get("type")
+    kw = dict(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m.get("vdim") or m["dim"]))
+    if kind == "hgrn2":
+        kw.update(mixer=MIXER_HGRN2)
+    elif kind == "latent_attention":
+        kw.update(mixer=MIXER_LATENT_ATTENTION, rot_dim=int(m["rot_dim"]), kv_rank=int(m["kv_rank"]), q_rank=int(m["q_rank"]),
+                  rot_base=float(m["rot"]["base"]), rot_dims=int(m["rot"].get("dims") or m["rot_dim"]), rot_pairs=1,
+                  scale=float(m["scale"]), window=int((m.get("mask") or {}).get("size") or 0),
+                  kv_from=int(m["kv_from"]) if m.get("kv_from") is not None else -1)
+    else:
+        raise ValueError(f"layer {i}: unknown layer type {kind!r}")
+    mlp = lc.get("mlp")
+    if mlp is None:
+        pass
+    elif mlp["kind"] == "dense":
+        kw.update(mlp=MLP_DENSE, act=FFN_POLYNORM, ff=int(mlp["ff"]))
+    elif mlp["kind"] == "moe":
+        r = mlp["router"]
+        kw.update(mlp=MLP_MOE, act=FFN_SWIGLU, ff=int(mlp["expert"]["ff"]), experts=int(r["experts"]), top=int(r["top"]),
+                  route_norm=1, route_bias=1, shared_ff=int((mlp.get("shared") or {}).get("ff") or 0))
+    else:
+        raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
+    return LayerSpec(**kw)
+
+
+def sozurax_from_json(j: dict) -> ListedModelConfig:
+    """config.json of the Sozurax design: HGRN2 layers and latent attention over a sliding window
+    (cache rows may be another layer's) in any order, pre-norm blocks with LayerNorms, a short causal
+    convolution added to what every mixer and feed-forward reads, PolyNorm dense feed-forwards or
+    softmax-routed gated experts with a plain always-on one, logits through a head of its own."""
+    taps = int((j.get("canon") or {}).get("taps") or 0)
+    return ListedModelConfig(
+        name="sozurax", vocab_size=int(j["vocab"]), hidden=int(j["width"]),
+        layers=tuple(_sozurax_layer(i, lc) for i, lc in enumerate(j["layers"])),
+        norm_eps=float(j["norm"]["eps"]), embedding_scale=float((j.get("embedding") or {}).get("scale", 1.0)),
+        arch=ARCH_SOZURAX, block_style=LBLOCK_SEQUENTIAL_PRENORM, layer_norm=True, mixer_conv=taps, ffn_conv=taps)
+
+
 def safetensors_shapes(model_dir: str) -> dict:
     """Tensor name -> shape from the header of model.safetensors (8-byte little-endian length,
     then that many bytes of JSON)."""
@@ -835,7 +914,7 @@ def safetensors_shapes(model_dir: str) -> dict:
 
 # model registry: config.json "architecture" -> config builder
 ARCHITECTURES = {"Dugopel": dugopel_from_json, "Zozonex": zozonex_from_json, "Lazovik": lazovik_from_json,
-                 "Sutuvik": sutuvik_from_json}
+                 "Sutuvik": sutuvik_from_json, "Sozurax": sozurax_from_json}
 # builders that also want the checkpoint's tensor shapes
 _WANTS_SHAPES = {"Lazovik"}
 

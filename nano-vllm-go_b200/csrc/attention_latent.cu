@@ -19,6 +19,8 @@
 //                         latent rows; one warp per item, a CTA's items share each key tile;
 //                         optional key splits (decode) merged by latent_combine_kernel
 //                         the head's sigmoid gate is applied where the sum is normalised
+// A window (LatentArgs::window) moves the first key tile of a CTA up and masks the keys before each
+// item's window in the tiles where they can occur.  Without `gate` the heads have no gate.
 // All arithmetic is fp32 (double for the angles); QT / KT are the activation / cache dtypes.
 #include <stdlib.h>
 
@@ -63,7 +65,7 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(LatentArgs a, Trace tr
   extern __shared__ float row[];  // [n_in]
   __shared__ float red[32];
   const int t = blockIdx.x;
-  const int n_in = a.q_rank + (a.own_kv ? a.R + a.rot : 0) + a.H;
+  const int n_in = a.q_rank + (a.own_kv ? a.R + a.rot : 0) + (a.gate ? a.H : 0);
   pdl_wait();
   if ((n_in & 7) == 0 && (a.in_stride & 7) == 0) {
     for (int i = threadIdx.x * 8; i < n_in; i += blockDim.x * 8) {
@@ -96,12 +98,17 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(LatentArgs a, Trace tr
     const float inv_k = 1.0f / sqrtf(s2 / (float)a.R + a.eps);
     KT* pr = (KT*)a.pool + (size_t)a.slots[t] * (a.R + a.rot);
     for (int i = threadIdx.x; i < a.R; i += blockDim.x) pr[i] = from_f32<KT>(v[i] * inv_k * a.dkv_norm[i]);
-    // shared key part: entry i pairs with i + half inside the first rot_dims entries
+    // shared key part: entry i pairs with i + half (rot_pairs: with its neighbour) inside the first rot_dims entries
     const float* kr = v + a.R;
     const int half = a.rot_dims / 2;
     for (int i = threadIdx.x; i < a.rot; i += blockDim.x) {
       float o = kr[i];
-      if (i < half) {
+      if (a.rot_pairs) {
+        if (i < a.rot_dims) {
+          const float c = a.cosT[(size_t)t * half + (i >> 1)], s = a.sinT[(size_t)t * half + (i >> 1)];
+          o = (i & 1) ? kr[i] * c + kr[i - 1] * s : kr[i] * c - kr[i + 1] * s;
+        }
+      } else if (i < half) {
         const float c = a.cosT[(size_t)t * half + i], s = a.sinT[(size_t)t * half + i];
         o = kr[i] * c - kr[i + half] * s;
       } else if (i < a.rot_dims) {
@@ -113,6 +120,7 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(LatentArgs a, Trace tr
     }
   }
   const float* g = row + a.q_rank + (a.own_kv ? a.R + a.rot : 0);
+  if (a.gate)
   for (int i = threadIdx.x; i < a.H; i += blockDim.x) a.gate[(size_t)t * a.H + i] = 1.0f / (1.0f + expf(-g[i]));
   TRACE_EXIT(tr);
 }
@@ -158,12 +166,15 @@ __global__ void __launch_bounds__(256) latent_q_kernel(LatentArgs a, Trace tr) {
     const int i = vec ? (i0 / a.rot) * Dk + a.R + i0 % a.rot : i0;
     const int d = i % Dk - a.R;  // index inside the rotated part (negative: absorbed part)
     float v = 0.f, pair = 0.f;
-    const int j = d < 0 || d >= a.rot_dims ? i : (d < half ? i + half : i - half);
+    const int j = d < 0 || d >= a.rot_dims ? i : a.rot_pairs ? i + ((d & 1) ? -1 : 1) : (d < half ? i + half : i - half);
     for (int k = 0; k < a.q_S; k++) {
       v += src[(size_t)k * a.q_stride + i];
       if (j != i) pair += src[(size_t)k * a.q_stride + j];
     }
-    if (j != i) v = d < half ? v * cs[d] - pair * sn[d] : v * cs[d - half] + pair * sn[d - half];
+    if (j != i) {
+      const int f = a.rot_pairs ? d >> 1 : d < half ? d : d - half;
+      v = j > i ? v * cs[f] - pair * sn[f] : v * cs[f] + pair * sn[f];
+    }
     out[i] = from_f32<QT>(v);
   }
   TRACE_EXIT(tr);
@@ -261,9 +272,11 @@ __global__ void __launch_bounds__(LAT_WARPS * 32) latent_attn_kernel(LatentArgs 
   // keys this CTA needs: up to its last item's position; a split takes a contiguous share
   const int last_q = min(nq - 1, (item0 + LAT_WARPS - 1) / a.H);
   const int kv_end = start + q0 + last_q + 1;
+  // ... from the first key inside its first item's window
+  const int first = a.window > 0 ? max(0, start + q0 + item0 / a.H - a.window + 1) / LAT_KT : 0;
   const int n_tiles_k = ceil_div(kv_end, LAT_KT);
-  const int per = ceil_div(n_tiles_k, (int)gridDim.z);
-  const int kt0 = blockIdx.z * per, kt1 = min(n_tiles_k, kt0 + per);
+  const int per = ceil_div(n_tiles_k - first, (int)gridDim.z);
+  const int kt0 = first + blockIdx.z * per, kt1 = min(n_tiles_k, kt0 + per);
   const int* bt = a.block_tables + (size_t)seq * a.max_blocks;
   const KT* pool = (const KT*)a.pool;
 
@@ -286,10 +299,11 @@ __global__ void __launch_bounds__(LAT_WARPS * 32) latent_attn_kernel(LatentArgs 
     for (int i = threadIdx.x; i < nk * Dk; i += blockDim.x) Ks[(i / Dk) * ldk + (i % Dk)] = to_f32(src[i]);
     __syncthreads();
     if (!valid) continue;
-    const int vis = min(nk, qpos - k0 + 1);  // keys of this tile the item sees
-    if (vis <= 0) continue;
+    const int vis = min(nk, qpos - k0 + 1);  // keys [lo, vis) of this tile are the item's
+    const int lo = a.window > 0 ? max(0, qpos - a.window + 1 - k0) : 0;
+    if (vis <= lo) continue;
     float s = -INFINITY;
-    if (lane < vis) {
+    if (lane >= lo && lane < vis) {
       const float* kr = Ks + lane * ldk;
       float d0 = 0.f, d1 = 0.f;
       int d = 0;
@@ -302,11 +316,11 @@ __global__ void __launch_bounds__(LAT_WARPS * 32) latent_attn_kernel(LatentArgs 
     }
     const float m_new = fmaxf(m, warp_max(s));
     const float corr = expf(m - m_new);  // m = -inf on the first visible tile -> 0
-    const float p = lane < vis ? expf(s - m_new) : 0.f;
+    const float p = lane >= lo && lane < vis ? expf(s - m_new) : 0.f;
     l = l * corr + warp_sum(p);
 #pragma unroll
     for (int i = 0; i < LAT_NACC; i++) acc[i] *= corr;
-    for (int j = 0; j < vis; j++) {
+    for (int j = lo; j < vis; j++) {
       const float pj = __shfl_sync(0xffffffffu, p, j);
       const float* vr = Ks + j * ldk;
 #pragma unroll
@@ -321,7 +335,7 @@ __global__ void __launch_bounds__(LAT_WARPS * 32) latent_attn_kernel(LatentArgs 
   TRACE_EXIT(tr);
   if (!valid) return;
   if (gridDim.z == 1) {
-    const float inv = a.gate[(size_t)row * a.H + head] / l;  // the head's sigmoid gate rides on the normalisation
+    const float inv = (a.gate ? a.gate[(size_t)row * a.H + head] : 1.f) / l;  // the head's sigmoid gate rides on the normalisation
     QT* op = (QT*)a.olat + (size_t)row * a.o_ld + head * a.R;
 #pragma unroll
     for (int i = 0; i < LAT_NACC; i++) {
@@ -383,9 +397,10 @@ latent_attn_mma_kernel(LatentArgs a, int two_stage, Trace tr) {
   if (item0 >= n_items) return;
   const int last_q = min(nq - 1, (item0 + LM_ROWS - 1) / a.H);
   const int kv_end = start + q0 + last_q + 1;
+  const int first = a.window > 0 ? max(0, start + q0 + item0 / a.H - a.window + 1) / LM_KT : 0;
   const int n_tiles_k = ceil_div(kv_end, LM_KT);
-  const int per = ceil_div(n_tiles_k, (int)gridDim.z);
-  const int kt0 = blockIdx.z * per, kt1 = min(n_tiles_k, kt0 + per);
+  const int per = ceil_div(n_tiles_k - first, (int)gridDim.z);
+  const int kt0 = first + blockIdx.z * per, kt1 = min(n_tiles_k, kt0 + per);
   const int* bt = a.block_tables + (size_t)seq * a.max_blocks;
   const bf16* pool = (const bf16*)a.pool;
   const bf16* qsrc = (const bf16*)a.qabs + ((size_t)(row0 + q0) * a.H + item0) * Dk;
@@ -411,13 +426,16 @@ latent_attn_mma_kernel(LatentArgs a, int two_stage, Trace tr) {
   if (kt0 < kt1) load_keys(kt0, 0);
   else cp_async_commit();
 
-  // rows g and g + 8 of this warp's 16: the last key position each may see (-1: no such item)
-  int limit[2];
+  // rows g and g + 8 of this warp's 16: the last key position each may see (-1: no such item) and the
+  // first one (its window's); the CTA's rows share tiles whose keys all lie inside every window
+  int limit[2], low[2];
 #pragma unroll
   for (int i = 0; i < 2; i++) {
     const int item = item0 + warp * 16 + g + 8 * i;
     limit[i] = item < n_items ? start + q0 + item / a.H : -1;
+    low[i] = a.window > 0 ? limit[i] - a.window + 1 : 0;
   }
+  const int low_max = a.window > 0 ? start + q0 + last_q - a.window + 1 : 0;
   float o[NR][4];
 #pragma unroll
   for (int dn = 0; dn < NR; dn++)
@@ -470,6 +488,16 @@ latent_attn_mma_kernel(LatentArgs a, int two_stage, Trace tr) {
         if (kp + 1 > limit[0]) s[nt][1] = -INFINITY;
         if (kp > limit[1]) s[nt][2] = -INFINITY;
         if (kp + 1 > limit[1]) s[nt][3] = -INFINITY;
+      }
+      if (kpos0 < low_max) {  // some row's window starts inside or past this tile
+#pragma unroll
+        for (int nt = 0; nt < 8; nt++) {
+          const int kp = kpos0 + nt * 8 + 2 * t;
+          if (kp < low[0]) s[nt][0] = -INFINITY;
+          if (kp + 1 < low[0]) s[nt][1] = -INFINITY;
+          if (kp < low[1]) s[nt][2] = -INFINITY;
+          if (kp + 1 < low[1]) s[nt][3] = -INFINITY;
+        }
       }
 #pragma unroll
       for (int i = 0; i < 2; i++) {
@@ -534,7 +562,7 @@ latent_attn_mma_kernel(LatentArgs a, int two_stage, Trace tr) {
     const size_t it = (size_t)(row0 + q0) * a.H + item;  // row * H + head
     if (gridDim.z == 1) {
       const int row = row0 + q0 + item / a.H, head = item % a.H;
-      const float inv = a.gate[it] / l[i];  // the head's sigmoid gate rides on the normalisation
+      const float inv = (a.gate ? a.gate[it] : 1.f) / l[i];  // the head's sigmoid gate rides on the normalisation
       bf16* op = (bf16*)a.olat + (size_t)row * a.o_ld + head * a.R;
 #pragma unroll
       for (int dn = 0; dn < NR; dn++)
@@ -620,7 +648,7 @@ __global__ void latent_combine_kernel(LatentArgs a, int n_splits, Trace tr) {
   const size_t row = item / a.H;
   const int head = (int)(item % a.H);
   QT* op = (QT*)a.olat + row * a.o_ld + head * a.R;
-  const float inv = a.gate[item] / l;
+  const float inv = (a.gate ? a.gate[item] : 1.f) / l;
   for (int r = threadIdx.x; r < a.R; r += blockDim.x) {
     float o = 0.f;
     for (int s = 0; s < n_splits; s++) {
@@ -637,12 +665,13 @@ __global__ void latent_combine_kernel(LatentArgs a, int n_splits, Trace tr) {
 
 int latent_attn_qtile() { return LAT_QTILE; }
 
-int latent_attn_splits(int n_seqs, int H, int max_len, int sm_count) {
+int latent_attn_splits(int n_seqs, int H, int max_len, int window, int sm_count) {
   static const int forced = getenv("NVLLM_LATENT_SPLITS") ? atoi(getenv("NVLLM_LATENT_SPLITS")) : 0;
   if (forced > 0) return min(forced, 64);
   // decode is latency-bound per key tile (a cached row is a few hundred bytes for all heads):
   // about three 64-key tiles per split, as long as all CTAs of the step stay resident
   const int ctas = n_seqs * ceil_div(H, 64);
+  if (window > 0) max_len = min(max_len, window + LM_KT - 1);  // tiles a window can touch
   int ns = ceil_div(ceil_div(max_len, 64), 3);
   ns = min(ns, max(1, 4 * sm_count / max(1, ctas)));
   return max(1, min(ns, 32));

@@ -92,7 +92,11 @@ cudaError_t launch_embed(cudaStream_t st, int wdt, const int* tokens, const int*
 // residual combine of generic_model.go:320-326 / :359-365 / :405-416:
 //   x <- x + m1 * (sum_s p1[s] + bias1) + m2 * (sum_s p2[s] + bias2);  y = norm(x)
 // The updated row is staged in shared memory so x is read once and written once.
-template <typename YT>
+// TAPS != 0 (NormArgs::conv_taps; > 0 at compile time, -1 read from the arguments): the normed row passes the
+// causal convolution of a step with one row per sequence before it goes out.  Its tail in the state slot was
+// last written in an earlier step, which the step's first kernel has waited for: it is fetched, like
+// the weights, before this kernel's own dependency resolves.
+template <typename YT, int TAPS>
 __global__ void __launch_bounds__(512) norm_kernel(NormArgs a, Trace tr) {
   const unsigned long long t_entry = trace_on(tr) ? gtime() : 0ull;
   pdl_launch_dependents();
@@ -115,6 +119,24 @@ __global__ void __launch_bounds__(512) norm_kernel(NormArgs a, Trace tr) {
     }
     if (a.p1 && a.bias1) load8(a.bias1 + i0, bias1_0);
     if (a.p2 && a.bias2) load8(a.bias2 + i0, bias2_0);
+  }
+  constexpr int KEEP0 = TAPS > 1 ? TAPS - 1 : 1;  // earlier rows fetched ahead
+  float tail0[KEEP0][8], cw0[TAPS > 0 ? TAPS : 1][8];
+  float* tail = nullptr;
+  int cpos = 0;
+  if constexpr (TAPS != 0) {
+    if (TAPS > 1 || a.conv_taps > 1) {  // (one tap: no earlier rows, a model without state slots)
+      tail = a.conv_pool + (size_t)a.conv_slots[blockIdx.x] * a.conv_slot_floats + a.conv_tail_off;
+      cpos = a.conv_pos[blockIdx.x];
+    }
+    if constexpr (TAPS > 0) {
+      if (i0 < H) {
+#pragma unroll
+        for (int j = 0; j < TAPS; j++) load8(a.conv_w + (size_t)j * H + i0, cw0[j]);
+#pragma unroll
+        for (int j = 0; j + 1 < TAPS; j++) load8(tail + (size_t)j * H + i0, tail0[j]);
+      }
+    }
   }
   pdl_wait();
   const unsigned long long t_wait = trace_on(tr) ? gtime() : 0ull;
@@ -248,6 +270,55 @@ __global__ void __launch_bounds__(512) norm_kernel(NormArgs a, Trace tr) {
     return;
   }
   unsigned long long t_loads = 0ull, t_red = 0ull;
+  // eight entries of the normed row -> convolution -> outputs
+  auto emit = [&](int i, float (&o)[8]) {
+    if constexpr (TAPS != 0) {
+      const int taps = TAPS > 0 ? TAPS : a.conv_taps, keep = taps - 1;
+      float y[8], prev[8];
+#pragma unroll
+      for (int e = 0; e < 8; e++) y[e] = o[e];
+      auto tap = [&](int j, const float (&u)[8], const float (&cw)[8]) {
+#pragma unroll
+        for (int e = 0; e < 8; e++) y[e] = fmaf(cw[e], u[e], y[e]);
+        if (j > 0) store8(tail + (size_t)(j - 1) * H + i, u);  // this row is one position further back next time
+      };
+      if constexpr (TAPS > 0) {
+        if (i != i0) {
+#pragma unroll
+          for (int j = 0; j < TAPS; j++) load8(a.conv_w + (size_t)j * H + i, cw0[j]);
+#pragma unroll
+          for (int j = 0; j + 1 < TAPS; j++) load8(tail + (size_t)j * H + i, tail0[j]);
+        }
+#pragma unroll
+        for (int j = 0; j + 1 < TAPS; j++) {
+          if (TAPS - 1 - j > cpos) {  // before the sequence's start: whatever the slot held counts as zero
+#pragma unroll
+            for (int e = 0; e < 8; e++) tail0[j][e] = 0.f;
+          }
+          tap(j, tail0[j], cw0[j]);
+        }
+        tap(TAPS - 1, o, cw0[TAPS - 1]);
+      } else {
+        float cw[8];
+        for (int j = 0; j < keep; j++) {
+          load8(a.conv_w + (size_t)j * H + i, cw);
+          load8(tail + (size_t)j * H + i, prev);
+          if (keep - j > cpos) {
+#pragma unroll
+            for (int e = 0; e < 8; e++) prev[e] = 0.f;
+          }
+          tap(j, prev, cw);
+        }
+        load8(a.conv_w + (size_t)keep * H + i, cw);
+        tap(keep, o, cw);
+      }
+#pragma unroll
+      for (int e = 0; e < 8; e++) o[e] = y[e];
+    }
+    if (a.y) store8((YT*)a.y + (size_t)orow * H + i, o);
+    if (a.y_f32) store8(a.y_f32 + (size_t)orow * H + i, o);
+    if (a.router || a.gate_w) store8(row + i, o);  // each thread overwrites only what it alone reads
+  };
   if (a.groups > 1 && !ln) {
     // RMS norm in equal parts: a warp sums the squares of one part at a time
     __shared__ float ginv[64];
@@ -264,7 +335,6 @@ __global__ void __launch_bounds__(512) norm_kernel(NormArgs a, Trace tr) {
       if (lane == 0) ginv[g] = 1.0f / sqrtf(sq / (float)part + a.eps);
     }
     __syncthreads();
-    YT* yg = a.y ? (YT*)a.y + (size_t)orow * H : nullptr;
     for (int i = i0; i < H; i += blockDim.x * 8) {
       float w[8], o[8];
       if (i == i0) {
@@ -276,9 +346,7 @@ __global__ void __launch_bounds__(512) norm_kernel(NormArgs a, Trace tr) {
         for (int j = 0; j < 8; j++) w[j] = 1.f;
 #pragma unroll
       for (int j = 0; j < 8; j++) o[j] = row[i + j] * ginv[(i + j) / part] * w[j];
-      if (yg) store8(yg + i, o);
-      if (a.y_f32) store8(a.y_f32 + (size_t)orow * H + i, o);
-      if (a.router || a.gate_w) store8(row + i, o);
+      emit(i, o);
     }
   } else {
   t_loads = tr.buf ? gtime() : 0ull;
@@ -300,7 +368,6 @@ __global__ void __launch_bounds__(512) norm_kernel(NormArgs a, Trace tr) {
   } else {
     inv = 1.0f / sqrtf(tot / (float)H + a.eps);
   }
-  YT* yr = a.y ? (YT*)a.y + (size_t)orow * H : nullptr;
   for (int i = i0; i < H; i += blockDim.x * 8) {
     float w[8], bb[8], o[8];
     if (i == i0) {
@@ -326,9 +393,7 @@ __global__ void __launch_bounds__(512) norm_kernel(NormArgs a, Trace tr) {
 #pragma unroll
       for (int j = 0; j < 8; j++) o[j] = row[i + j] * inv * w[j];
     }
-    if (yr) store8(yr + i, o);
-    if (a.y_f32) store8(a.y_f32 + (size_t)orow * H + i, o);
-    if (a.router || a.gate_w) store8(row + i, o);  // each thread overwrites only what it alone reads
+    emit(i, o);
   }
   }
   if (a.gate_w) {  // one number per token: sigmoid(normed row . gate_w), fp32
@@ -360,10 +425,19 @@ cudaError_t launch_norm(cudaStream_t st, const NormArgs& a) {
   // occupancy of the narrow CTA (measured: 512 threads cost cfg3 prefill 35 -> 44 ms)
   if (a.router && a.n_rows <= 1024) threads = 512;
   size_t smem = (size_t)a.H * sizeof(float);
-  if (a.ydt == DT_F32)
-    (void)launch_k(norm_kernel<float>, dim3(a.n_rows), dim3(threads), smem, st, a, next_trace(2));
-  else
-    (void)launch_k(norm_kernel<bf16>, dim3(a.n_rows), dim3(threads), smem, st, a, next_trace(2));
+  if (a.conv_taps < 0 || a.conv_taps > INPUT_CONV_MAX_TAPS || (a.conv_taps > 0 && (a.post || a.plain || a.row_idx)))
+    return cudaErrorInvalidValue;
+#define NK(TP_)                                                                                                        \
+  do {                                                                                                                 \
+    if (a.ydt == DT_F32) (void)launch_k(norm_kernel<float, TP_>, dim3(a.n_rows), dim3(threads), smem, st, a, next_trace(2)); \
+    else (void)launch_k(norm_kernel<bf16, TP_>, dim3(a.n_rows), dim3(threads), smem, st, a, next_trace(2));             \
+  } while (0)
+  if (a.conv_taps == 0) NK(0);
+  else if (a.conv_taps == 2) NK(2);
+  else if (a.conv_taps == 3) NK(3);
+  else if (a.conv_taps == 4) NK(4);
+  else NK(-1);
+#undef NK
   return cudaGetLastError();
 }
 
@@ -438,6 +512,65 @@ cudaError_t launch_act(cudaStream_t st, int odt, int T, int F, const float* h, i
     (void)launch_k(act_kernel<float>, dim3(blocks), dim3(threads), 0, st, T, F, h, S, stride, bias, swiglu, (float*)out, glu_limit, next_trace(6));
   else
     (void)launch_k(act_kernel<bf16>, dim3(blocks), dim3(threads), 0, st, T, F, h, S, stride, bias, swiglu, (bf16*)out, glu_limit, next_trace(6));
+  return cudaGetLastError();
+}
+
+// ------------------------------------------------------------------ PolyNorm
+// CTA per token: the row's split-K slices summed into shared memory while its sums of z^2, z^4 and z^6 are taken,
+// then one pass that applies the cubic with its three normalisers.
+template <typename OT>
+__global__ void __launch_bounds__(256) poly_norm_kernel(int n, int ld, const float* __restrict__ h, int S, size_t stride,
+                                                        const float* __restrict__ coef, float eps, OT* __restrict__ out,
+                                                        Trace tr) {
+  TRACE_ENTRY(tr);
+  pdl_launch_dependents();
+  extern __shared__ float row[];  // [ld]
+  __shared__ float red[32];
+  const float ca = coef[0], cb = coef[1], cc = coef[2], ce = coef[3];
+  pdl_wait();
+  const size_t t = blockIdx.x;
+  float s1 = 0.f, s2 = 0.f, s3 = 0.f;
+  for (int i = threadIdx.x * 8; i < ld; i += blockDim.x * 8) {
+    float z[8];
+    sum_partials8(h + t * ld + i, S, stride, z);
+    store8(row + i, z);
+#pragma unroll
+    for (int e = 0; e < 8; e++)
+      if (i + e < n) {
+        const float q = z[e] * z[e], c = q * z[e];
+        s1 += q;
+        s2 = fmaf(q, q, s2);
+        s3 = fmaf(c, c, s3);
+      }
+  }
+  s1 = block_sum(s1, red);
+  s2 = block_sum(s2, red);
+  s3 = block_sum(s3, red);
+  const float inv_n = 1.0f / (float)n;
+  const float n1 = ca / sqrtf(s1 * inv_n + eps), n2 = cb / sqrtf(s2 * inv_n + eps), n3 = cc / sqrtf(s3 * inv_n + eps);
+  for (int i = threadIdx.x * 8; i < ld; i += blockDim.x * 8) {
+    float z[8], o[8];
+    load8(row + i, z);
+#pragma unroll
+    for (int e = 0; e < 8; e++) o[e] = i + e < n ? fmaf(fmaf(fmaf(n3, z[e], n2), z[e], n1), z[e], ce) : 0.f;
+    store8(out + t * ld + i, o);
+  }
+  TRACE_EXIT(tr);
+}
+
+cudaError_t launch_poly_norm(cudaStream_t st, int odt, int T, int n, int ld, const float* h, int S, size_t stride,
+                             const float* coef, float eps, void* out) {
+  if (T <= 0) return cudaSuccess;
+  if (n <= 0 || n > ld || (ld & 7) || S < 1) return cudaErrorInvalidValue;
+  const size_t smem = (size_t)ld * sizeof(float);
+  const int threads = min(256, max(64, ((ld / 8 + 31) / 32) * 32));
+  if (odt == DT_F32) {
+    if (smem > 48 * 1024) cudaFuncSetAttribute(poly_norm_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    (void)launch_k(poly_norm_kernel<float>, dim3(T), dim3(threads), smem, st, n, ld, h, S, stride, coef, eps, (float*)out, next_trace(6));
+  } else {
+    if (smem > 48 * 1024) cudaFuncSetAttribute(poly_norm_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    (void)launch_k(poly_norm_kernel<bf16>, dim3(T), dim3(threads), smem, st, n, ld, h, S, stride, coef, eps, (bf16*)out, next_trace(6));
+  }
   return cudaGetLastError();
 }
 

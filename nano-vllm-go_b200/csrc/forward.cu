@@ -23,7 +23,7 @@ namespace nvllm {
 void free_workspace(nvllm_handle* h) {
   Workspace& w = h->ws;
   h->drop_graphs();  // the captured decode steps hold these pointers
-  void* ptrs[] = {w.tp_buf, w.x, w.xn, w.xn_f32, w.ws_a, w.ws_b, w.ws_c, w.q, w.attn_out, w.hbuf, w.xn_last,
+  void* ptrs[] = {w.tp_buf, w.x, w.xn, w.xn_f32, w.xn2_f32, w.ws_a, w.ws_b, w.ws_c, w.q, w.attn_out, w.hbuf, w.xn_last,
                   w.xb, w.ssq, w.chain_ctr, w.lat_cq, w.lat_gate, w.lat_o, w.dl_qkv, w.dl_bg, w.dl_o, w.m_xbc, w.m_dt, w.m_y, w.m_yn, w.logits_p, w.logits, w.attn_ws, w.out_tokens, w.amax, w.amax_ticket, w.topk_idx, w.topk_w,
                   w.sort.counts, w.sort.offsets, w.sort.cursor, w.sort.sorted_pair, w.sort.pair_row,
                   w.sort.a_rows, w.sort.tile_expert, w.sort.tile_row0, w.sort.tile_rows,
@@ -131,7 +131,7 @@ int ensure_workspace(nvllm_handle* h, int T, int n) {
         if (s.v_mix) vfirst = std::max(vfirst, (size_t)s.kv_heads * s.vdim);
         split_g = std::max(split_g, (size_t)s.kv_heads);
         split_v = std::max(split_v, (size_t)s.vdim);
-      } else if (s.mixer == NVLLM_MIXER_GLA) {
+      } else if (s.mixer == NVLLM_MIXER_GLA || s.mixer == NVLLM_MIXER_HGRN2) {
         lhd = std::max(lhd, (size_t)s.heads * s.dim);
         lhv = std::max(lhv, (size_t)s.heads * s.vdim);
       } else if (s.mixer == NVLLM_MIXER_ATTN_TMIX) {
@@ -159,6 +159,7 @@ int ensure_workspace(nvllm_handle* h, int T, int n) {
       w.att_split_pairs = (int)pairs;
     }
     if (h->mixer_conv && !h->moe) WS(w.xn_f32, Tc * H * 4);
+    if (h->ffn_conv) WS(w.xn2_f32, Tc * H * 4);
     if (tmix) WS(w.mx_in, (size_t)5 * Tc * H * asz);
     if (shared) WS(w.sh_gate, (size_t)Tc * 4);
     for (auto& r : h->ropes) {

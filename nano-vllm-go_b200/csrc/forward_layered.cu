@@ -17,7 +17,12 @@
 //     (attention_window.cu: whole-row norms, interpolated rotation, score cap, chunked mask, output
 //     gate) beside time mixing with a token shift (linrec.cu), their outputs summed with two scales.
 //     Feed-forward: a mixture of squared-ReLU experts chosen by sigmoid scores, the weight on the
-//     expert's input, plus an always-on expert with a per-token gate.
+//     expert's input, plus an always-on expert with a per-token gate.  Further mixers: attention with
+//     options, Mamba-2, HGRN2 (linrec.cu), latent attention (below; window, neighbouring pairs rotated, no
+//     gate); further feed-forwards: gated experts (+ a plain always-on one), a PolyNorm dense layer.  The
+//     norms may be LayerNorms with an additive term, and what a mixer or a feed-forward reads may pass a
+//     short causal convolution first: inside the norm kernel in steps with one row per sequence, as a launch
+//     of its own (which then also routes) otherwise.
 // Mixer "latent attention" (attention_latent.cu): one fused input projection [W_dq | W_dkv | W_g]
 // of h, RMS-normed latents, the query up projection with W_uk folded in, the absorbed-query
 // attention over the paged latent cache (per-head sigmoid gate applied to its result), the output
@@ -48,6 +53,7 @@ void layered_free(nvllm_handle* h) {
     F(y.post1_w); F(y.post2_w); F(y.conv_w); F(y.a_log); F(y.dt_bias); F(y.onorm_w);
     F(y.bias_in); F(y.o_bias); F(y.qnorm_w); F(y.knorm_w); F(y.lr_w2); F(y.lr_b); F(y.mu); F(y.bonus);
     F(y.w_in2); F(y.w_o2); F(y.sh_gate);
+    F(y.canon2_w); F(y.norm1_b); F(y.norm2_b); F(y.f_lower); F(y.route_bias); F(y.poly);
     F(y.sink_w); F(y.head_temp); F(y.vmix); F(y.conv_b); F(y.d_skip); F(y.route_corr); F(y.canon_w);
     F(y.side_gate); F(y.side_proj); F(y.side_norm);
   }
@@ -83,6 +89,7 @@ struct Dst {
   int64_t rows = 0, cols = 0;  // expected shape ([rows] when cols == 0)
   int ld = 0;            // destination row stride (elements)
   int row_mul = 1, row_add = 0;
+  bool transposed = false;     // [rows, cols] of the file becomes [cols, ld = rows] here
   float add = 0.f;       // vectors: constant added to every element (norm weights stored around zero)
 };
 __global__ void add_const_kernel(float* p, size_t n, float c) {
@@ -90,6 +97,12 @@ __global__ void add_const_kernel(float* p, size_t n, float c) {
   if (i < n) p[i] += c;
 }
 }  // namespace
+
+// layers of the sequential pre-norm blocks whose tensors follow one naming (see layered_set_weight)
+static bool option_block(const nvllm_handle* h, const nvllm_layer_spec& s) {
+  return s.mixer == NVLLM_MIXER_ATTENTION || s.mixer == NVLLM_MIXER_MAMBA2 || s.mixer == NVLLM_MIXER_HGRN2 ||
+         (s.mixer == NVLLM_MIXER_LATENT_ATTENTION && h->block_style == NVLLM_LBLOCK_SEQUENTIAL_PRENORM);
+}
 
 static bool parse_layer_name(const std::string& name, int* layer, std::string* rest) {
   if (name.size() < 3 || name[0] != 'l' || name[1] < '0' || name[1] > '9') return false;
@@ -129,22 +142,28 @@ int layered_set_weight(nvllm_handle* h, const char* cname, int dtype, const void
   if (name == "embed") mat(h->wte, h->V, W, W);
   else if (name == "head" && h->lm_head_owned) mat(h->lm_head, h->V, W, W);
   else if (name == "final.norm") { vec(h->lnf_w, W); d.add = noff; }
+  else if (name == "final.norm.b" && h->lnf_b) vec(h->lnf_b, W);
   else if (name == "embed.norm" && h->embed_norm_w) vec(h->embed_norm_w, W);
   else if (name == "side.embed" && h->side_embed) mat(h->side_embed, h->V, (int64_t)h->L * h->side_dim, h->L * h->side_dim);
   else if (name == "loop.step" && h->loop_step) {
     mat(h->loop_step, h->loop_times, W, W);
     d.ddt = DT_F32; d.p = h->loop_step;
-  } else if (parse_layer_name(name, &l, &rest) && l < h->L &&
-             (h->ll[l].s.mixer == NVLLM_MIXER_ATTENTION || h->ll[l].s.mixer == NVLLM_MIXER_MAMBA2)) {
-    // sequential pre-norm blocks: attention with options / Mamba-2, mixture of gated experts, the
-    // convolution on the mixer's input and the per-layer token input
+  } else if (parse_layer_name(name, &l, &rest) && l < h->L && option_block(h, h->ll[l].s)) {
+    // sequential pre-norm blocks: attention with options / Mamba-2 / HGRN2 / latent attention, mixture of
+    // gated experts or PolyNorm dense layer, the convolutions on the sublayers' inputs, the per-layer token input
     ListedLayer& y = h->ll[l];
     const nvllm_layer_spec& s = y.s;
     auto f32mat = [&](float* p, int64_t rows, int64_t cols) { mat(p, rows, cols, (int)cols); d.ddt = DT_F32; d.p = p; };
     const int hv = s.heads * s.vdim;
+    auto taps = [&](float* p, int n) { mat(p, W, n, W); d.ddt = DT_F32; d.p = p; d.transposed = true; };
     if (rest == "norm1") vec(y.post1_w, W);
     else if (rest == "norm2" && s.mlp != NVLLM_MLP_NONE) vec(y.post2_w, W);
-    else if (rest == "canon1" && y.canon_w) f32mat(y.canon_w, W, h->mixer_conv);
+    else if (rest == "norm1.b" && y.norm1_b) vec(y.norm1_b, W);
+    else if (rest == "norm2.b" && y.norm2_b) vec(y.norm2_b, W);
+    else if (rest == "canon1" && y.canon_w) taps(y.canon_w, h->mixer_conv);
+    else if (rest == "canon2" && y.canon2_w) taps(y.canon2_w, h->ffn_conv);
+    // (a layer without feed-forward reads none of the tensors ahead of one)
+    else if (s.mlp == NVLLM_MLP_NONE && (rest == "norm2" || rest == "norm2.b" || rest == "canon2")) return NVLLM_OK;
     else if (rest == "side.gate" && y.side_gate) mat(y.side_gate, h->side_dim, W, W);
     else if (rest == "side.proj" && y.side_proj) mat(y.side_proj, W, h->side_dim, h->side_p);
     else if (rest == "side.norm" && y.side_norm) vec(y.side_norm, W);
@@ -159,6 +178,24 @@ int layered_set_weight(nvllm_handle* h, const char* cname, int dtype, const void
       else if (rest == "mix.vmix" && s.v_mix) vec(y.vmix, 1);
       else if (rest == "mix.sink" && s.sink_learned) vec(y.sink_w, s.heads);
       else if (rest == "mix.temp" && s.head_temp) vec(y.head_temp, s.heads);
+    } else if (s.mixer == NVLLM_MIXER_HGRN2) {
+      const int hd = s.heads * s.dim;
+      if (rest == "mix.q") mat(y.w_in, hd, W, W, 0);
+      else if (rest == "mix.f") mat(y.w_in, hd, W, W, hd);
+      else if (rest == "mix.v") mat(y.w_in, hv, W, W, 2 * hd);
+      else if (rest == "mix.f.b") vec(y.lr_b, hd);
+      else if (rest == "mix.lower") vec(y.f_lower, hd);
+      else if (rest == "mix.norm") vec(y.onorm_w, s.vdim);
+    } else if (s.mixer == NVLLM_MIXER_LATENT_ATTENTION) {
+      const int own = s.kv_from < 0;
+      if (rest == "mix.dq") mat(y.w_in, s.q_rank, W, W, 0);
+      else if (rest == "mix.dkv" && own) mat(y.w_in, y.Dk, W, W, s.q_rank);
+      else if (rest == "mix.g" && y.lat_gate) mat(y.w_in, s.heads, W, W, s.q_rank + (own ? y.Dk : 0));
+      else if (rest == "mix.dq.norm") vec(y.dq_norm, s.q_rank);
+      else if (rest == "mix.dkv.norm" && own) vec(y.dkv_norm, s.kv_rank);
+      else if (rest == "mix.uq") mat(y.w_uq, y.q_cols, s.q_rank, y.q_rank_p);
+      else if (rest == "mix.uk") mat(y.w_uk, (int64_t)s.heads * s.dim, s.kv_rank, s.kv_rank);
+      else if (rest == "mix.uv") mat(y.w_uv, (int64_t)s.heads * s.vdim, s.kv_rank, s.kv_rank);
     } else {
       if (rest == "mix.in") mat(y.w_in, y.n_in, W, W);
       else if (rest == "mix.conv") f32mat(y.conv_w, y.conv_ch, s.conv);
@@ -168,8 +205,17 @@ int layered_set_weight(nvllm_handle* h, const char* cname, int dtype, const void
       else if (rest == "mix.D") vec(y.d_skip, s.heads);
       else if (rest == "mix.norm") vec(y.onorm_w, hv);
     }
+    if (!d.p && s.mlp == NVLLM_MLP_DENSE) {
+      if (rest == "mlp.up") mat(y.w1, s.ff, W, W);
+      else if (rest == "mlp.down") mat(y.w2, W, s.ff, y.ff_p);
+      else if (rest == "mlp.act") vec(y.poly, 4);
+    }
     if (!d.p && s.mlp == NVLLM_MLP_MOE) {
       if (rest == "mlp.router") f32mat(y.router, s.experts, W);
+      else if (rest == "mlp.router.b" && s.route_bias) vec(y.route_bias, s.experts);
+      else if (rest == "mlp.shared.gate" && s.shared_ff > 0) mat(y.w1, s.shared_ff, W, W, 0, 2, 0);
+      else if (rest == "mlp.shared.up" && s.shared_ff > 0) mat(y.w1, s.shared_ff, W, W, 0, 2, 1);
+      else if (rest == "mlp.shared.down" && s.shared_ff > 0) mat(y.w2, W, s.shared_ff, y.sff_p);
       else if (rest == "mlp.correction" && s.route_correction) vec(y.route_corr, s.experts);
       else if (rest.compare(0, 5, "mlp.e") == 0) {
         size_t i = 5;
@@ -321,6 +367,8 @@ int layered_set_weight(nvllm_handle* h, const char* cname, int dtype, const void
         add_const_kernel<<<(unsigned)((numel + 255) / 256), 256, 0, h->stream>>>((float*)d.p, numel, d.add);
         e = cudaGetLastError();
       }
+    } else if (d.transposed) {
+      e = launch_transpose_convert(h->stream, dtype, stage, (size_t)d.cols, (int)d.rows, (int)d.cols, d.ddt, d.p, d.ld);
     } else e = launch_copy_rows(h->stream, dtype, stage, (size_t)d.cols, (int)d.rows, (int)d.cols, d.ddt, d.p,
                               d.ld, d.row_mul, d.row_add);
   }
@@ -339,15 +387,26 @@ int layered_finalize(nvllm_handle* h) {
   };
   std::vector<std::string> need = {"embed", "final.norm"};
   if (h->lm_head_owned) need.push_back("head");
+  if (h->layer_norm) need.push_back("final.norm.b");
   if (h->loop_step) need.push_back("loop.step");
   if (h->embed_norm_w) need.push_back("embed.norm");
   if (h->side_embed) need.push_back("side.embed");
   for (int l = 0; l < h->L; l++) {
     const nvllm_layer_spec& s = h->ll[l].s;
     const std::string p = "l" + std::to_string(l) + ".";
-    if (s.mixer == NVLLM_MIXER_ATTENTION || s.mixer == NVLLM_MIXER_MAMBA2) {
+    if (option_block(h, s)) {
       need.push_back(p + "norm1");
       need.push_back(p + "mix.o");
+      if (h->ll[l].norm1_b) need.push_back(p + "norm1.b");
+      if (h->ll[l].norm2_b) need.push_back(p + "norm2.b");
+      if (h->ll[l].canon2_w) need.push_back(p + "canon2");
+      if (s.mixer == NVLLM_MIXER_HGRN2) {
+        for (const char* n : {"mix.q", "mix.f", "mix.v", "mix.f.b", "mix.lower", "mix.norm"}) need.push_back(p + n);
+      } else if (s.mixer == NVLLM_MIXER_LATENT_ATTENTION) {
+        for (const char* n : {"mix.dq", "mix.dq.norm", "mix.uq", "mix.uk", "mix.uv"}) need.push_back(p + n);
+        if (s.kv_from < 0) { need.push_back(p + "mix.dkv"); need.push_back(p + "mix.dkv.norm"); }
+        if (h->ll[l].lat_gate) need.push_back(p + "mix.g");
+      } else
       if (s.mixer == NVLLM_MIXER_ATTENTION) {
         for (const char* n : {"mix.q", "mix.k", "mix.v"}) need.push_back(p + n);
         if (s.qk_norm == 3) { need.push_back(p + "mix.q.norm"); need.push_back(p + "mix.k.norm"); }
@@ -365,9 +424,14 @@ int layered_finalize(nvllm_handle* h) {
       if (s.mlp == NVLLM_MLP_MOE) {
         need.push_back(p + "norm2");
         need.push_back(p + "mlp.router");
+        if (s.route_bias) need.push_back(p + "mlp.router.b");
+        if (s.shared_ff > 0)
+          for (const char* n : {"mlp.shared.gate", "mlp.shared.up", "mlp.shared.down"}) need.push_back(p + n);
         if (s.route_correction) need.push_back(p + "mlp.correction");
         for (int e = 0; e < s.experts; e++)
           for (const char* n : {".gate", ".up", ".down"}) need.push_back(p + "mlp.e" + std::to_string(e) + n);
+      } else if (s.mlp == NVLLM_MLP_DENSE) {
+        for (const char* n : {"norm2", "mlp.up", "mlp.down", "mlp.act"}) need.push_back(p + n);
       }
       continue;
     }
@@ -690,13 +754,35 @@ static LinSeg seg_of(const Pending& p, int ld, int col) {
   return g;
 }
 
-// x += pending sublayer results (+ the vector that opens a pass); xn = RMSNorm(x) * w.  With `moe`
-// the kernel also routes the normed row and computes the always-on expert's gate.
-// f32_out: the normed row goes out in fp32 (to xn_f32) instead of the activation dtype — the input of the
-// convolution that precedes a mixer.  plain: no norm, xn = the updated x itself.
+// The routing of a layer with a mixture of experts: fields shared by the kernels that can do it
+template <typename Args>
+static void set_router(nvllm_handle* h, const ListedLayer& y, float* topk_w, Args* a) {
+  const nvllm_layer_spec& s = y.s;
+  a->router = y.router; a->E = s.experts; a->topk = s.top;
+  a->topk_idx = h->ws.topk_idx; a->topk_w = topk_w;
+  a->route = RouteOpts{s.groups, s.keep_groups, s.route_norm ? 0 : 1, 1.f, s.route_sigmoid, s.weight_on_input,
+                       s.route_correction ? y.route_corr : nullptr, s.group_top2, y.route_bias};
+}
+
+// A convolution between a norm and the sublayer that reads it
+struct InputConv {
+  const float* w = nullptr;  // [taps, W]; null: none
+  int taps = 0;
+  size_t off = 0;            // its tail inside a state slot
+  float* buf = nullptr;      // fp32 normed rows of a step with several rows per sequence
+};
+
+// x += pending sublayer results (+ the vector that opens a pass); xn = norm(x) * w (+ b).  With `moe`
+// the kernel also routes the normed row (weights to topk_w) and computes the always-on expert's gate.
+// conv: the row passes a convolution first (and is routed after it).  In steps with one row per sequence
+// that happens in the norm kernel, the tail in the slot included; otherwise the normed rows stay in
+// conv->buf, *tail_job (n_jobs + 1) moves the tail once they have been read.  plain: no norm, xn = the updated x itself.
 static int run_prenorm(nvllm_handle* h, Pending* p1, Pending* p2, const float* row_m2, const float* xadd, const float* w,
-                       const ListedLayer* moe, int T, bool f32_out = false, bool plain = false) {
+                       const float* b, const ListedLayer* moe, float* topk_w, int T, const InputConv* conv = nullptr,
+                       TailJob* tail_job = nullptr, int* n_jobs = nullptr, bool plain = false) {
   Workspace& ws = h->ws;
+  const int32_t* d = h->lay.d;
+  const bool fused = conv && T == h->lay.n;  // one row per sequence
   NormArgs a{};
   a.x = ws.x;
   a.groups = h->norm_groups;
@@ -715,22 +801,60 @@ static int run_prenorm(nvllm_handle* h, Pending* p1, Pending* p2, const float* r
     impl += (double)T * h->H * 4 * (p2->S - 1);
   }
   a.xadd = xadd;
-  a.w = w; a.eps = h->cfg.norm_eps; a.y = ws.xn; a.ydt = h->adt;
-  if (f32_out) { a.y = nullptr; a.y_f32 = ws.xn_f32; }
-  a.n_rows = T; a.H = h->H;
-  if (moe) {
-    const nvllm_layer_spec& s = moe->s;
-    a.router = moe->router; a.E = s.experts; a.topk = s.top;
-    a.topk_idx = ws.topk_idx; a.topk_w = ws.topk_w;
-    a.route = RouteOpts{s.groups, s.keep_groups, s.route_norm ? 0 : 1, 1.f, s.route_sigmoid, s.weight_on_input,
-                        s.route_correction ? moe->route_corr : nullptr, s.group_top2};
-    if (s.shared_ff > 0) { a.gate_w = moe->sh_gate; a.gate_out = ws.sh_gate; }
-    bytes += (double)s.experts * h->H * 4;
+  a.w = w; a.b = b; a.eps = h->cfg.norm_eps; a.y = ws.xn; a.ydt = h->adt;
+  if (fused) {
+    a.conv_w = conv->w; a.conv_taps = conv->taps;
+    a.conv_pos = d + h->lay.positions; a.conv_slots = d + h->lay.state_slots;
+    a.conv_pool = h->state_pool; a.conv_slot_floats = h->state_slot_floats; a.conv_tail_off = conv->off;
+    bytes += (double)T * (conv->taps - 1) * h->H * 8;
+  } else if (conv) {
+    a.y = nullptr; a.y_f32 = conv->buf;
+    bytes += (double)T * h->H * (4 - (double)dt_size(h->adt));
   }
-  ProfScope ps(h, NVLLM_K_NORM, bytes, 0, impl);
-  LAUNCH(h, launch_norm(h->stream, a));
+  a.n_rows = T; a.H = h->H;
+  if (moe && (fused || !conv)) {
+    set_router(h, *moe, topk_w, &a);
+    if (moe->sh_gate) { a.gate_w = moe->sh_gate; a.gate_out = ws.sh_gate; }
+    bytes += (double)moe->s.experts * h->H * 4;
+  }
+  {
+    ProfScope ps(h, NVLLM_K_NORM, bytes, 0, impl);
+    LAUNCH(h, launch_norm(h->stream, a));
+  }
   *p1 = Pending();
   *p2 = Pending();
+  if (!conv || fused) return NVLLM_OK;
+  InputConvArgs c{};
+  c.T = T; c.n_seqs = h->lay.n; c.W = h->H; c.taps = conv->taps;
+  c.h = conv->buf; c.w = conv->w;
+  c.cu_q = d + h->lay.cu_q; c.positions = d + h->lay.positions; c.state_slots = d + h->lay.state_slots;
+  c.state_pool = h->state_pool; c.slot_floats = h->state_slot_floats; c.tail_off = conv->off;
+  c.out = ws.xn;
+  if (moe) set_router(h, *moe, topk_w, &c);
+  {
+    ProfScope ps(h, NVLLM_K_RECUR, (double)T * h->H * (4 + dt_size(h->adt)) + (moe ? (double)moe->s.experts * h->H * 4 : 0.0),
+                 2.0 * T * h->H * (conv->taps + (moe ? moe->s.experts : 0)), (double)T * h->H * 4 * (conv->taps - 1));
+    LAUNCH(h, launch_input_conv(h->stream, h->adt, c));
+  }
+  if (conv->taps > 1) {
+    TailJob& j = tail_job[(*n_jobs)++];
+    j.seg = LinSeg{conv->buf, 1, 0, h->H}; j.bias = nullptr; j.act = nullptr;
+    j.channels = h->H; j.taps = conv->taps; j.tail_off = conv->off;
+  }
+  return NVLLM_OK;
+}
+
+// The tails of the step's convolutions move on (their inputs are still in place)
+static int run_roll_tails(nvllm_handle* h, const TailJob* jobs, int* n_jobs) {
+  if (*n_jobs == 0) return NVLLM_OK;
+  const StepLayout& L = h->lay;
+  const int32_t* d = L.d;
+  double bytes = 0;
+  for (int i = 0; i < *n_jobs; i++) bytes += (double)L.n * (jobs[i].taps - 1) * jobs[i].channels * 8;
+  ProfScope ps(h, NVLLM_K_RECUR, bytes, 0);
+  LAUNCH(h, launch_roll_tails(h->stream, h->adt, L.n, jobs, *n_jobs, d + L.cu_q, d + L.positions, d + L.state_slots,
+                              h->state_pool, h->state_slot_floats));
+  *n_jobs = 0;
   return NVLLM_OK;
 }
 
@@ -755,19 +879,27 @@ static int run_linrec(nvllm_handle* h, const LinRecArgs& a, double in_cols, int 
     LAUNCH(h, launch_linrec_decode(h->stream, h->adt, a));
     return NVLLM_OK;
   }
+  LinRecArgs sc = a;  // what the scan reads
   {
     ProfScope ps(h, NVLLM_K_RECUR, (double)T * (in_cols * 4 + (3 * hd + hv) * 4) + hd * a.rank * 4, 2.0 * T * hd * a.rank,
                  (double)T * in_cols * 4 * (in_S - 1));
-    LAUNCH(h, launch_linrec_prep(h->stream, a));
+    if (a.lower) {
+      LAUNCH(h, launch_hgrn_prep(h->stream, a));
+      sc.q = LinSeg{a.qkw, 1, 0, (int)(3 * hd)};
+      sc.k = LinSeg{a.qkw + (size_t)hd, 1, 0, (int)(3 * hd)};
+      if (a.v.S > 1) sc.v = LinSeg{a.vv, 1, 0, (int)hv};
+    } else {
+      LAUNCH(h, launch_linrec_prep(h->stream, a));
+    }
   }
   {
     // algorithmic: every sequence's state once in and once out, the token inputs once, the read-outs once
     const double state = (double)a.n_seqs * hd * a.vdim * 4 * 2;
     ProfScope ps(h, NVLLM_K_RECUR, state + (double)T * (3 * hd + 2 * hv) * 4, 4.0 * T * hv * a.dim);
-    LAUNCH(h, launch_linrec_scan(h->stream, a));
+    LAUNCH(h, launch_linrec_scan(h->stream, sc));
   }
   {
-    ProfScope ps(h, NVLLM_K_RECUR, (double)T * hv * (4 + 4 + asz), 0, (double)T * hv * 4 * (a.gate.S - 1));
+    ProfScope ps(h, NVLLM_K_RECUR, (double)T * hv * (4 + (a.gate.p ? 4 : 0) + asz), 0, (double)T * hv * 4 * std::max(0, a.gate.S - 1));
     LAUNCH(h, launch_linrec_out(h->stream, h->adt, a));
   }
   return NVLLM_OK;
@@ -789,6 +921,24 @@ static int mixer_gla(nvllm_handle* h, const ListedLayer& y, const LayerRun& r, P
   a.gate = seg_of(pin, y.n_in, 2 * hd + hv); a.lr = seg_of(pin, y.n_in, 2 * hd + 2 * hv);
   a.rank = s.lowrank; a.w2 = y.lr_w2; a.w2b = y.lr_b;
   a.onorm_w = y.onorm_w; a.onorm_ld = 0;
+  a.o_ld = y.ov_p;
+  if ((rc = run_linrec(h, a, y.n_in, pin.S))) return rc;
+  return run_gemm(h, w.attn_out, y.ov_p, y.w_o, T, H, y.ov_p, 1.f, w.ws_b, w.ws_b_floats, H, out);
+}
+
+static int mixer_hgrn2(nvllm_handle* h, const ListedLayer& y, const LayerRun& r, Pending* out) {
+  Workspace& w = h->ws;
+  const nvllm_layer_spec& s = y.s;
+  const int T = h->lay.T, H = h->H, hd = s.heads * s.dim;
+  int rc;
+  Pending pin;
+  if ((rc = run_gemm(h, w.xn, H, y.w_in, T, y.n_in, H, 1.f, w.ws_a, w.ws_a_floats, y.n_in, &pin))) return rc;
+  LinRecArgs a{};
+  linrec_common(h, &a, r);
+  a.H = s.heads; a.dim = s.dim; a.vdim = s.vdim; a.tau = 1.f; a.qmul = 1.f;
+  a.q = seg_of(pin, y.n_in, 0); a.lr = seg_of(pin, y.n_in, hd); a.v = seg_of(pin, y.n_in, 2 * hd);
+  a.w2b = y.lr_b; a.lower = y.f_lower;
+  a.onorm_w = y.onorm_w;
   a.o_ld = y.ov_p;
   if ((rc = run_linrec(h, a, y.n_in, pin.S))) return rc;
   return run_gemm(h, w.attn_out, y.ov_p, y.w_o, T, H, y.ov_p, 1.f, w.ws_b, w.ws_b_floats, H, out);
@@ -899,13 +1049,13 @@ static int mixer_attn_tmix(nvllm_handle* h, const ListedLayer& y, const LayerRun
 
 // Mixture of squared-ReLU experts (+ the always-on expert): *p1 = the experts' outputs, combined
 // by the next norm kernel with the squared scores; *p2 = the always-on expert, times its gate there.
-static int ffn_moe_relu2(nvllm_handle* h, const ListedLayer& y, Pending* p1, Pending* p2) {
+static int ffn_moe_relu2(nvllm_handle* h, const ListedLayer& y, float* topk_w, Pending* p1, Pending* p2) {
   Workspace& w = h->ws;
   const nvllm_layer_spec& s = y.s;
   const int T = h->lay.T, H = h->H;
   const double asz = dt_size(h->adt);
   int rc;
-  if ((rc = run_moe_ffn(h, T, w.xn, s.experts, s.top, y.ff_p, 0.f, y.moe_in, y.moe_out, w.topk_w, p1, 2))) return rc;
+  if ((rc = run_moe_ffn(h, T, w.xn, s.experts, s.top, y.ff_p, 0.f, y.moe_in, y.moe_out, topk_w, p1, 2))) return rc;
   if (s.shared_ff <= 0) return NVLLM_OK;
   const int ff = y.sff_p;
   Pending h1;
@@ -922,6 +1072,50 @@ static int ffn_moe_relu2(nvllm_handle* h, const ListedLayer& y, Pending* p1, Pen
   if (h1.S > 0) {
     ProfScope ps(h, NVLLM_K_ACT, (double)T * ff * (4 + asz), 0, (double)T * ff * 4 * (h1.S - 1));
     LAUNCH(h, launch_act(h->stream, h->adt, T, ff, h1.p, h1.S, h1.stride, nullptr, 2, w.hbuf));
+  }
+  return run_gemm(h, w.hbuf, ff, y.w2, T, H, ff, 1.f, w.ws_b, w.ws_b_floats, H, p2);
+}
+
+// W_down P(W_up h), P the cubic whose powers are normed over the row: both GEMMs with the library's
+// split-K partials between them, the activation needs the whole row
+static int ffn_poly(nvllm_handle* h, const ListedLayer& y, Pending* out) {
+  Workspace& w = h->ws;
+  const int T = h->lay.T, H = h->H, ff = y.ff_p;
+  int rc;
+  Pending h1;
+  if ((rc = run_gemm(h, w.xn, H, y.w1, T, ff, H, 1.f, w.ws_a, w.ws_a_floats, ff, &h1))) return rc;
+  {
+    ProfScope ps(h, NVLLM_K_ACT, (double)T * ff * (4 + dt_size(h->adt)), 0, (double)T * ff * 4 * (h1.S - 1));
+    LAUNCH(h, launch_poly_norm(h->stream, h->adt, T, y.s.ff, ff, h1.p, h1.S, h1.stride, y.poly, h->cfg.norm_eps, w.hbuf));
+  }
+  return run_gemm(h, w.hbuf, ff, y.w2, T, H, ff, 1.f, w.ws_b, w.ws_b_floats, H, out);
+}
+
+// Mixture of gated experts: *p1 = the experts' outputs, combined by the next norm kernel; *p2 = the
+// always-on expert of the same form, if the layer has one
+static int ffn_moe_gated(nvllm_handle* h, const ListedLayer& y, float* topk_w, Pending* p1, Pending* p2) {
+  Workspace& w = h->ws;
+  const nvllm_layer_spec& s = y.s;
+  const int T = h->lay.T, H = h->H;
+  const double asz = dt_size(h->adt);
+  int rc;
+  if ((rc = run_moe_ffn(h, T, w.xn, s.experts, s.top, y.ff_p, 0.f, y.moe_in, y.moe_out, topk_w, p1))) return rc;
+  if (s.shared_ff <= 0) return NVLLM_OK;
+  const int ff = y.sff_p;
+  Pending h1;
+  if ((rc = run_gemm(h, w.xn, H, y.w1, T, 2 * ff, H, 1.f, w.ws_a, w.ws_a_floats, 2 * ff, &h1, TC5_EPI_SWIGLU, w.hbuf, ff, nullptr)))
+    return rc;
+  // steps of <= 8 rows: the gated unit is built inside the down projection's GEMV (one launch less)
+  const char* gpre_env = getenv("NVLLM_GEMV_PRE");
+  if (h1.S > 0 && T <= 8 && !(gpre_env && atoi(gpre_env) == 0)) {
+    GemvPre ga{};
+    ga.mode = 2; ga.hp = h1.p; ga.Sh = h1.S; ga.hstride = h1.stride; ga.hld = 2 * ff; ga.swiglu = 1;
+    return run_gemm(h, w.hbuf, ff, y.w2, T, H, ff, 1.f, w.ws_b, w.ws_b_floats, H, p2, 0, nullptr, 0, nullptr, nullptr, 0,
+                    0.0, nullptr, nullptr, &ga);
+  }
+  if (h1.S > 0) {
+    ProfScope ps(h, NVLLM_K_ACT, (double)T * ff * (8 + asz), 0, (double)T * 2 * ff * 4 * (h1.S - 1));
+    LAUNCH(h, launch_act(h->stream, h->adt, T, ff, h1.p, h1.S, h1.stride, nullptr, 1, w.hbuf));
   }
   return run_gemm(h, w.hbuf, ff, y.w2, T, H, ff, 1.f, w.ws_b, w.ws_b_floats, H, p2);
 }
@@ -1078,6 +1272,71 @@ static int mixer_mamba2(nvllm_handle* h, const ListedLayer& y, const LayerRun& r
   return run_gemm(h, w.attn_out, y.ov_p, y.w_o, T, H, y.ov_p, 1.f, w.ws_b, w.ws_b_floats, H, out);
 }
 
+// Latent attention on the normed rows in xn; its result stays pending in *out
+static int mixer_latent(nvllm_handle* h, const ListedLayer& y, Pending* out) {
+  const StepLayout& L = h->lay;
+  Workspace& w = h->ws;
+  const nvllm_layer_spec& s = y.s;
+  const int T = L.T, n = L.n, H = h->H;
+  const int32_t* d = L.d;
+  cudaStream_t st = h->stream;
+  const double asz = dt_size(h->adt), kvsz = dt_size(h->kvdt);
+  int rc;
+  const int own = s.kv_from < 0;
+  Pending pin;
+  if ((rc = run_gemm(h, w.xn, H, y.w_in, T, y.n_in, H, 1.f, w.ws_a, w.ws_a_floats, y.n_in, &pin))) return rc;
+  const RopeTable& rt = h->ropes[y.rope];
+  LatentArgs a{};
+  a.T = T; a.H = s.heads; a.dim = s.dim; a.rot = s.rot_dim; a.rot_dims = s.rot_dims; a.vdim = s.vdim;
+  a.R = s.kv_rank; a.q_rank = s.q_rank; a.q_rank_p = y.q_rank_p; a.o_ld = y.ovr_p; a.own_kv = own; a.window = s.window; a.rot_pairs = s.rot_pairs;
+  a.eps = h->cfg.norm_eps; a.scale = s.scale;
+  a.in_p = pin.p; a.in_S = pin.S; a.in_stride = pin.stride; a.in_ld = y.n_in;
+  a.dq_norm = y.dq_norm; a.dkv_norm = y.dkv_norm;
+  a.cosT = rt.cosT; a.sinT = rt.sinT;
+  a.slots = d + L.slots;
+  a.pool = h->lat_pools[y.pool];
+  a.cq = w.lat_cq; a.gate = y.lat_gate ? w.lat_gate : nullptr;
+  a.qabs = w.q;
+  a.block_tables = d + L.block_tables; a.max_blocks = L.max_blocks;
+  a.cu_q = d + L.cu_q; a.seq_start = d + L.seq_start; a.seq_len = d + L.seq_len;
+  a.olat = w.lat_o;
+  a.split_ws = w.attn_ws;
+  a.sm_count = h->sm_count;
+  if (L.prefill) {
+    a.tile_seq = d + L.tile_seq; a.tile_q0 = d + L.tile_q0; a.n_tiles = L.n_qtiles;
+    a.qtile = h->attn_qtile; a.n_splits = 1;
+  } else {
+    a.n_tiles = n; a.qtile = 1;
+    a.n_splits = latent_attn_splits(n, s.heads, L.max_len, s.window, h->sm_count);
+    while (a.n_splits > 1 && (size_t)T * s.heads * a.n_splits * (s.kv_rank + 2) > w.attn_ws_floats) a.n_splits--;
+  }
+  {
+    ProfScope ps(h, NVLLM_K_ROPE_KV, (double)T * y.n_in * 4 + (double)T * (y.q_rank_p * asz + own * y.Dk * kvsz), 0,
+                 (double)T * y.n_in * 4 * (pin.S - 1));
+    LAUNCH(h, launch_latent_prep(st, h->adt, h->kvdt, a));
+  }
+  const int qn = s.heads * y.Dk;
+  Pending pq;
+  if ((rc = run_gemm(h, w.lat_cq, y.q_rank_p, y.w_q, T, qn, y.q_rank_p, 1.f, w.ws_a, w.ws_a_floats, qn, &pq)))
+    return rc;
+  a.q_p = pq.p; a.q_S = pq.S; a.q_stride = pq.stride; a.q_ld = qn;
+  {
+    ProfScope ps(h, NVLLM_K_ROPE_KV, (double)T * qn * (4 + asz), 0, (double)T * qn * 4 * (pq.S - 1));
+    LAUNCH(h, launch_latent_q(st, h->adt, a));
+  }
+  {
+    // algorithmic: every cached row the queries can see once; flops: scores over Dk, sums over R
+    const double win = s.window > 0 ? s.window : 1e30;
+    const double bytes = std::min((double)L.sum_len, (double)n * (win - 1) + (double)T) * y.Dk * kvsz;
+    const double flops = 2.0 * s.heads * (y.Dk + s.kv_rank) * std::min(L.attn_pairs, (double)T * win);
+    ProfScope ps(h, L.prefill ? NVLLM_K_ATTN_PREFILL : NVLLM_K_ATTN_DECODE, bytes, flops,
+                 (double)T * (qn + y.ovr_p) * asz);
+    LAUNCH(h, launch_latent_attn(st, h->adt, h->kvdt, a));
+    if (a.n_splits > 1) h->launches++;
+  }
+  return run_gemm(h, w.lat_o, y.ovr_p, y.w_ov, T, H, y.ovr_p, 1.f, w.ws_b, w.ws_b_floats, H, out);
+}
+
 // Per-layer token input after the feed-forward: x += rmsnorm(W_proj (gelu_tanh(W_gate x) * e)) * w, e = the
 // token's entries of this layer's part of the side table.  The pending results join x first (the
 // gate reads the updated stream itself, not a normed copy).
@@ -1086,7 +1345,8 @@ static int token_side_input(nvllm_handle* h, const ListedLayer& y, int layer, Pe
   Workspace& w = h->ws;
   const int T = L.T, H = h->H, sp = h->side_p;
   int rc;
-  if ((rc = run_prenorm(h, p1, p2, row_m2, nullptr, nullptr, nullptr, T, false, true))) return rc;
+  if ((rc = run_prenorm(h, p1, p2, row_m2, nullptr, nullptr, nullptr, nullptr, nullptr, T, nullptr, nullptr, nullptr, true)))
+    return rc;
   Pending pg;
   if ((rc = run_gemm(h, w.xn, H, y.side_gate, T, sp, H, 1.f, w.ws_a, w.ws_a_floats, sp, &pg))) return rc;
   {
@@ -1103,60 +1363,50 @@ static int token_side_input(nvllm_handle* h, const ListedLayer& y, int layer, Pe
 static int forward_layers_prenorm(nvllm_handle* h, Pending* p1, Pending* p2, const float** row_m2_out) {
   const int T = h->lay.T;
   const float* row_m2 = nullptr;  // per-row multiplier of the pending second addend
+  int routed = 0;                 // routed layers so far
   int rc;
   for (size_t ri = 0; ri < h->runs.size(); ri++) {
     const LayerRun& r = h->runs[ri];
     const ListedLayer& y = h->ll[r.layer];
     const float* xadd = r.pass_start >= 0 ? h->loop_step + (size_t)r.pass_start * h->H : nullptr;
-    const bool conv_in = y.canon_w != nullptr;  // the mixer reads h + conv(h)
-    if ((rc = run_prenorm(h, p1, p2, row_m2, xadd, y.post1_w, nullptr, T, conv_in))) return rc;
+    TailJob jobs[TAIL_MAX_JOBS];
+    int n_jobs = 0;
+    const InputConv c1{y.canon_w, h->mixer_conv, r.canon_off, h->ws.xn_f32}, c2{y.canon2_w, h->ffn_conv, r.canon2_off, h->ws.xn2_f32};
+    if ((rc = run_prenorm(h, p1, p2, row_m2, xadd, y.post1_w, y.norm1_b, nullptr, nullptr, T, c1.w ? &c1 : nullptr, jobs, &n_jobs)))
+      return rc;
     row_m2 = nullptr;
-    const StepLayout& L = h->lay;
-    const int32_t* d = L.d;
-    if (conv_in) {
-      ProfScope ps(h, NVLLM_K_RECUR, (double)T * h->H * (4 + dt_size(h->adt)), 2.0 * T * h->H * h->mixer_conv,
-                   (double)T * h->H * 4 * (h->mixer_conv - 1));
-      LAUNCH(h, launch_mixer_conv(h->stream, h->adt, T, L.n, h->H, h->mixer_conv, h->ws.xn_f32, y.canon_w, d + L.cu_q,
-                                  d + L.positions, d + L.state_slots, h->state_pool, h->state_slot_floats, r.canon_off,
-                                  h->ws.xn));
-    }
     Pending pa, pb, pin;
     if (y.s.mixer == NVLLM_MIXER_GLA) rc = mixer_gla(h, y, r, &pa);
     else if (y.s.mixer == NVLLM_MIXER_ATTENTION) rc = mixer_attention(h, y, (int)ri, &pa);
     else if (y.s.mixer == NVLLM_MIXER_MAMBA2) rc = mixer_mamba2(h, y, r, &pin, &pa);
+    else if (y.s.mixer == NVLLM_MIXER_HGRN2) rc = mixer_hgrn2(h, y, r, &pa);
+    else if (y.s.mixer == NVLLM_MIXER_LATENT_ATTENTION) rc = mixer_latent(h, y, &pa);
     else rc = mixer_attn_tmix(h, y, r, (int)ri, &pa, &pb);
     if (rc) return rc;
-    if (conv_in || y.s.mixer == NVLLM_MIXER_MAMBA2) {
-      // the slot's tails move on: the normed rows the mixer's convolution read (still in xn_f32) and Mamba-2's
-      // convolution inputs (still in ws_a: the output projection wrote elsewhere)
-      TailJob jobs[2];
-      int nj = 0;
-      double bytes = 0;
-      if (conv_in) {
-        TailJob& j = jobs[nj++];
-        j.seg = LinSeg{h->ws.xn_f32, 1, 0, h->H}; j.bias = nullptr; j.act = nullptr;
-        j.channels = h->H; j.taps = h->mixer_conv; j.tail_off = r.canon_off;
-        bytes += (double)L.n * (h->mixer_conv - 1) * h->H * 8;
-      }
-      if (y.s.mixer == NVLLM_MIXER_MAMBA2 && y.s.conv > 1) {
-        TailJob& j = jobs[nj++];
-        j.seg = seg_of(pin, y.n_in, y.s.heads * y.s.vdim); j.bias = nullptr; j.act = nullptr;
-        j.channels = y.conv_ch; j.taps = y.s.conv; j.tail_off = r.tail_off;
-        bytes += (double)L.n * (y.s.conv - 1) * y.conv_ch * 8;
-      }
-      if (nj) {
-        ProfScope ps(h, NVLLM_K_RECUR, bytes, 0);
-        LAUNCH(h, launch_roll_tails(h->stream, h->adt, L.n, jobs, nj, d + L.cu_q, d + L.positions, d + L.state_slots,
-                                    h->state_pool, h->state_slot_floats));
-      }
+    if (y.s.mixer == NVLLM_MIXER_MAMBA2 && y.s.conv > 1) {
+      // Mamba-2's convolution inputs are still in ws_a (the output projection wrote elsewhere)
+      TailJob& j = jobs[n_jobs++];
+      j.seg = seg_of(pin, y.n_in, y.s.heads * y.s.vdim); j.bias = nullptr; j.act = nullptr;
+      j.channels = y.conv_ch; j.taps = y.s.conv; j.tail_off = r.tail_off;
     }
-    if (y.s.mlp == NVLLM_MLP_MOE && y.s.act == NVLLM_FFN_SWIGLU) {
-      if ((rc = run_prenorm(h, &pa, &pb, nullptr, nullptr, y.post2_w, &y, T))) return rc;
-      if ((rc = run_moe_ffn(h, T, h->ws.xn, y.s.experts, y.s.top, y.ff_p, 0.f, y.moe_in, y.moe_out, h->ws.topk_w, p1))) return rc;
-    } else if (y.s.mlp == NVLLM_MLP_MOE) {
-      if ((rc = run_prenorm(h, &pa, &pb, nullptr, nullptr, y.post2_w, &y, T))) return rc;
-      if ((rc = ffn_moe_relu2(h, y, p1, p2))) return rc;
-      row_m2 = p2->p ? h->ws.sh_gate : nullptr;
+    // without a convolution ahead of the feed-forward the tails move now; with one, its rows have a buffer of
+    // their own and the mixer's are moved in the same launch — unless ws_a holds a tail
+    if (!c2.w || y.s.mixer == NVLLM_MIXER_MAMBA2)
+      if ((rc = run_roll_tails(h, jobs, &n_jobs))) return rc;
+    if (y.s.mlp != NVLLM_MLP_NONE) {
+      // a routed layer's norm kernel combines the previous routed layer's experts while it writes its own
+      // routing weights: the two halves of topk_w alternate
+      const bool moe = y.s.mlp == NVLLM_MLP_MOE;
+      float* topk_w = h->ws.topk_w + (moe ? (size_t)(routed++ & 1) * h->ws.topk_pairs : 0);
+      if ((rc = run_prenorm(h, &pa, &pb, nullptr, nullptr, y.post2_w, y.norm2_b, moe ? &y : nullptr, topk_w, T,
+                            c2.w ? &c2 : nullptr, jobs, &n_jobs)))
+        return rc;
+      if ((rc = run_roll_tails(h, jobs, &n_jobs))) return rc;
+      if (!moe) rc = ffn_poly(h, y, p1);
+      else if (y.s.act == NVLLM_FFN_SWIGLU) rc = ffn_moe_gated(h, y, topk_w, p1, p2);
+      else rc = ffn_moe_relu2(h, y, topk_w, p1, p2);
+      if (rc) return rc;
+      row_m2 = moe && y.s.act == NVLLM_FFN_RELU2 && p2->p ? h->ws.sh_gate : nullptr;
     } else {
       *p1 = pa;
       *p2 = pb;
@@ -1220,60 +1470,8 @@ int forward_step_layered(nvllm_handle* h) {
     if ((rc = run_norm(h, w.x, &p1, &p2, y.norm_w, nullptr, w.xn, nullptr, nullptr, T,
                        s.mlp == NVLLM_MLP_MOE ? &ra : nullptr, true)))
       return rc;
-    // ---- mixer: latent attention
-    const int own = s.kv_from < 0;
-    Pending pin;
-    if ((rc = run_gemm(h, w.xn, H, y.w_in, T, y.n_in, H, 1.f, w.ws_a, w.ws_a_floats, y.n_in, &pin))) return rc;
-    const RopeTable& rt = h->ropes[y.rope];
-    LatentArgs a{};
-    a.T = T; a.H = s.heads; a.dim = s.dim; a.rot = s.rot_dim; a.rot_dims = s.rot_dims; a.vdim = s.vdim;
-    a.R = s.kv_rank; a.q_rank = s.q_rank; a.q_rank_p = y.q_rank_p; a.o_ld = y.ovr_p; a.own_kv = own;
-    a.eps = h->cfg.norm_eps; a.scale = s.scale;
-    a.in_p = pin.p; a.in_S = pin.S; a.in_stride = pin.stride; a.in_ld = y.n_in;
-    a.dq_norm = y.dq_norm; a.dkv_norm = y.dkv_norm;
-    a.cosT = rt.cosT; a.sinT = rt.sinT;
-    a.slots = d + L.slots;
-    a.pool = h->lat_pools[y.pool];
-    a.cq = w.lat_cq; a.gate = w.lat_gate;
-    a.qabs = w.q;
-    a.block_tables = d + L.block_tables; a.max_blocks = L.max_blocks;
-    a.cu_q = d + L.cu_q; a.seq_start = d + L.seq_start; a.seq_len = d + L.seq_len;
-    a.olat = w.lat_o;
-    a.split_ws = w.attn_ws;
-    a.sm_count = h->sm_count;
-    if (L.prefill) {
-      a.tile_seq = d + L.tile_seq; a.tile_q0 = d + L.tile_q0; a.n_tiles = L.n_qtiles;
-      a.qtile = LAT_QTILE; a.n_splits = 1;
-    } else {
-      a.n_tiles = n; a.qtile = 1;
-      a.n_splits = latent_attn_splits(n, s.heads, L.max_len, h->sm_count);
-      while (a.n_splits > 1 && (size_t)T * s.heads * a.n_splits * (s.kv_rank + 2) > w.attn_ws_floats) a.n_splits--;
-    }
-    {
-      ProfScope ps(h, NVLLM_K_ROPE_KV, (double)T * y.n_in * 4 + (double)T * (y.q_rank_p * asz + own * y.Dk * kvsz), 0,
-                   (double)T * y.n_in * 4 * (pin.S - 1));
-      LAUNCH(h, launch_latent_prep(st, h->adt, h->kvdt, a));
-    }
-    const int qn = s.heads * y.Dk;
-    Pending pq;
-    if ((rc = run_gemm(h, w.lat_cq, y.q_rank_p, y.w_q, T, qn, y.q_rank_p, 1.f, w.ws_a, w.ws_a_floats, qn, &pq)))
-      return rc;
-    a.q_p = pq.p; a.q_S = pq.S; a.q_stride = pq.stride; a.q_ld = qn;
-    {
-      ProfScope ps(h, NVLLM_K_ROPE_KV, (double)T * qn * (4 + asz), 0, (double)T * qn * 4 * (pq.S - 1));
-      LAUNCH(h, launch_latent_q(st, h->adt, a));
-    }
-    {
-      // algorithmic: every cached row of the contexts once; flops: scores over Dk, sums over R
-      const double bytes = (double)L.sum_len * y.Dk * kvsz;
-      const double flops = 2.0 * s.heads * (y.Dk + s.kv_rank) * L.attn_pairs;
-      ProfScope ps(h, L.prefill ? NVLLM_K_ATTN_PREFILL : NVLLM_K_ATTN_DECODE, bytes, flops,
-                   (double)T * (qn + y.ovr_p) * asz);
-      LAUNCH(h, launch_latent_attn(st, h->adt, h->kvdt, a));
-      if (a.n_splits > 1) h->launches++;
-    }
     Pending pa;
-    if ((rc = run_gemm(h, w.lat_o, y.ovr_p, y.w_ov, T, H, y.ovr_p, 1.f, w.ws_b, w.ws_b_floats, H, &pa))) return rc;
+    if ((rc = mixer_latent(h, y, &pa))) return rc;
     // ---- feed-forward on the same normed input
     Pending pm;
     if (s.mlp == NVLLM_MLP_DENSE) {
@@ -1313,7 +1511,7 @@ int forward_step_layered(nvllm_handle* h) {
     }
   }
   // final norm + LM head on the rows that were asked for: each sequence's last, then the extra ones
-  if ((rc = run_norm(h, w.x, &p1, &p2, h->lnf_w, nullptr, w.xn_last, nullptr, d + L.last_row, n_out, nullptr,
+  if ((rc = run_norm(h, w.x, &p1, &p2, h->lnf_w, h->lnf_b, w.xn_last, nullptr, d + L.last_row, n_out, nullptr,
                      h->block_style == NVLLM_LBLOCK_PARALLEL_PRENORM, row_m2)))
     return rc;
   Pending lg;
@@ -1342,6 +1540,22 @@ int forward_step_layered(nvllm_handle* h) {
 
 using namespace nvllm;
 
+// what is wrong with a latent-attention layer's sizes (null: nothing)
+static const char* latent_spec_error(const nvllm_layer_spec* layers, int l) {
+  const nvllm_layer_spec& s = layers[l];
+  if (s.heads <= 0 || s.dim <= 0 || s.rot_dim <= 0 || s.vdim <= 0 || s.kv_rank <= 0 || s.q_rank <= 0) return "non-positive mixer size";
+  if (s.kv_rank > 512) return "kv_rank above 512";
+  if (s.rot_dims < 2 || s.rot_dims > s.rot_dim || (s.rot_dims & 1)) return "rotated entries must be even and <= rot_dim";
+  if (s.window < 0) return "negative window";
+  if (s.kv_from >= 0) {
+    if (s.kv_from >= l) return "kv_from must name an earlier layer";
+    const nvllm_layer_spec& j = layers[s.kv_from];
+    if (j.mixer != NVLLM_MIXER_LATENT_ATTENTION || j.kv_from >= 0) return "kv_from must name a layer with its own down projection";
+    if (j.kv_rank != s.kv_rank || j.rot_dim != s.rot_dim) return "kv_from layer has other cache sizes";
+  }
+  return nullptr;
+}
+
 extern "C" int nvllm_create_layered(const nvllm_layered_config* c, const nvllm_layer_spec* layers,
                                     nvllm_handle** out) {
   if (!c || !layers || !out) return set_err(nullptr, NVLLM_ERR_INVALID, "null argument");
@@ -1358,19 +1572,27 @@ extern "C" int nvllm_create_layered(const nvllm_layered_config* c, const nvllm_l
   const bool has_loop = c->loop_times >= 1 && c->loop_stop > c->loop_start;
   if (has_loop && (!pre_style || c->loop_start < 0 || c->loop_stop > c->num_layers))
     return bad(-1, "a repeated run of layers needs the sequential pre-norm block style and 0 <= start < stop <= layers");
-  if ((c->norm_groups > 1 || c->embed_norm || c->mixer_conv > 1 || c->side_dim > 0) && !pre_style)
-    return bad(-1, "grouped norms, a normed embedding, the convolution on the mixers' input and the per-layer token input need the sequential pre-norm block style");
+  if ((c->norm_groups > 1 || c->embed_norm || c->mixer_conv > 0 || c->ffn_conv > 0 || c->side_dim > 0 || c->layer_norm) && !pre_style)
+    return bad(-1, "grouped norms, a normed embedding, convolutions on the sublayers' inputs, LayerNorms with an additive term and the per-layer token input need the sequential pre-norm block style");
+  if (c->layer_norm && (c->norm_groups > 1 || c->embed_norm)) return bad(-1, "LayerNorms are not split in parts and have no form on the embedding");
   if (c->norm_groups > 64 || (c->norm_groups > 1 && c->hidden % c->norm_groups)) return bad(-1, "norm groups must divide the width (at most 64)");
-  if (c->mixer_conv < 0 || c->mixer_conv > 8) return bad(-1, "convolution on the mixers' input: at most 8 taps");
+  if (c->mixer_conv < 0 || c->mixer_conv > INPUT_CONV_MAX_TAPS || c->ffn_conv < 0 || c->ffn_conv > INPUT_CONV_MAX_TAPS)
+    return bad(-1, "convolution on a sublayer's input: at most 8 taps");
   if (c->side_dim < 0) return bad(-1, "negative side_dim");
   int vmix_first = -1;
   for (int l = 0; l < c->num_layers; l++) {
     const nvllm_layer_spec& s = layers[l];
     const bool seq_style = c->block_style == NVLLM_LBLOCK_SEQUENTIAL_POSTNORM;
-    if (s.mixer == NVLLM_MIXER_ATTENTION || s.mixer == NVLLM_MIXER_MAMBA2) {
-      if (!pre_style) return bad(l, "attention with options / Mamba-2 need the sequential pre-norm block style");
+    if (s.mixer == NVLLM_MIXER_ATTENTION || s.mixer == NVLLM_MIXER_MAMBA2 || s.mixer == NVLLM_MIXER_HGRN2 ||
+        (s.mixer == NVLLM_MIXER_LATENT_ATTENTION && pre_style)) {
+      if (!pre_style) return bad(l, "attention with options / Mamba-2 / HGRN2 need the sequential pre-norm block style");
       if (s.heads <= 0 || s.vdim <= 0) return bad(l, "non-positive mixer size");
-      if (s.mixer == NVLLM_MIXER_ATTENTION) {
+      if (s.mixer == NVLLM_MIXER_LATENT_ATTENTION) {
+        if (const char* what = latent_spec_error(layers, l)) return bad(l, what);
+        if (has_loop) return bad(l, "latent attention has one cache per layer: no repeated run of layers");
+      } else if (s.mixer == NVLLM_MIXER_HGRN2) {
+        if (s.dim <= 0 || s.dim > LINREC_MAX_DIM) return bad(l, "HGRN2: 0 < dim <= 256");
+      } else if (s.mixer == NVLLM_MIXER_ATTENTION) {
         if (s.kv_heads <= 0 || s.dim <= 0 || s.heads % s.kv_heads) return bad(l, "heads must be a multiple of kv_heads");
         if (s.vdim > 512 || s.dim > 1024) return bad(l, "attention: dim <= 1024, vdim <= 512");
         if (s.qk_norm != 0 && s.qk_norm != 1 && s.qk_norm != 3) return bad(l, "attention: qk_norm 0, 1 (per head) or 3 (per head, weighted)");
@@ -1390,8 +1612,11 @@ extern "C" int nvllm_create_layered(const nvllm_layered_config* c, const nvllm_l
         if (s.norm_groups <= 0 || s.norm_groups > 64 || (s.heads * s.vdim) % s.norm_groups) return bad(l, "Mamba-2: norm groups must divide heads * vdim (at most 64)");
         if (s.conv < 1 || s.conv > 8) return bad(l, "convolution taps 1..8");
       }
-      if (s.mlp != NVLLM_MLP_NONE && s.mlp != NVLLM_MLP_MOE) return bad(l, "pre-norm blocks: feed-forward none or mixture of experts");
+      if (s.mlp < NVLLM_MLP_NONE || s.mlp > NVLLM_MLP_MOE) return bad(l, "unknown feed-forward kind");
+      if (s.mlp == NVLLM_MLP_DENSE && (s.ff <= 0 || s.act != NVLLM_FFN_POLYNORM)) return bad(l, "pre-norm blocks: a dense feed-forward has ff > 0 and the PolyNorm activation");
+      if (s.mlp == NVLLM_MLP_DENSE && s.ff > 48 * 1024) return bad(l, "PolyNorm: ff <= 49152");
       if (s.mlp == NVLLM_MLP_MOE) {
+        if (s.shared_ff < 0) return bad(l, "negative shared_ff");
         if (s.act != NVLLM_FFN_SWIGLU) return bad(l, "these blocks take gated experts W_down (silu(W_gate h) * W_up h)");
         if (s.ff <= 0 || s.experts <= 0 || s.experts > 256 || s.top <= 0 || s.top > 32 || s.top > s.experts)
           return bad(l, "ff > 0, experts 1..256, top 1..32");
@@ -1451,16 +1676,8 @@ extern "C" int nvllm_create_layered(const nvllm_layered_config* c, const nvllm_l
     }
     if (s.mixer != NVLLM_MIXER_LATENT_ATTENTION) return bad(l, "unknown mixer kind");
     if (seq_style) return bad(l, "latent attention needs the parallel pre-norm block style");
-    if (s.heads <= 0 || s.dim <= 0 || s.rot_dim <= 0 || s.vdim <= 0 || s.kv_rank <= 0 || s.q_rank <= 0)
-      return bad(l, "non-positive mixer size");
-    if (s.kv_rank > 512) return bad(l, "kv_rank above 512");
-    if (s.rot_dims < 2 || s.rot_dims > s.rot_dim || (s.rot_dims & 1)) return bad(l, "rotated entries must be even and <= rot_dim");
-    if (s.kv_from >= 0) {
-      if (s.kv_from >= l) return bad(l, "kv_from must name an earlier layer");
-      const nvllm_layer_spec& j = layers[s.kv_from];
-      if (j.kv_from >= 0) return bad(l, "kv_from must name a layer with its own down projection");
-      if (j.kv_rank != s.kv_rank || j.rot_dim != s.rot_dim) return bad(l, "kv_from layer has other cache sizes");
-    }
+    if (const char* what = latent_spec_error(layers, l)) return bad(l, what);
+    if (s.window > 0 || s.rot_pairs) return bad(l, "latent attention in parallel blocks: no window, halves rotated");
     if (s.mlp < NVLLM_MLP_NONE || s.mlp > NVLLM_MLP_MOE) return bad(l, "unknown feed-forward kind");
     if (s.mlp != NVLLM_MLP_NONE && s.ff <= 0) return bad(l, "ff must be positive");
     if (s.mlp != NVLLM_MLP_NONE && !(s.limit > 0.f)) return bad(l, "limit must be positive");
@@ -1516,7 +1733,9 @@ extern "C" int nvllm_create_layered(const nvllm_layered_config* c, const nvllm_l
   h->position_kind = c->position;
   h->norm_offset = c->norm_offset;
   h->norm_groups = c->norm_groups > 1 ? c->norm_groups : 0;
-  h->mixer_conv = c->mixer_conv > 1 ? c->mixer_conv : 0;
+  h->mixer_conv = c->mixer_conv;
+  h->ffn_conv = c->ffn_conv;
+  h->layer_norm = c->layer_norm != 0;
   h->side_dim = c->side_dim;
   h->side_p = (int)up8((size_t)c->side_dim);
   h->logit_scale = c->logit_scale;
@@ -1560,22 +1779,65 @@ extern "C" int nvllm_create_layered(const nvllm_layered_config* c, const nvllm_l
     h->lm_head_owned = true;
   }
   AL(h->lnf_w, (size_t)W * 4);
+  if (h->layer_norm) AL(h->lnf_b, (size_t)W * 4);
   if (c->embed_norm) AL(h->embed_norm_w, (size_t)W * 4);
   if (h->side_dim > 0) AL(h->side_embed, (size_t)h->V * h->L * h->side_dim * wsz);
   h->ll.resize(h->L);
   int qkv_cols = 0, q_cols = 0, win_qtile = 0;
+  // sizes and tensors of a latent-attention mixer (ov_p is set, w_o is the caller's), its rotation table, and the
+  // extents the shared workspace is sized by (forward.cu ensure_workspace)
+  auto alloc_latent = [&](ListedLayer& y, int l) -> cudaError_t {
+    const nvllm_layer_spec& s = y.s;
+    y.lat_gate = !pre_style || s.head_gate;
+    y.Dk = s.kv_rank + s.rot_dim;
+    y.n_in = s.q_rank + (s.kv_from < 0 ? y.Dk : 0) + (y.lat_gate ? s.heads : 0);
+    y.q_cols = s.heads * (s.dim + s.rot_dim);
+    y.q_rank_p = (int)up8(s.q_rank);
+    y.ovr_p = (int)up8((size_t)s.heads * s.kv_rank);
+    y.pool = s.kv_from < 0 ? l : s.kv_from;
+    for (size_t r = 0; r < h->ropes.size(); r++) {
+      const RopeTable& t = h->ropes[r];
+      if (t.base == (double)s.rot_base && t.dims == s.rot_dims && t.factor == 0) y.rope = (int)r;
+    }
+    if (y.rope < 0) {
+      RopeTable rt;
+      rt.base = s.rot_base;
+      rt.dims = s.rot_dims;
+      y.rope = (int)h->ropes.size();
+      h->ropes.push_back(rt);
+    }
+    cudaError_t ce = alloc(&y.w_in, (size_t)y.n_in * W * wsz);
+    if (ce == cudaSuccess) ce = alloc((void**)&y.dq_norm, (size_t)s.q_rank * 4);
+    if (ce == cudaSuccess && s.kv_from < 0) ce = alloc((void**)&y.dkv_norm, (size_t)s.kv_rank * 4);
+    if (ce == cudaSuccess) ce = alloc(&y.w_uq, (size_t)y.q_cols * y.q_rank_p * wsz);
+    if (ce == cudaSuccess) ce = alloc(&y.w_uk, (size_t)s.heads * s.dim * s.kv_rank * wsz);
+    if (ce == cudaSuccess) ce = alloc(&y.w_uv, (size_t)s.heads * s.vdim * s.kv_rank * wsz);
+    if (ce == cudaSuccess) ce = alloc(&y.w_q, (size_t)s.heads * y.Dk * y.q_rank_p * wsz);
+    if (ce == cudaSuccess) ce = alloc(&y.w_ov, (size_t)W * y.ovr_p * wsz);
+    qkv_cols = std::max(qkv_cols, std::max(y.n_in, s.heads * y.Dk));
+    q_cols = std::max(q_cols, s.heads * y.Dk);
+    h->nh = std::max(h->nh, s.heads);
+    h->hd = std::max(h->hd, s.kv_rank);
+    return ce;
+  };
   for (int l = 0; l < h->L; l++) {
     ListedLayer& y = h->ll[l];
     y.s = layers[l];
     const nvllm_layer_spec& s = y.s;
+    const bool has_ffn = s.mlp != NVLLM_MLP_NONE;
     if (pre_style && h->mixer_conv) AL(y.canon_w, (size_t)W * h->mixer_conv * 4);
+    if (pre_style && h->ffn_conv && has_ffn) AL(y.canon2_w, (size_t)W * h->ffn_conv * 4);
+    if (pre_style && h->layer_norm) {
+      AL(y.norm1_b, (size_t)W * 4);
+      if (has_ffn) AL(y.norm2_b, (size_t)W * 4);
+    }
     if (pre_style && h->side_dim > 0) {
       AL(y.side_gate, (size_t)h->side_p * W * wsz);
       AL(y.side_proj, (size_t)W * h->side_p * wsz);
       AL(y.side_norm, (size_t)W * 4);
       qkv_cols = std::max(qkv_cols, h->side_p);
     }
-    if (s.mixer == NVLLM_MIXER_ATTENTION || s.mixer == NVLLM_MIXER_MAMBA2) {
+    if (option_block(h, s)) {
       const int hv = s.heads * s.vdim;
       y.ov_p = (int)up8((size_t)hv);
       y.ff_p = (int)up8((size_t)std::max(s.ff, 0));
@@ -1615,6 +1877,15 @@ extern "C" int nvllm_create_layered(const nvllm_layered_config* c, const nvllm_l
         const int qt = attention_on_tc5(h, s) ? 128 : winattn_qtile(h->adt, h->kvdt, s.dim, s.vdim);
         win_qtile = win_qtile ? std::min(win_qtile, qt) : qt;
         q_cols = std::max(q_cols, std::max(y.n_q, y.ov_p));
+      } else if (s.mixer == NVLLM_MIXER_HGRN2) {
+        y.n_in = 2 * s.heads * s.dim + hv;  // q | f | v
+        AL(y.w_in, (size_t)y.n_in * W * wsz);
+        AL(y.lr_b, (size_t)s.heads * s.dim * 4);
+        AL(y.f_lower, (size_t)s.heads * s.dim * 4);
+        AL(y.onorm_w, (size_t)s.vdim * 4);
+        q_cols = std::max(q_cols, y.ov_p);
+      } else if (s.mixer == NVLLM_MIXER_LATENT_ATTENTION) {
+        if ((e = alloc_latent(y, l)) != cudaSuccess) return fail(e, "cudaMalloc(weights)");
       } else {
         const int gn = s.ssm_groups * s.state;
         y.conv_ch = hv + 2 * gn;
@@ -1629,9 +1900,25 @@ extern "C" int nvllm_create_layered(const nvllm_layered_config* c, const nvllm_l
         q_cols = std::max(q_cols, y.ov_p);
       }
       AL(y.w_o, (size_t)W * y.ov_p * wsz);
+      if (s.mlp == NVLLM_MLP_DENSE) {
+        AL(y.post2_w, (size_t)W * 4);
+        AL(y.w1, (size_t)y.ff_p * W * wsz);
+        AL(y.w2, (size_t)W * y.ff_p * wsz);
+        AL(y.poly, 4 * 4);
+        h->F = std::max(h->F, y.ff_p);
+        qkv_cols = std::max(qkv_cols, y.ff_p);
+      }
       if (s.mlp == NVLLM_MLP_MOE) {
         AL(y.post2_w, (size_t)W * 4);
         AL(y.router, (size_t)s.experts * W * 4);
+        if (s.route_bias) AL(y.route_bias, (size_t)s.experts * 4);
+        if (s.shared_ff > 0) {
+          y.sff_p = (int)up8((size_t)s.shared_ff);
+          AL(y.w1, (size_t)2 * y.sff_p * W * wsz);
+          AL(y.w2, (size_t)W * y.sff_p * wsz);
+          h->F = std::max(h->F, y.sff_p);
+          qkv_cols = std::max(qkv_cols, 2 * y.sff_p);
+        }
         if (s.route_correction) AL(y.route_corr, (size_t)s.experts * 4);
         AL(y.moe_in, (size_t)s.experts * 2 * y.ff_p * W * wsz);
         AL(y.moe_out, (size_t)s.experts * W * y.ff_p * wsz);
@@ -1770,33 +2057,11 @@ extern "C" int nvllm_create_layered(const nvllm_layered_config* c, const nvllm_l
       h->hd = std::max(h->hd, s.vdim);
       continue;
     }
-    y.Dk = s.kv_rank + s.rot_dim;
-    y.n_in = s.q_rank + (s.kv_from < 0 ? y.Dk : 0) + s.heads;
-    y.q_cols = s.heads * (s.dim + s.rot_dim);
-    y.q_rank_p = (int)up8(s.q_rank);
     y.ov_p = (int)up8((size_t)s.heads * s.vdim);
-    y.ovr_p = (int)up8((size_t)s.heads * s.kv_rank);
     y.ff_p = (int)up8((size_t)std::max(s.ff, 0));
-    y.pool = s.kv_from < 0 ? l : s.kv_from;
-    for (size_t r = 0; r < h->ropes.size(); r++)
-      if (h->ropes[r].base == (double)s.rot_base && h->ropes[r].dims == s.rot_dims) y.rope = (int)r;
-    if (y.rope < 0) {
-      RopeTable rt;
-      rt.base = s.rot_base;
-      rt.dims = s.rot_dims;
-      y.rope = (int)h->ropes.size();
-      h->ropes.push_back(rt);
-    }
+    if ((e = alloc_latent(y, l)) != cudaSuccess) return fail(e, "cudaMalloc(weights)");
     AL(y.norm_w, (size_t)W * 4);
-    AL(y.w_in, (size_t)y.n_in * W * wsz);
-    AL(y.dq_norm, (size_t)s.q_rank * 4);
-    if (s.kv_from < 0) AL(y.dkv_norm, (size_t)s.kv_rank * 4);
-    AL(y.w_uq, (size_t)y.q_cols * y.q_rank_p * wsz);
-    AL(y.w_uk, (size_t)s.heads * s.dim * s.kv_rank * wsz);
-    AL(y.w_uv, (size_t)s.heads * s.vdim * s.kv_rank * wsz);
     AL(y.w_o, (size_t)W * y.ov_p * wsz);
-    AL(y.w_q, (size_t)s.heads * y.Dk * y.q_rank_p * wsz);
-    AL(y.w_ov, (size_t)W * y.ovr_p * wsz);
     if (s.mlp == NVLLM_MLP_DENSE) {
       AL(y.w1, (size_t)2 * y.ff_p * W * wsz);
       AL(y.w2, (size_t)W * y.ff_p * wsz);
@@ -1811,11 +2076,6 @@ extern "C" int nvllm_create_layered(const nvllm_layered_config* c, const nvllm_l
       h->topk = std::max(h->topk, s.top);
       h->F = std::max(h->F, y.ff_p);
     }
-    // extents the shared workspace is sized by (forward.cu ensure_workspace)
-    qkv_cols = std::max(qkv_cols, std::max(y.n_in, s.heads * y.Dk));
-    q_cols = std::max(q_cols, s.heads * y.Dk);
-    h->nh = std::max(h->nh, s.heads);
-    h->hd = std::max(h->hd, s.kv_rank);
   }
   if (pre_style) {
     // the executions of a step in order; every one gets its own piece of a state slot
@@ -1831,12 +2091,17 @@ extern "C" int nvllm_create_layered(const nvllm_layered_config* c, const nvllm_l
         h->state_slot_floats = up4(r.canon_off + (size_t)(h->mixer_conv - 1) * W);
         r.state_off = h->state_slot_floats;
       }
-      if (s.mixer == NVLLM_MIXER_ATTENTION) {
+      if (h->ffn_conv && s.mlp != NVLLM_MLP_NONE) {  // and of the one on the feed-forward's input
+        r.canon2_off = r.state_off;
+        h->state_slot_floats = up4(r.canon2_off + (size_t)(h->ffn_conv - 1) * W);
+        r.state_off = h->state_slot_floats;
+      }
+      if (s.mixer == NVLLM_MIXER_ATTENTION || s.mixer == NVLLM_MIXER_LATENT_ATTENTION) {
         // no state of its own
       } else if (s.mixer == NVLLM_MIXER_MAMBA2) {
         r.tail_off = up4(r.state_off + (size_t)s.heads * s.state * s.vdim);
         h->state_slot_floats = up4(r.tail_off + (size_t)(s.conv - 1) * h->ll[l].conv_ch);
-      } else if (s.mixer == NVLLM_MIXER_GLA) {
+      } else if (s.mixer == NVLLM_MIXER_GLA || s.mixer == NVLLM_MIXER_HGRN2) {
         h->state_slot_floats = up4(r.state_off + (size_t)s.heads * s.dim * s.vdim);
       } else {
         r.tail_off = up4(r.state_off + (size_t)s.heads2 * s.dim2 * s.dim2);

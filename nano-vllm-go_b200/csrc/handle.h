@@ -91,7 +91,13 @@ struct ListedLayer {
   float *conv_b = nullptr, *d_skip = nullptr;
   // ---- options of the sequential pre-norm blocks
   float* route_corr = nullptr;      // [experts]: added to the scores for the choice of experts only
-  float* canon_w = nullptr;         // [W, taps]: convolution on what the mixer reads
+  float *canon_w = nullptr, *canon2_w = nullptr;  // [taps, W]: convolution on what the mixer / the feed-forward reads
+  float *norm1_b = nullptr, *norm2_b = nullptr;   // [W]: additive terms of LayerNorms
+  // HGRN2: fused projection rows [q | f | v] in w_in, the gate's additive term in lr_b, its lower bound [heads dim] here
+  float* f_lower = nullptr;
+  float* route_bias = nullptr;      // [experts]: added to the router's logits
+  float* poly = nullptr;            // [4]: coefficients of the PolyNorm activation
+  int lat_gate = 0;                 // latent attention: the fused input projection holds gate rows
   void *side_gate = nullptr, *side_proj = nullptr;  // per-layer token input: [side_p, W], [W, side_p]
   float* side_norm = nullptr;       // [W]
 };
@@ -103,7 +109,7 @@ struct LayerRun {
   size_t state_off = 0;  // recurrent state [heads][dim][vdim] (time mixing: [heads2][dim2][dim2]) inside a slot
   size_t tail_off = 0;   // attention side: convolution tail [taps - 1][n_q + n_k + n_v]
   size_t shift_off = 0;  // time mixing: the previous token's input [W]
-  size_t canon_off = 0;  // tail [taps - 1][W] of the convolution on the mixer's input
+  size_t canon_off = 0, canon2_off = 0;  // tails [taps - 1][W] of the convolutions on the mixer's / the feed-forward's input
 };
 struct RopeTable {
   double base = 0;
@@ -138,7 +144,7 @@ struct Workspace {
   int T_cap = 0, n_cap = 0;
   float* x = nullptr;        // [T, H] fp32 residual stream
   void* xn = nullptr;        // [T, H] act dtype
-  float* xn_f32 = nullptr;   // [T, H] (MoE router input)
+  float *xn_f32 = nullptr, *xn2_f32 = nullptr;  // [T, H] fp32 normed rows (MoE router input; inputs of the convolutions)
   float *ws_a = nullptr, *ws_b = nullptr, *ws_c = nullptr;
   size_t ws_a_floats = 0, ws_b_floats = 0;
   void* q = nullptr;         // [T, nh hd]
@@ -260,7 +266,8 @@ struct nvllm_handle {
   float* loop_step = nullptr;
   int loop_start = 0, loop_stop = 0, loop_times = 0;  // times >= 1 with stop > start: a repeated run exists
   // further options of the sequential pre-norm blocks (nvllm_layered_config)
-  int norm_groups = 0, mixer_conv = 0, side_dim = 0, side_p = 0;
+  int norm_groups = 0, mixer_conv = 0, ffn_conv = 0, side_dim = 0, side_p = 0;
+  bool layer_norm = false;
   float* embed_norm_w = nullptr;   // [W] or null
   void* side_embed = nullptr;      // [V, L * side_dim] weight dtype
   float logit_scale = 0.f;

@@ -51,6 +51,7 @@ struct RouteOpts {
   int sigmoid, square;
   const float* correction;
   int group_top2;
+  const float* bias;  // [E] or null: added to the router's logits (choice and weights)
 };
 struct NormArgs {
   float* x;            // [*, H] residual stream, updated in place when p1/p2 given
@@ -107,6 +108,15 @@ struct NormArgs {
   // only; y_f32 == x normalises the stream in place).
   int groups;
   int plain;
+  // conv_taps > 0 (steps with ONE row per sequence, no row_idx): the row that goes out — and is routed — is
+  // o + sum_j conv_w[j] * o_(t - taps + 1 + j), o = the normed row; conv_w [taps][H] (last tap = the row
+  // itself).  Earlier rows come from the sequence's state slot (tail [taps - 1][H], zeros before position 0),
+  // which moves on by this row in the same launch.
+  const float* conv_w;
+  int conv_taps;
+  const int *conv_pos, *conv_slots;  // [rows] position, state slot
+  float* conv_pool;
+  size_t conv_slot_floats, conv_tail_off;
 };
 cudaError_t launch_norm(cudaStream_t st, const NormArgs& a);
 
@@ -117,6 +127,10 @@ cudaError_t launch_norm(cudaStream_t st, const NormArgs& a);
 // swiglu == 2: out[t,j] = relu(h[t,j])^2
 cudaError_t launch_act(cudaStream_t st, int odt, int T, int F, const float* h, int S, size_t stride,
                        const float* bias, int swiglu, void* out, float glu_limit = 0.f);
+// out[t, j] = a N(z) + b N(z^2) + c N(z^3) + e for j < n, z = sum_s h[s][t] (rows ld apart), powers element by
+// element, N(u) = u / sqrt(mean over the row's n entries of u^2 + eps), coef = {a, b, c, e}; zero for n <= j < ld
+cudaError_t launch_poly_norm(cudaStream_t st, int odt, int T, int n, int ld, const float* h, int S, size_t stride,
+                             const float* coef, float eps, void* out);
 // Per-layer token input: out[t, j] = gelu_tanh(sum_s h[s][t][j]) * table[tokens[t]][col0 + j] for j < n,
 // zero for n <= j < ld_out (h rows ld_h apart, table rows ld_table apart in the weight dtype)
 cudaError_t launch_token_gate(cudaStream_t st, int odt, int wdt, int T, int n, const float* h, int S, size_t stride, int ld_h,
@@ -397,15 +411,17 @@ struct LatentArgs {
   int T, H, dim, rot, rot_dims, vdim, R, q_rank, q_rank_p;
   int o_ld;              // row stride of olat: heads * R rounded up to 8 (padding written as zeros)
   int own_kv;            // the layer has its own key/value down projection (writes the pool)
+  int window;            // position i sees j with 0 <= i - j < window; 0: every j <= i
+  int rot_pairs;         // entry 2i rotates with entry 2i + 1 instead of i with i + rot_dims / 2
   float eps, scale;
-  // fused input projection [dq | dkv | g]: split-K partials [S][T][in_ld]
+  // fused input projection [dq | dkv | g] (no g columns without `gate`): split-K partials [S][T][in_ld]
   const float* in_p; int in_S; size_t in_stride; int in_ld;
   const float *dq_norm, *dkv_norm;   // [q_rank], [R] fp32
   const float *cosT, *sinT;          // [T, rot_dims / 2] of the step's rows
   const int* slots;                  // [T] pool row of each new token
   void* pool;                        // [blocks * 256][R + rot] cache dtype
   void* cq;                          // [T, q_rank_p] act dtype (zero padded)
-  float* gate;                       // [T, H] sigmoid of the head gates
+  float* gate;                       // [T, H] sigmoid of the head gates; null: the heads have none
   // folded query projection partials [S][T][q_ld] -> absorbed queries [T, H, R + rot] act dtype
   const float* q_p; int q_S; size_t q_stride; int q_ld;
   void* qabs;
@@ -428,7 +444,7 @@ cudaError_t launch_latent_fold(cudaStream_t st, int wdt, const void* w_uq, const
                                const void* w_uv, void* wo, int W, int H, int dim, int rot, int vdim, int R,
                                int q_rank, int q_rank_p, int ov_p, int ovr_p);
 int latent_attn_qtile();
-int latent_attn_splits(int n_seqs, int H, int max_len, int sm_count);
+int latent_attn_splits(int n_seqs, int H, int max_len, int window, int sm_count);
 cudaError_t launch_latent_attn(cudaStream_t st, int qdt, int kvdt, const LatentArgs& a);
 // out[i] = cap * tanh(sum_s p[s * stride + i] / cap)   (cap <= 0: plain sum)
 cudaError_t launch_softcap(cudaStream_t st, const float* p, int S, size_t stride, size_t n, float cap,
@@ -537,6 +553,7 @@ cudaError_t launch_delta_out(cudaStream_t st, int odt, const DeltaArgs& a);
 // Linear recurrences with a diagonal decay, per head a dim x vdim state in fp32 kept per state slot:
 //   gated linear attention   S <- diag(a_t) S + k_t v_t^T,  o_t = S^T q_t
 //   time mixing              o_t = (S + diag(u) k_t v_t^T)^T r_t,  then S <- diag(w_t) S + k_t v_t^T
+//   HGRN2                    S <- diag(f_t) S + (1 - f_t) v_t^T,  o_t = S^T silu(q_t),  f_t = l + (1 - l) sigmoid(z_t)
 // between their projections.  A projection's result is a segment of split-K partials.
 struct LinSeg {
   const float* p;   // element (t, c) = sum_s p[s * stride + t * ld + c]
@@ -548,13 +565,15 @@ struct LinRecArgs {
   int T, n_seqs;
   int H, dim, vdim;
   int tmix;              // 0: gated linear attention, 1: time mixing (read before the update, bonus u)
+  const float* lower;    // [H dim] or null; set: HGRN2 — lr holds the gate's projection itself (z = lr + w2b, one column
+                         // per key entry, no second step), `lower` its lower bound l, k is not read
   float eps, tau, qmul;  // read-outs times qmul (= q scaled); gated linear attention: decay = sigmoid(z)^(1 / tau)
   LinSeg q, k, v, lr, gate;  // lr [T, rank]: inner result of the decay's two-step projection
   int rank;
   const float* w2;       // [H dim, rank] fp32; z = w2 f(lr) + w2b, f = tanh for time mixing
   const float* w2b;      // [H dim]
   const float* bonus;    // [H, dim] (time mixing)
-  const float* onorm_w;  // weight of the read-out's RMS norm over vdim
+  const float* onorm_w;  // weight of the read-out's RMS norm over vdim (gate.p null: norm and weight only)
   int onorm_ld;          // 0: one [vdim] weight shared by the heads; vdim: a weight per head
   const int *cu_q, *positions, *state_slots;  // [n_seqs + 1], [T], [n_seqs]
   float* state_pool; size_t slot_floats, state_off;  // this layer's [H][dim][vdim] inside a slot
@@ -569,6 +588,8 @@ struct LinRecArgs {
   void* out; int o_ld;   // [T, o_ld] act dtype: normed, gated read-outs = input of the output projection
 };
 cudaError_t launch_linrec_prep(cudaStream_t st, const LinRecArgs& a);
+// HGRN2's: qkw rows [silu(q) | 1 - f | f], vv = v's slices summed (not written when v is one slice)
+cudaError_t launch_hgrn_prep(cudaStream_t st, const LinRecArgs& a);
 cudaError_t launch_linrec_scan(cudaStream_t st, const LinRecArgs& a);
 cudaError_t launch_linrec_out(cudaStream_t st, int odt, const LinRecArgs& a);
 // One row per sequence (T == n_seqs) and vdim <= 128: prep + scan + out as one launch (a CTA per sequence and head)
@@ -580,11 +601,21 @@ constexpr int LINREC_MAX_DIM = 256;
 cudaError_t launch_token_shift(cudaStream_t st, int adt, int T, int n_seqs, int W, int n_mix, const void* h,
                                const float* mu, const int* cu_q, const int* positions, const int* state_slots,
                                const float* state_pool, size_t slot_floats, size_t tail_off, void* out);
-// What a mixer reads: out[t] = h[t] + sum_j w[:, j] h[t - taps + 1 + j] per channel (h fp32 [T, W], w [W, taps],
+// What a sublayer reads: out[t] = h[t] + sum_j w[j] h[t - taps + 1 + j] per channel (h fp32 [T, W], w [taps][W],
 // out act dtype); rows before a step's first one come from the slot's tail [taps - 1][W], zeros before position 0.
-cudaError_t launch_mixer_conv(cudaStream_t st, int adt, int T, int n_seqs, int W, int taps, const float* h, const float* w,
-                              const int* cu_q, const int* positions, const int* state_slots, const float* state_pool,
-                              size_t slot_floats, size_t tail_off, void* out);
+// router != null: the fp32 row is routed as in the norm kernel (NormArgs::router).
+struct InputConvArgs {
+  int T, n_seqs, W, taps;
+  const float *h, *w;
+  const int *cu_q, *positions, *state_slots;
+  const float* state_pool; size_t slot_floats, tail_off;
+  void* out;
+  const float* router; int E, topk;
+  int* topk_idx; float* topk_w;
+  RouteOpts route;
+};
+cudaError_t launch_input_conv(cudaStream_t st, int adt, const InputConvArgs& a);
+constexpr int INPUT_CONV_MAX_TAPS = 8;
 // After a step: the last taps - 1 inputs of every sequence become its slot's tail [taps - 1][channels].
 // Source: split-K partials (+ bias) when seg.p, else rows of `act` (act dtype, row stride channels).
 struct TailJob {
@@ -594,6 +625,7 @@ struct TailJob {
   int channels, taps;
   size_t tail_off;
 };
+constexpr int TAIL_MAX_JOBS = 3;
 cudaError_t launch_roll_tails(cudaStream_t st, int adt, int n_seqs, const TailJob* jobs, int n_jobs, const int* cu_q,
                               const int* positions, const int* state_slots, float* state_pool, size_t slot_floats);
 

@@ -4,13 +4,17 @@
 // Per head a dim x vdim state S in fp32, zero at a sequence's start, kept per state slot:
 //   gated linear attention   a_t = sigmoid(z_t)^(1 / tau),  S <- diag(a_t) S + k_t v_t^T,  o_t = S^T q_t
 //   time mixing              w_t = exp(-exp(z_t)),  o_t = (S + diag(u) k_t v_t^T)^T r_t,  S <- diag(w_t) S + k_t v_t^T
+//   HGRN2                    f_t = l + (1 - l) sigmoid(z_t),  S <- diag(f_t) S + (1 - f_t) v_t^T,  o_t = S^T silu(q_t)
 // with z_t = W_2 f(W_1 x_t) + b per (head, key entry): f = identity / tanh.  The decay rows belong to
-// key entries.  The read-out of a head is divided by its root mean square, multiplied by a weight
-// and by silu(gate) and goes to the output projection.
+// key entries.  (HGRN2: z_t = W_f x_t + b, one projection, and the
+// gate also is the key.)  The read-out of a head is divided by its root mean square, multiplied by a weight
+// and (HGRN2: not) by silu(gate) and goes to the output projection.
 //
 //   linrec_prep_kernel   per tile of tokens: split-K sums of the projections, q scaled, the second step of
 //                        the decay's projection (fp32 FMA, the inner size is small) and the decay itself —
 //                        logarithms, exponentials and sigmoids in fp32 (log-sigmoid form, no overflow).
+//   hgrn_prep_kernel     HGRN2's epilogue: silu(q), the bounded gate and its complement (neither by a
+//                        subtraction from one: both sides of the sigmoid come from one exponential).
 //   linrec_scan_kernel   CTA = (sequence, head, 32 CC value columns), NW warps.  A column of the state is
 //                        independent of the others; a warp holds a slice of the rows (RPL each, dealt in
 //                        groups of four), a lane CC columns of that slice in registers.  Per token one pass
@@ -31,6 +35,7 @@
 #include "common.cuh"
 #include "kernels.h"
 #include "mma.cuh"
+#include "moe_route.cuh"
 
 namespace nvllm {
 
@@ -65,7 +70,6 @@ __device__ __forceinline__ void lr_cp_async4(uint32_t dst, const void* src, bool
 // at a time, in registers) for all TT tokens, whose inner vectors sit in shared memory and are
 // read as broadcasts — the matrix crosses L2 once per TT tokens instead of once per token.
 constexpr int LP_RC = 16;  // inner entries per register chunk
-constexpr int TAIL_MAX_TAPS_C = 8;  // most taps of a short convolution
 
 template <int TT>
 __global__ void __launch_bounds__(256) linrec_prep_kernel(LinRecArgs a, Trace tr) {
@@ -177,6 +181,74 @@ cudaError_t launch_linrec_prep(cudaStream_t st, const LinRecArgs& a) {
     if (smem > 48 * 1024) cudaFuncSetAttribute(linrec_prep_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     (void)launch_k(linrec_prep_kernel<1>, dim3(a.T, std::min(16, ceil_div(big, 256))), dim3(256), smem, st, a, next_trace(40));
   }
+  return cudaGetLastError();
+}
+
+// f = l + (1 - l) sigmoid(z) and 1 - f = (1 - l) sigmoid(-z)
+__device__ __forceinline__ void bounded_gate(float z, float l, float* f, float* w) {
+  const float e = expf(-fabsf(z)), big = 1.0f / (1.0f + e), small = e * big;
+  *f = fmaf(1.0f - l, z >= 0.f ? big : small, l);
+  *w = (1.0f - l) * (z >= 0.f ? small : big);
+}
+
+// grid (T, Y), a thread per VEC neighbouring key entries (VEC = 4: 16-byte accesses; every row must allow them)
+template <int VEC>
+__global__ void __launch_bounds__(256) hgrn_prep_kernel(LinRecArgs a, Trace tr) {
+  TRACE_ENTRY(tr);
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x, hd = a.H * a.dim, hv = a.H * a.vdim;
+  auto take = [&](const LinSeg& g, int c, float (&v)[VEC]) {
+    const float* p = g.p + (size_t)t * g.ld + c;
+    if constexpr (VEC == 4) {
+      float4 x = *reinterpret_cast<const float4*>(p);
+      for (int s = 1; s < g.S; s++) {
+        const float4 y = *reinterpret_cast<const float4*>(p + (size_t)s * g.stride);
+        x.x += y.x; x.y += y.y; x.z += y.z; x.w += y.w;
+      }
+      v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
+    } else {
+      v[0] = seg_at(g, t, c);
+    }
+  };
+  auto put = [&](float* p, const float (&v)[VEC]) {
+    if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    else *p = v[0];
+  };
+  float* qkw = a.qkw + (size_t)t * 3 * hd;
+  for (int c = (blockIdx.y * blockDim.x + threadIdx.x) * VEC; c < hd; c += gridDim.y * blockDim.x * VEC) {
+    float q[VEC], z[VEC], k[VEC], f[VEC];
+    take(a.q, c, q);
+    take(a.lr, c, z);
+#pragma unroll
+    for (int e = 0; e < VEC; e++) {
+      bounded_gate(z[e] + a.w2b[c + e], a.lower[c + e], &f[e], &k[e]);
+      q[e] = silu(q[e]);
+    }
+    put(qkw + c, q);
+    put(qkw + hd + c, k);
+    put(qkw + 2 * hd + c, f);
+  }
+  if (a.v.S > 1)
+    for (int c = (blockIdx.y * blockDim.x + threadIdx.x) * VEC; c < hv; c += gridDim.y * blockDim.x * VEC) {
+      float v[VEC];
+      take(a.v, c, v);
+      put(a.vv + (size_t)t * hv + c, v);
+    }
+  TRACE_EXIT(tr);
+}
+
+cudaError_t launch_hgrn_prep(cudaStream_t st, const LinRecArgs& a) {
+  if (a.T <= 0) return cudaSuccess;
+  if (!a.lower) return cudaErrorInvalidValue;
+  const int hd = a.H * a.dim, hv = a.H * a.vdim;
+  auto ok = [](const LinSeg& g) { return g.ld % 4 == 0 && g.stride % 4 == 0 && reinterpret_cast<size_t>(g.p) % 16 == 0; };
+  const bool vec = hd % 4 == 0 && hv % 4 == 0 && ok(a.q) && ok(a.lr) && ok(a.v);
+  const int per = 256 * (vec ? 4 : 1);
+  const dim3 grid(a.T, a.T >= 1024 ? 1 : std::min(8, ceil_div(std::max(hd, hv), per)));
+  const int threads = std::min(256, std::max(32, ceil_div(ceil_div(std::max(hd, hv), vec ? 4 : 1), 32) * 32));
+  if (vec) (void)launch_k(hgrn_prep_kernel<4>, grid, dim3(threads), 0, st, a, next_trace(40));
+  else (void)launch_k(hgrn_prep_kernel<1>, grid, dim3(threads), 0, st, a, next_trace(40));
   return cudaGetLastError();
 }
 
@@ -350,10 +422,12 @@ cudaError_t launch_linrec_scan(cudaStream_t st, const LinRecArgs& a) {
 // decay), the state update with its read-out, the head's RMS norm, weight and gate run as ONE
 // launch per layer instead of three.  CTA = (sequence, head); the state slice of a thread is as
 // in linrec_scan_kernel and its loads are in flight while the row's inputs are prepared.
-template <int RPL, int NW, int CC, bool TMIX>
+// KIND: 0 gated linear attention, 1 time mixing, 2 HGRN2
+template <int RPL, int NW, int CC, int KIND>
 __global__ void __launch_bounds__(32 * NW) linrec_decode_kernel(LinRecArgs a, int out_bf16, Trace tr) {
   TRACE_ENTRY(tr);
   pdl_launch_dependents();
+  constexpr bool TMIX = KIND == 1;
   constexpr int NT = 32 * NW;
   constexpr int DP = RPL * NW;
   constexpr int VC = 32 * CC;
@@ -391,7 +465,13 @@ __global__ void __launch_bounds__(32 * NW) linrec_decode_kernel(LinRecArgs a, in
   const float inv_tau = 1.0f / a.tau;
   for (int i = tid; i < DP; i += NT) {
     float q = 0.f, k = 0.f, decay = 0.f;
-    if (i < dim) {
+    if (KIND == 2) {
+      if (i < dim) {
+        const int c = head * dim + i;
+        bounded_gate(seg_at(a.lr, t, c) + a.w2b[c], a.lower[c], &decay, &k);
+        q = silu(seg_at(a.q, t, c));
+      }
+    } else if (i < dim) {
       const int c = head * dim + i;
       const float* w = a.w2 + (size_t)c * a.rank;
       float z = 0.f;
@@ -472,11 +552,11 @@ __global__ void __launch_bounds__(32 * NW) linrec_decode_kernel(LinRecArgs a, in
 #pragma unroll
     for (int w = 0; w < NW; w++) o += part[w * VC + tid];
     o *= a.qmul;
-    gt = seg_at(a.gate, t, head * vdim + tid);
+    if (KIND != 2) gt = seg_at(a.gate, t, head * vdim + tid);
     wn = a.onorm_w[(size_t)head * a.onorm_ld + tid];
   }
   const float inv = 1.0f / sqrtf(block_sum(o * o, red) / (float)vdim + a.eps);
-  const float res = o * inv * wn * silu(gt);
+  const float res = KIND == 2 ? o * inv * wn : o * inv * wn * silu(gt);
   if (out_bf16) {
     bf16* out = (bf16*)a.out + (size_t)t * a.o_ld;
     if (mine) out[head * vdim + tid] = __float2bfloat16_rn(res);
@@ -495,13 +575,16 @@ template <int RPL, int NW, int CC>
 static cudaError_t linrec_decode_launch_cc(cudaStream_t st, int odt, const LinRecArgs& a) {
   const size_t smem = (size_t)(3 * RPL * NW + 32 * CC + NW * 32 * CC + a.rank) * sizeof(float);
   const int bf = odt == DT_BF16;
-  if (a.tmix) {
-    if (smem > 48 * 1024) cudaFuncSetAttribute(linrec_decode_kernel<RPL, NW, CC, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    (void)launch_k(linrec_decode_kernel<RPL, NW, CC, true>, dim3(a.T, a.H), dim3(32 * NW), smem, st, a, bf, next_trace(45));
-  } else {
-    if (smem > 48 * 1024) cudaFuncSetAttribute(linrec_decode_kernel<RPL, NW, CC, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    (void)launch_k(linrec_decode_kernel<RPL, NW, CC, false>, dim3(a.T, a.H), dim3(32 * NW), smem, st, a, bf, next_trace(45));
-  }
+#define LD(KIND_)                                                                                                        \
+  do {                                                                                                                   \
+    if (smem > 48 * 1024)                                                                                                \
+      cudaFuncSetAttribute(linrec_decode_kernel<RPL, NW, CC, KIND_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+    (void)launch_k(linrec_decode_kernel<RPL, NW, CC, KIND_>, dim3(a.T, a.H), dim3(32 * NW), smem, st, a, bf, next_trace(45)); \
+  } while (0)
+  if (a.lower) LD(2);
+  else if (a.tmix) LD(1);
+  else LD(0);
+#undef LD
   return cudaGetLastError();
 }
 template <int RPL, int NW>
@@ -538,6 +621,7 @@ __global__ void __launch_bounds__(256) linrec_out_kernel(LinRecArgs a, Trace tr)
   const int vdim = a.vdim;
   OT* out = (OT*)a.out + (size_t)t * a.o_ld;
   // 16-byte loads when every row and head starts on a 16-byte boundary
+  const bool gated = a.gate.p != nullptr;
   const bool vec = (vdim % 4) == 0 && vdim <= 512 && (a.gate.ld % 4) == 0 && (a.gate.stride % 4) == 0 &&
                    (reinterpret_cast<size_t>(a.gate.p) % 16) == 0 && (a.onorm_ld % 4) == 0;
   for (int h = blockIdx.y * nw + warp; h < a.H; h += gridDim.y * nw) {
@@ -552,13 +636,14 @@ __global__ void __launch_bounds__(256) linrec_out_kernel(LinRecArgs a, Trace tr)
         const int i = lane * 4 + 128 * j;
         if (i < vdim) {
           ov[j] = *reinterpret_cast<const float4*>(o + i);
+          ss += ov[j].x * ov[j].x + ov[j].y * ov[j].y + ov[j].z * ov[j].z + ov[j].w * ov[j].w;
+          if (!gated) continue;
           const float* gp = a.gate.p + (size_t)t * a.gate.ld + h * vdim + i;
           gv[j] = *reinterpret_cast<const float4*>(gp);
           for (int sl = 1; sl < a.gate.S; sl++) {
             const float4 x = *reinterpret_cast<const float4*>(gp + (size_t)sl * a.gate.stride);
             gv[j].x += x.x; gv[j].y += x.y; gv[j].z += x.z; gv[j].w += x.w;
           }
-          ss += ov[j].x * ov[j].x + ov[j].y * ov[j].y + ov[j].z * ov[j].z + ov[j].w * ov[j].w;
         }
       }
       const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)vdim + a.eps);
@@ -568,8 +653,10 @@ __global__ void __launch_bounds__(256) linrec_out_kernel(LinRecArgs a, Trace tr)
         const int i = lane * 4 + 128 * j;
         if (i < vdim) {
           const float4 w4 = *reinterpret_cast<const float4*>(w + i);
-          const float r[4] = {ov[j].x * inv * w4.x * silu(gv[j].x), ov[j].y * inv * w4.y * silu(gv[j].y),
-                              ov[j].z * inv * w4.z * silu(gv[j].z), ov[j].w * inv * w4.w * silu(gv[j].w)};
+          float r[4] = {ov[j].x * inv * w4.x, ov[j].y * inv * w4.y, ov[j].z * inv * w4.z, ov[j].w * inv * w4.w};
+          if (gated) {
+            r[0] *= silu(gv[j].x); r[1] *= silu(gv[j].y); r[2] *= silu(gv[j].z); r[3] *= silu(gv[j].w);
+          }
 #pragma unroll
           for (int e = 0; e < 4; e++) out[h * vdim + i + e] = from_f32<OT>(r[e]);
         }
@@ -581,8 +668,8 @@ __global__ void __launch_bounds__(256) linrec_out_kernel(LinRecArgs a, Trace tr)
     const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)vdim + a.eps);
     const float* w = a.onorm_w + (size_t)h * a.onorm_ld;
     for (int i = lane; i < vdim; i += 32) {
-      const float gt = seg_at(a.gate, t, h * vdim + i);
-      out[h * vdim + i] = from_f32<OT>(o[i] * inv * w[i] * silu(gt));
+      const float r = o[i] * inv * w[i];
+      out[h * vdim + i] = from_f32<OT>(gated ? r * silu(seg_at(a.gate, t, h * vdim + i)) : r);
     }
   }
   if (blockIdx.y == 0)
@@ -656,78 +743,99 @@ cudaError_t launch_token_shift(cudaStream_t st, int adt, int T, int n_seqs, int 
   return cudaGetLastError();
 }
 
-// ------------------------------------------------------------------ convolution on a mixer's input
-// One CTA per token; TAPS > 0: the number of taps at compile time.  Where tap j's input lives is the
-// same for every channel of the row: a row of this step, a row of the slot's tail, or nowhere
-// (before the sequence's start).
+// ------------------------------------------------------------------ convolution on a sublayer's input
+// One CTA per token, eight channels per thread; TAPS > 0: the number of taps at compile time.  Where tap
+// j's input lives is the same for every channel of the row: a row of this step, a row of the slot's
+// tail, or nowhere (before the sequence's start).  With a router the fp32 row is routed here.
 template <typename AT, int TAPS>
-__global__ void __launch_bounds__(256) mixer_conv_kernel(int T, int n_seqs, int W, int taps_rt, const float* __restrict__ h,
-                                                         const float* __restrict__ w, const int* __restrict__ cu_q,
-                                                         const int* __restrict__ positions,
-                                                         const int* __restrict__ state_slots,
-                                                         const float* __restrict__ state_pool, size_t slot_floats,
-                                                         size_t tail_off, AT* __restrict__ out, Trace tr) {
+__global__ void __launch_bounds__(512) input_conv_kernel(InputConvArgs a, Trace tr) {
   TRACE_ENTRY(tr);
   pdl_launch_dependents();
-  pdl_wait();
-  constexpr int MT = TAPS > 0 ? TAPS : TAIL_MAX_TAPS_C;
-  const int taps = TAPS > 0 ? TAPS : taps_rt;
-  const int t = blockIdx.x;
+  extern __shared__ __align__(16) float row[];  // [W] with a router
   __shared__ int s_seq;
-  if (T == n_seqs) {
+  constexpr int MT = TAPS > 0 ? TAPS : INPUT_CONV_MAX_TAPS;
+  const int taps = TAPS > 0 ? TAPS : a.taps, W = a.W;
+  const int t = blockIdx.x;
+  // (the step's integer inputs are in place before any kernel of the step starts)
+  if (a.T == a.n_seqs) {
     if (threadIdx.x == 0) s_seq = t;
   } else {
-    for (int i = threadIdx.x; i < n_seqs; i += blockDim.x)
-      if (cu_q[i] <= t && t < cu_q[i + 1]) s_seq = i;
+    for (int i = threadIdx.x; i < a.n_seqs; i += blockDim.x)
+      if (a.cu_q[i] <= t && t < a.cu_q[i + 1]) s_seq = i;
   }
   __syncthreads();
   const int s = s_seq;
-  const int li = t - cu_q[s], pos = positions[t], keep = taps - 1;
-  const float* tail = state_pool + (size_t)state_slots[s] * slot_floats + tail_off;
+  const int li = t - a.cu_q[s], pos = a.positions[t], keep = taps - 1;
+  const float* tail = taps > 1 ? a.state_pool + (size_t)a.state_slots[s] * a.slot_floats + a.tail_off : nullptr;
   const float* src[MT];
 #pragma unroll
   for (int j = 0; j < MT; j++) {
     src[j] = nullptr;
     if (j < taps) {
       const int back = keep - j;  // input `back` positions before this token
-      if (back <= li) src[j] = h + (size_t)(t - back) * W;
+      if (back <= li) src[j] = a.h + (size_t)(t - back) * W;
       else if (back <= pos) src[j] = tail + (size_t)(keep - (back - li)) * W;
     }
   }
-  for (int c = threadIdx.x; c < W; c += blockDim.x) {
-    float u[MT], wv[MT];
+  pdl_wait();
+  for (int c = threadIdx.x * 8; c < W; c += blockDim.x * 8) {
+    float y[8];
+    if constexpr (TAPS > 0) {
+      float u[MT][8], wv[MT][8];
 #pragma unroll
-    for (int j = 0; j < MT; j++) {  // all the loads first
-      u[j] = (j < taps && src[j]) ? src[j][c] : 0.f;
-      wv[j] = j < taps ? w[(size_t)c * taps + j] : 0.f;
+      for (int j = 0; j < MT; j++) {  // all the loads first
+        if (src[j]) load8(src[j] + c, u[j]);
+        else
+#pragma unroll
+          for (int e = 0; e < 8; e++) u[j][e] = 0.f;
+        load8(a.w + (size_t)j * W + c, wv[j]);
+      }
+#pragma unroll
+      for (int e = 0; e < 8; e++) y[e] = u[MT - 1][e];
+#pragma unroll
+      for (int j = 0; j < MT; j++)
+#pragma unroll
+        for (int e = 0; e < 8; e++) y[e] = fmaf(wv[j][e], u[j][e], y[e]);
+    } else {
+      load8(a.h + (size_t)t * W + c, y);
+#pragma unroll
+      for (int j = 0; j < MT; j++)
+        if (j < taps && src[j]) {
+          float u[8], wv[8];
+          load8(src[j] + c, u);
+          load8(a.w + (size_t)j * W + c, wv);
+#pragma unroll
+          for (int e = 0; e < 8; e++) y[e] = fmaf(wv[e], u[e], y[e]);
+        }
     }
-    float y = h[(size_t)t * W + c];
-#pragma unroll
-    for (int j = 0; j < MT; j++) y = fmaf(wv[j], u[j], y);
-    out[(size_t)t * W + c] = from_f32<AT>(y);
+    store8((AT*)a.out + (size_t)t * W + c, y);
+    if (a.router) store8(row + c, y);
+  }
+  if (a.router) {
+    __shared__ float probs[MOE_MAX_E];
+    __syncthreads();
+    moe_route_row(row, a.router, W, a.E, a.topk, probs, (size_t)t, a.topk_idx, a.topk_w, a.route);
   }
   TRACE_EXIT(tr);
 }
 
-cudaError_t launch_mixer_conv(cudaStream_t st, int adt, int T, int n_seqs, int W, int taps, const float* h, const float* w,
-                              const int* cu_q, const int* positions, const int* state_slots, const float* state_pool,
-                              size_t slot_floats, size_t tail_off, void* out) {
-  if (T <= 0) return cudaSuccess;
-  if (taps < 1 || taps > TAIL_MAX_TAPS_C) return cudaErrorInvalidValue;
-#define MC(AT_, TP_)                                                                                                  \
-  (void)launch_k(mixer_conv_kernel<AT_, TP_>, dim3(T), dim3(256), 0, st, T, n_seqs, W, taps, h, w, cu_q, positions,    \
-                 state_slots, state_pool, slot_floats, tail_off, (AT_*)out, next_trace(43))
+cudaError_t launch_input_conv(cudaStream_t st, int adt, const InputConvArgs& a) {
+  if (a.T <= 0) return cudaSuccess;
+  if (a.taps < 1 || a.taps > INPUT_CONV_MAX_TAPS || (a.W & 7)) return cudaErrorInvalidValue;
+  int threads = std::min(512, std::max(64, ceil_div(a.W / 8, 32) * 32));
+  if (a.router && a.T <= 1024) threads = 512;  // few rows: 16 warps share a row's experts (see launch_norm)
+  const size_t smem = a.router ? (size_t)a.W * sizeof(float) : 0;
+#define IC(AT_, TP_) (void)launch_k(input_conv_kernel<AT_, TP_>, dim3(a.T), dim3(threads), smem, st, a, next_trace(43))
   if (adt == DT_F32) {
-    if (taps == 2) MC(float, 2); else if (taps == 3) MC(float, 3); else if (taps == 4) MC(float, 4); else MC(float, 0);
+    if (a.taps == 2) IC(float, 2); else if (a.taps == 3) IC(float, 3); else if (a.taps == 4) IC(float, 4); else IC(float, 0);
   } else {
-    if (taps == 2) MC(bf16, 2); else if (taps == 3) MC(bf16, 3); else if (taps == 4) MC(bf16, 4); else MC(bf16, 0);
+    if (a.taps == 2) IC(bf16, 2); else if (a.taps == 3) IC(bf16, 3); else if (a.taps == 4) IC(bf16, 4); else IC(bf16, 0);
   }
-#undef MC
+#undef IC
   return cudaGetLastError();
 }
 
 // ------------------------------------------------------------------ tails of short convolutions
-constexpr int TAIL_MAX_JOBS = 2;
 constexpr int TAIL_MAX_TAPS = 8;
 struct TailArgs {
   TailJob j[TAIL_MAX_JOBS];

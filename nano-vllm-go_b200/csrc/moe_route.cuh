@@ -58,8 +58,8 @@ __device__ __forceinline__ void moe_route_row(const float* y, const float* __res
     acc1 = warp_sum(acc1);
     acc2 = warp_sum(acc2);
     if (lane == 0) {
-      probs[e] = acc1;
-      if (two) probs[e2] = acc2;
+      probs[e] = ro.bias ? acc1 + ro.bias[e] : acc1;
+      if (two) probs[e2] = ro.bias ? acc2 + ro.bias[e2] : acc2;
     }
   }
   __syncthreads();

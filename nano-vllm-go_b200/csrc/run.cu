@@ -105,7 +105,7 @@ static int graphed_step(nvllm_handle* h, int slot, Pre pre, bool* used) {
     // every layer picks its own key split from (batch, its heads, longest context)
     for (auto& y : h->ll)
       if (y.s.mixer == NVLLM_MIXER_LATENT_ATTENTION)
-        sig.n_splits += latent_attn_splits(L.n, y.s.heads, L.max_len, h->sm_count);
+        sig.n_splits += latent_attn_splits(L.n, y.s.heads, L.max_len, y.s.window, h->sm_count);
   } else {
     sig.n_splits = attn_decode_splits(h->adt, h->kvdt, L.n, h->nh, h->nkv, h->hd, L.max_len, h->sm_count);
   }
