@@ -153,6 +153,24 @@ __global__ void __launch_bounds__(256) latent_q_kernel(LatentArgs a, Trace tr) {
   const float* sn = a.sinT + (size_t)t * half;
   // absorbed part, 8 entries at a time when the sizes allow (sum of the slices, one rounding)
   const bool vec = (a.R & 7) == 0 && (Dk & 7) == 0 && (a.q_stride & 7) == 0 && (a.q_ld & 7) == 0;
+  if (vec && a.rot_pairs) {
+    // pairs are neighbours: a vector of the rotated part holds whole pairs, so every vector goes the same way
+    for (int i = threadIdx.x * 8; i < n; i += blockDim.x * 8) {
+      const int d = i % Dk - a.R;
+      float acc[8];
+      sum_partials8(src + i, a.q_S, a.q_stride, acc);
+#pragma unroll
+      for (int e = 0; e < 8; e += 2)
+        if (d >= 0 && d + e < a.rot_dims) {
+          const float c = cs[(d + e) >> 1], s = sn[(d + e) >> 1], u = acc[e], v = acc[e + 1];
+          acc[e] = u * c - v * s;
+          acc[e + 1] = v * c + u * s;
+        }
+      store8(out + i, acc);
+    }
+    TRACE_EXIT(tr);
+    return;
+  }
   if (vec) {
     const int vph = a.R / 8;  // vectors per head
     for (int v = threadIdx.x; v < a.H * vph; v += blockDim.x) {
@@ -637,23 +655,41 @@ __global__ void latent_combine_kernel(LatentArgs a, int n_splits, Trace tr) {
   pdl_launch_dependents();
   pdl_wait();
   const size_t item = blockIdx.x;  // row * H + head
-  const float* rec = a.split_ws + item * n_splits * (a.R + 2);
-  float m = -INFINITY;
-  for (int s = 0; s < n_splits; s++) m = fmaxf(m, rec[(size_t)s * (a.R + 2) + a.R]);
-  float l = 0.f;
-  for (int s = 0; s < n_splits; s++) {
-    const float ms = rec[(size_t)s * (a.R + 2) + a.R];
-    if (ms != -INFINITY) l += rec[(size_t)s * (a.R + 2) + a.R + 1] * expf(ms - m);
+  const int ld = a.R + 2;
+  const float* rec = a.split_ws + item * n_splits * ld;
+  // a lane per split (two when there are more than 32): one round trip for all maxima and sums
+  __shared__ float wgt[64];
+  const int lane = threadIdx.x & 31;
+  float ms[2], ls[2];
+#pragma unroll
+  for (int i = 0; i < 2; i++) {
+    const int s = lane + 32 * i;
+    ms[i] = s < n_splits ? rec[(size_t)s * ld + a.R] : -INFINITY;
+    ls[i] = s < n_splits ? rec[(size_t)s * ld + a.R + 1] : 0.f;
   }
+  const float m = warp_max(fmaxf(ms[0], ms[1]));
+  float part = 0.f;
+#pragma unroll
+  for (int i = 0; i < 2; i++) {
+    const float e = ms[i] == -INFINITY ? 0.f : expf(ms[i] - m);  // a split without visible keys has no weight
+    part += ls[i] * e;
+    if (threadIdx.x < 32) wgt[lane + 32 * i] = e;
+  }
+  const float l = warp_sum(part);
+  __syncthreads();
   const size_t row = item / a.H;
   const int head = (int)(item % a.H);
   QT* op = (QT*)a.olat + row * a.o_ld + head * a.R;
   const float inv = (a.gate ? a.gate[item] : 1.f) / l;
   for (int r = threadIdx.x; r < a.R; r += blockDim.x) {
     float o = 0.f;
-    for (int s = 0; s < n_splits; s++) {
-      const float ms = rec[(size_t)s * (a.R + 2) + a.R];
-      if (ms != -INFINITY) o += rec[(size_t)s * (a.R + 2) + r] * expf(ms - m);
+    for (int s0 = 0; s0 < n_splits; s0 += 8) {
+      float v[8];
+#pragma unroll
+      for (int q = 0; q < 8; q++) v[q] = s0 + q < n_splits ? rec[(size_t)(s0 + q) * ld + r] : 0.f;
+#pragma unroll
+      for (int q = 0; q < 8; q++)
+        if (s0 + q < n_splits) o = fmaf(v[q], wgt[s0 + q], o);
     }
     op[r] = from_f32<QT>(o * inv);
   }

@@ -460,28 +460,12 @@ __global__ void act_kernel(int T, int F, const float* __restrict__ h, int S, siz
     float g[8], o[8];
 #pragma unroll
     for (int i = 0; i < 8; i++) g[i] = 0.f;
-    if (!swiglu)
-      for (int s = 0; s < S; s++) {
-        float p[8];
-        load8(h + (size_t)s * stride + (size_t)t * ld + j, p);
-#pragma unroll
-        for (int i = 0; i < 8; i++) g[i] += p[i];
-      }
+    if (!swiglu) sum_partials8(h + (size_t)t * ld + j, S, stride, g);
     if (swiglu) {
       // W1 rows are stored interleaved (weights.cu): column 2j = gate j, 2j + 1 = up j
       float a[8], b[8];
-#pragma unroll
-      for (int i = 0; i < 8; i++) a[i] = b[i] = 0.f;
-      for (int s = 0; s < S; s++) {
-        float p[8];
-        const float* base = h + (size_t)s * stride + (size_t)t * ld + 2 * j;
-        load8(base, p);
-#pragma unroll
-        for (int i = 0; i < 8; i++) a[i] += p[i];
-        load8(base + 8, p);
-#pragma unroll
-        for (int i = 0; i < 8; i++) b[i] += p[i];
-      }
+      sum_partials8(h + (size_t)t * ld + 2 * j, S, stride, a);
+      sum_partials8(h + (size_t)t * ld + 2 * j + 8, S, stride, b);
 #pragma unroll
       for (int i = 0; i < 4; i++) {
         o[i] = glu_unit(a[2 * i], a[2 * i + 1], glu_limit);

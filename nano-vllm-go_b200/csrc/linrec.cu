@@ -15,14 +15,12 @@
 //                        logarithms, exponentials and sigmoids in fp32 (log-sigmoid form, no overflow).
 //   hgrn_prep_kernel     HGRN2's epilogue: silu(q), the bounded gate and its complement (neither by a
 //                        subtraction from one: both sides of the sigmoid come from one exponential).
-//   linrec_scan_kernel   CTA = (sequence, head, 32 CC value columns), NW warps.  A column of the state is
-//                        independent of the others; a warp holds a slice of the rows (RPL each, dealt in
-//                        groups of four), a lane CC columns of that slice in registers.  Per token one pass
-//                        over the rows; the lanes of a warp read the same q / k / decay entries (broadcast
-//                        16-byte loads).  Token inputs are staged through shared memory in chunks, the next
-//                        chunk's loads in flight (cp.async) while the current one is scanned; the warps'
-//                        partial read-outs meet in shared memory once per chunk.  State read from the slot
-//                        when the sequence has earlier tokens, written back at the end.
+//   linrec_scan_kernel   CTA = (sequence, head, range of value columns).  The state sits in registers, a tile of
+//                        8 rows by CN columns per lane, updated with packed fp32 instructions.  Token inputs are
+//                        staged through shared memory in chunks, the next chunk's loads in flight (cp.async)
+//                        while the current one is scanned; the row groups' partial read-outs meet by
+//                        shuffles, the warps' in shared memory once per chunk.  State read from the slot when the
+//                        sequence has earlier tokens, written back at the end.
 //   linrec_out_kernel    per token, a warp per head: RMS over vdim, weight, silu(gate) -> act dtype.
 //   linrec_decode_kernel steps with one row per sequence (decode): the three kernels above as one launch per layer.
 //   token_shift_kernel   the inputs of time mixing's projections: h_t + (h_{t-1} - h_t) mu_s.
@@ -253,24 +251,47 @@ cudaError_t launch_hgrn_prep(cudaStream_t st, const LinRecArgs& a) {
 }
 
 // ------------------------------------------------------------------ scan over tokens
-// A warp holds one slice of the state's rows (RPL rows, dealt in groups of four), its lanes the
-// value columns (CC each): all lanes of a warp read the SAME q / k / decay entries — one
-// broadcast per 16-byte load instead of a pass per quarter warp — and the NW warps' partial
-// read-outs of a chunk of tokens meet in shared memory once per chunk.
-template <int RPL, int NW, int CC, bool TMIX>
-__global__ void __launch_bounds__(32 * NW) linrec_scan_kernel(LinRecArgs a, Trace tr) {
+// A lane holds a tile of the state, 8 rows (four packed pairs of neighbouring rows) by CN value columns, in
+// registers; a warp covers 8 RG rows by (32 / RG) CN columns, a CTA's WR warps the rows of the head.  Per token a
+// lane reads its 8 entries of q, k and decay and its CN values (16-byte shared-memory loads, broadcast among the
+// lanes that share them) for 8 CN state entries, and updates two rows with one packed fp32 instruction
+// (f32x2: two independent IEEE fp32 operations).  The row groups' partial read-outs are summed by shuffles that
+// scatter the columns over the lanes, the warps' in shared memory once per chunk of tokens.
+__device__ __forceinline__ unsigned long long fma2(unsigned long long a, unsigned long long b, unsigned long long c) {
+  unsigned long long d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ unsigned long long mul2(unsigned long long a, unsigned long long b) {
+  unsigned long long d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+__device__ __forceinline__ unsigned long long pack2(float lo, float hi) {
+  unsigned long long d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
+  return d;
+}
+__device__ __forceinline__ void unpack2(unsigned long long v, float& lo, float& hi) {
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
+}
+
+// DP: rows of the state, padded (RG * 8 * WR); TMIX: read before the update, with a bonus; SD: one decay per
+// (token, head) instead of one per row
+template <int RG, int WR, int CN, bool TMIX, bool SD>
+__global__ void __launch_bounds__(32 * WR) linrec_scan_kernel(LinRecArgs a, int vec16, Trace tr) {
   TRACE_ENTRY(tr);
   pdl_launch_dependents();
-  constexpr int NT = 32 * NW;
-  constexpr int DP = RPL * NW;            // rows of the state, padded
-  constexpr int VC = 32 * CC;             // value columns of this CTA
-  constexpr int TC = DP >= 256 ? 4 : 8;   // tokens per staged chunk
-  constexpr int ROW = 3 * DP + VC;        // floats of one staged token: q | k | decay | v
+  constexpr int NT = 32 * WR, CG = 32 / RG, DP = 8 * RG * WR, VC = CG * CN;
+  constexpr int TC = DP >= 256 ? 4 : 8;                        // tokens per staged chunk
+  constexpr int ROW = 3 * DP + VC;                             // floats of one staged token: q | k | decay | v
+  constexpr int NO = CN >= RG ? CN / RG : 1;                   // columns a lane holds after the shuffles
   __shared__ __align__(16) float stage[2][TC][ROW];
-  __shared__ float part[NW][TC][VC];
+  __shared__ float part[WR][TC][VC];
   const int seq = blockIdx.x, head = blockIdx.y, col0 = blockIdx.z * VC;
-  const int tid = threadIdx.x;
-  const int l = tid >> 5, lane = tid & 31;  // row slice, column group
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int rg = lane / CG, cg = lane % CG;
+  const int row0 = (warp * RG + rg) * 8;                       // this lane's first row
   const int dim = a.dim, vdim = a.vdim, hd = a.H * dim, hv = a.H * vdim;
   pdl_wait();
   const int r0 = a.cu_q[seq], n_new = a.cu_q[seq + 1] - r0;
@@ -280,44 +301,67 @@ __global__ void __launch_bounds__(32 * NW) linrec_scan_kernel(LinRecArgs a, Trac
 
   // q | k | decay | v of the step's rows: the projections' own output when it needs no summing
   const bool direct = linrec_direct(a);
-  const float* part_p[3] = {direct ? a.q.p : a.qkw, direct ? a.k.p : a.qkw + hd, a.qkw + 2 * hd};
-  const size_t part_ld[3] = {direct ? (size_t)a.q.ld : (size_t)3 * hd, direct ? (size_t)a.k.ld : (size_t)3 * hd, (size_t)3 * hd};
-  const float* v_p = direct ? a.v.p : a.vv;
-  const size_t v_ld = direct ? (size_t)a.v.ld : (size_t)hv;
   const int qk_head = a.qk_div > 1 ? head / a.qk_div : head;
+  const float* part_p[3] = {(direct ? a.q.p : a.qkw) + qk_head * dim, (direct ? a.k.p : a.qkw + hd) + qk_head * dim,
+                            SD ? a.decay_p + head : a.qkw + 2 * hd + head * dim};
+  const size_t part_ld[3] = {direct ? (size_t)a.q.ld : (size_t)3 * hd, direct ? (size_t)a.k.ld : (size_t)3 * hd,
+                             SD ? (size_t)a.decay_ld : (size_t)3 * hd};
+  const float* v_p = (direct ? a.v.p : a.vv) + head * vdim + col0;
+  const size_t v_ld = direct ? (size_t)a.v.ld : (size_t)hv;
   auto load_chunk = [&](int t0, int buf) {
     const int nt = min(TC, n_new - t0);
-    for (int i = tid; i < TC * 3 * DP; i += NT) {
-      const int tt = i / (3 * DP), j = i % (3 * DP), pt = j / DP, r = j % DP;
-      const bool ok = tt < nt && r < dim;
-      const size_t trow = (size_t)(r0 + t0 + (ok ? tt : 0));
-      const float* src = (pt == 2 && a.decay_p) ? a.decay_p + trow * a.decay_ld + head
-                                                : part_p[pt] + trow * part_ld[pt] + (pt < 2 ? qk_head : head) * dim + (ok ? r : 0);
-      lr_cp_async4(smem_addr(&stage[buf][tt][j]), src, ok);
+    if (vec16) {  // every row, head and column range starts on a 16-byte boundary and is whole 16-byte pieces long
+      constexpr int NP = SD ? 2 : 3;
+#pragma unroll
+      for (int pt = 0; pt < NP; pt++)
+        for (int i = tid; i < TC * (DP / 4); i += NT) {
+          const int tt = i / (DP / 4), r = (i % (DP / 4)) * 4;
+          const bool ok = tt < nt && r < dim;
+          cp_async16(smem_addr(&stage[buf][tt][pt * DP + r]), part_p[pt] + (size_t)(r0 + t0 + (ok ? tt : 0)) * part_ld[pt] + (ok ? r : 0), ok);
+        }
+      for (int i = tid; i < TC * (VC / 4); i += NT) {
+        const int tt = i / (VC / 4), c = (i % (VC / 4)) * 4;
+        const bool ok = tt < nt && col0 + c < vdim;
+        cp_async16(smem_addr(&stage[buf][tt][3 * DP + c]), v_p + (size_t)(r0 + t0 + (ok ? tt : 0)) * v_ld + (ok ? c : 0), ok);
+      }
+    } else {
+      for (int i = tid; i < TC * 3 * DP; i += NT) {
+        const int tt = i / (3 * DP), j = i % (3 * DP), pt = j / DP, r = j % DP;
+        if (SD && pt == 2) continue;
+        const bool ok = tt < nt && r < dim;
+        lr_cp_async4(smem_addr(&stage[buf][tt][j]), part_p[pt] + (size_t)(r0 + t0 + (ok ? tt : 0)) * part_ld[pt] + (ok ? r : 0), ok);
+      }
+      for (int i = tid; i < TC * VC; i += NT) {
+        const int tt = i / VC, c = i % VC;
+        const bool ok = tt < nt && col0 + c < vdim;
+        lr_cp_async4(smem_addr(&stage[buf][tt][3 * DP + c]), v_p + (size_t)(r0 + t0 + (ok ? tt : 0)) * v_ld + (ok ? c : 0), ok);
+      }
     }
-    for (int i = tid; i < TC * VC; i += NT) {
-      const int tt = i / VC, c = i % VC;
-      const bool ok = tt < nt && col0 + c < vdim;
-      const float* src = v_p + (size_t)(r0 + t0 + (ok ? tt : 0)) * v_ld + head * vdim + (ok ? col0 + c : 0);
-      lr_cp_async4(smem_addr(&stage[buf][tt][3 * DP + c]), src, ok);
-    }
+    if (SD)
+      for (int tt = tid; tt < TC; tt += NT)
+        lr_cp_async4(smem_addr(&stage[buf][tt][2 * DP]), part_p[2] + (size_t)(r0 + t0 + (tt < nt ? tt : 0)) * part_ld[2], tt < nt);
   };
   load_chunk(0, 0);
   cp_async_commit();
 
-  float S[CC][RPL], U[TMIX ? RPL : 1];
+  unsigned long long S[4][CN], U[TMIX ? 4 : 1];
 #pragma unroll
-  for (int g = 0; g < RPL / 4; g++)
+  for (int p = 0; p < 4; p++) {
+    float s[2][CN];
 #pragma unroll
-    for (int e = 0; e < 4; e++) {
-      const int r = (g * NW + l) * 4 + e;
+    for (int e = 0; e < 2; e++)
 #pragma unroll
-      for (int cc = 0; cc < CC; cc++) {
-        const int col = col0 + cc * 32 + lane;
-        S[cc][g * 4 + e] = (r < dim && col < vdim && has_prev) ? state[(size_t)r * vdim + col] : 0.f;
+      for (int c = 0; c < CN; c++) {
+        const int r = row0 + 2 * p + e, col = col0 + cg * CN + c;
+        s[e][c] = (r < dim && col < vdim && has_prev) ? state[(size_t)r * vdim + col] : 0.f;
       }
-      if (TMIX) U[g * 4 + e] = r < dim ? a.bonus[head * dim + r] : 0.f;
+#pragma unroll
+    for (int c = 0; c < CN; c++) S[p][c] = pack2(s[0][c], s[1][c]);
+    if (TMIX) {
+      const int r = row0 + 2 * p;
+      U[p] = pack2(r < dim ? a.bonus[head * dim + r] : 0.f, r + 1 < dim ? a.bonus[head * dim + r + 1] : 0.f);
     }
+  }
 
   const int n_chunks = (n_new + TC - 1) / TC;
   for (int ch = 0; ch < n_chunks; ch++) {
@@ -327,93 +371,139 @@ __global__ void __launch_bounds__(32 * NW) linrec_scan_kernel(LinRecArgs a, Trac
     cp_async_wait<1>();
     __syncthreads();
     const int nt = min(TC, n_new - ch * TC);
-#pragma unroll
-    for (int tt = 0; tt < TC; tt++) {
-      if (tt >= nt) break;
+#pragma unroll 2
+    for (int tt = 0; tt < nt; tt++) {
       const float* row = stage[buf][tt];
-      float v[CC], acc[CC];
+      unsigned long long q[4], k[4], w[4], acc[CN];
+      float v[CN];
 #pragma unroll
-      for (int cc = 0; cc < CC; cc++) {
-        v[cc] = row[3 * DP + cc * 32 + lane];
-        acc[cc] = 0.f;
+      for (int p = 0; p < 2; p++) {
+        const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(row + row0 + 4 * p);
+        const ulonglong2 y = *reinterpret_cast<const ulonglong2*>(row + DP + row0 + 4 * p);
+        q[2 * p] = x.x; q[2 * p + 1] = x.y;
+        k[2 * p] = y.x; k[2 * p + 1] = y.y;
+        if (!SD) {
+          const ulonglong2 z = *reinterpret_cast<const ulonglong2*>(row + 2 * DP + row0 + 4 * p);
+          w[2 * p] = z.x; w[2 * p + 1] = z.y;
+        }
+      }
+      if (SD) {
+        const float d = row[2 * DP];
+        w[0] = w[1] = w[2] = w[3] = pack2(d, d);
+      }
+      const float* vr = row + 3 * DP + cg * CN;
+      if constexpr (CN >= 4) {
+#pragma unroll
+        for (int c = 0; c < CN; c += 4) {
+          const float4 x = *reinterpret_cast<const float4*>(vr + c);
+          v[c] = x.x; v[c + 1] = x.y; v[c + 2] = x.z; v[c + 3] = x.w;
+        }
+      } else {
+#pragma unroll
+        for (int c = 0; c < CN; c++) v[c] = vr[c];
       }
 #pragma unroll
-      for (int g = 0; g < RPL / 4; g++) {
-        const int rb = (g * NW + l) * 4;
-        const float4 q4 = *reinterpret_cast<const float4*>(row + rb);
-        const float4 k4 = *reinterpret_cast<const float4*>(row + DP + rb);
-        const float4 w4 = *reinterpret_cast<const float4*>(row + 2 * DP + rb);
-        const float qq[4] = {q4.x, q4.y, q4.z, q4.w}, kk[4] = {k4.x, k4.y, k4.z, k4.w}, ww[4] = {w4.x, w4.y, w4.z, w4.w};
+      for (int c = 0; c < CN; c++) {
+        const unsigned long long vd = pack2(v[c], v[c]);
+        unsigned long long ac = 0ull;  // (+0, +0)
 #pragma unroll
-        for (int e = 0; e < 4; e++) {
-#pragma unroll
-          for (int cc = 0; cc < CC; cc++) {
-            float& s = S[cc][g * 4 + e];
-            if (TMIX) {
-              const float kv = kk[e] * v[cc];
-              acc[cc] = fmaf(qq[e], fmaf(U[g * 4 + e], kv, s), acc[cc]);
-              s = fmaf(ww[e], s, kv);
-            } else {
-              s = fmaf(ww[e], s, kk[e] * v[cc]);
-              acc[cc] = fmaf(qq[e], s, acc[cc]);
-            }
+        for (int p = 0; p < 4; p++) {
+          const unsigned long long kv = mul2(k[p], vd);
+          if (TMIX) {
+            ac = fma2(q[p], fma2(U[p], kv, S[p][c]), ac);
+            S[p][c] = fma2(w[p], S[p][c], kv);
+          } else {
+            S[p][c] = fma2(w[p], S[p][c], kv);
+            ac = fma2(q[p], S[p][c], ac);
           }
+        }
+        acc[c] = ac;
+      }
+      float o[CN];
+#pragma unroll
+      for (int c = 0; c < CN; c++) {
+        float lo, hi;
+        unpack2(acc[c], lo, hi);
+        o[c] = lo + hi;
+      }
+      // sum over the row groups: every exchange halves the columns a lane is responsible for
+      int n = CN, cofs = 0;
+#pragma unroll
+      for (int off = 16; off >= CG; off >>= 1) {
+        if (n > 1) {
+          n >>= 1;
+          const bool up = lane & off;
+#pragma unroll
+          for (int i = 0; i < CN / 2; i++)
+            if (i < n) {
+              const float send = up ? o[i] : o[i + n], mine = up ? o[i + n] : o[i];
+              o[i] = mine + __shfl_xor_sync(0xffffffffu, send, off);
+            }
+          cofs += up ? n : 0;
+        } else {
+          o[0] += __shfl_xor_sync(0xffffffffu, o[0], off);
         }
       }
 #pragma unroll
-      for (int cc = 0; cc < CC; cc++) part[l][tt][cc * 32 + lane] = acc[cc];
+      for (int i = 0; i < NO; i++) part[warp][tt][cg * CN + cofs + i] = o[i];
     }
-    __syncthreads();  // the slices' partial read-outs are in; the staged chunk has been consumed
+    __syncthreads();  // the warps' partial read-outs are in; the staged chunk has been consumed
     for (int i = tid; i < nt * VC; i += NT) {
       const int tt = i / VC, c = i % VC;
       float t = 0.f;
 #pragma unroll
-      for (int w = 0; w < NW; w++) t += part[w][tt][c];
+      for (int w = 0; w < WR; w++) t += part[w][tt][c];
       if (col0 + c < vdim) a.o[(size_t)(r0 + ch * TC + tt) * hv + head * vdim + col0 + c] = t * a.qmul;
     }
   }
   cp_async_wait<0>();
 #pragma unroll
-  for (int g = 0; g < RPL / 4; g++)
+  for (int p = 0; p < 4; p++)
 #pragma unroll
-    for (int e = 0; e < 4; e++) {
-      const int r = (g * NW + l) * 4 + e;
-#pragma unroll
-      for (int cc = 0; cc < CC; cc++) {
-        const int col = col0 + cc * 32 + lane;
-        if (r < dim && col < vdim) state[(size_t)r * vdim + col] = S[cc][g * 4 + e];
-      }
+    for (int c = 0; c < CN; c++) {
+      float lo, hi;
+      unpack2(S[p][c], lo, hi);
+      const int r = row0 + 2 * p, col = col0 + cg * CN + c;
+      if (r < dim && col < vdim) state[(size_t)r * vdim + col] = lo;
+      if (r + 1 < dim && col < vdim) state[(size_t)(r + 1) * vdim + col] = hi;
     }
   TRACE_EXIT(tr);
 }
 
-template <int RPL, int NW, int CC>
-static cudaError_t linrec_scan_launch_cc(cudaStream_t st, const LinRecArgs& a) {
-  const dim3 grid(a.n_seqs, a.H, ceil_div(a.vdim, 32 * CC));
-  if (a.tmix) (void)launch_k(linrec_scan_kernel<RPL, NW, CC, true>, grid, dim3(32 * NW), 0, st, a, next_trace(41));
-  else (void)launch_k(linrec_scan_kernel<RPL, NW, CC, false>, grid, dim3(32 * NW), 0, st, a, next_trace(41));
+template <int RG, int WR, int CN>
+static cudaError_t linrec_scan_launch_cn(cudaStream_t st, const LinRecArgs& a) {
+  const dim3 grid(a.n_seqs, a.H, ceil_div(a.vdim, 32 / RG * CN));
+  auto ok = [](const void* p, size_t ld) { return reinterpret_cast<size_t>(p) % 16 == 0 && ld % 4 == 0; };
+  const int hd = a.H * a.dim;
+  bool vec = a.dim % 4 == 0 && a.vdim % 4 == 0;
+  if (linrec_direct(a)) vec = vec && ok(a.q.p, a.q.ld) && ok(a.k.p, a.k.ld) && ok(a.v.p, a.v.ld);
+  else vec = vec && ok(a.qkw, 3 * (size_t)hd) && ok(a.vv, (size_t)a.H * a.vdim);
+  if (!a.decay_p) vec = vec && ok(a.qkw, 3 * (size_t)hd);
+  const int v16 = vec ? 1 : 0;
+  if (a.tmix) (void)launch_k(linrec_scan_kernel<RG, WR, CN, true, false>, grid, dim3(32 * WR), 0, st, a, v16, next_trace(41));
+  else if (a.decay_p) (void)launch_k(linrec_scan_kernel<RG, WR, CN, false, true>, grid, dim3(32 * WR), 0, st, a, v16, next_trace(41));
+  else (void)launch_k(linrec_scan_kernel<RG, WR, CN, false, false>, grid, dim3(32 * WR), 0, st, a, v16, next_trace(41));
   return cudaGetLastError();
 }
-template <int RPL, int NW>
+template <int RG, int WR>
 static cudaError_t linrec_scan_launch(cudaStream_t st, const LinRecArgs& a) {
-  // more columns per lane where a head has that many (a row's q / k / decay is read once for all of
-  // them) — as long as the grid still fills the GPU twice over: a sequence's tokens are scanned in
-  // order, so few long sequences want many narrow CTAs
+  // more columns per lane: fewer shared-memory reads per state entry.  A sequence's tokens are scanned in order,
+  // so few long sequences want many narrow CTAs instead
+  constexpr int CG = 32 / RG;
   const long units = (long)a.n_seqs * a.H;
-  const long want = 2 * 148;
-  if (RPL <= 16 && a.vdim >= 128 && units * ceil_div(a.vdim, 128) >= want) return linrec_scan_launch_cc<RPL, NW, 4>(st, a);
-  if (a.vdim >= 64 && units * ceil_div(a.vdim, 64) >= want) return linrec_scan_launch_cc<RPL, NW, 2>(st, a);
-  return linrec_scan_launch_cc<RPL, NW, 1>(st, a);
+  if (a.vdim > CG * 4 && units * ceil_div(a.vdim, CG * 8) >= 148) return linrec_scan_launch_cn<RG, WR, 8>(st, a);
+  if (a.vdim > CG * 2 && units * ceil_div(a.vdim, CG * 4) >= 148) return linrec_scan_launch_cn<RG, WR, 4>(st, a);
+  return linrec_scan_launch_cn<RG, WR, 2>(st, a);
 }
 
 cudaError_t launch_linrec_scan(cudaStream_t st, const LinRecArgs& a) {
   if (a.T <= 0 || a.n_seqs <= 0) return cudaSuccess;
   if (a.dim > LINREC_MAX_DIM || (a.tmix && !a.bonus)) return cudaErrorInvalidValue;
-  if (a.dim <= 16) return linrec_scan_launch<4, 4>(st, a);
-  if (a.dim <= 32) return linrec_scan_launch<8, 4>(st, a);
-  if (a.dim <= 64) return linrec_scan_launch<16, 4>(st, a);
-  if (a.dim <= 128) return linrec_scan_launch<32, 4>(st, a);
-  return linrec_scan_launch<32, 8>(st, a);
+  if (a.dim <= 16) return linrec_scan_launch<2, 1>(st, a);
+  if (a.dim <= 32) return linrec_scan_launch<4, 1>(st, a);
+  if (a.dim <= 64) return linrec_scan_launch<4, 2>(st, a);
+  if (a.dim <= 128) return linrec_scan_launch<4, 4>(st, a);
+  return linrec_scan_launch<4, 8>(st, a);
 }
 
 // ------------------------------------------------------------------ one token per sequence: everything in one kernel
@@ -611,6 +701,13 @@ cudaError_t launch_linrec_decode(cudaStream_t st, int odt, const LinRecArgs& a) 
 }
 
 // ------------------------------------------------------------------ gated norm of the read-out
+__device__ __forceinline__ void store4(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void store4(bf16* p, const float (&v)[4]) {
+  uint2 u;
+  reinterpret_cast<__nv_bfloat162*>(&u)[0] = __floats2bfloat162_rn(v[0], v[1]);
+  reinterpret_cast<__nv_bfloat162*>(&u)[1] = __floats2bfloat162_rn(v[2], v[3]);
+  *reinterpret_cast<uint2*>(p) = u;
+}
 template <typename OT>
 __global__ void __launch_bounds__(256) linrec_out_kernel(LinRecArgs a, Trace tr) {
   TRACE_ENTRY(tr);
@@ -657,8 +754,7 @@ __global__ void __launch_bounds__(256) linrec_out_kernel(LinRecArgs a, Trace tr)
           if (gated) {
             r[0] *= silu(gv[j].x); r[1] *= silu(gv[j].y); r[2] *= silu(gv[j].z); r[3] *= silu(gv[j].w);
           }
-#pragma unroll
-          for (int e = 0; e < 4; e++) out[h * vdim + i + e] = from_f32<OT>(r[e]);
+          store4(out + h * vdim + i, r);
         }
       }
       continue;
@@ -819,11 +915,112 @@ __global__ void __launch_bounds__(512) input_conv_kernel(InputConvArgs a, Trace 
   TRACE_EXIT(tr);
 }
 
+// The same for steps of many rows with a router: a CTA takes TT tokens, their convolved rows stay in
+// shared memory, and a warp accumulates four experts against all of them — a router row crosses L2 once per TT tokens
+// instead of once per token.  Every dot product is summed in moe_route_row's order.
+template <typename AT, int TAPS, int TT>
+__global__ void __launch_bounds__(256) input_conv_route_kernel(InputConvArgs a, Trace tr) {
+  TRACE_ENTRY(tr);
+  pdl_launch_dependents();
+  extern __shared__ __align__(16) float rows[];  // [TT][W], then probs | chs | gsc [TT][E] each
+  __shared__ int s_seq[TT];
+  constexpr int EB = 4;
+  const int W = a.W, E = a.E, t0 = blockIdx.x * TT, nt = min(TT, a.T - t0), keep = a.taps - 1;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  for (int i = threadIdx.x; i < a.n_seqs; i += blockDim.x) {
+    const int lo = max(a.cu_q[i], t0), hi = min(a.cu_q[i + 1], t0 + nt);
+    for (int t = lo; t < hi; t++) s_seq[t - t0] = i;
+  }
+  __syncthreads();
+  pdl_wait();
+  const int vpr = W / 8;
+  for (int it = threadIdx.x; it < TT * vpr; it += blockDim.x) {
+    const int tt = it / vpr, c = (it % vpr) * 8;
+    float y[8];
+    if (tt < nt) {
+      const int t = t0 + tt, s = s_seq[tt], li = t - a.cu_q[s], pos = a.positions[t];
+      load8(a.h + (size_t)t * W + c, y);
+#pragma unroll
+      for (int j = 0; j < (TAPS > 0 ? TAPS : INPUT_CONV_MAX_TAPS); j++) {
+        if (TAPS == 0 && j >= a.taps) break;
+        const int back = keep - j;
+        float u[8], wv[8];
+        if (back <= li) load8(a.h + (size_t)(t - back) * W + c, u);
+        else if (back <= pos)
+          load8(a.state_pool + (size_t)a.state_slots[s] * a.slot_floats + a.tail_off + (size_t)(keep - (back - li)) * W + c, u);
+        else continue;
+        load8(a.w + (size_t)j * W + c, wv);
+#pragma unroll
+        for (int e = 0; e < 8; e++) y[e] = fmaf(wv[e], u[e], y[e]);
+      }
+      store8((AT*)a.out + (size_t)t * W + c, y);
+    } else {
+#pragma unroll
+      for (int e = 0; e < 8; e++) y[e] = 0.f;
+    }
+    store8(rows + (size_t)tt * W + c, y);
+  }
+  __syncthreads();
+  float* probs = rows + (size_t)TT * W;
+  for (int e0 = warp * EB; e0 < E; e0 += nw * EB) {
+    float acc[EB][TT];
+#pragma unroll
+    for (int q = 0; q < EB; q++)
+#pragma unroll
+      for (int tt = 0; tt < TT; tt++) acc[q][tt] = 0.f;
+    for (int i = lane * 8; i < W; i += 256) {
+      float r[EB][8];
+#pragma unroll
+      for (int q = 0; q < EB; q++) load8(a.router + (size_t)min(e0 + q, E - 1) * W + i, r[q]);
+#pragma unroll
+      for (int tt = 0; tt < TT; tt++) {
+        float y[8];
+        load8(rows + (size_t)tt * W + i, y);
+#pragma unroll
+        for (int q = 0; q < EB; q++)
+#pragma unroll
+          for (int e = 0; e < 8; e++) acc[q][tt] = fmaf(y[e], r[q][e], acc[q][tt]);
+      }
+    }
+#pragma unroll
+    for (int q = 0; q < EB; q++)
+#pragma unroll
+      for (int tt = 0; tt < TT; tt++) {
+        const float z = warp_sum(acc[q][tt]);
+        if (lane == 0 && e0 + q < E) probs[tt * E + e0 + q] = a.route.bias ? z + a.route.bias[e0 + q] : z;
+      }
+  }
+  __syncthreads();
+  for (int tt = warp; tt < nt; tt += nw)
+    moe_select_row(probs + tt * E, probs + (size_t)(TT + tt) * E, probs + (size_t)(2 * TT + tt) * E, E, a.topk, (size_t)(t0 + tt),
+                   a.topk_idx, a.topk_w, a.route);
+  TRACE_EXIT(tr);
+}
+
+constexpr int IC_TT = 8;             // tokens per CTA of input_conv_route_kernel
+constexpr size_t IC_SMEM = 96 * 1024;  // ... as long as their rows fit (two CTAs per SM)
+
+template <typename AT, int TAPS>
+static void input_conv_route(cudaStream_t st, const InputConvArgs& a, size_t smem) {
+  if (smem > 48 * 1024)
+    cudaFuncSetAttribute(input_conv_route_kernel<AT, TAPS, IC_TT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  (void)launch_k(input_conv_route_kernel<AT, TAPS, IC_TT>, dim3(ceil_div(a.T, IC_TT)), dim3(256), smem, st, a, next_trace(43));
+}
+
 cudaError_t launch_input_conv(cudaStream_t st, int adt, const InputConvArgs& a) {
   if (a.T <= 0) return cudaSuccess;
   if (a.taps < 1 || a.taps > INPUT_CONV_MAX_TAPS || (a.W & 7)) return cudaErrorInvalidValue;
   int threads = std::min(512, std::max(64, ceil_div(a.W / 8, 32) * 32));
   if (a.router && a.T <= 1024) threads = 512;  // few rows: 16 warps share a row's experts (see launch_norm)
+  const size_t tile_smem = ((size_t)IC_TT * a.W + 3 * (size_t)IC_TT * a.E) * sizeof(float);
+  if (a.router && a.T >= 1024 && tile_smem <= IC_SMEM) {
+    if (adt == DT_F32) {
+      if (a.taps == 4) input_conv_route<float, 4>(st, a, tile_smem); else input_conv_route<float, 0>(st, a, tile_smem);
+    } else {
+      if (a.taps == 4) input_conv_route<bf16, 4>(st, a, tile_smem); else input_conv_route<bf16, 0>(st, a, tile_smem);
+    }
+    return cudaGetLastError();
+  }
   const size_t smem = a.router ? (size_t)a.W * sizeof(float) : 0;
 #define IC(AT_, TP_) (void)launch_k(input_conv_kernel<AT_, TP_>, dim3(a.T), dim3(threads), smem, st, a, next_trace(43))
   if (adt == DT_F32) {

@@ -8,62 +8,15 @@ namespace nvllm {
 
 constexpr int MOE_MAX_E = 256;
 
-// All warps of the CTA: warp w computes the logits of experts w, w + nw, ... from the
-// normed row y (shared or global memory, fp32) and R [E, H]; warp 0 then does the softmax
-// over ALL E experts (tensor.go:128-155), k rounds of first-max selection (ties -> lower
-// index, which is what a stable descending sort gives; the reference's sort.Slice is unstable,
-// ties have measure zero with random-init weights) and the renormalisation over the chosen k
-// (moe.go:88-103).  probs: shared scratch of >= E floats.  Contains __syncthreads.
-__device__ __forceinline__ void moe_route_row(const float* y, const float* __restrict__ R, int H,
-                                              int E, int k, float* probs, size_t t,
-                                              int* __restrict__ topk_idx,
-                                              float* __restrict__ topk_w,
-                                              RouteOpts ro = RouteOpts{}) {
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
-  // Two experts per pass with the k loop unrolled four deep: up to 8 independent 32-byte loads
-  // of R per lane in flight, so the E / nw passes cost one L2 round trip each instead of one
-  // per 256 columns per expert (measured 10 us per row CTA with the rolled loop at E = 32).
-  // The per-expert accumulation order (ascending i, then the warp tree) is unchanged.
-  for (int e = warp; e < E; e += 2 * nw) {
-    const int e2 = e + nw;
-    const bool two = e2 < E;
-    const float* r1 = R + (size_t)e * H;
-    const float* r2 = R + (size_t)(two ? e2 : e) * H;
-    float acc1 = 0.f, acc2 = 0.f;
-    for (int i0 = lane * 8; i0 < H; i0 += 1024) {
-      float b1[4][8], b2[4][8];
-#pragma unroll
-      for (int u = 0; u < 4; u++) {
-        const int i = i0 + u * 256;
-        if (i < H) {
-          load8(r1 + i, b1[u]);
-          if (two) load8(r2 + i, b2[u]);
-        }
-      }
-#pragma unroll
-      for (int u = 0; u < 4; u++) {
-        const int i = i0 + u * 256;
-        if (i < H) {
-          float a[8];
-          load8(y + i, a);
-#pragma unroll
-          for (int j = 0; j < 8; j++) acc1 = fmaf(a[j], b1[u][j], acc1);
-          if (two) {
-#pragma unroll
-            for (int j = 0; j < 8; j++) acc2 = fmaf(a[j], b2[u][j], acc2);
-          }
-        }
-      }
-    }
-    acc1 = warp_sum(acc1);
-    acc2 = warp_sum(acc2);
-    if (lane == 0) {
-      probs[e] = ro.bias ? acc1 + ro.bias[e] : acc1;
-      if (two) probs[e2] = ro.bias ? acc2 + ro.bias[e2] : acc2;
-    }
-  }
-  __syncthreads();
-  if (warp != 0) return;
+// ONE warp: from the logits in probs (overwritten) the softmax over ALL E experts
+// (tensor.go:128-155), k rounds of first-max selection (ties -> lower index, which is what a
+// stable descending sort gives; the reference's sort.Slice is unstable, ties have measure zero
+// with random-init weights) and the renormalisation over the chosen k (moe.go:88-103).
+// probs, chs, gsc: shared scratch of E floats each, this warp's own.
+__device__ __forceinline__ void moe_select_row(float* probs, float* chs, float* gsc, int E, int k, size_t t,
+                                               int* __restrict__ topk_idx, float* __restrict__ topk_w,
+                                               RouteOpts ro) {
+  const int lane = threadIdx.x & 31;
   if (ro.sigmoid) {
     // every expert scores on its own
     for (int e = lane; e < E; e += 32) probs[e] = 1.0f / (1.0f + expf(-probs[e]));
@@ -85,7 +38,6 @@ __device__ __forceinline__ void moe_route_row(const float* y, const float* __res
   }
   // The choice may go by other numbers than the weights: ch[e] = probs[e] + correction[e] (any sign;
   // an expert taken out of the choice is -inf), while the weights stay probs[e].
-  __shared__ float chs[MOE_MAX_E];
   const bool corr = ro.correction != nullptr;
   float* ch = corr ? chs : probs;
   const float OUT = corr ? -INFINITY : -2.f;   // marks an expert that cannot be chosen (plain scores are >= 0)
@@ -97,7 +49,6 @@ __device__ __forceinline__ void moe_route_row(const float* y, const float* __res
   // stays iff fewer than `keep` groups beat it (higher score, or equal score and lower index).
   // Experts of the other groups are taken out of the selection below.
   if (ro.groups > 1 && ro.keep < ro.groups) {
-    __shared__ float gsc[MOE_MAX_E];
     const int per = E / ro.groups;
     for (int g = lane; g < ro.groups; g += 32) {
       float b1 = -INFINITY, b2 = -INFINITY;
@@ -160,6 +111,63 @@ __device__ __forceinline__ void moe_route_row(const float* y, const float* __res
     const float wgt = ro.raw ? sel_p * ro.scale : sel_p / ksum;
     topk_w[t * k + lane] = ro.square ? wgt * wgt : wgt;
   }
+}
+
+// All warps of the CTA: warp w computes the logits of experts w, w + nw, ... from the
+// normed row y (shared or global memory, fp32) and R [E, H]; warp 0 then selects.
+// probs: shared scratch of >= E floats.  Contains __syncthreads.
+__device__ __forceinline__ void moe_route_row(const float* y, const float* __restrict__ R, int H,
+                                              int E, int k, float* probs, size_t t,
+                                              int* __restrict__ topk_idx,
+                                              float* __restrict__ topk_w,
+                                              RouteOpts ro = RouteOpts{}) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  // Two experts per pass with the k loop unrolled four deep: up to 8 independent 32-byte loads
+  // of R per lane in flight, so the E / nw passes cost one L2 round trip each instead of one
+  // per 256 columns per expert (measured 10 us per row CTA with the rolled loop at E = 32).
+  // The per-expert accumulation order (ascending i, then the warp tree) is unchanged.
+  for (int e = warp; e < E; e += 2 * nw) {
+    const int e2 = e + nw;
+    const bool two = e2 < E;
+    const float* r1 = R + (size_t)e * H;
+    const float* r2 = R + (size_t)(two ? e2 : e) * H;
+    float acc1 = 0.f, acc2 = 0.f;
+    for (int i0 = lane * 8; i0 < H; i0 += 1024) {
+      float b1[4][8], b2[4][8];
+#pragma unroll
+      for (int u = 0; u < 4; u++) {
+        const int i = i0 + u * 256;
+        if (i < H) {
+          load8(r1 + i, b1[u]);
+          if (two) load8(r2 + i, b2[u]);
+        }
+      }
+#pragma unroll
+      for (int u = 0; u < 4; u++) {
+        const int i = i0 + u * 256;
+        if (i < H) {
+          float a[8];
+          load8(y + i, a);
+#pragma unroll
+          for (int j = 0; j < 8; j++) acc1 = fmaf(a[j], b1[u][j], acc1);
+          if (two) {
+#pragma unroll
+            for (int j = 0; j < 8; j++) acc2 = fmaf(a[j], b2[u][j], acc2);
+          }
+        }
+      }
+    }
+    acc1 = warp_sum(acc1);
+    acc2 = warp_sum(acc2);
+    if (lane == 0) {
+      probs[e] = ro.bias ? acc1 + ro.bias[e] : acc1;
+      if (two) probs[e2] = ro.bias ? acc2 + ro.bias[e2] : acc2;
+    }
+  }
+  __syncthreads();
+  if (warp != 0) return;
+  __shared__ float chs[MOE_MAX_E], gsc[MOE_MAX_E];
+  moe_select_row(probs, chs, gsc, E, k, t, topk_idx, topk_w, ro);
 }
 
 }  // namespace nvllm
