@@ -490,7 +490,8 @@ cudaError_t launch_act(cudaStream_t st, int odt, int T, int F, const float* h, i
                        const float* bias, int swiglu, void* out, float glu_limit) {
   if (T <= 0) return cudaSuccess;
   size_t nvec = (size_t)T * (F / 8);
-  int threads = 256;
+  // few rows: small CTAs, so that the slices come in through many SMs
+  int threads = nvec < (size_t)148 * 512 ? 64 : 256;
   int blocks = (int)min((size_t)148 * 16, (nvec + threads - 1) / threads);
   if (odt == DT_F32)
     (void)launch_k(act_kernel<float>, dim3(blocks), dim3(threads), 0, st, T, F, h, S, stride, bias, swiglu, (float*)out, glu_limit, next_trace(6));

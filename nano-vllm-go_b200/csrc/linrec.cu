@@ -487,11 +487,10 @@ static cudaError_t linrec_scan_launch_cn(cudaStream_t st, const LinRecArgs& a) {
 }
 template <int RG, int WR>
 static cudaError_t linrec_scan_launch(cudaStream_t st, const LinRecArgs& a) {
-  // more columns per lane: fewer shared-memory reads per state entry.  A sequence's tokens are scanned in order,
-  // so few long sequences want many narrow CTAs instead
+  // four columns per lane (eight were slower: too few warps to cover the latency of a token); a sequence's tokens
+  // are scanned in order, so few long sequences want narrower, more CTAs
   constexpr int CG = 32 / RG;
   const long units = (long)a.n_seqs * a.H;
-  if (a.vdim > CG * 4 && units * ceil_div(a.vdim, CG * 8) >= 148) return linrec_scan_launch_cn<RG, WR, 8>(st, a);
   if (a.vdim > CG * 2 && units * ceil_div(a.vdim, CG * 4) >= 148) return linrec_scan_launch_cn<RG, WR, 4>(st, a);
   return linrec_scan_launch_cn<RG, WR, 2>(st, a);
 }
@@ -708,7 +707,8 @@ __device__ __forceinline__ void store4(bf16* p, const float (&v)[4]) {
   reinterpret_cast<__nv_bfloat162*>(&u)[1] = __floats2bfloat162_rn(v[2], v[3]);
   *reinterpret_cast<uint2*>(p) = u;
 }
-template <typename OT>
+// MJ: 16-byte pieces per lane (vdim <= 128 MJ)
+template <typename OT, int MJ, bool GATED>
 __global__ void __launch_bounds__(256) linrec_out_kernel(LinRecArgs a, Trace tr) {
   TRACE_ENTRY(tr);
   pdl_launch_dependents();
@@ -718,15 +718,13 @@ __global__ void __launch_bounds__(256) linrec_out_kernel(LinRecArgs a, Trace tr)
   const int vdim = a.vdim;
   OT* out = (OT*)a.out + (size_t)t * a.o_ld;
   // 16-byte loads when every row and head starts on a 16-byte boundary
-  const bool gated = a.gate.p != nullptr;
-  const bool vec = (vdim % 4) == 0 && vdim <= 512 && (a.gate.ld % 4) == 0 && (a.gate.stride % 4) == 0 &&
+  const bool vec = (vdim % 4) == 0 && vdim <= 128 * MJ && (a.gate.ld % 4) == 0 && (a.gate.stride % 4) == 0 &&
                    (reinterpret_cast<size_t>(a.gate.p) % 16) == 0 && (a.onorm_ld % 4) == 0;
   for (int h = blockIdx.y * nw + warp; h < a.H; h += gridDim.y * nw) {
     const float* o = a.o + (size_t)t * a.H * vdim + (size_t)h * vdim;
     if (vec) {
       // four neighbouring columns per lane, all loads (read-outs, gate slices, weights) before the arithmetic
-      constexpr int MJ = 4;  // vdim <= 512
-      float4 ov[MJ], gv[MJ];
+      float4 ov[MJ], gv[GATED ? MJ : 1];
       float ss = 0.f;
 #pragma unroll
       for (int j = 0; j < MJ; j++) {
@@ -734,12 +732,13 @@ __global__ void __launch_bounds__(256) linrec_out_kernel(LinRecArgs a, Trace tr)
         if (i < vdim) {
           ov[j] = *reinterpret_cast<const float4*>(o + i);
           ss += ov[j].x * ov[j].x + ov[j].y * ov[j].y + ov[j].z * ov[j].z + ov[j].w * ov[j].w;
-          if (!gated) continue;
-          const float* gp = a.gate.p + (size_t)t * a.gate.ld + h * vdim + i;
-          gv[j] = *reinterpret_cast<const float4*>(gp);
-          for (int sl = 1; sl < a.gate.S; sl++) {
-            const float4 x = *reinterpret_cast<const float4*>(gp + (size_t)sl * a.gate.stride);
-            gv[j].x += x.x; gv[j].y += x.y; gv[j].z += x.z; gv[j].w += x.w;
+          if constexpr (GATED) {
+            const float* gp = a.gate.p + (size_t)t * a.gate.ld + h * vdim + i;
+            gv[j] = *reinterpret_cast<const float4*>(gp);
+            for (int sl = 1; sl < a.gate.S; sl++) {
+              const float4 x = *reinterpret_cast<const float4*>(gp + (size_t)sl * a.gate.stride);
+              gv[j].x += x.x; gv[j].y += x.y; gv[j].z += x.z; gv[j].w += x.w;
+            }
           }
         }
       }
@@ -751,7 +750,7 @@ __global__ void __launch_bounds__(256) linrec_out_kernel(LinRecArgs a, Trace tr)
         if (i < vdim) {
           const float4 w4 = *reinterpret_cast<const float4*>(w + i);
           float r[4] = {ov[j].x * inv * w4.x, ov[j].y * inv * w4.y, ov[j].z * inv * w4.z, ov[j].w * inv * w4.w};
-          if (gated) {
+          if constexpr (GATED) {
             r[0] *= silu(gv[j].x); r[1] *= silu(gv[j].y); r[2] *= silu(gv[j].z); r[3] *= silu(gv[j].w);
           }
           store4(out + h * vdim + i, r);
@@ -765,7 +764,7 @@ __global__ void __launch_bounds__(256) linrec_out_kernel(LinRecArgs a, Trace tr)
     const float* w = a.onorm_w + (size_t)h * a.onorm_ld;
     for (int i = lane; i < vdim; i += 32) {
       const float r = o[i] * inv * w[i];
-      out[h * vdim + i] = from_f32<OT>(gated ? r * silu(seg_at(a.gate, t, h * vdim + i)) : r);
+      out[h * vdim + i] = from_f32<OT>(GATED ? r * silu(seg_at(a.gate, t, h * vdim + i)) : r);
     }
   }
   if (blockIdx.y == 0)
@@ -776,8 +775,17 @@ __global__ void __launch_bounds__(256) linrec_out_kernel(LinRecArgs a, Trace tr)
 cudaError_t launch_linrec_out(cudaStream_t st, int odt, const LinRecArgs& a) {
   if (a.T <= 0) return cudaSuccess;
   const dim3 grid(a.T, a.T >= 1024 ? 1 : ceil_div(a.H, 8));
-  if (odt == DT_F32) (void)launch_k(linrec_out_kernel<float>, grid, dim3(256), 0, st, a, next_trace(42));
-  else (void)launch_k(linrec_out_kernel<bf16>, grid, dim3(256), 0, st, a, next_trace(42));
+#define LO(OT_, MJ_)                                                                                           \
+  do {                                                                                                         \
+    if (a.gate.p) (void)launch_k(linrec_out_kernel<OT_, MJ_, true>, grid, dim3(256), 0, st, a, next_trace(42)); \
+    else (void)launch_k(linrec_out_kernel<OT_, MJ_, false>, grid, dim3(256), 0, st, a, next_trace(42));         \
+  } while (0)
+  if (odt == DT_F32) {
+    if (a.vdim <= 128) LO(float, 1); else LO(float, 4);
+  } else {
+    if (a.vdim <= 128) LO(bf16, 1); else LO(bf16, 4);
+  }
+#undef LO
   return cudaGetLastError();
 }
 
@@ -917,7 +925,7 @@ __global__ void __launch_bounds__(512) input_conv_kernel(InputConvArgs a, Trace 
 
 // The same for steps of many rows with a router: a CTA takes TT tokens, their convolved rows stay in
 // shared memory, and a warp accumulates four experts against all of them — a router row crosses L2 once per TT tokens
-// instead of once per token.  Every dot product is summed in moe_route_row's order.
+// instead of once per token.
 template <typename AT, int TAPS, int TT>
 __global__ void __launch_bounds__(256) input_conv_route_kernel(InputConvArgs a, Trace tr) {
   TRACE_ENTRY(tr);
@@ -968,18 +976,21 @@ __global__ void __launch_bounds__(256) input_conv_route_kernel(InputConvArgs a, 
     for (int q = 0; q < EB; q++)
 #pragma unroll
       for (int tt = 0; tt < TT; tt++) acc[q][tt] = 0.f;
-    for (int i = lane * 8; i < W; i += 256) {
-      float r[EB][8];
+#pragma unroll 2
+    for (int i = lane * 4; i < W; i += 128) {  // neighbouring lanes, neighbouring 16-byte pieces: no bank conflicts
+      float4 r[EB];
 #pragma unroll
-      for (int q = 0; q < EB; q++) load8(a.router + (size_t)min(e0 + q, E - 1) * W + i, r[q]);
+      for (int q = 0; q < EB; q++) r[q] = *reinterpret_cast<const float4*>(a.router + (size_t)min(e0 + q, E - 1) * W + i);
 #pragma unroll
       for (int tt = 0; tt < TT; tt++) {
-        float y[8];
-        load8(rows + (size_t)tt * W + i, y);
+        const float4 y = *reinterpret_cast<const float4*>(rows + (size_t)tt * W + i);
 #pragma unroll
-        for (int q = 0; q < EB; q++)
-#pragma unroll
-          for (int e = 0; e < 8; e++) acc[q][tt] = fmaf(y[e], r[q][e], acc[q][tt]);
+        for (int q = 0; q < EB; q++) {
+          acc[q][tt] = fmaf(y.x, r[q].x, acc[q][tt]);
+          acc[q][tt] = fmaf(y.y, r[q].y, acc[q][tt]);
+          acc[q][tt] = fmaf(y.z, r[q].z, acc[q][tt]);
+          acc[q][tt] = fmaf(y.w, r[q].w, acc[q][tt]);
+        }
       }
     }
 #pragma unroll
