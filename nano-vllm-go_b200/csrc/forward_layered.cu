@@ -2,7 +2,7 @@
 // (nvllm_create_layered): handle set-up, tensors by checkpoint name, the cache pools and the
 // forward pass of one engine step.
 //
-// Two block styles on the fp32 residual stream x (nvllm_layered_config::block_style):
+// Three block styles on the fp32 residual stream x (nvllm_layered_config::block_style):
 //   parallel, pre-norm:      h = LayerNorm(x) (weight only);  x += mixer(h) + feed_forward(h)
 //   sequential, post-norm:   x += RMSNorm(mixer(x));  x += RMSNorm(feed_forward(x))  — the
 //     sublayers read x itself (kept beside the fp32 stream in the activation dtype), the norm
