@@ -191,9 +191,11 @@ int nvllm_create(const nvllm_config* cfg, const uint8_t* tp_id, nvllm_handle** o
  *   NVLLM_LBLOCK_SEQUENTIAL_PRENORM   x += mixer(RMSNorm(x)), then x += feed_forward(RMSNorm(x)); a run of
  *                                   layers may repeat with the same weights (loop_*), every pass with caches and
  *                                   state of its own and a learned vector added to x at its start (Lazovik, Sutuvik);
- *                                   with layer_norm = 1 LayerNorm (weight and additive term) instead (Sozurax)
+ *                                   with layer_norm = 1 LayerNorm (weight and additive term) instead (Sozurax); with loop_embed = 1 the
+ *                                   passes after the first open with the embedding instead (Defilorn)
  * Tensors are handed in by checkpoint name (nvllm_set_named_weight, or nvllm_load_safetensors
- * with NVLLM_ARCH_DUGOPEL / NVLLM_ARCH_ZOZONEX / NVLLM_ARCH_LAZOVIK / NVLLM_ARCH_SUTUVIK / NVLLM_ARCH_SOZURAX). */
+ * with NVLLM_ARCH_DUGOPEL / NVLLM_ARCH_ZOZONEX / NVLLM_ARCH_LAZOVIK / NVLLM_ARCH_SUTUVIK / NVLLM_ARCH_SOZURAX /
+ * NVLLM_ARCH_DEFILORN). */
 enum nvllm_mixer_kind {
   NVLLM_MIXER_LATENT_ATTENTION = 1,
   NVLLM_MIXER_WINDOW_ATTENTION = 2, /* grouped-query attention over a sliding window of the paged K / V cache */
@@ -209,15 +211,20 @@ enum nvllm_mixer_kind {
                                        learned one per head, values mixed with an earlier layer's, a gate per head */
   NVLLM_MIXER_MAMBA2 = 7,           /* Mamba-2: per head S <- exp(-exp(A_log) dt) S + dt B x^T (state x vdim), y = S^T C + D x,
                                        gated by silu(z) and then normed in groups; state and convolution tail per state slot */
-  NVLLM_MIXER_HGRN2 = 8             /* per head S <- diag(f) S + (1 - f) v^T (dim x vdim), o = S^T silu(q), f = l + (1 - l)
+  NVLLM_MIXER_HGRN2 = 8,            /* per head S <- diag(f) S + (1 - f) v^T (dim x vdim), o = S^T silu(q), f = l + (1 - l)
                                        sigmoid(W_f h + b) per key entry with a lower bound l; read-outs RMS-normed per
                                        head; state per slot */
+  NVLLM_MIXER_MLSTM = 9             /* matrix memory with scalar gates per head, given as capped logarithms i and f: S and a
+                                       vector n decay by exp(f) and take exp(i) k v^T and exp(i) k, both kept relative to a
+                                       running maximum m of the log gates (0 at the start); o = S^T q / (max(|n . q|,
+                                       exp(-m)) + 1e-6), RMS-normed per head, times a weight and sigmoid(W_g h); state per slot */
 };
 enum nvllm_mlp_kind { NVLLM_MLP_NONE = 0, NVLLM_MLP_DENSE = 1, NVLLM_MLP_MOE = 2 };
 enum nvllm_ffn_act {
   NVLLM_FFN_GLU_CLAMPED = 0, /* W_down (g sigmoid(1.702 g) (u + 1)), g / u clamped by `limit` */
   NVLLM_FFN_RELU2 = 1,       /* W_down relu(W_up h)^2 */
   NVLLM_FFN_SWIGLU = 2,      /* W_down (silu(W_gate h) * (W_up h)) */
+  NVLLM_FFN_GEGLU = 4,       /* W_down (gelu_tanh(W_gate h) * (W_up h)) */
   NVLLM_FFN_POLYNORM = 3     /* W_down (a N(z) + b N(z^2) + c N(z^3) + e), z = W_up h, powers element by element, N divides
                                 the row by its root mean square; {a, b, c, e} = tensor "mlp.act" */
 };
@@ -298,6 +305,18 @@ typedef struct nvllm_layer_spec {
   int32_t group_top2;       /* 1: a group of experts scores as the sum of its two best choice scores (else its best) */
   int32_t route_norm;       /* 1 (with route_sigmoid): the weights are the chosen scores divided by their sum (+ 1e-20) */
   int32_t route_bias;       /* 1: tensor "mlp.router.b" [experts] is added to the logits */
+  /* NVLLM_MIXER_ATTENTION also takes window (0: every j <= i); latent attention in sequential pre-norm blocks also takes
+   * sink / sink_learned, out_gate (every entry of the concatenated heads times sigmoid(W_g h)) and rot_factor /
+   * rot_original / rot_fast / rot_slow */
+  int32_t diff_maps;        /* 1: two score maps per head over the same values (q and k rows hold [map 1, map 2] per head,
+                               dim entries each), o = N(map 1 - l * map 2) * (1 - diff), N divides a head's vdim entries by
+                               their root mean square, l = exp(lq1 . lk1) - exp(lq2 . lk2) + diff (tensors "mix.lq1" ...) */
+  float diff;
+  float gate_cap;           /* NVLLM_MIXER_MLSTM: log gates are cap * tanh(z / cap) */
+  int32_t route_identity;   /* the router has this many more outputs after the experts: an expert without tensors whose
+                               output is its input (softmax scores only) */
+  int32_t route_raw;        /* 1: the weights are the chosen experts' scores as they are (times router_scale) */
+  int32_t shared_gate;      /* 1 (with shared_ff, act = NVLLM_FFN_SWIGLU): that expert's output times sigmoid(W_sg h) */
 } nvllm_layer_spec;
 
 typedef struct nvllm_layered_config {
@@ -330,6 +349,8 @@ typedef struct nvllm_layered_config {
   int32_t ffn_conv;        /* taps >= 1: the same on what a feed-forward reads (tensor "l<i>.canon2"; the router reads it too) */
   int32_t layer_norm;      /* 1: the norms of the stream are LayerNorms with weight and additive term (tensors "<norm>",
                               "<norm>.b") */
+  int32_t loop_embed;      /* 1: a repeated run has no "loop.step"; every pass but the first opens with x += the embedding
+                              of the token (as it entered layer 0) */
 } nvllm_layered_config;
 
 int nvllm_create_layered(const nvllm_layered_config* cfg, const nvllm_layer_spec* layers,
@@ -376,7 +397,8 @@ enum nvllm_arch {
   NVLLM_ARCH_ZOZONEX = 5,     /* layered handle, likewise */
   NVLLM_ARCH_LAZOVIK = 6,     /* layered handle, likewise */
   NVLLM_ARCH_SUTUVIK = 7,     /* layered handle, likewise */
-  NVLLM_ARCH_SOZURAX = 8      /* layered handle, likewise */
+  NVLLM_ARCH_SOZURAX = 8,     /* layered handle, likewise */
+  NVLLM_ARCH_DEFILORN = 9     /* layered handle, likewise */
 };
 
 /* Load every weight of the model straight from `model_dir` — model.safetensors, or the shards

@@ -27,11 +27,11 @@ BLOCK_SEQUENTIAL, BLOCK_PARALLEL = 0, 1
 PREC_FP32, PREC_BF16 = 0, 1
 # enum nvllm_arch (checkpoint families of generic_loader.go:60-182)
 ARCH_GPT2, ARCH_FALCON, ARCH_LLAMA, ARCH_GRANITE_MOE, ARCH_DUGOPEL, ARCH_ZOZONEX, ARCH_LAZOVIK, ARCH_SUTUVIK = 0, 1, 2, 3, 4, 5, 6, 7
-ARCH_SOZURAX = 8
+ARCH_SOZURAX, ARCH_DEFILORN = 8, 9
 MIXER_LATENT_ATTENTION, MIXER_WINDOW_ATTENTION, MIXER_DELTA, MIXER_GLA, MIXER_ATTN_TMIX = 1, 2, 3, 4, 5
-MIXER_ATTENTION, MIXER_MAMBA2, MIXER_HGRN2 = 6, 7, 8
+MIXER_ATTENTION, MIXER_MAMBA2, MIXER_HGRN2, MIXER_MLSTM = 6, 7, 8, 9
 MLP_NONE, MLP_DENSE, MLP_MOE = 0, 1, 2
-FFN_GLU_CLAMPED, FFN_RELU2, FFN_SWIGLU, FFN_POLYNORM = 0, 1, 2, 3
+FFN_GLU_CLAMPED, FFN_RELU2, FFN_SWIGLU, FFN_POLYNORM, FFN_GEGLU = 0, 1, 2, 3, 4
 LBLOCK_PARALLEL_PRENORM, LBLOCK_SEQUENTIAL_POSTNORM, LBLOCK_SEQUENTIAL_PRENORM = 0, 1, 2
 LPOS_NONE, LPOS_SINUSOIDAL = 0, 1
 DT_F32, DT_BF16, DT_F16 = 0, 1, 2
@@ -318,6 +318,8 @@ class CLayerSpec(ctypes.Structure):
         ("state", ctypes.c_int32), ("ssm_groups", ctypes.c_int32), ("norm_groups", ctypes.c_int32),
         ("route_correction", ctypes.c_int32), ("group_top2", ctypes.c_int32), ("route_norm", ctypes.c_int32),
         ("route_bias", ctypes.c_int32),
+        ("diff_maps", ctypes.c_int32), ("diff", ctypes.c_float), ("gate_cap", ctypes.c_float),
+        ("route_identity", ctypes.c_int32), ("route_raw", ctypes.c_int32), ("shared_gate", ctypes.c_int32),
     ]
 
 
@@ -336,7 +338,7 @@ class CLayeredConfig(ctypes.Structure):
         ("loop_start", ctypes.c_int32), ("loop_stop", ctypes.c_int32), ("loop_times", ctypes.c_int32),
         ("norm_groups", ctypes.c_int32), ("embed_norm", ctypes.c_int32), ("mixer_conv", ctypes.c_int32),
         ("side_dim", ctypes.c_int32), ("logit_scale", ctypes.c_float),
-        ("ffn_conv", ctypes.c_int32), ("layer_norm", ctypes.c_int32),
+        ("ffn_conv", ctypes.c_int32), ("layer_norm", ctypes.c_int32), ("loop_embed", ctypes.c_int32),
     ]
 
 
@@ -402,6 +404,12 @@ class LayerSpec:
     group_top2: int = 0
     route_norm: int = 0
     route_bias: int = 0
+    diff_maps: int = 0
+    diff: float = 0.0
+    gate_cap: float = 0.0
+    route_identity: int = 0
+    route_raw: int = 0
+    shared_gate: int = 0
 
     def to_c(self) -> CLayerSpec:
         c = CLayerSpec()
@@ -415,7 +423,7 @@ class LayerSpec:
         p = f"l{layer}."
         if self.mixer in (MIXER_GLA, MIXER_ATTN_TMIX):
             return self._prenorm_shapes(p, width)
-        if self.mixer in (MIXER_ATTENTION, MIXER_MAMBA2, MIXER_HGRN2) or (self.mixer == MIXER_LATENT_ATTENTION and prenorm):
+        if self.mixer in (MIXER_ATTENTION, MIXER_MAMBA2, MIXER_HGRN2, MIXER_MLSTM) or (self.mixer == MIXER_LATENT_ATTENTION and prenorm):
             return self._prenorm2_shapes(p, width)
         if self.mixer == MIXER_WINDOW_ATTENTION:
             d = {p + "norm1": (width,), p + "mix.q": (self.heads * self.dim, width),
@@ -493,14 +501,17 @@ LayerSpec._prenorm_shapes = _prenorm_shapes
 
 
 def _prenorm2_shapes(self, p: str, width: int) -> dict:
-    """Attention with its options / Mamba-2 / HGRN2 / latent attention, and the mixture of gated
-    experts or the PolyNorm dense layer."""
+    """Attention with its options / Mamba-2 / HGRN2 / mLSTM / latent attention, and the mixture of gated
+    experts or a dense layer (PolyNorm, gated)."""
     d = {p + "norm1": (width,)}
     m = p + "mix."
     if self.mixer == MIXER_ATTENTION:
         hv = self.heads * self.vdim
-        d.update({m + "q": (self.heads * self.dim, width), m + "k": (self.kv_heads * self.dim, width),
+        maps = 2 if self.diff_maps else 1
+        d.update({m + "q": (self.heads * maps * self.dim, width), m + "k": (self.kv_heads * maps * self.dim, width),
                   m + "v": (self.kv_heads * self.vdim, width), m + "o": (width, hv)})
+        if self.diff_maps:
+            d.update({m + n: (self.dim,) for n in ("lq1", "lk1", "lq2", "lk2")})
         if self.qk_norm == 3:
             d.update({m + "q.norm": (self.dim,), m + "k.norm": (self.dim,)})
         if self.v_mix:
@@ -515,6 +526,11 @@ def _prenorm2_shapes(self, p: str, width: int) -> dict:
         hd, hv = self.heads * self.dim, self.heads * self.vdim
         d.update({m + "q": (hd, width), m + "f": (hd, width), m + "f.b": (hd,), m + "lower": (hd,), m + "v": (hv, width),
                   m + "norm": (self.vdim,), m + "o": (width, hv)})
+    elif self.mixer == MIXER_MLSTM:
+        hd, hv = self.heads * self.dim, self.heads * self.vdim
+        d.update({m + "q": (hd, width), m + "k": (hd, width), m + "v": (hv, width), m + "g": (hv, width), m + "o": (width, hv),
+                  m + "norm": (hv,), m + "i": (self.heads, width), m + "i.b": (self.heads,), m + "f": (self.heads, width),
+                  m + "f.b": (self.heads,)})
     elif self.mixer == MIXER_LATENT_ATTENTION:
         d.update({m + "dq": (self.q_rank, width), m + "dq.norm": (self.q_rank,),
                   m + "uq": (self.heads * (self.dim + self.rot_dim), self.q_rank),
@@ -522,25 +538,31 @@ def _prenorm2_shapes(self, p: str, width: int) -> dict:
                   m + "o": (width, self.heads * self.vdim)})
         if self.kv_from < 0:
             d.update({m + "dkv": (self.kv_rank + self.rot_dim, width), m + "dkv.norm": (self.kv_rank,)})
-        if self.head_gate:
-            d[m + "g"] = (self.heads, width)
+        if self.head_gate or self.out_gate:
+            d[m + "g"] = (self.heads * (self.vdim if self.out_gate else 1), width)
+        if self.sink_learned:
+            d[m + "sink"] = (self.heads,)
     else:
         inner, gn = self.heads * self.vdim, self.ssm_groups * self.state
         d.update({m + "in": (2 * inner + 2 * gn + self.heads, width), m + "conv": (inner + 2 * gn, self.conv),
                   m + "conv.b": (inner + 2 * gn,), m + "dt_bias": (self.heads,), m + "A_log": (self.heads,),
                   m + "D": (self.heads,), m + "norm": (inner,), m + "o": (width, inner)})
     if self.mlp == MLP_DENSE:
-        d.update({p + "norm2": (width,), p + "mlp.up": (self.ff, width), p + "mlp.down": (width, self.ff), p + "mlp.act": (4,)})
+        d.update({p + "norm2": (width,), p + "mlp.up": (self.ff, width), p + "mlp.down": (width, self.ff)})
+        d[p + "mlp.act" if self.act == FFN_POLYNORM else p + "mlp.gate"] = (4,) if self.act == FFN_POLYNORM else (self.ff, width)
     if self.mlp == MLP_MOE:
         d[p + "norm2"] = (width,)
-        d[p + "mlp.router"] = (self.experts, width)
+        outs = self.experts + self.route_identity
+        d[p + "mlp.router"] = (outs, width)
         if self.route_bias:
-            d[p + "mlp.router.b"] = (self.experts,)
+            d[p + "mlp.router.b"] = (outs,)
         if self.shared_ff > 0:
             d.update({p + "mlp.shared.gate": (self.shared_ff, width), p + "mlp.shared.up": (self.shared_ff, width),
                       p + "mlp.shared.down": (width, self.shared_ff)})
+            if self.shared_gate:
+                d[p + "mlp.shared.sg"] = (1, width)
         if self.route_correction:
-            d[p + "mlp.correction"] = (self.experts,)
+            d[p + "mlp.correction"] = (outs,)
         for e in range(self.experts):
             d.update({f"{p}mlp.e{e}.gate": (self.ff, width), f"{p}mlp.e{e}.up": (self.ff, width),
                       f"{p}mlp.e{e}.down": (width, self.ff)})
@@ -552,7 +574,8 @@ LayerSpec._prenorm2_shapes = _prenorm2_shapes
 
 @dataclass(frozen=True)
 class ListedModelConfig:
-    """A model whose config.json lists its layers (architectures "Dugopel", "Zozonex", "Lazovik", "Sutuvik", "Sozurax")."""
+    """A model whose config.json lists its layers (architectures "Dugopel", "Zozonex", "Lazovik", "Sutuvik", "Sozurax",
+    "Defilorn")."""
     name: str
     vocab_size: int
     hidden: int
@@ -576,6 +599,7 @@ class ListedModelConfig:
     logit_scale: float = 0.0
     ffn_conv: int = 0     # taps of the causal convolution added to what every feed-forward reads
     layer_norm: bool = False  # the stream's norms are LayerNorms with weight and additive term
+    loop_embed: bool = False  # passes of a repeated run after the first open with the embedding, not a learned vector
 
     @property
     def has_loop(self) -> bool:
@@ -598,14 +622,14 @@ class ListedModelConfig:
     def needs_state_slots(self) -> bool:
         """True when some layer keeps state per sequence: a recurrence, the tail of a short convolution."""
         return self.mixer_conv > 1 or any(
-            l.mixer in (MIXER_DELTA, MIXER_GLA, MIXER_ATTN_TMIX, MIXER_MAMBA2, MIXER_HGRN2) or
+            l.mixer in (MIXER_DELTA, MIXER_GLA, MIXER_ATTN_TMIX, MIXER_MAMBA2, MIXER_HGRN2, MIXER_MLSTM) or
             (self.ffn_conv > 1 and l.mlp != MLP_NONE) for l in self.layers)
 
     def tensor_shapes(self) -> dict:
         d = {"embed": (self.vocab_size, self.hidden), "final.norm": (self.hidden,)}
         if not self.tied_head:
             d["head"] = (self.vocab_size, self.hidden)
-        if self.has_loop:
+        if self.has_loop and not self.loop_embed:
             d["loop.step"] = (self.loop_times, self.hidden)
         if self.layer_norm:
             d["final.norm.b"] = (self.hidden,)
@@ -637,7 +661,7 @@ class ListedModelConfig:
         n = 0
         for l in (self.layers[i] for i in self.runs):
             if l.mixer in (MIXER_ATTN_TMIX, MIXER_ATTENTION):
-                n += l.kv_heads * (l.dim + l.vdim) * bytes_per_el
+                n += l.kv_heads * (l.dim * (2 if l.diff_maps else 1) + l.vdim) * bytes_per_el
             elif l.mixer == MIXER_LATENT_ATTENTION and l.kv_from < 0:
                 n += (l.kv_rank + l.rot_dim) * bytes_per_el
             elif l.mixer == MIXER_WINDOW_ATTENTION and l.kv_from < 0:
@@ -651,6 +675,8 @@ class ListedModelConfig:
         for l in (self.layers[i] for i in self.runs):
             if l.mixer in (MIXER_GLA, MIXER_HGRN2):
                 n += 4 * l.heads * l.dim * l.vdim
+            elif l.mixer == MIXER_MLSTM:
+                n += 4 * l.heads * (l.dim * l.vdim + l.dim + 1)
             elif l.mixer == MIXER_ATTN_TMIX:
                 n += 4 * (l.heads2 * l.dim2 * l.dim2 + self.hidden +
                           (l.conv - 1) * (l.heads * l.dim + l.kv_heads * (l.dim + l.vdim)))
@@ -675,7 +701,7 @@ class ListedModelConfig:
         c.loop_start, c.loop_stop, c.loop_times = self.loop_start, self.loop_stop, self.loop_times
         c.norm_groups, c.embed_norm, c.mixer_conv = self.norm_groups, int(self.embed_norm), self.mixer_conv
         c.side_dim, c.logit_scale = self.side_dim, self.logit_scale
-        c.ffn_conv, c.layer_norm = self.ffn_conv, int(self.layer_norm)
+        c.ffn_conv, c.layer_norm, c.loop_embed = self.ffn_conv, int(self.layer_norm), int(self.loop_embed)
         specs = (CLayerSpec * len(self.layers))(*[l.to_c() for l in self.layers])
         return c, specs
 
@@ -900,6 +926,56 @@ def sozurax_from_json(j: dict) -> ListedModelConfig:
         arch=ARCH_SOZURAX, block_style=LBLOCK_SEQUENTIAL_PRENORM, layer_norm=True, mixer_conv=taps, ffn_conv=taps)
 
 
+def _defilorn_layer(i: int, lc: dict) -> LayerSpec:
+    m = lc["mixer"]
+    kind = lc.get("type")
+    kw = dict(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m.get("vdim") or m["dim"]))
+    if kind == "mlstm":
+        kw.update(mixer=MIXER_MLSTM, gate_cap=float(m["gate_cap"]))
+    elif kind == "attention":
+        kw.update(mixer=MIXER_ATTENTION, kv_heads=int(m.get("kv_heads") or m["heads"]), scale=float(m["scale"]), qk_norm=3,
+                  window=int((m.get("mask") or {}).get("size") or 0), diff_maps=1, diff=float(m["diff"]))
+    elif kind == "latent_attention":
+        rot = m["rot"]
+        sc = rot.get("scaling") or {}
+        kw.update(mixer=MIXER_LATENT_ATTENTION, rot_dim=int(m["rot_dim"]), kv_rank=int(m["kv_rank"]), q_rank=int(m["q_rank"]),
+                  rot_base=float(rot["base"]), rot_dims=int(rot.get("dims") or m["rot_dim"]), rot_pairs=1, scale=float(m["scale"]),
+                  rot_factor=float(sc.get("factor") or 0.0), rot_original=float(sc.get("original") or 0.0),
+                  rot_fast=float(sc.get("fast") or 0.0), rot_slow=float(sc.get("slow") or 0.0),
+                  sink=1, sink_learned=1, out_gate=1)
+    else:
+        raise ValueError(f"layer {i}: unknown layer type {kind!r}")
+    mlp = lc.get("mlp")
+    if mlp is None:
+        pass
+    elif mlp["kind"] == "dense":
+        kw.update(mlp=MLP_DENSE, act=FFN_GEGLU, ff=int(mlp["ff"]))
+    elif mlp["kind"] == "moe":
+        r = mlp["router"]
+        kw.update(mlp=MLP_MOE, act=FFN_SWIGLU, ff=int(mlp["expert"]["ff"]), experts=int(r["experts"]), top=int(r["top"]),
+                  route_identity=int(r.get("identity") or 0), route_correction=1, route_raw=1,
+                  shared_ff=int((mlp.get("shared") or {}).get("ff") or 0), shared_gate=1)
+    else:
+        raise ValueError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
+    return LayerSpec(**kw)
+
+
+def defilorn_from_json(j: dict) -> ListedModelConfig:
+    """config.json of the Defilorn design: mLSTM layers, latent attention with sinks and an output gate,
+    and differential attention over a sliding window in any order, pre-norm blocks with norm weights
+    stored around zero; a run of layers may repeat, its later passes open with the embedding; tanh-GELU
+    gated dense feed-forwards or softmax-routed gated experts among which some are the identity, with a
+    gated always-on expert; logits through a head of its own."""
+    lp = j.get("loop") or {}
+    times = int(lp.get("times") or 0)
+    return ListedModelConfig(
+        name="defilorn", vocab_size=int(j["vocab"]), hidden=int(j["width"]),
+        layers=tuple(_defilorn_layer(i, lc) for i, lc in enumerate(j["layers"])),
+        norm_eps=float(j["norm"]["eps"]), arch=ARCH_DEFILORN, block_style=LBLOCK_SEQUENTIAL_PRENORM, norm_offset=1.0,
+        loop_start=int(lp.get("start") or 0) if times >= 1 else 0,
+        loop_stop=int(lp.get("stop") or 0) if times >= 1 else 0, loop_times=times, loop_embed=True)
+
+
 def safetensors_shapes(model_dir: str) -> dict:
     """Tensor name -> shape from the header of model.safetensors (8-byte little-endian length,
     then that many bytes of JSON)."""
@@ -914,7 +990,7 @@ def safetensors_shapes(model_dir: str) -> dict:
 
 # model registry: config.json "architecture" -> config builder
 ARCHITECTURES = {"Dugopel": dugopel_from_json, "Zozonex": zozonex_from_json, "Lazovik": lazovik_from_json,
-                 "Sutuvik": sutuvik_from_json, "Sozurax": sozurax_from_json}
+                 "Sutuvik": sutuvik_from_json, "Sozurax": sozurax_from_json, "Defilorn": defilorn_from_json}
 # builders that also want the checkpoint's tensor shapes
 _WANTS_SHAPES = {"Lazovik"}
 

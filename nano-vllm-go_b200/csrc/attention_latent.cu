@@ -19,8 +19,12 @@
 //                         latent rows; one warp per item, a CTA's items share each key tile;
 //                         optional key splits (decode) merged by latent_combine_kernel
 //                         the head's sigmoid gate is applied where the sum is normalised
+//  latent_expand_kernel   layers whose output gate sits between the value expansion and the output projection:
+//                         out = sigmoid(gate) * (W_uv o) per head (W_uv is not folded into W_o there); decode steps
+//                         with key splits do it inside latent_combine_kernel
 // A window (LatentArgs::window) moves the first key tile of a CTA up and masks the keys before each
-// item's window in the tiles where they can occur.  Without `gate` the heads have no gate.
+// item's window in the tiles where they can occur.  Without `gate` the heads have no gate.  A learned sink
+// (LatentArgs::sink_w) is one more term of the softmax denominator; it joins where the sum is normalised.
 // All arithmetic is fp32 (double for the angles); QT / KT are the activation / cache dtypes.
 #include <stdlib.h>
 
@@ -65,9 +69,30 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(LatentArgs a, Trace tr
   extern __shared__ float row[];  // [n_in]
   __shared__ float red[32];
   const int t = blockIdx.x;
+  // (per-entry output gates are many columns: they go straight through, the rest is staged)
   const int n_in = a.q_rank + (a.own_kv ? a.R + a.rot : 0) + (a.gate ? a.H : 0);
   pdl_wait();
-  if ((n_in & 7) == 0 && (a.in_stride & 7) == 0) {
+  if (a.out_gate) {
+    const int n_g = a.H * a.vdim;
+    const float* gp = a.in_p + (size_t)t * a.in_ld + n_in;
+    float* go = a.out_gate + (size_t)t * n_g;
+    if ((n_g & 7) == 0 && (n_in & 7) == 0 && (a.in_ld & 7) == 0 && (a.in_stride & 7) == 0) {
+      for (int i = threadIdx.x * 8; i < n_g; i += blockDim.x * 8) {
+        float v[8];
+        sum_partials8(gp + i, a.in_S, a.in_stride, v);
+#pragma unroll
+        for (int j = 0; j < 8; j++) v[j] = 1.0f / (1.0f + expf(-v[j]));
+        store8(go + i, v);
+      }
+    } else {
+      for (int i = threadIdx.x; i < n_g; i += blockDim.x) {
+        float s = 0.f;
+        for (int k = 0; k < a.in_S; k++) s += gp[(size_t)k * a.in_stride + i];
+        go[i] = 1.0f / (1.0f + expf(-s));
+      }
+    }
+  }
+  if ((n_in & 7) == 0 && (a.in_stride & 7) == 0 && (a.in_ld & 7) == 0) {
     for (int i = threadIdx.x * 8; i < n_in; i += blockDim.x * 8) {
       float v[8];
       sum_partials8(a.in_p + (size_t)t * a.in_ld + i, a.in_S, a.in_stride, v);
@@ -245,18 +270,24 @@ cudaError_t launch_latent_fold(cudaStream_t st, int wdt, const void* w_uq, const
   if (wdt == DT_F32) {
     latent_fold_q_kernel<float><<<148 * 8, 256, 0, st>>>((const float*)w_uq, (const float*)w_uk, (float*)wq, H, dim,
                                                          rot, R, q_rank, q_rank_p);
-    latent_fold_o_kernel<float><<<148 * 8, 256, 0, st>>>((const float*)w_o, (const float*)w_uv, (float*)wo, W, H,
+    if (wo) latent_fold_o_kernel<float><<<148 * 8, 256, 0, st>>>((const float*)w_o, (const float*)w_uv, (float*)wo, W, H,
                                                          vdim, R, ov_p, ovr_p);
   } else {
     latent_fold_q_kernel<bf16><<<148 * 8, 256, 0, st>>>((const bf16*)w_uq, (const bf16*)w_uk, (bf16*)wq, H, dim, rot,
                                                         R, q_rank, q_rank_p);
-    latent_fold_o_kernel<bf16><<<148 * 8, 256, 0, st>>>((const bf16*)w_o, (const bf16*)w_uv, (bf16*)wo, W, H, vdim, R,
+    if (wo) latent_fold_o_kernel<bf16><<<148 * 8, 256, 0, st>>>((const bf16*)w_o, (const bf16*)w_uv, (bf16*)wo, W, H, vdim, R,
                                                         ov_p, ovr_p);
   }
   return cudaGetLastError();
 }
 
 // ---------------------------------------------------------------- attention
+// 1 / (softmax denominator), the sink's term included: m, l are the running maximum (of scaled scores) and sum
+__device__ __forceinline__ float inv_denom(const LatentArgs& a, int head, float m, float l) {
+  if (!a.sink_w) return 1.0f / l;
+  const float s = a.sink_w[head], top = fmaxf(m, s), e = expf(m - top);
+  return e / (l * e + expf(s - top));
+}
 // grid (tiles, item chunks, key splits).  A tile is LAT_QTILE consecutive new tokens of one
 // sequence (the host's tile list; without one, tile = sequence and its single new token).  The
 // tile's (query, head) items are dealt to warps, LAT_WARPS per CTA; all of them read the same
@@ -353,7 +384,8 @@ __global__ void __launch_bounds__(LAT_WARPS * 32) latent_attn_kernel(LatentArgs 
   TRACE_EXIT(tr);
   if (!valid) return;
   if (gridDim.z == 1) {
-    const float inv = (a.gate ? a.gate[(size_t)row * a.H + head] : 1.f) / l;  // the head's sigmoid gate rides on the normalisation
+    // the head's sigmoid gate rides on the normalisation
+    const float inv = (a.gate ? a.gate[(size_t)row * a.H + head] : 1.f) * inv_denom(a, head, m, l);
     QT* op = (QT*)a.olat + (size_t)row * a.o_ld + head * a.R;
 #pragma unroll
     for (int i = 0; i < LAT_NACC; i++) {
@@ -580,7 +612,8 @@ latent_attn_mma_kernel(LatentArgs a, int two_stage, Trace tr) {
     const size_t it = (size_t)(row0 + q0) * a.H + item;  // row * H + head
     if (gridDim.z == 1) {
       const int row = row0 + q0 + item / a.H, head = item % a.H;
-      const float inv = (a.gate ? a.gate[it] : 1.f) / l[i];  // the head's sigmoid gate rides on the normalisation
+      // the head's sigmoid gate rides on the normalisation
+      const float inv = (a.gate ? a.gate[it] : 1.f) * inv_denom(a, head, m[i] * a.scale, l[i]);
       bf16* op = (bf16*)a.olat + (size_t)row * a.o_ld + head * a.R;
 #pragma unroll
       for (int dn = 0; dn < NR; dn++)
@@ -649,10 +682,50 @@ static cudaError_t launch_latent_mma(cudaStream_t st, const LatentArgs& a, int n
   return launch_latent_mma_r<NR, 64>(st, a, ns);
 }
 
+// One head of one row: out[head vdim + e] = out_gate * sum_r W_uv[head vdim + e, r] o[r] (o in shared memory, fp32);
+// a warp takes four entries at a time, its lanes 8 neighbouring latent entries each (16-byte loads) when R allows
 template <typename QT>
-__global__ void latent_combine_kernel(LatentArgs a, int n_splits, Trace tr) {
+__device__ __forceinline__ void expand_head(const LatentArgs& a, const QT* __restrict__ w_uv, const float* o, size_t row, int head,
+                                            QT* __restrict__ out) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  const float* gt = a.out_gate + (row * a.H + head) * a.vdim;
+  const QT* w0 = w_uv + (size_t)head * a.vdim * a.R;
+  for (int e0 = warp * 4; e0 < a.vdim; e0 += nw * 4) {
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    if ((a.R & 7) == 0) {
+      for (int r = lane * 8; r < a.R; r += 256) {
+        float w[4][8], x[8];
+#pragma unroll
+        for (int q = 0; q < 4; q++)
+          if (e0 + q < a.vdim) load8(w0 + (size_t)(e0 + q) * a.R + r, w[q]);
+        load8(o + r, x);
+#pragma unroll
+        for (int q = 0; q < 4; q++)
+          if (e0 + q < a.vdim)
+#pragma unroll
+            for (int j = 0; j < 8; j++) acc[q] = fmaf(w[q][j], x[j], acc[q]);
+      }
+    } else {
+      for (int r = lane; r < a.R; r += 32)
+#pragma unroll
+        for (int q = 0; q < 4; q++)
+          if (e0 + q < a.vdim) acc[q] = fmaf(to_f32(w0[(size_t)(e0 + q) * a.R + r]), o[r], acc[q]);
+    }
+#pragma unroll
+    for (int q = 0; q < 4; q++) {
+      const float s = warp_sum(acc[q]);
+      if (lane == 0 && e0 + q < a.vdim) out[head * a.vdim + e0 + q] = from_f32<QT>(s * gt[e0 + q]);
+    }
+  }
+}
+
+// exp_out != null: the merged sum is expanded and gated here as well (latent_expand_kernel's job), rows exp_ld apart
+template <typename QT>
+__global__ void __launch_bounds__(256) latent_combine_kernel(LatentArgs a, int n_splits, const QT* __restrict__ w_uv,
+                                                             QT* __restrict__ exp_out, int exp_ld, Trace tr) {
   TRACE_ENTRY(tr);
   pdl_launch_dependents();
+  extern __shared__ __align__(16) float merged[];  // [R] with exp_out
   pdl_wait();
   const size_t item = blockIdx.x;  // row * H + head
   const int ld = a.R + 2;
@@ -680,7 +753,7 @@ __global__ void latent_combine_kernel(LatentArgs a, int n_splits, Trace tr) {
   const size_t row = item / a.H;
   const int head = (int)(item % a.H);
   QT* op = (QT*)a.olat + row * a.o_ld + head * a.R;
-  const float inv = (a.gate ? a.gate[item] : 1.f) / l;
+  const float inv = (a.gate ? a.gate[item] : 1.f) * inv_denom(a, head, m, l);
   for (int r = threadIdx.x; r < a.R; r += blockDim.x) {
     float o = 0.f;
     for (int s0 = 0; s0 < n_splits; s0 += 8) {
@@ -691,12 +764,152 @@ __global__ void latent_combine_kernel(LatentArgs a, int n_splits, Trace tr) {
       for (int q = 0; q < 8; q++)
         if (s0 + q < n_splits) o = fmaf(v[q], wgt[s0 + q], o);
     }
-    op[r] = from_f32<QT>(o * inv);
+    if (exp_out) merged[r] = to_f32(from_f32<QT>(o * inv));  // (rounded as it would be on the way through memory)
+    else op[r] = from_f32<QT>(o * inv);
   }
-  if (head == a.H - 1)
+  if (exp_out) {
+    __syncthreads();
+    expand_head<QT>(a, w_uv, merged, row, head, exp_out + row * exp_ld);
+    if (head == a.H - 1)
+      for (int c = a.H * a.vdim + threadIdx.x; c < exp_ld; c += blockDim.x) exp_out[row * exp_ld + c] = from_f32<QT>(0.f);
+  } else if (head == a.H - 1) {
     for (int r = a.H * a.R + threadIdx.x; r < a.o_ld; r += blockDim.x)
       ((QT*)a.olat)[row * a.o_ld + r] = from_f32<QT>(0.f);
+  }
   TRACE_EXIT(tr);
+}
+
+template <typename QT>
+static void launch_latent_combine(cudaStream_t st, const LatentArgs& a, int ns) {
+  const bool ex = a.exp_out != nullptr;
+  (void)launch_k(latent_combine_kernel<QT>, dim3(a.T * a.H), dim3(ex ? 256 : 64), ex ? a.R * sizeof(float) : 0, st, a, ns,
+                 (const QT*)a.exp_w, (QT*)a.exp_out, a.exp_ld, next_trace(23));
+}
+
+// ---------------------------------------------------------------- value expansion with an output gate
+// grid (T, H): one head of one row per CTA, fp32 arithmetic, any sizes
+template <typename QT>
+__global__ void __launch_bounds__(256) latent_expand_kernel(LatentArgs a, const QT* __restrict__ w_uv, QT* __restrict__ out, int o_ld,
+                                                            Trace tr) {
+  TRACE_ENTRY(tr);
+  pdl_launch_dependents();
+  extern __shared__ __align__(16) float o[];  // [R]
+  pdl_wait();
+  const size_t row = blockIdx.x;
+  const int head = blockIdx.y;
+  const QT* src = (const QT*)a.olat + row * a.o_ld + (size_t)head * a.R;
+  for (int r = threadIdx.x; r < a.R; r += blockDim.x) o[r] = to_f32(src[r]);
+  __syncthreads();
+  expand_head<QT>(a, w_uv, o, row, head, out + row * o_ld);
+  if (head == a.H - 1)
+    for (int c = a.H * a.vdim + threadIdx.x; c < o_ld; c += blockDim.x) out[row * o_ld + c] = from_f32<QT>(0.f);
+  TRACE_EXIT(tr);
+}
+
+// bf16, R a multiple of 16, vdim of 8: CTA = 64 rows x one head x EN value entries on mma.sync.  Row and weight tiles
+// of LE_K latent entries by cp.async, double buffered; rows padded by 8 elements (ldmatrix without bank conflicts).
+constexpr int LE_M = 64;
+template <int EN, int LE_K>
+__global__ void __launch_bounds__(128) latent_expand_mma_kernel(LatentArgs a, const bf16* __restrict__ w_uv, bf16* __restrict__ out,
+                                                                int o_ld, Trace tr) {
+  constexpr int LE_LD = LE_K + 8;
+  TRACE_ENTRY(tr);
+  pdl_launch_dependents();
+  __shared__ __align__(16) bf16 As[2][LE_M * LE_LD];
+  __shared__ __align__(16) bf16 Ws[2][EN * LE_LD];
+  pdl_wait();
+  const int m0 = blockIdx.x * LE_M, head = blockIdx.y, e0 = blockIdx.z * EN;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const bf16* src = (const bf16*)a.olat + (size_t)head * a.R;
+  const bf16* wsrc = w_uv + ((size_t)head * a.vdim + e0) * a.R;
+  const int nm = min(LE_M, a.T - m0), ne = min(EN, a.vdim - e0);
+  auto load = [&](int kt, int buf) {
+    const int k0 = kt * LE_K;
+    for (int i = threadIdx.x; i < LE_M * (LE_K / 8); i += 128) {
+      const int r = i / (LE_K / 8), c = (i % (LE_K / 8)) * 8;
+      const bool ok = r < nm && k0 + c < a.R;
+      cp_async16(smem_addr(&As[buf][r * LE_LD + c]), ok ? src + (size_t)(m0 + r) * a.o_ld + k0 + c : src, ok);
+    }
+    for (int i = threadIdx.x; i < EN * (LE_K / 8); i += 128) {
+      const int r = i / (LE_K / 8), c = (i % (LE_K / 8)) * 8;
+      const bool ok = r < ne && k0 + c < a.R;
+      cp_async16(smem_addr(&Ws[buf][r * LE_LD + c]), ok ? wsrc + (size_t)r * a.R + k0 + c : wsrc, ok);
+    }
+    cp_async_commit();
+  };
+  float acc[EN / 8][4];
+#pragma unroll
+  for (int i = 0; i < EN / 8; i++) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+  const int nk = (a.R + LE_K - 1) / LE_K;
+  load(0, 0);
+  for (int kt = 0; kt < nk; kt++) {
+    const int buf = kt & 1;
+    if (kt + 1 < nk) {
+      load(kt + 1, buf ^ 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncthreads();
+#pragma unroll
+    for (int kk = 0; kk < LE_K / 16; kk++) {
+      uint32_t a0, a1, a2, a3;
+      ldsm_x4(smem_addr(&As[buf][(warp * 16 + (lane & 15)) * LE_LD + kk * 16 + (lane >> 4) * 8]), a0, a1, a2, a3);
+#pragma unroll
+      for (int nb = 0; nb < EN / 16; nb++) {
+        uint32_t b0, b1, b2, b3;
+        ldsm_x4(smem_addr(&Ws[buf][(nb * 16 + (lane & 7) + ((lane >> 4) << 3)) * LE_LD + kk * 16 + ((lane >> 3) & 1) * 8]), b0, b1, b2, b3);
+        mma16816(acc[2 * nb], a0, a1, a2, a3, b0, b1);
+        mma16816(acc[2 * nb + 1], a0, a1, a2, a3, b2, b3);
+      }
+    }
+    __syncthreads();
+  }
+  const int g = lane >> 2, t2 = (lane & 3) * 2;
+#pragma unroll
+  for (int hf = 0; hf < 2; hf++) {
+    const int row = m0 + warp * 16 + g + 8 * hf;
+    if (row >= a.T) continue;
+    const float* gt = a.out_gate + ((size_t)row * a.H + head) * a.vdim + e0;
+    bf16* op = out + (size_t)row * o_ld + (size_t)head * a.vdim + e0;
+#pragma unroll
+    for (int i = 0; i < EN / 8; i++) {
+      const int c = i * 8 + t2;
+      if (c < ne) {  // ne is a multiple of 8
+        const float2 gv = *reinterpret_cast<const float2*>(gt + c);
+        *reinterpret_cast<uint32_t*>(op + c) = pack_bf16(acc[i][2 * hf] * gv.x, acc[i][2 * hf + 1] * gv.y);
+      }
+    }
+    if (head == a.H - 1 && blockIdx.z == 0)
+      for (int c = a.H * a.vdim + (lane & 3); c < o_ld; c += 4) out[(size_t)row * o_ld + c] = __float2bfloat16_rn(0.f);
+  }
+  TRACE_EXIT(tr);
+}
+
+cudaError_t launch_latent_expand(cudaStream_t st, int qdt, const LatentArgs& a, const void* w_uv, void* out, int o_ld) {
+  if (a.T <= 0) return cudaSuccess;
+  if (!a.out_gate) return cudaErrorInvalidValue;
+  const size_t smem = (size_t)a.R * sizeof(float);
+  if (qdt == DT_BF16 && a.T > 8 && (a.R % 16) == 0 && (a.vdim % 8) == 0 && (a.o_ld % 8) == 0) {
+    // narrow column ranges while the rows alone do not fill the GPU
+    const long ctas = (long)ceil_div(a.T, LE_M) * a.H;
+    if (a.vdim > 64 && ctas >= 2L * a.sm_count)
+      (void)launch_k(latent_expand_mma_kernel<128, 32>, dim3(ceil_div(a.T, LE_M), a.H, ceil_div(a.vdim, 128)), dim3(128), 0, st, a,
+                     (const bf16*)w_uv, (bf16*)out, o_ld, next_trace(24));
+    else if (a.vdim > 32 && ctas >= a.sm_count)
+      (void)launch_k(latent_expand_mma_kernel<64, 64>, dim3(ceil_div(a.T, LE_M), a.H, ceil_div(a.vdim, 64)), dim3(128), 0, st, a,
+                     (const bf16*)w_uv, (bf16*)out, o_ld, next_trace(24));
+    else
+      (void)launch_k(latent_expand_mma_kernel<32, 64>, dim3(ceil_div(a.T, LE_M), a.H, ceil_div(a.vdim, 32)), dim3(128), 0, st, a,
+                     (const bf16*)w_uv, (bf16*)out, o_ld, next_trace(24));
+  } else if (qdt == DT_BF16) {
+    (void)launch_k(latent_expand_kernel<bf16>, dim3(a.T, a.H), dim3(256), smem, st, a, (const bf16*)w_uv, (bf16*)out, o_ld,
+                   next_trace(24));
+  } else {
+    (void)launch_k(latent_expand_kernel<float>, dim3(a.T, a.H), dim3(256), smem, st, a, (const float*)w_uv, (float*)out, o_ld,
+                   next_trace(24));
+  }
+  return cudaGetLastError();
 }
 
 int latent_attn_qtile() { return LAT_QTILE; }
@@ -724,19 +937,19 @@ cudaError_t launch_latent_attn(cudaStream_t st, int qdt, int kvdt, const LatentA
     cudaError_t e = a.R <= 64 ? launch_latent_mma<8>(st, a, ns)
                     : a.R <= 128 ? launch_latent_mma<16>(st, a, ns) : launch_latent_mma<32>(st, a, ns);
     if (e != cudaSuccess) return e;
-    if (ns > 1) (void)launch_k(latent_combine_kernel<bf16>, dim3(a.T * a.H), dim3(64), 0, st, a, ns, next_trace(23));
+    if (ns > 1) launch_latent_combine<bf16>(st, a, ns);
     return cudaGetLastError();
   }
   if (qdt == DT_F32 && kvdt == DT_F32) {
     if (smem > 48 * 1024)
       cudaFuncSetAttribute(latent_attn_kernel<float, float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     (void)launch_k(latent_attn_kernel<float, float>, grid, dim3(LAT_WARPS * 32), smem, st, a, next_trace(22));
-    if (ns > 1) (void)launch_k(latent_combine_kernel<float>, dim3(a.T * a.H), dim3(64), 0, st, a, ns, next_trace(23));
+    if (ns > 1) launch_latent_combine<float>(st, a, ns);
   } else if (qdt == DT_BF16 && kvdt == DT_BF16) {
     if (smem > 48 * 1024)
       cudaFuncSetAttribute(latent_attn_kernel<bf16, bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     (void)launch_k(latent_attn_kernel<bf16, bf16>, grid, dim3(LAT_WARPS * 32), smem, st, a, next_trace(22));
-    if (ns > 1) (void)launch_k(latent_combine_kernel<bf16>, dim3(a.T * a.H), dim3(64), 0, st, a, ns, next_trace(23));
+    if (ns > 1) launch_latent_combine<bf16>(st, a, ns);
   } else {
     return cudaErrorInvalidValue;
   }

@@ -9,7 +9,10 @@
 // Options of the same kernels (WinAttnArgs): chunk > 0 replaces the window by a chunked mask — i sees
 // j <= i with i / chunk == j / chunk, chunks counted from position 0 of the sequence —, softcap > 0
 // caps the score, s <- softcap * tanh(s / softcap), before the mask, and gate multiplies the
-// normalised output element by element.  Both masks give every query a contiguous key range
+// normalised output element by element.  maps = 2: every head has two score maps (two queries and two keys of `dim`
+// entries, side by side) over the same values, and its output is N(o_1 - lambda o_2) times a constant, N dividing the
+// head's vdim entries by their root mean square (differential attention); the fp32 states of both maps meet inside
+// the attention kernels.  Both masks give every query a contiguous key range
 // [first_key(i), i] whose start does not decrease with i, which is all the tile logic relies on.
 //
 //  * winattn_prep_kernel: epilogue of the fused projection [Q | K | V] — split-K sum, the
@@ -62,6 +65,10 @@ __device__ __forceinline__ float head_slope(const WinAttnArgs& a, int head) {
 }
 // score of the sink (a term of the softmax denominator without a key or a value): 0 or learned per head
 __device__ __forceinline__ float sink_score(const WinAttnArgs& a, int head) { return a.sink_w ? a.sink_w[head] : 0.f; }
+// two maps: what the entries of map 1 - lambda map 2 are multiplied by, given their sum of squares
+__device__ __forceinline__ float diff_factor(const WinAttnArgs& a, float ss) {
+  return a.out_mul / sqrtf(ss / (float)a.vdim + a.eps);
+}
 __device__ __forceinline__ const float* gate_row(const WinAttnArgs& a, size_t row, int head, int vdim) {
   return a.gate ? a.gate + row * a.gate_ld + (a.gate_head ? head : head * vdim) : nullptr;
 }
@@ -80,7 +87,8 @@ __global__ void __launch_bounds__(256) winattn_prep_kernel(WinAttnArgs a, Trace 
   pdl_wait();
   const int t = blockIdx.x;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
-  const int n_qkv = a.H + (a.own_kv ? 2 * a.G : 0);
+  const int maps = max(1, a.maps), HQ = a.H * maps, GK = a.G * maps;  // query / key vectors of the row
+  const int n_qkv = HQ + (a.own_kv ? GK + a.G : 0);
   const int n_items = n_qkv + (a.gate_out ? 1 : 0);
   const float* row = a.in_p + (size_t)t * a.in_ld;
   const int slot = a.slots[t];
@@ -95,15 +103,15 @@ __global__ void __launch_bounds__(256) winattn_prep_kernel(WinAttnArgs a, Trace 
   const float lam = a.vmix ? a.vmix[0] : 0.f;
   for (int it = blockIdx.y * nw + warp; it < n_items; it += gridDim.y * nw) {
     if (it == n_qkv) {  // the heads' gates: sigmoid of the H columns after Q | K | V
-      const float* gp = row + (a.H + (a.own_kv ? a.G : 0)) * a.dim + (a.own_kv ? a.G : 0) * a.vdim;
+      const float* gp = row + (HQ + (a.own_kv ? GK : 0)) * a.dim + (a.own_kv ? a.G : 0) * a.vdim;
       for (int i = lane; i < a.H; i += 32)
         a.gate_out[(size_t)t * a.H + i] = 1.0f / (1.0f + expf(-sum_slices(gp + i, a.in_S, a.in_stride)));
       continue;
     }
     int col, n, kind;  // 0 = query, 1 = key, 2 = value
-    if (it < a.H) { kind = 0; n = a.dim; col = it * a.dim; }
-    else if (it < a.H + a.G) { kind = 1; n = a.dim; col = a.H * a.dim + (it - a.H) * a.dim; }
-    else { kind = 2; n = a.vdim; col = (a.H + a.G) * a.dim + (it - a.H - a.G) * a.vdim; }
+    if (it < HQ) { kind = 0; n = a.dim; col = it * a.dim; }
+    else if (it < HQ + GK) { kind = 1; n = a.dim; col = it * a.dim; }
+    else { kind = 2; n = a.vdim; col = (HQ + GK) * a.dim + (it - HQ - GK) * a.vdim; }
     // the rotation of (i, i + rot_half) pairs reaches across lanes: those heads take the second path
     const bool in_regs = n <= 32 * WP_MAXV && !(rot > 0 && !a.rot_pairs && kind != 2);
     float v[WP_MAXV];
@@ -131,12 +139,12 @@ __global__ void __launch_bounds__(256) winattn_prep_kernel(WinAttnArgs a, Trace 
     if (kind != 2 && a.qk_norm) inv = 1.0f / sqrtf(warp_sum(ss) / (float)n + a.eps);
     if (kind == 0) inv *= qmul * (a.head_scale ? a.head_scale[it] : 1.f);
     const float* nw_ = (kind == 2 || a.qk_norm != 3) ? nullptr : (kind == 0 ? a.qnorm_w : a.knorm_w);
-    float* vf = (kind == 2 && a.vfirst) ? a.vfirst + (size_t)t * a.G * a.vdim + (size_t)(it - a.H - a.G) * a.vdim : nullptr;
+    float* vf = (kind == 2 && a.vfirst) ? a.vfirst + (size_t)t * a.G * a.vdim + (size_t)(it - HQ - GK) * a.vdim : nullptr;
     QT* qd = nullptr;
     KT* kd = nullptr;
-    if (kind == 0) qd = (QT*)a.q + (size_t)t * a.H * a.dim + col;
-    else if (kind == 1) kd = (KT*)a.kpool + (((size_t)blk * a.G + (it - a.H)) * KV_BLOCK + off) * a.dim;
-    else kd = (KT*)a.vpool + (((size_t)blk * a.G + (it - a.H - a.G)) * KV_BLOCK + off) * a.vdim;
+    if (kind == 0) qd = (QT*)a.q + (size_t)t * HQ * a.dim + col;
+    else if (kind == 1) kd = (KT*)a.kpool + ((((size_t)blk * a.G + (it - HQ) / maps) * KV_BLOCK + off) * maps + (it - HQ) % maps) * a.dim;
+    else kd = (KT*)a.vpool + (((size_t)blk * a.G + (it - HQ - GK)) * KV_BLOCK + off) * a.vdim;
     if (in_regs) {
 #pragma unroll
       for (int c = 0; c < WP_MAXV; c++) {
@@ -185,7 +193,8 @@ cudaError_t launch_winattn_prep(cudaStream_t st, int qdt, int kvdt, const WinAtt
   if (a.T <= 0) return cudaSuccess;
   if (2 * a.rot_half > a.dim || (a.vfirst && !a.own_kv)) return cudaErrorInvalidValue;
   // few rows (decode): the heads of a row spread over several CTAs
-  const int n_items = a.H + (a.own_kv ? 2 * a.G : 0) + (a.gate_out ? 1 : 0);
+  const int maps = std::max(1, a.maps);
+  const int n_items = a.H * maps + (a.own_kv ? a.G * (maps + 1) : 0) + (a.gate_out ? 1 : 0);
   const int ny = a.T >= 1024 ? 1 : ceil_div(n_items, 8);
   const dim3 grid(a.T, ny);
   const int big = std::max(a.dim, a.vdim);
@@ -354,7 +363,7 @@ cudaError_t launch_winattn_prep_conv(cudaStream_t st, int qdt, int kvdt, const W
 constexpr int WA_KT = 32;  // keys per tile (divides KV_BLOCK)
 constexpr int WA_QS = 16;  // queries per sub-tile: 8 warps x 2
 
-template <typename QT, typename KT, int VPL>
+template <typename QT, typename KT, int VPL, int MAPS>
 __global__ void __launch_bounds__(256) winattn_kernel(WinAttnArgs a, Trace tr) {
   TRACE_ENTRY(tr);
   pdl_launch_dependents();
@@ -388,91 +397,118 @@ __global__ void __launch_bounds__(256) winattn_kernel(WinAttnArgs a, Trace tr) {
 
   for (int qb = 0; qb < nq; qb += WA_QS) {
     const int nqs = min(WA_QS, nq - qb);
-    __syncthreads();  // the previous sub-tile's Qs / Ks / Vs have been consumed
-    for (int i = threadIdx.x; i < nqs * dim; i += blockDim.x) {
-      const int qi = i / dim, d = i % dim;
-      Qs[i] = to_f32(((const QT*)a.q)[(size_t)(row0 + qb + qi) * a.H * dim + head * dim + d]) * a.scale;
-    }
-    float m[2], l[2], acc[2][VPL];
+    float first[2][MAPS > 1 ? VPL : 1];  // two maps: the first one's normalised output
 #pragma unroll
-    for (int qq = 0; qq < 2; qq++) {
-      m[qq] = m0;
-      l[qq] = l0;
-#pragma unroll
-      for (int c = 0; c < VPL; c++) acc[qq][c] = 0.f;
-    }
-    const int p_first = qpos0 + qb, p_last = qpos0 + qb + nqs - 1;
-    int k_lo = first_key(a, p_first);
-    k_lo = k_lo / WA_KT * WA_KT;
-    const int k_hi = p_last + 1;
-    for (int k0 = k_lo; k0 < k_hi; k0 += WA_KT) {
-      const int nk = min(WA_KT, k_hi - k0);
-      const int blk = bt[k0 / KV_BLOCK];
-      const size_t kb = (((size_t)blk * a.G + g) * KV_BLOCK + (k0 % KV_BLOCK));
-      __syncthreads();
-      for (int i = threadIdx.x; i < nk * dim; i += blockDim.x) {
-        const int r = i / dim, d = i % dim;
-        Ks[r * kld + d] = to_f32(kpool[(kb + r) * dim + d]);
+    for (int map = 0; map < MAPS; map++) {
+      __syncthreads();  // the previous pass's Qs / Ks / Vs have been consumed
+      for (int i = threadIdx.x; i < nqs * dim; i += blockDim.x) {
+        const int qi = i / dim, d = i % dim;
+        Qs[i] = to_f32(((const QT*)a.q)[((size_t)(row0 + qb + qi) * a.H + head) * MAPS * dim + map * dim + d]) * a.scale;
       }
-      for (int i = threadIdx.x; i < nk * vdim; i += blockDim.x) Vs[i] = to_f32(vpool[kb * vdim + i]);
-      __syncthreads();
+      float m[2], l[2], acc[2][VPL];
+#pragma unroll
+      for (int qq = 0; qq < 2; qq++) {
+        m[qq] = m0;
+        l[qq] = l0;
+#pragma unroll
+        for (int c = 0; c < VPL; c++) acc[qq][c] = 0.f;
+      }
+      const int p_first = qpos0 + qb, p_last = qpos0 + qb + nqs - 1;
+      int k_lo = first_key(a, p_first);
+      k_lo = k_lo / WA_KT * WA_KT;
+      const int k_hi = p_last + 1;
+      for (int k0 = k_lo; k0 < k_hi; k0 += WA_KT) {
+        const int nk = min(WA_KT, k_hi - k0);
+        const int blk = bt[k0 / KV_BLOCK];
+        const size_t kb = (((size_t)blk * a.G + g) * KV_BLOCK + (k0 % KV_BLOCK));
+        __syncthreads();
+        for (int i = threadIdx.x; i < nk * dim; i += blockDim.x) {
+          const int r = i / dim, d = i % dim;
+          Ks[r * kld + d] = to_f32(kpool[((kb + r) * MAPS + map) * dim + d]);
+        }
+        for (int i = threadIdx.x; i < nk * vdim; i += blockDim.x) Vs[i] = to_f32(vpool[kb * vdim + i]);
+        __syncthreads();
+#pragma unroll
+        for (int qq = 0; qq < 2; qq++) {
+          const int qi = warp + 8 * qq;
+          if (qi >= nqs) continue;  // warp-uniform
+          const int qp = p_first + qi;
+          const int j = k0 + lane;
+          const bool vis = lane < nk && j <= qp && j >= first_key(a, qp);
+          float s = -INFINITY;
+          if (vis) {
+            const float* qr = Qs + qi * dim;
+            const float* kr = Ks + lane * kld;
+            float d = 0.f;
+            for (int i = 0; i < dim; i++) d = fmaf(qr[i], kr[i], d);
+            s = a.softcap > 0.f ? cap_score<sizeof(QT) == 2>(d, a.softcap) : d;
+            s -= slope * (float)(qp - j);
+          }
+          const float cmax = warp_max(s);
+          if (cmax == -INFINITY) continue;  // no key of this tile is visible to the query
+          const float mn = fmaxf(m[qq], cmax);
+          const float corr = (m[qq] == -INFINITY) ? 0.f : expf(m[qq] - mn);
+          const float p = vis ? expf(s - mn) : 0.f;
+          l[qq] = l[qq] * corr + warp_sum(p);
+#pragma unroll
+          for (int c = 0; c < VPL; c++) acc[qq][c] *= corr;
+          for (int jj = 0; jj < nk; jj++) {
+            const float pj = __shfl_sync(0xffffffffu, p, jj);
+            if (pj == 0.f) continue;  // warp-uniform
+            const float* vr = Vs + jj * vdim;
+#pragma unroll
+            for (int c = 0; c < VPL; c++) {
+              const int col = lane + 32 * c;
+              if (col < vdim) acc[qq][c] = fmaf(pj, vr[col], acc[qq][c]);
+            }
+          }
+          m[qq] = mn;
+        }
+      }
 #pragma unroll
       for (int qq = 0; qq < 2; qq++) {
         const int qi = warp + 8 * qq;
-        if (qi >= nqs) continue;  // warp-uniform
-        const int qp = p_first + qi;
-        const int j = k0 + lane;
-        const bool vis = lane < nk && j <= qp && j >= first_key(a, qp);
-        float s = -INFINITY;
-        if (vis) {
-          const float* qr = Qs + qi * dim;
-          const float* kr = Ks + lane * kld;
-          float d = 0.f;
-          for (int i = 0; i < dim; i++) d = fmaf(qr[i], kr[i], d);
-          s = a.softcap > 0.f ? cap_score<sizeof(QT) == 2>(d, a.softcap) : d;
-          s -= slope * (float)(qp - j);
-        }
-        const float cmax = warp_max(s);
-        if (cmax == -INFINITY) continue;  // no key of this tile is visible to the query
-        const float mn = fmaxf(m[qq], cmax);
-        const float corr = (m[qq] == -INFINITY) ? 0.f : expf(m[qq] - mn);
-        const float p = vis ? expf(s - mn) : 0.f;
-        l[qq] = l[qq] * corr + warp_sum(p);
+        if (qi >= nqs) continue;
+        const float inv = 1.0f / l[qq];
+        if (MAPS > 1) {
+          if (map == 0) {
 #pragma unroll
-        for (int c = 0; c < VPL; c++) acc[qq][c] *= corr;
-        for (int jj = 0; jj < nk; jj++) {
-          const float pj = __shfl_sync(0xffffffffu, p, jj);
-          if (pj == 0.f) continue;  // warp-uniform
-          const float* vr = Vs + jj * vdim;
+            for (int c = 0; c < VPL; c++) first[qq][c] = acc[qq][c] * inv;
+            continue;
+          }
+          float ss = 0.f;
+#pragma unroll
+          for (int c = 0; c < VPL; c++) {  // (columns past vdim are zero in both)
+            acc[qq][c] = first[qq][c] - a.diff_lambda * (acc[qq][c] * inv);
+            ss += acc[qq][c] * acc[qq][c];
+          }
+          const float f = diff_factor(a, warp_sum(ss));
+          QT* op = (QT*)a.out + (size_t)(row0 + qb + qi) * a.o_ld;
 #pragma unroll
           for (int c = 0; c < VPL; c++) {
             const int col = lane + 32 * c;
-            if (col < vdim) acc[qq][c] = fmaf(pj, vr[col], acc[qq][c]);
+            if (col < vdim) op[head * vdim + col] = from_f32<QT>(acc[qq][c] * f);
           }
+          if (head == 0)
+            for (int col = a.H * vdim + lane; col < a.o_ld; col += 32) op[col] = from_f32<QT>(0.f);
+          continue;
         }
-        m[qq] = mn;
-      }
-    }
+        QT* op = (QT*)a.out + (size_t)(row0 + qb + qi) * a.o_ld;
+        const float* gt = gate_row(a, (size_t)(row0 + qb + qi), head, vdim);
 #pragma unroll
-    for (int qq = 0; qq < 2; qq++) {
-      const int qi = warp + 8 * qq;
-      if (qi >= nqs) continue;
-      const float inv = 1.0f / l[qq];
-      QT* op = (QT*)a.out + (size_t)(row0 + qb + qi) * a.o_ld;
-      const float* gt = gate_row(a, (size_t)(row0 + qb + qi), head, vdim);
-#pragma unroll
-      for (int c = 0; c < VPL; c++) {
-        const int col = lane + 32 * c;
-        if (col < vdim) op[head * vdim + col] = from_f32<QT>(acc[qq][c] * inv * (gt ? gt[a.gate_head ? 0 : col] : 1.f));
+        for (int c = 0; c < VPL; c++) {
+          const int col = lane + 32 * c;
+          if (col < vdim) op[head * vdim + col] = from_f32<QT>(acc[qq][c] * inv * (gt ? gt[a.gate_head ? 0 : col] : 1.f));
+        }
+        if (head == 0)  // padding columns of the output projection's input stay zero
+          for (int col = a.H * vdim + lane; col < a.o_ld; col += 32) op[col] = from_f32<QT>(0.f);
       }
-      if (head == 0)  // padding columns of the output projection's input stay zero
-        for (int col = a.H * vdim + lane; col < a.o_ld; col += 32) op[col] = from_f32<QT>(0.f);
     }
   }
   TRACE_EXIT(tr);
 }
 
-template <typename QT, typename KT>
+template <typename QT, typename KT, int MAPS>
 static cudaError_t winattn_dispatch(cudaStream_t st, const WinAttnArgs& a) {
   const dim3 grid(a.n_tiles, a.H);
   const size_t smem = ((size_t)WA_QS * a.dim + (size_t)WA_KT * (a.dim | 1) + (size_t)WA_KT * a.vdim) * sizeof(float);
@@ -480,8 +516,8 @@ static cudaError_t winattn_dispatch(cudaStream_t st, const WinAttnArgs& a) {
 #define WA(V)                                                                                               \
   {                                                                                                         \
     if (smem > 48 * 1024)                                                                                   \
-      cudaFuncSetAttribute(winattn_kernel<QT, KT, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
-    (void)launch_k(winattn_kernel<QT, KT, V>, grid, dim3(256), smem, st, a, next_trace(31));                \
+      cudaFuncSetAttribute(winattn_kernel<QT, KT, V, MAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+    (void)launch_k(winattn_kernel<QT, KT, V, MAPS>, grid, dim3(256), smem, st, a, next_trace(31));                \
   }
   if (vpl <= 1) WA(1)
   else if (vpl <= 2) WA(2)
@@ -499,15 +535,16 @@ static cudaError_t winattn_dispatch(cudaStream_t st, const WinAttnArgs& a) {
 // its own key (a cached row is contiguous), the chunk's probabilities are then broadcast lane
 // by lane for the weighted sum over the value rows (coalesced); the four partial states meet in
 // shared memory, where the sink joins once.
-template <typename QT, typename KT, int VPL>
+template <typename QT, typename KT, int VPL, int MAPS>
 __global__ void __launch_bounds__(128) winattn_decode_kernel(WinAttnArgs a, Trace tr) {
   TRACE_ENTRY(tr);
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ float smem[];
   const int dim = a.dim, vdim = a.vdim;
-  float* qs = smem;             // [dim], scaled
-  float* part = smem + dim;     // [4][vdim + 2]
+  float* qs = smem;                    // [MAPS][dim], scaled
+  float* part = smem + MAPS * dim;     // [4][MAPS][vdim + 2]
+  __shared__ float red[32];
   const int seq = blockIdx.x, head = blockIdx.y;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int g = head / (a.H / a.G);
@@ -517,53 +554,105 @@ __global__ void __launch_bounds__(128) winattn_decode_kernel(WinAttnArgs a, Trac
   const int* bt = a.block_tables + (size_t)seq * a.max_blocks;
   const KT* kpool = (const KT*)a.kpool;
   const KT* vpool = (const KT*)a.vpool;
-  for (int i = threadIdx.x; i < dim; i += blockDim.x)
-    qs[i] = to_f32(((const QT*)a.q)[(size_t)seq * a.H * dim + head * dim + i]) * a.scale;
+  for (int i = threadIdx.x; i < MAPS * dim; i += blockDim.x)
+    qs[i] = to_f32(((const QT*)a.q)[((size_t)seq * a.H + head) * MAPS * dim + i]) * a.scale;
   __syncthreads();
-  float m = -INFINITY, l = 0.f, acc[VPL];
+  float m[MAPS], l[MAPS], acc[MAPS][VPL];
 #pragma unroll
-  for (int c = 0; c < VPL; c++) acc[c] = 0.f;
+  for (int u = 0; u < MAPS; u++) {
+    m[u] = -INFINITY;
+    l[u] = 0.f;
+#pragma unroll
+    for (int c = 0; c < VPL; c++) acc[u][c] = 0.f;
+  }
   for (int k0 = k_lo + warp * 32; k0 <= qp; k0 += 4 * 32) {
     const int j = k0 + lane;
     const bool vis = j <= qp;
-    float s = -INFINITY;
-    if (vis) {
-      const KT* kr = kpool + (((size_t)bt[j / KV_BLOCK] * a.G + g) * KV_BLOCK + (j % KV_BLOCK)) * dim;
-      float d = 0.f;
-      for (int i = 0; i < dim; i++) d = fmaf(qs[i], to_f32(kr[i]), d);
-      s = a.softcap > 0.f ? cap_score<sizeof(QT) == 2>(d, a.softcap) : d;
-      s -= slope * (float)(qp - j);
-    }
-    const float mn = fmaxf(m, warp_max(s));  // lane 0 of the chunk is always visible
-    const float corr = (m == -INFINITY) ? 0.f : expf(m - mn);
-    const float p = vis ? expf(s - mn) : 0.f;
-    l = l * corr + warp_sum(p);
+    float p[MAPS];
 #pragma unroll
-    for (int c = 0; c < VPL; c++) acc[c] *= corr;
+    for (int u = 0; u < MAPS; u++) {
+      float s = -INFINITY;
+      if (vis) {
+        const KT* kr = kpool + ((((size_t)bt[j / KV_BLOCK] * a.G + g) * KV_BLOCK + (j % KV_BLOCK)) * MAPS + u) * dim;
+        float d = 0.f;
+        for (int i = 0; i < dim; i++) d = fmaf(qs[u * dim + i], to_f32(kr[i]), d);
+        s = a.softcap > 0.f ? cap_score<sizeof(QT) == 2>(d, a.softcap) : d;
+        s -= slope * (float)(qp - j);
+      }
+      const float mn = fmaxf(m[u], warp_max(s));  // lane 0 of the chunk is always visible
+      const float corr = (m[u] == -INFINITY) ? 0.f : expf(m[u] - mn);
+      p[u] = vis ? expf(s - mn) : 0.f;
+      l[u] = l[u] * corr + warp_sum(p[u]);
+#pragma unroll
+      for (int c = 0; c < VPL; c++) acc[u][c] *= corr;
+      m[u] = mn;
+    }
     const int nk = min(32, qp + 1 - k0);
     for (int jj = 0; jj < nk; jj++) {
-      const float pj = __shfl_sync(0xffffffffu, p, jj);
+      float pj[MAPS];
+#pragma unroll
+      for (int u = 0; u < MAPS; u++) pj[u] = __shfl_sync(0xffffffffu, p[u], jj);
       const int jp = k0 + jj;
       const KT* vr = vpool + (((size_t)bt[jp / KV_BLOCK] * a.G + g) * KV_BLOCK + (jp % KV_BLOCK)) * vdim;
 #pragma unroll
       for (int c = 0; c < VPL; c++) {
         const int col = lane + 32 * c;
-        if (col < vdim) acc[c] = fmaf(pj, to_f32(vr[col]), acc[c]);
+        if (col < vdim) {
+          const float v = to_f32(vr[col]);
+#pragma unroll
+          for (int u = 0; u < MAPS; u++) acc[u][c] = fmaf(pj[u], v, acc[u][c]);
+        }
       }
     }
-    m = mn;
   }
-  float* mine = part + warp * (vdim + 2);
 #pragma unroll
-  for (int c = 0; c < VPL; c++) {
-    const int col = lane + 32 * c;
-    if (col < vdim) mine[col] = acc[c];
-  }
-  if (lane == 0) {
-    mine[vdim] = m;
-    mine[vdim + 1] = l;
+  for (int u = 0; u < MAPS; u++) {
+    float* mine = part + (warp * MAPS + u) * (vdim + 2);
+#pragma unroll
+    for (int c = 0; c < VPL; c++) {
+      const int col = lane + 32 * c;
+      if (col < vdim) mine[col] = acc[u][c];
+    }
+    if (lane == 0) {
+      mine[vdim] = m[u];
+      mine[vdim + 1] = l[u];
+    }
   }
   __syncthreads();
+  if (MAPS > 1) {  // (no sink, no gate)
+    constexpr int NC = VPL > 4 ? VPL / 4 : 1;  // columns per thread
+    float v[NC], ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < NC; e++) {
+      const int col = threadIdx.x + 128 * e;
+      v[e] = 0.f;
+      if (col < vdim)
+#pragma unroll
+        for (int u = 0; u < MAPS; u++) {
+          float mt = -INFINITY, lt = 0.f, o = 0.f;
+          for (int w = 0; w < 4; w++) mt = fmaxf(mt, part[(w * MAPS + u) * (vdim + 2) + vdim]);
+          for (int w = 0; w < 4; w++) {
+            const float* pw = part + (w * MAPS + u) * (vdim + 2);
+            const float cw = (pw[vdim] == -INFINITY) ? 0.f : expf(pw[vdim] - mt);
+            lt += pw[vdim + 1] * cw;
+            o += pw[col] * cw;
+          }
+          v[e] += (u ? -a.diff_lambda : 1.f) * (o / lt);
+        }
+      ss += v[e] * v[e];
+    }
+    const float f = diff_factor(a, block_sum(ss, red));
+    QT* op = (QT*)a.out + (size_t)seq * a.o_ld;
+#pragma unroll
+    for (int e = 0; e < NC; e++) {
+      const int col = threadIdx.x + 128 * e;
+      if (col < vdim) op[head * vdim + col] = from_f32<QT>(v[e] * f);
+    }
+    if (head == 0)
+      for (int col = a.H * vdim + threadIdx.x; col < a.o_ld; col += blockDim.x) op[col] = from_f32<QT>(0.f);
+    TRACE_EXIT(tr);
+    return;
+  }
   const float sk = sink_score(a, head);
   float mt = a.sink ? sk : -INFINITY;
   for (int w = 0; w < 4; w++) mt = fmaxf(mt, part[w * (vdim + 2) + vdim]);
@@ -623,9 +712,12 @@ __global__ void __launch_bounds__(256, (GQMAX * VPT <= 16) ? 2 : 1) winattn_deco
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) float smem[];
-  const int dim = a.dim, vdim = 32 * VPT;
+  // two maps: a head is two neighbouring queries against the whole cached row [map 1 | map 2], each with zeros where
+  // the other map's entries are (both sit in one chunk: GQMAX is even)
+  const int maps = max(1, a.maps), qdim = a.dim;
+  const int dim = qdim * maps, vdim = 32 * VPT;
   const int seq = blockIdx.x, g = blockIdx.y;
-  const int GQ = a.H / a.G;
+  const int GQ = a.H / a.G * maps;
   const int gq0 = blockIdx.z * GQMAX;         // first query head of the chunk within the group
   const int gqn = min(GQMAX, GQ - gq0);
   const int h0 = g * GQ + gq0;
@@ -637,8 +729,11 @@ __global__ void __launch_bounds__(256, (GQMAX * VPT <= 16) ? 2 : 1) winattn_deco
   const int* bt = a.block_tables + (size_t)seq * a.max_blocks;
   const KT* kpool = (const KT*)a.kpool;
   const KT* vpool = (const KT*)a.vpool;
-  for (int i = threadIdx.x; i < gqn * dim; i += blockDim.x)
-    qs[i] = to_f32(((const QT*)a.q)[(size_t)seq * a.H * dim + (size_t)(h0 + i / dim) * dim + i % dim]) * a.scale;
+  for (int i = threadIdx.x; i < gqn * dim; i += blockDim.x) {
+    const int q = h0 + i / dim, d = i % dim;
+    const bool own = maps == 1 || d / qdim == q % maps;
+    qs[i] = own ? to_f32(((const QT*)a.q)[((size_t)seq * a.H * maps + q) * qdim + d % qdim]) * a.scale : 0.f;
+  }
   __syncthreads();
   float m[GQMAX], l[GQMAX], acc[GQMAX][VPT];
 #pragma unroll
@@ -729,6 +824,36 @@ __global__ void __launch_bounds__(256, (GQMAX * VPT <= 16) ? 2 : 1) winattn_deco
     }
   }
   __syncthreads();
+  if (maps > 1) {  // a warp per head: both maps' outputs, their difference, its norm (no sink, no gate)
+    for (int hq = warp; hq < gqn / 2; hq += WD_WARPS) {
+      float v[VPT], ss = 0.f;
+#pragma unroll
+      for (int c = 0; c < VPT; c++) v[c] = 0.f;
+#pragma unroll
+      for (int u = 0; u < 2; u++) {
+        float mt = -INFINITY, lt = 0.f, o[VPT];
+#pragma unroll
+        for (int c = 0; c < VPT; c++) o[c] = 0.f;
+        for (int w = 0; w < WD_WARPS; w++) mt = fmaxf(mt, part[((size_t)w * GQMAX + 2 * hq + u) * ps + vdim]);
+        for (int w = 0; w < WD_WARPS; w++) {
+          const float* pw = part + ((size_t)w * GQMAX + 2 * hq + u) * ps;
+          const float cw = (pw[vdim] == -INFINITY) ? 0.f : expf(pw[vdim] - mt);
+          lt += pw[vdim + 1] * cw;
+#pragma unroll
+          for (int c = 0; c < VPT; c++) o[c] += pw[lane + 32 * c] * cw;
+        }
+        const float f = (u ? -a.diff_lambda : 1.f) / lt;
+#pragma unroll
+        for (int c = 0; c < VPT; c++) v[c] = fmaf(o[c], f, v[c]);
+      }
+#pragma unroll
+      for (int c = 0; c < VPT; c++) ss += v[c] * v[c];
+      const float f = diff_factor(a, warp_sum(ss));
+      QT* op = (QT*)a.out + (size_t)seq * a.o_ld + (size_t)(h0 / 2 + hq) * vdim;
+#pragma unroll
+      for (int c = 0; c < VPT; c++) op[lane + 32 * c] = from_f32<QT>(v[c] * f);
+    }
+  } else
   for (int i = threadIdx.x; i < gqn * vdim; i += blockDim.x) {
     const int q = i / vdim, col = i % vdim;
     const float sk = sink_score(a, h0 + q);
@@ -752,10 +877,10 @@ __global__ void __launch_bounds__(256, (GQMAX * VPT <= 16) ? 2 : 1) winattn_deco
 
 template <typename QT, typename KT, int VPT>
 static cudaError_t winattn_decode_group_vpt(cudaStream_t st, const WinAttnArgs& a) {
-  const int GQ = a.H / a.G;
+  const int maps = std::max(1, a.maps), GQ = a.H / a.G * maps;
   const int gmax = GQ <= 1 ? 1 : GQ <= 2 ? 2 : GQ <= 4 ? 4 : 8;
   const dim3 grid(a.n_tiles, a.G, ceil_div(GQ, gmax));
-  const size_t smem = ((size_t)gmax * a.dim + WD_WARPS * (size_t)gmax * (a.vdim + 2)) * sizeof(float);
+  const size_t smem = ((size_t)gmax * a.dim * maps + WD_WARPS * (size_t)gmax * (a.vdim + 2)) * sizeof(float);
   if (smem > 48 * 1024) return cudaErrorInvalidValue;
   if (gmax == 1) (void)launch_k(winattn_decode_group_kernel<QT, KT, VPT, 1>, grid, dim3(32 * WD_WARPS), smem, st, a, next_trace(33));
   else if (gmax == 2) (void)launch_k(winattn_decode_group_kernel<QT, KT, VPT, 2>, grid, dim3(32 * WD_WARPS), smem, st, a, next_trace(33));
@@ -769,9 +894,10 @@ static bool winattn_decode_group_ok(const WinAttnArgs& a) {
     return e ? atoi(e) != 0 : true;
   }();
   const int vpt = a.vdim / 32;
-  const int gmax = std::min(8, a.H / a.G);
+  const int maps = std::max(1, a.maps), GQ = a.H / a.G * maps;
+  const int gmax = GQ <= 1 ? 1 : GQ <= 2 ? 2 : GQ <= 4 ? 4 : 8;
   return on && a.dim % 8 == 0 && a.vdim % 32 == 0 && (vpt == 1 || vpt == 2 || vpt == 4 || vpt == 8) &&
-         ((size_t)gmax * a.dim + WD_WARPS * (size_t)gmax * (a.vdim + 2)) * sizeof(float) <= 48 * 1024;
+         ((size_t)gmax * a.dim * maps + WD_WARPS * (size_t)gmax * (a.vdim + 2)) * sizeof(float) <= 48 * 1024;
 }
 template <typename QT, typename KT>
 static cudaError_t winattn_decode_group(cudaStream_t st, const WinAttnArgs& a) {
@@ -783,12 +909,12 @@ static cudaError_t winattn_decode_group(cudaStream_t st, const WinAttnArgs& a) {
   }
 }
 
-template <typename QT, typename KT>
+template <typename QT, typename KT, int MAPS>
 static cudaError_t winattn_decode_dispatch(cudaStream_t st, const WinAttnArgs& a) {
   const dim3 grid(a.n_tiles, a.H);
-  const size_t smem = ((size_t)a.dim + 4 * ((size_t)a.vdim + 2)) * sizeof(float);
+  const size_t smem = MAPS * ((size_t)a.dim + 4 * ((size_t)a.vdim + 2)) * sizeof(float);
   const int vpl = ceil_div(a.vdim, 32);
-#define WD(V) (void)launch_k(winattn_decode_kernel<QT, KT, V>, grid, dim3(128), smem, st, a, next_trace(33));
+#define WD(V) (void)launch_k(winattn_decode_kernel<QT, KT, V, MAPS>, grid, dim3(128), smem, st, a, next_trace(33));
   if (smem > 48 * 1024) return cudaErrorInvalidValue;
   if (vpl <= 1) WD(1)
   else if (vpl <= 2) WD(2)
@@ -810,12 +936,13 @@ static cudaError_t winattn_decode_dispatch(cudaStream_t st, const WinAttnArgs& a
 // are never loaded; K / V of tile i + 1 arrive by cp.async while tile i is computed.
 constexpr int WM_Q = 64, WM_K = 64;
 
-template <int DIM, int VDIM>
+template <int DIM, int VDIM, int MAPS>
 __global__ void __launch_bounds__(128) winattn_mma_kernel(WinAttnArgs a, Trace tr) {
   TRACE_ENTRY(tr);
   pdl_launch_dependents();
   pdl_wait();
-  constexpr int DP = DIM + 8, VP = VDIM + 8;
+  constexpr int KD = DIM * MAPS;  // a cached key row: the maps side by side
+  constexpr int DP = KD + 8, VP = VDIM + 8;
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* Qs = reinterpret_cast<bf16*>(smem_raw);  // [64][DP]
   bf16* Ks = Qs + WM_Q * DP;                      // [2][64][DP]
@@ -838,13 +965,13 @@ __global__ void __launch_bounds__(128) winattn_mma_kernel(WinAttnArgs a, Trace t
   const int* bt = a.block_tables + (size_t)seq * a.max_blocks;
   const bf16* kpool = (const bf16*)a.kpool;
   const bf16* vpool = (const bf16*)a.vpool;
-  const bf16* qg = (const bf16*)a.q + (size_t)row0 * a.H * DIM + head * DIM;
+  const bf16* qg = (const bf16*)a.q + (size_t)row0 * a.H * KD + head * KD;
 
   // Q tile: rows past nq are zero
-  for (int i = threadIdx.x; i < WM_Q * (DIM / 8); i += blockDim.x) {
-    const int r = i / (DIM / 8), c = i % (DIM / 8);
+  for (int i = threadIdx.x; i < WM_Q * (KD / 8); i += blockDim.x) {
+    const int r = i / (KD / 8), c = i % (KD / 8);
     const bool ok = r < nq;
-    cp_async16(smem_addr(Qs + r * DP + c * 8), ok ? (const void*)(qg + (size_t)r * a.H * DIM + c * 8) : (const void*)qg, ok);
+    cp_async16(smem_addr(Qs + r * DP + c * 8), ok ? (const void*)(qg + (size_t)r * a.H * KD + c * 8) : (const void*)qg, ok);
   }
   int k_lo = first_key(a, qpos0);
   k_lo = k_lo / WM_K * WM_K;
@@ -857,10 +984,10 @@ __global__ void __launch_bounds__(128) winattn_mma_kernel(WinAttnArgs a, Trace t
     const size_t kb = (((size_t)blk * a.G + g) * KV_BLOCK + (k0 % KV_BLOCK));
     bf16* kd = Ks + buf * WM_K * DP;
     bf16* vd = Vs + buf * WM_K * VP;
-    for (int i = threadIdx.x; i < WM_K * (DIM / 8); i += blockDim.x) {
-      const int r = i / (DIM / 8), c = i % (DIM / 8);
+    for (int i = threadIdx.x; i < WM_K * (KD / 8); i += blockDim.x) {
+      const int r = i / (KD / 8), c = i % (KD / 8);
       const bool ok = r < nk;
-      cp_async16(smem_addr(kd + r * DP + c * 8), ok ? (const void*)(kpool + (kb + r) * DIM + c * 8) : (const void*)kpool, ok);
+      cp_async16(smem_addr(kd + r * DP + c * 8), ok ? (const void*)(kpool + (kb + r) * KD + c * 8) : (const void*)kpool, ok);
     }
     for (int i = threadIdx.x; i < WM_K * (VDIM / 8); i += blockDim.x) {
       const int r = i / (VDIM / 8), c = i % (VDIM / 8);
@@ -874,13 +1001,20 @@ __global__ void __launch_bounds__(128) winattn_mma_kernel(WinAttnArgs a, Trace t
   const int gid = lane >> 2, tig = lane & 3;
   const int r_lo = warp * 16 + gid, r_hi = r_lo + 8;     // the thread's two query rows in the tile
   const int qp_lo = qpos0 + r_lo, qp_hi = qpos0 + r_hi;  // their positions
-  float m_lo, m_hi, l_lo, l_hi;
-  m_lo = m_hi = a.sink ? sink_score(a, head) * 1.4426950408889634f : -INFINITY;  // base-2 domain, like the scores
-  l_lo = l_hi = a.sink ? 1.f : 0.f;
-  const float slope2 = head_slope(a, head) * 1.4426950408889634f;
-  float o[VDIM / 8][4];
+  float m_lo[MAPS], m_hi[MAPS], l_lo[MAPS], l_hi[MAPS];
+  m_lo[0] = m_hi[0] = a.sink ? sink_score(a, head) * 1.4426950408889634f : -INFINITY;  // base-2 domain, like the scores
+  l_lo[0] = l_hi[0] = a.sink ? 1.f : 0.f;
 #pragma unroll
-  for (int i = 0; i < VDIM / 8; i++) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  for (int u = 1; u < MAPS; u++) {
+    m_lo[u] = m_hi[u] = m_lo[0];
+    l_lo[u] = l_hi[u] = l_lo[0];
+  }
+  const float slope2 = head_slope(a, head) * 1.4426950408889634f;
+  float o[MAPS][VDIM / 8][4];
+#pragma unroll
+  for (int u = 0; u < MAPS; u++)
+#pragma unroll
+    for (int i = 0; i < VDIM / 8; i++) o[u][i][0] = o[u][i][1] = o[u][i][2] = o[u][i][3] = 0.f;
   const float sc = a.scale * 1.4426950408889634f;  // log2(e): softmax in base 2
 
   for (int kt = 0; kt < n_kt; kt++) {
@@ -896,113 +1030,136 @@ __global__ void __launch_bounds__(128) winattn_mma_kernel(WinAttnArgs a, Trace t
     const int w_qlo = qpos0 + warp * 16, w_qhi = w_qlo + 15;
     const bool warp_sees = warp * 16 < nq && k0 <= w_qhi && k0 + WM_K - 1 >= first_key(a, w_qlo);
     if (warp_sees) {
-      float s[WM_K / 8][4];
 #pragma unroll
-      for (int i = 0; i < WM_K / 8; i++) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
+      for (int u = 0; u < MAPS; u++) {
+        float s[WM_K / 8][4];
 #pragma unroll
-      for (int kk = 0; kk < DIM / 16; kk++) {
-        uint32_t a0, a1, a2, a3;
-        // A fragment (16 query rows x 16 dims): matrices (rows 0-7, k 0-7), (rows 8-15, k 0-7),
-        // (rows 0-7, k 8-15), (rows 8-15, k 8-15)
-        ldsm_x4(smem_addr(Qs + (warp * 16 + (lane & 15)) * DP + kk * 16 + (lane >> 4) * 8), a0, a1, a2, a3);
+        for (int i = 0; i < WM_K / 8; i++) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
 #pragma unroll
-        for (int nb = 0; nb < WM_K / 16; nb++) {
-          // B fragments of two 8-key blocks: K rows are the n index, dims the k index
-          uint32_t b0, b1, b2, b3;
-          ldsm_x4(smem_addr(kd + (nb * 16 + (lane & 7) + ((lane >> 4) << 3)) * DP + kk * 16 + ((lane >> 3) & 1) * 8),
-                  b0, b1, b2, b3);
-          mma16816(s[2 * nb], a0, a1, a2, a3, b0, b1);
-          mma16816(s[2 * nb + 1], a0, a1, a2, a3, b2, b3);
-        }
-      }
-      // scale (scores live in the base-2 domain: exp2 of a difference is one instruction), mask
-      // (only on tiles that some row of the warp sees partly), running max
-      const bool interior = k0 + WM_K - 1 <= w_qlo && k0 + WM_K <= k_hi && k0 >= first_key(a, w_qhi);
-      float mx_lo = -INFINITY, mx_hi = -INFINITY;
-      if (a.softcap > 0.f) {  // the cap works on the scaled score; back to the base-2 domain afterwards
+        for (int kk = 0; kk < DIM / 16; kk++) {
+          uint32_t a0, a1, a2, a3;
+          // A fragment (16 query rows x 16 dims): matrices (rows 0-7, k 0-7), (rows 8-15, k 0-7),
+          // (rows 0-7, k 8-15), (rows 8-15, k 8-15)
+          ldsm_x4(smem_addr(Qs + (warp * 16 + (lane & 15)) * DP + u * DIM + kk * 16 + (lane >> 4) * 8), a0, a1, a2, a3);
 #pragma unroll
-        for (int nb = 0; nb < WM_K / 8; nb++)
-#pragma unroll
-          for (int e = 0; e < 4; e++) s[nb][e] = cap_score<true>(s[nb][e] * a.scale, a.softcap) * (1.4426950408889634f / sc);
-      }
-      if (interior) {
-#pragma unroll
-        for (int nb = 0; nb < WM_K / 8; nb++) {
-          s[nb][0] *= sc; s[nb][1] *= sc; s[nb][2] *= sc; s[nb][3] *= sc;
-          if (slope2 != 0.f) {
-            const int j = k0 + nb * 8 + tig * 2;
-            s[nb][0] -= slope2 * (float)(qp_lo - j); s[nb][1] -= slope2 * (float)(qp_lo - j - 1);
-            s[nb][2] -= slope2 * (float)(qp_hi - j); s[nb][3] -= slope2 * (float)(qp_hi - j - 1);
-          }
-          mx_lo = fmaxf(mx_lo, fmaxf(s[nb][0], s[nb][1]));
-          mx_hi = fmaxf(mx_hi, fmaxf(s[nb][2], s[nb][3]));
-        }
-      } else {
-#pragma unroll
-        for (int nb = 0; nb < WM_K / 8; nb++) {
-#pragma unroll
-          for (int e = 0; e < 4; e++) {
-            const int j = k0 + nb * 8 + tig * 2 + (e & 1);
-            const int qp = (e & 2) ? qp_hi : qp_lo;
-            const bool vis = j <= qp && j < k_hi && j >= first_key(a, qp);
-            const float v = vis ? s[nb][e] * sc - slope2 * (float)(qp - j) : -INFINITY;
-            s[nb][e] = v;
-            if (e & 2) mx_hi = fmaxf(mx_hi, v);
-            else mx_lo = fmaxf(mx_lo, v);
+          for (int nb = 0; nb < WM_K / 16; nb++) {
+            // B fragments of two 8-key blocks: K rows are the n index, dims the k index
+            uint32_t b0, b1, b2, b3;
+            ldsm_x4(smem_addr(kd + (nb * 16 + (lane & 7) + ((lane >> 4) << 3)) * DP + u * DIM + kk * 16 + ((lane >> 3) & 1) * 8),
+                    b0, b1, b2, b3);
+            mma16816(s[2 * nb], a0, a1, a2, a3, b0, b1);
+            mma16816(s[2 * nb + 1], a0, a1, a2, a3, b2, b3);
           }
         }
-      }
-      mx_lo = fmaxf(mx_lo, __shfl_xor_sync(0xffffffffu, mx_lo, 1));
-      mx_lo = fmaxf(mx_lo, __shfl_xor_sync(0xffffffffu, mx_lo, 2));
-      mx_hi = fmaxf(mx_hi, __shfl_xor_sync(0xffffffffu, mx_hi, 1));
-      mx_hi = fmaxf(mx_hi, __shfl_xor_sync(0xffffffffu, mx_hi, 2));
-      const float mn_lo = fmaxf(m_lo, mx_lo), mn_hi = fmaxf(m_hi, mx_hi);
-      // a row that has seen nothing yet (and has no sink) keeps max -inf: every p below is 0
-      const float c_lo = (mn_lo == -INFINITY) ? 1.f : exp2f(m_lo - mn_lo);  // exp2(-inf) = 0
-      const float c_hi = (mn_hi == -INFINITY) ? 1.f : exp2f(m_hi - mn_hi);
-      const float sub_lo = (mn_lo == -INFINITY) ? 0.f : mn_lo, sub_hi = (mn_hi == -INFINITY) ? 0.f : mn_hi;
-      float ps_lo = 0.f, ps_hi = 0.f;
-      uint32_t pa[WM_K / 8][2];
+        // scale (scores live in the base-2 domain: exp2 of a difference is one instruction), mask
+        // (only on tiles that some row of the warp sees partly), running max
+        const bool interior = k0 + WM_K - 1 <= w_qlo && k0 + WM_K <= k_hi && k0 >= first_key(a, w_qhi);
+        float mx_lo = -INFINITY, mx_hi = -INFINITY;
+        if (a.softcap > 0.f) {  // the cap works on the scaled score; back to the base-2 domain afterwards
 #pragma unroll
-      for (int nb = 0; nb < WM_K / 8; nb++) {
-        const float p0 = exp2f(s[nb][0] - sub_lo), p1 = exp2f(s[nb][1] - sub_lo);  // masked scores are -inf: 0
-        const float p2 = exp2f(s[nb][2] - sub_hi), p3 = exp2f(s[nb][3] - sub_hi);
-        ps_lo += p0 + p1;
-        ps_hi += p2 + p3;
-        pa[nb][0] = pack_bf16(p0, p1);
-        pa[nb][1] = pack_bf16(p2, p3);
-      }
-      ps_lo += __shfl_xor_sync(0xffffffffu, ps_lo, 1);
-      ps_lo += __shfl_xor_sync(0xffffffffu, ps_lo, 2);
-      ps_hi += __shfl_xor_sync(0xffffffffu, ps_hi, 1);
-      ps_hi += __shfl_xor_sync(0xffffffffu, ps_hi, 2);
-      l_lo = l_lo * c_lo + ps_lo;
-      l_hi = l_hi * c_hi + ps_hi;
-      m_lo = mn_lo;
-      m_hi = mn_hi;
+          for (int nb = 0; nb < WM_K / 8; nb++)
 #pragma unroll
-      for (int i = 0; i < VDIM / 8; i++) {
-        o[i][0] *= c_lo; o[i][1] *= c_lo;
-        o[i][2] *= c_hi; o[i][3] *= c_hi;
-      }
-      // O += P V: P (16 x 64 keys) as A fragments of 16 keys each, V [key][vdim] through ldmatrix.trans
+            for (int e = 0; e < 4; e++) s[nb][e] = cap_score<true>(s[nb][e] * a.scale, a.softcap) * (1.4426950408889634f / sc);
+        }
+        if (interior) {
 #pragma unroll
-      for (int kk = 0; kk < WM_K / 16; kk++) {
-        const uint32_t a0 = pa[2 * kk][0], a1 = pa[2 * kk][1], a2 = pa[2 * kk + 1][0], a3 = pa[2 * kk + 1][1];
+          for (int nb = 0; nb < WM_K / 8; nb++) {
+            s[nb][0] *= sc; s[nb][1] *= sc; s[nb][2] *= sc; s[nb][3] *= sc;
+            if (slope2 != 0.f) {
+              const int j = k0 + nb * 8 + tig * 2;
+              s[nb][0] -= slope2 * (float)(qp_lo - j); s[nb][1] -= slope2 * (float)(qp_lo - j - 1);
+              s[nb][2] -= slope2 * (float)(qp_hi - j); s[nb][3] -= slope2 * (float)(qp_hi - j - 1);
+            }
+            mx_lo = fmaxf(mx_lo, fmaxf(s[nb][0], s[nb][1]));
+            mx_hi = fmaxf(mx_hi, fmaxf(s[nb][2], s[nb][3]));
+          }
+        } else {
 #pragma unroll
-        for (int nb = 0; nb < VDIM / 16; nb++) {
-          uint32_t b0, b1, b2, b3;
-          // matrices: (keys 0-7, cols 0-7), (keys 8-15, cols 0-7), (keys 0-7, cols 8-15), (keys 8-15, cols 8-15)
-          ldsm_x4_t(smem_addr(vd + (kk * 16 + (lane & 15)) * VP + nb * 16 + (lane >> 4) * 8), b0, b1, b2, b3);
-          mma16816(o[2 * nb], a0, a1, a2, a3, b0, b1);
-          mma16816(o[2 * nb + 1], a0, a1, a2, a3, b2, b3);
+          for (int nb = 0; nb < WM_K / 8; nb++) {
+#pragma unroll
+            for (int e = 0; e < 4; e++) {
+              const int j = k0 + nb * 8 + tig * 2 + (e & 1);
+              const int qp = (e & 2) ? qp_hi : qp_lo;
+              const bool vis = j <= qp && j < k_hi && j >= first_key(a, qp);
+              const float v = vis ? s[nb][e] * sc - slope2 * (float)(qp - j) : -INFINITY;
+              s[nb][e] = v;
+              if (e & 2) mx_hi = fmaxf(mx_hi, v);
+              else mx_lo = fmaxf(mx_lo, v);
+            }
+          }
+        }
+        mx_lo = fmaxf(mx_lo, __shfl_xor_sync(0xffffffffu, mx_lo, 1));
+        mx_lo = fmaxf(mx_lo, __shfl_xor_sync(0xffffffffu, mx_lo, 2));
+        mx_hi = fmaxf(mx_hi, __shfl_xor_sync(0xffffffffu, mx_hi, 1));
+        mx_hi = fmaxf(mx_hi, __shfl_xor_sync(0xffffffffu, mx_hi, 2));
+        const float mn_lo = fmaxf(m_lo[u], mx_lo), mn_hi = fmaxf(m_hi[u], mx_hi);
+        // a row that has seen nothing yet (and has no sink) keeps max -inf: every p below is 0
+        const float c_lo = (mn_lo == -INFINITY) ? 1.f : exp2f(m_lo[u] - mn_lo);  // exp2(-inf) = 0
+        const float c_hi = (mn_hi == -INFINITY) ? 1.f : exp2f(m_hi[u] - mn_hi);
+        const float sub_lo = (mn_lo == -INFINITY) ? 0.f : mn_lo, sub_hi = (mn_hi == -INFINITY) ? 0.f : mn_hi;
+        float ps_lo = 0.f, ps_hi = 0.f;
+        uint32_t pa[WM_K / 8][2];
+#pragma unroll
+        for (int nb = 0; nb < WM_K / 8; nb++) {
+          const float p0 = exp2f(s[nb][0] - sub_lo), p1 = exp2f(s[nb][1] - sub_lo);  // masked scores are -inf: 0
+          const float p2 = exp2f(s[nb][2] - sub_hi), p3 = exp2f(s[nb][3] - sub_hi);
+          ps_lo += p0 + p1;
+          ps_hi += p2 + p3;
+          pa[nb][0] = pack_bf16(p0, p1);
+          pa[nb][1] = pack_bf16(p2, p3);
+        }
+        ps_lo += __shfl_xor_sync(0xffffffffu, ps_lo, 1);
+        ps_lo += __shfl_xor_sync(0xffffffffu, ps_lo, 2);
+        ps_hi += __shfl_xor_sync(0xffffffffu, ps_hi, 1);
+        ps_hi += __shfl_xor_sync(0xffffffffu, ps_hi, 2);
+        l_lo[u] = l_lo[u] * c_lo + ps_lo;
+        l_hi[u] = l_hi[u] * c_hi + ps_hi;
+        m_lo[u] = mn_lo;
+        m_hi[u] = mn_hi;
+#pragma unroll
+        for (int i = 0; i < VDIM / 8; i++) {
+          o[u][i][0] *= c_lo; o[u][i][1] *= c_lo;
+          o[u][i][2] *= c_hi; o[u][i][3] *= c_hi;
+        }
+        // O += P V: P (16 x 64 keys) as A fragments of 16 keys each, V [key][vdim] through ldmatrix.trans
+#pragma unroll
+        for (int kk = 0; kk < WM_K / 16; kk++) {
+          const uint32_t a0 = pa[2 * kk][0], a1 = pa[2 * kk][1], a2 = pa[2 * kk + 1][0], a3 = pa[2 * kk + 1][1];
+#pragma unroll
+          for (int nb = 0; nb < VDIM / 16; nb++) {
+            uint32_t b0, b1, b2, b3;
+            // matrices: (keys 0-7, cols 0-7), (keys 8-15, cols 0-7), (keys 0-7, cols 8-15), (keys 8-15, cols 8-15)
+            ldsm_x4_t(smem_addr(vd + (kk * 16 + (lane & 15)) * VP + nb * 16 + (lane >> 4) * 8), b0, b1, b2, b3);
+            mma16816(o[u][2 * nb], a0, a1, a2, a3, b0, b1);
+            mma16816(o[u][2 * nb + 1], a0, a1, a2, a3, b2, b3);
+          }
         }
       }
     }
     __syncthreads();  // the buffer is free for the load of tile kt + 2
   }
   cp_async_wait<0>();
-  const float i_lo = 1.0f / l_lo, i_hi = 1.0f / l_hi;
+  float i_lo = 1.0f / l_lo[0], i_hi = 1.0f / l_hi[0];
+  if constexpr (MAPS > 1) {
+    // o_1 - lambda o_2 and what its entries are multiplied by; a row's entries lie in the four lanes of a quad
+    const float j_lo = a.diff_lambda / l_lo[1], j_hi = a.diff_lambda / l_hi[1];
+    float ss_lo = 0.f, ss_hi = 0.f;
+#pragma unroll
+    for (int i = 0; i < VDIM / 8; i++)
+#pragma unroll
+      for (int e = 0; e < 2; e++) {
+        o[0][i][e] = o[0][i][e] * i_lo - o[1][i][e] * j_lo;
+        o[0][i][e + 2] = o[0][i][e + 2] * i_hi - o[1][i][e + 2] * j_hi;
+        ss_lo += o[0][i][e] * o[0][i][e];
+        ss_hi += o[0][i][e + 2] * o[0][i][e + 2];
+      }
+    ss_lo += __shfl_xor_sync(0xffffffffu, ss_lo, 1);
+    ss_lo += __shfl_xor_sync(0xffffffffu, ss_lo, 2);
+    ss_hi += __shfl_xor_sync(0xffffffffu, ss_hi, 1);
+    ss_hi += __shfl_xor_sync(0xffffffffu, ss_hi, 2);
+    i_lo = diff_factor(a, ss_lo);
+    i_hi = diff_factor(a, ss_hi);
+  }
   bf16* ob = (bf16*)a.out + (size_t)row0 * a.o_ld + head * VDIM;
   const float* gb = gate_row(a, (size_t)row0, head, VDIM);
 #pragma unroll
@@ -1016,8 +1173,8 @@ __global__ void __launch_bounds__(128) winattn_mma_kernel(WinAttnArgs a, Trace t
       if (r_lo < nq) { g0 = gb[(size_t)r_lo * a.gate_ld + col]; g1 = gb[(size_t)r_lo * a.gate_ld + col + 1]; }
       if (r_hi < nq) { g2 = gb[(size_t)r_hi * a.gate_ld + col]; g3 = gb[(size_t)r_hi * a.gate_ld + col + 1]; }
     }
-    if (r_lo < nq) *reinterpret_cast<uint32_t*>(ob + (size_t)r_lo * a.o_ld + col) = pack_bf16(o[i][0] * i_lo * g0, o[i][1] * i_lo * g1);
-    if (r_hi < nq) *reinterpret_cast<uint32_t*>(ob + (size_t)r_hi * a.o_ld + col) = pack_bf16(o[i][2] * i_hi * g2, o[i][3] * i_hi * g3);
+    if (r_lo < nq) *reinterpret_cast<uint32_t*>(ob + (size_t)r_lo * a.o_ld + col) = pack_bf16(o[0][i][0] * i_lo * g0, o[0][i][1] * i_lo * g1);
+    if (r_hi < nq) *reinterpret_cast<uint32_t*>(ob + (size_t)r_hi * a.o_ld + col) = pack_bf16(o[0][i][2] * i_hi * g2, o[0][i][3] * i_hi * g3);
   }
   if (head == 0) {
     bf16* orow = (bf16*)a.out + (size_t)row0 * a.o_ld;
@@ -1038,18 +1195,21 @@ __global__ void __launch_bounds__(128) winattn_mma_kernel(WinAttnArgs a, Trace t
 constexpr int WDM_ST = 3;
 constexpr int WDM_MIN_TILES = 4;  // a split range holds at least this many key tiles
 
-template <int DIM, int VDIM>
+// MAPS = 2: a head is two rows of the tile, one per map, each with zeros where the other map's entries are, scored
+// against the whole cached row [map 1 | map 2]; KD = its length
+template <int KD, int VDIM, int MAPS>
 __global__ void __launch_bounds__(128) winattn_decode_mma_kernel(WinAttnArgs a, Trace tr) {
   TRACE_ENTRY(tr);
   pdl_launch_dependents();
   pdl_wait();
-  constexpr int DP = DIM + 8, VP = VDIM + 8;
+  constexpr int DIM = KD / MAPS;
+  constexpr int DP = KD + 8, VP = VDIM + 8;
   extern __shared__ __align__(16) unsigned char smem_raw[];
   bf16* Qs = reinterpret_cast<bf16*>(smem_raw);  // [16][DP]
   bf16* Ks = Qs + 16 * DP;                        // [WDM_ST][64][DP]
   bf16* Vs = Ks + WDM_ST * WM_K * DP;             // [WDM_ST][64][VP]
   const int seq = blockIdx.x, g = blockIdx.y;
-  const int GQ = a.H / a.G, h0 = g * GQ;
+  const int GQ = a.H / a.G * MAPS, h0 = g * GQ;  // rows of the group, the first one's index
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int qp = a.seq_len[seq] - 1;
   const int k_lo = first_key(a, qp);
@@ -1067,11 +1227,11 @@ __global__ void __launch_bounds__(128) winattn_decode_mma_kernel(WinAttnArgs a, 
   const int* bt = a.block_tables + (size_t)seq * a.max_blocks;
   const bf16* kpool = (const bf16*)a.kpool;
   const bf16* vpool = (const bf16*)a.vpool;
-  const bf16* qg = (const bf16*)a.q + ((size_t)seq * a.H + h0) * DIM;  // the group's heads are neighbours
-  for (int i = threadIdx.x; i < 16 * (DIM / 8); i += blockDim.x) {
-    const int r = i / (DIM / 8), c = i % (DIM / 8);
-    const bool ok = r < GQ;
-    cp_async16(smem_addr(Qs + r * DP + c * 8), ok ? (const void*)(qg + (size_t)r * DIM + c * 8) : (const void*)qg, ok);
+  const bf16* qg = (const bf16*)a.q + ((size_t)seq * a.H * MAPS + h0) * DIM;  // the group's rows are neighbours
+  for (int i = threadIdx.x; i < 16 * (KD / 8); i += blockDim.x) {
+    const int r = i / (KD / 8), c = i % (KD / 8);
+    const bool ok = r < GQ && (MAPS == 1 || c / (DIM / 8) == r % MAPS);
+    cp_async16(smem_addr(Qs + r * DP + c * 8), ok ? (const void*)(qg + (size_t)r * DIM + c % (DIM / 8) * 8) : (const void*)qg, ok);
   }
   auto load_kv = [&](int kt) {
     const int buf = kt % WDM_ST;
@@ -1080,10 +1240,10 @@ __global__ void __launch_bounds__(128) winattn_decode_mma_kernel(WinAttnArgs a, 
     const size_t kb = (((size_t)bt[k0 / KV_BLOCK] * a.G + g) * KV_BLOCK + (k0 % KV_BLOCK));
     bf16* kd = Ks + buf * WM_K * DP;
     bf16* vd = Vs + buf * WM_K * VP;
-    for (int i = threadIdx.x; i < WM_K * (DIM / 8); i += blockDim.x) {
-      const int r = i / (DIM / 8), c = i % (DIM / 8);
+    for (int i = threadIdx.x; i < WM_K * (KD / 8); i += blockDim.x) {
+      const int r = i / (KD / 8), c = i % (KD / 8);
       const bool ok = r < nk;
-      cp_async16(smem_addr(kd + r * DP + c * 8), ok ? (const void*)(kpool + (kb + r) * DIM + c * 8) : (const void*)kpool, ok);
+      cp_async16(smem_addr(kd + r * DP + c * 8), ok ? (const void*)(kpool + (kb + r) * KD + c * 8) : (const void*)kpool, ok);
     }
     for (int i = threadIdx.x; i < WM_K * (VDIM / 8); i += blockDim.x) {
       const int r = i / (VDIM / 8), c = i % (VDIM / 8);
@@ -1102,7 +1262,7 @@ __global__ void __launch_bounds__(128) winattn_decode_mma_kernel(WinAttnArgs a, 
   float o[VDIM / 8][4];
 #pragma unroll
   for (int i = 0; i < VDIM / 8; i++) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-  uint32_t qa[DIM / 16][4];
+  uint32_t qa[KD / 16][4];
   const float sc = a.scale * 1.4426950408889634f;  // log2(e): softmax in base 2
   // the thread's two rows are two heads of the group, each with its own slope
   const float slope_lo = gid < GQ ? head_slope(a, h0 + gid) * 1.4426950408889634f : 0.f;
@@ -1115,7 +1275,7 @@ __global__ void __launch_bounds__(128) winattn_decode_mma_kernel(WinAttnArgs a, 
     __syncthreads();
     if (kt == kt_b) {
 #pragma unroll
-      for (int kk = 0; kk < DIM / 16; kk++)
+      for (int kk = 0; kk < KD / 16; kk++)
         ldsm_x4(smem_addr(Qs + (lane & 15) * DP + kk * 16 + (lane >> 4) * 8), qa[kk][0], qa[kk][1], qa[kk][2], qa[kk][3]);
     }
     const int k0 = t_lo + kt * WM_K;
@@ -1127,7 +1287,7 @@ __global__ void __launch_bounds__(128) winattn_decode_mma_kernel(WinAttnArgs a, 
 #pragma unroll
       for (int i = 0; i < 2; i++) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
 #pragma unroll
-      for (int kk = 0; kk < DIM / 16; kk++) {
+      for (int kk = 0; kk < KD / 16; kk++) {
         uint32_t b0, b1, b2, b3;
         ldsm_x4(smem_addr(kd + (kb16 + (lane & 7) + ((lane >> 4) << 3)) * DP + kk * 16 + ((lane >> 3) & 1) * 8), b0, b1, b2, b3);
         mma16816(s[0], qa[kk][0], qa[kk][1], qa[kk][2], qa[kk][3], b0, b1);
@@ -1207,6 +1367,27 @@ __global__ void __launch_bounds__(128) winattn_decode_mma_kernel(WinAttnArgs a, 
     }
   }
   __syncthreads();
+  // two maps: the rows' normalised outputs are in mrg[row][VDIM]; a warp per head writes N(o_1 - lambda o_2)
+  auto write_difference = [&]() {
+    __syncthreads();
+    for (int hq = warp; hq < GQ / 2; hq += 4) {
+      constexpr int NC = (VDIM + 31) / 32;
+      const float *p1 = mrg + (size_t)(2 * hq) * MS, *p2 = p1 + MS;
+      float v[NC], ss = 0.f;
+#pragma unroll
+      for (int c = 0; c < NC; c++) {
+        const int col = lane + 32 * c;
+        v[c] = col < VDIM ? p1[col] - a.diff_lambda * p2[col] : 0.f;
+        ss += v[c] * v[c];
+      }
+      const float f = diff_factor(a, warp_sum(ss));
+#pragma unroll
+      for (int c = 0; c < NC; c++) {
+        const int col = lane + 32 * c;
+        if (col < VDIM) ((bf16*)a.out)[(size_t)seq * a.o_ld + (size_t)(h0 / 2 + hq) * VDIM + col] = __float2bfloat16_rn(v[c] * f);
+      }
+    }
+  };
   if (n_split > 1) {
     // the CTA's state (relative to its own maximum, without the sink) goes to its place among the pair's
     // n_split; the CTA that arrives last adds them up.  Nobody waits: the counter only tells who is last.
@@ -1256,8 +1437,10 @@ __global__ void __launch_bounds__(128) winattn_decode_mma_kernel(WinAttnArgs a, 
           v += __ldcg(pz + col) * cz;
         }
         if (a.gate) v *= gate_row(a, (size_t)seq, h0 + r, VDIM)[a.gate_head ? 0 : col];
-        ((bf16*)a.out)[(size_t)seq * a.o_ld + (size_t)(h0 + r) * VDIM + col] = __float2bfloat16_rn(v / lt);
+        if (MAPS > 1) mrg[(size_t)r * MS + col] = v / lt;
+        else ((bf16*)a.out)[(size_t)seq * a.o_ld + (size_t)(h0 + r) * VDIM + col] = __float2bfloat16_rn(v / lt);
       }
+      if (MAPS > 1) write_difference();
     }
   } else {
     for (int i = threadIdx.x; i < GQ * VDIM; i += blockDim.x) {
@@ -1273,8 +1456,11 @@ __global__ void __launch_bounds__(128) winattn_decode_mma_kernel(WinAttnArgs a, 
         v += pw[col] * cw;
       }
       if (a.gate) v *= gate_row(a, (size_t)seq, h0 + r, VDIM)[a.gate_head ? 0 : col];
-      ((bf16*)a.out)[(size_t)seq * a.o_ld + (size_t)(h0 + r) * VDIM + col] = __float2bfloat16_rn(v / lt);
+      // (two maps: warp 0's states become the rows' outputs — each of their entries is read by this thread only)
+      if (MAPS > 1) mrg[(size_t)r * MS + col] = v / lt;
+      else ((bf16*)a.out)[(size_t)seq * a.o_ld + (size_t)(h0 + r) * VDIM + col] = __float2bfloat16_rn(v / lt);
     }
+    if (MAPS > 1) write_difference();
   }
   if (g == 0 && blockIdx.z == 0)
     for (int col = a.H * VDIM + threadIdx.x; col < a.o_ld; col += blockDim.x)
@@ -1282,17 +1468,18 @@ __global__ void __launch_bounds__(128) winattn_decode_mma_kernel(WinAttnArgs a, 
   TRACE_EXIT(tr);
 }
 
-template <int DIM, int VDIM>
+template <int DIM, int VDIM, int MAPS>
 static cudaError_t winattn_decode_mma_launch(cudaStream_t st, const WinAttnArgs& a) {
-  const size_t tiles = (size_t)WDM_ST * WM_K * ((DIM + 8) + (VDIM + 8)) * 2;
+  constexpr int KD = DIM * MAPS;
+  const size_t tiles = (size_t)WDM_ST * WM_K * ((KD + 8) + (VDIM + 8)) * 2;
   const size_t merge = (size_t)4 * 16 * (VDIM + 2) * 4;
-  const size_t smem = (size_t)16 * (DIM + 8) * 2 + std::max(tiles, merge);
+  const size_t smem = (size_t)16 * (KD + 8) * 2 + std::max(tiles, merge);
   if (smem > 48 * 1024)
-    cudaFuncSetAttribute(winattn_decode_mma_kernel<DIM, VDIM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaFuncSetAttribute(winattn_decode_mma_kernel<KD, VDIM, MAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   const int n_split = a.n_split > 1 && a.split_ws && a.split_cnt ? std::min(a.n_split, WINATTN_MAX_SPLIT) : 1;
   WinAttnArgs b = a;
   b.n_split = n_split;
-  (void)launch_k(winattn_decode_mma_kernel<DIM, VDIM>, dim3(a.n_tiles, a.G, n_split), dim3(128), smem, st, b, next_trace(37));
+  (void)launch_k(winattn_decode_mma_kernel<KD, VDIM, MAPS>, dim3(a.n_tiles, a.G, n_split), dim3(128), smem, st, b, next_trace(37));
   return cudaGetLastError();
 }
 
@@ -1308,54 +1495,77 @@ static bool winattn_mma_shape(int dim, int vdim) {
   return (dim == 64 && vdim == 64) || (dim == 96 && vdim == 96) || (dim == 128 && vdim == 128) ||
          (dim == 32 && vdim == 32) || (dim == 64 && vdim == 128) || (dim == 128 && vdim == 64);
 }
-bool winattn_uses_mma(int qdt, int kvdt, int dim, int vdim) {
-  return winattn_mma_on() && qdt == DT_BF16 && kvdt == DT_BF16 && winattn_mma_shape(dim, vdim);
+// ... and of its form for two maps per head (`dim` entries each)
+static bool winattn_mma_shape2(int dim, int vdim) {
+  return (dim == 32 && vdim == 32) || (dim == 32 && vdim == 64) || (dim == 64 && vdim == 64) || (dim == 64 && vdim == 128) ||
+         (dim == 128 && vdim == 128);
 }
-int winattn_qtile(int qdt, int kvdt, int dim, int vdim) {
-  return winattn_uses_mma(qdt, kvdt, dim, vdim) ? WM_Q : WA_QS;
+bool winattn_uses_mma(int qdt, int kvdt, int dim, int vdim, int maps = 1) {
+  return winattn_mma_on() && qdt == DT_BF16 && kvdt == DT_BF16 && (maps > 1 ? winattn_mma_shape2(dim, vdim) : winattn_mma_shape(dim, vdim));
+}
+int winattn_qtile(int qdt, int kvdt, int dim, int vdim, int maps) {
+  return winattn_uses_mma(qdt, kvdt, dim, vdim, maps) ? WM_Q : WA_QS;
 }
 
-template <int DIM, int VDIM>
+template <int DIM, int VDIM, int MAPS>
 static cudaError_t winattn_mma_launch(cudaStream_t st, const WinAttnArgs& a) {
-  const size_t smem = ((size_t)WM_Q * (DIM + 8) + 2 * (size_t)WM_K * (DIM + 8) + 2 * (size_t)WM_K * (VDIM + 8)) * 2;
+  const size_t smem = ((size_t)WM_Q * (DIM * MAPS + 8) + 2 * (size_t)WM_K * (DIM * MAPS + 8) + 2 * (size_t)WM_K * (VDIM + 8)) * 2;
   if (smem > 48 * 1024)
-    cudaFuncSetAttribute(winattn_mma_kernel<DIM, VDIM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-  (void)launch_k(winattn_mma_kernel<DIM, VDIM>, dim3(a.n_tiles, a.H), dim3(128), smem, st, a, next_trace(32));
+    cudaFuncSetAttribute(winattn_mma_kernel<DIM, VDIM, MAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  (void)launch_k(winattn_mma_kernel<DIM, VDIM, MAPS>, dim3(a.n_tiles, a.H), dim3(128), smem, st, a, next_trace(32));
   return cudaGetLastError();
 }
 
 cudaError_t launch_winattn(cudaStream_t st, int qdt, int kvdt, const WinAttnArgs& a) {
   if (a.n_tiles <= 0) return cudaSuccess;
   if (a.H % a.G) return cudaErrorInvalidValue;
+  const int maps = std::max(1, a.maps);
+  if (maps > 2 || (maps == 2 && (a.sink || a.gate || a.softcap > 0.f || a.slope_exp > 0.f))) return cudaErrorInvalidValue;
   if (a.tile_seq == nullptr) {  // decode: one query per sequence
     static const bool dec_mma = !(getenv("NVLLM_WINATTN_DECODE_MMA") && atoi(getenv("NVLLM_WINATTN_DECODE_MMA")) == 0);
-    if (dec_mma && winattn_uses_mma(qdt, kvdt, a.dim, a.vdim) && a.H / a.G <= 16) {
-      if (a.dim == 64 && a.vdim == 64) return winattn_decode_mma_launch<64, 64>(st, a);
-      if (a.dim == 96 && a.vdim == 96) return winattn_decode_mma_launch<96, 96>(st, a);
-      if (a.dim == 128 && a.vdim == 128) return winattn_decode_mma_launch<128, 128>(st, a);
-      if (a.dim == 32 && a.vdim == 32) return winattn_decode_mma_launch<32, 32>(st, a);
-      if (a.dim == 64 && a.vdim == 128) return winattn_decode_mma_launch<64, 128>(st, a);
-      if (a.dim == 128 && a.vdim == 64) return winattn_decode_mma_launch<128, 64>(st, a);
+    if (dec_mma && maps == 2 && winattn_uses_mma(qdt, kvdt, a.dim, a.vdim, 2) && a.H / a.G <= 8) {
+      if (a.dim == 32 && a.vdim == 32) return winattn_decode_mma_launch<32, 32, 2>(st, a);
+      if (a.dim == 32 && a.vdim == 64) return winattn_decode_mma_launch<32, 64, 2>(st, a);
+      if (a.dim == 64 && a.vdim == 64) return winattn_decode_mma_launch<64, 64, 2>(st, a);
+      if (a.dim == 64 && a.vdim == 128) return winattn_decode_mma_launch<64, 128, 2>(st, a);
+      if (a.dim == 128 && a.vdim == 128) return winattn_decode_mma_launch<128, 128, 2>(st, a);
+    }
+    if (dec_mma && maps == 1 && winattn_uses_mma(qdt, kvdt, a.dim, a.vdim) && a.H / a.G <= 16) {
+      if (a.dim == 64 && a.vdim == 64) return winattn_decode_mma_launch<64, 64, 1>(st, a);
+      if (a.dim == 96 && a.vdim == 96) return winattn_decode_mma_launch<96, 96, 1>(st, a);
+      if (a.dim == 128 && a.vdim == 128) return winattn_decode_mma_launch<128, 128, 1>(st, a);
+      if (a.dim == 32 && a.vdim == 32) return winattn_decode_mma_launch<32, 32, 1>(st, a);
+      if (a.dim == 64 && a.vdim == 128) return winattn_decode_mma_launch<64, 128, 1>(st, a);
+      if (a.dim == 128 && a.vdim == 64) return winattn_decode_mma_launch<128, 64, 1>(st, a);
     }
     if (winattn_decode_group_ok(a)) {
       if (qdt == DT_F32 && kvdt == DT_F32) return winattn_decode_group<float, float>(st, a);
       if (qdt == DT_BF16 && kvdt == DT_BF16) return winattn_decode_group<bf16, bf16>(st, a);
     }
-    if (qdt == DT_F32 && kvdt == DT_F32) return winattn_decode_dispatch<float, float>(st, a);
-    if (qdt == DT_BF16 && kvdt == DT_BF16) return winattn_decode_dispatch<bf16, bf16>(st, a);
+    if (qdt == DT_F32 && kvdt == DT_F32)
+      return a.maps > 1 ? winattn_decode_dispatch<float, float, 2>(st, a) : winattn_decode_dispatch<float, float, 1>(st, a);
+    if (qdt == DT_BF16 && kvdt == DT_BF16)
+      return a.maps > 1 ? winattn_decode_dispatch<bf16, bf16, 2>(st, a) : winattn_decode_dispatch<bf16, bf16, 1>(st, a);
     return cudaErrorInvalidValue;
   }
   // the mma kernel's tile is 64 queries: prefill steps whose tile list was built for it
-  if (winattn_uses_mma(qdt, kvdt, a.dim, a.vdim) && a.qtile == WM_Q && (a.o_ld % 2) == 0) {
-    if (a.dim == 64 && a.vdim == 64) return winattn_mma_launch<64, 64>(st, a);
-    if (a.dim == 96 && a.vdim == 96) return winattn_mma_launch<96, 96>(st, a);
-    if (a.dim == 128 && a.vdim == 128) return winattn_mma_launch<128, 128>(st, a);
-    if (a.dim == 32 && a.vdim == 32) return winattn_mma_launch<32, 32>(st, a);
-    if (a.dim == 64 && a.vdim == 128) return winattn_mma_launch<64, 128>(st, a);
-    if (a.dim == 128 && a.vdim == 64) return winattn_mma_launch<128, 64>(st, a);
+  if (maps == 2 && winattn_uses_mma(qdt, kvdt, a.dim, a.vdim, 2) && a.qtile == WM_Q && (a.o_ld % 2) == 0) {
+    if (a.dim == 32 && a.vdim == 32) return winattn_mma_launch<32, 32, 2>(st, a);
+    if (a.dim == 32 && a.vdim == 64) return winattn_mma_launch<32, 64, 2>(st, a);
+    if (a.dim == 64 && a.vdim == 64) return winattn_mma_launch<64, 64, 2>(st, a);
+    if (a.dim == 64 && a.vdim == 128) return winattn_mma_launch<64, 128, 2>(st, a);
+    if (a.dim == 128 && a.vdim == 128) return winattn_mma_launch<128, 128, 2>(st, a);
   }
-  if (qdt == DT_F32 && kvdt == DT_F32) return winattn_dispatch<float, float>(st, a);
-  if (qdt == DT_BF16 && kvdt == DT_BF16) return winattn_dispatch<bf16, bf16>(st, a);
+  if (maps == 1 && winattn_uses_mma(qdt, kvdt, a.dim, a.vdim) && a.qtile == WM_Q && (a.o_ld % 2) == 0) {
+    if (a.dim == 64 && a.vdim == 64) return winattn_mma_launch<64, 64, 1>(st, a);
+    if (a.dim == 96 && a.vdim == 96) return winattn_mma_launch<96, 96, 1>(st, a);
+    if (a.dim == 128 && a.vdim == 128) return winattn_mma_launch<128, 128, 1>(st, a);
+    if (a.dim == 32 && a.vdim == 32) return winattn_mma_launch<32, 32, 1>(st, a);
+    if (a.dim == 64 && a.vdim == 128) return winattn_mma_launch<64, 128, 1>(st, a);
+    if (a.dim == 128 && a.vdim == 64) return winattn_mma_launch<128, 64, 1>(st, a);
+  }
+  if (qdt == DT_F32 && kvdt == DT_F32) return a.maps > 1 ? winattn_dispatch<float, float, 2>(st, a) : winattn_dispatch<float, float, 1>(st, a);
+  if (qdt == DT_BF16 && kvdt == DT_BF16) return a.maps > 1 ? winattn_dispatch<bf16, bf16, 2>(st, a) : winattn_dispatch<bf16, bf16, 1>(st, a);
   return cudaErrorInvalidValue;
 }
 

@@ -172,7 +172,8 @@ __global__ void __launch_bounds__(512) norm_kernel(NormArgs a, Trace tr) {
     if (threadIdx.x == 0 && trace_on(tr)) trace_rec(tr, t_entry, t_wait, 0ull);
     return;
   }
-  const bool upd = (a.p1 != nullptr) || (a.p2 != nullptr) || (a.xadd != nullptr);
+  const bool upd = (a.p1 != nullptr) || (a.p2 != nullptr) || (a.xadd != nullptr) || (a.xadd_table != nullptr);
+  const YT* xtab = a.xadd_table ? (const YT*)a.xadd_table + (size_t)a.xadd_tokens[r] * H : nullptr;
   const bool ln = a.b != nullptr || a.centered != 0;  // LayerNorm (with or without the additive term)
   float lsum = 0.f;
   for (int i = i0; i < H; i += blockDim.x * 8) {
@@ -197,10 +198,10 @@ __global__ void __launch_bounds__(512) norm_kernel(NormArgs a, Trace tr) {
             }
 #pragma unroll
           for (int q = 0; q < 4; q++)
-            if (s0 + q < a.comb_k) load8(a.p1 + (size_t)prow[q] * H + i, pv[q]);
+            if (s0 + q < a.comb_k && prow[q] >= 0) load8(a.p1 + (size_t)prow[q] * H + i, pv[q]);
 #pragma unroll
           for (int q = 0; q < 4; q++)
-            if (s0 + q < a.comb_k) {
+            if (s0 + q < a.comb_k && prow[q] >= 0) {
 #pragma unroll
               for (int j = 0; j < 8; j++) acc[j] += cw[q] * pv[q][j];
             }
@@ -247,6 +248,13 @@ __global__ void __launch_bounds__(512) norm_kernel(NormArgs a, Trace tr) {
       load8(a.xadd + i, p);
 #pragma unroll
       for (int j = 0; j < 8; j++) v[j] += p[j];
+    }
+    if (xtab) {
+      float p[8];
+      load8(xtab + i, p);
+      const float m = a.xadd_mult != 0.f ? a.xadd_mult : 1.f;
+#pragma unroll
+      for (int j = 0; j < 8; j++) v[j] = fmaf(p[j], m, v[j]);
     }
     if (upd) store8(xr + i, v);
     store8(row + i, v);
@@ -410,7 +418,23 @@ __global__ void __launch_bounds__(512) norm_kernel(NormArgs a, Trace tr) {
   if (a.router) {
     __shared__ float probs[MOE_MAX_E];
     __syncthreads();
-    moe_route_row(row, a.router, H, a.E, a.topk, probs, (size_t)orow, a.topk_idx, a.topk_w, a.route);
+    if (a.route.identity > 0) {
+      // the chosen identity experts return the row itself: their weight times it joins x here, where both are at hand
+      __shared__ float id_w;
+      moe_route_row(row, a.router, H, a.E, a.topk, probs, (size_t)orow, a.topk_idx, a.topk_w, a.route, &id_w);
+      __syncthreads();
+      const float wi = id_w;
+      if (wi != 0.f)
+        for (int i = i0; i < H; i += blockDim.x * 8) {
+          float v[8];
+          load8(xr + i, v);  // (this thread's own store above)
+#pragma unroll
+          for (int j = 0; j < 8; j++) v[j] = fmaf(wi, row[i + j], v[j]);
+          store8(xr + i, v);
+        }
+    } else {
+      moe_route_row(row, a.router, H, a.E, a.topk, probs, (size_t)orow, a.topk_idx, a.topk_w, a.route);
+    }
   }
   if (threadIdx.x == 0 && trace_on(tr))
     trace_rec(tr, t_entry, t_wait, ((t_loads - t_wait) << 32) | (t_red - t_wait));

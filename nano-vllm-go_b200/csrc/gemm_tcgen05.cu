@@ -70,7 +70,7 @@ struct Tc5Fuse {
   float m;
   const float* g;  // weight of the norm that reads x next: xb = bf16(x * g); null = ones
   int cl;          // > 1: the S k-splits of an output tile are one thread-block cluster of `cl` CTAs
-  float glu_limit; // > 0: the gated epilogue computes the clamped unit (common.cuh glu_unit)
+  float glu_limit; // != 0: the gated epilogue computes another unit than silu(g) u (common.cuh glu_unit)
 };
 // A second GEMM chained behind the first inside ONE launch (the FFN pair of a decode step:
 // W1 + activation, then W2): every CTA runs its units of problem 1, then its units of problem 2.
@@ -541,7 +541,7 @@ gemm_tc5_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__
             const float send = __uint_as_float(odd ? r[c] : r[c + 16]);
             const float got = __shfl_xor_sync(0xffffffffu, send, 1);
             const float g = alpha * (odd ? got : mine), u = alpha * (odd ? mine : got);
-            const float v = fz.glu_limit > 0.f ? glu_unit(g, u, fz.glu_limit)
+            const float v = fz.glu_limit != 0.f ? glu_unit(g, u, fz.glu_limit)
                                                : __fdividef(g, 1.0f + __expf(-g)) * u;
             *reinterpret_cast<bf16*>(stg + (c + (odd ? 16 : 0)) * 48 + p * 2) =
                 __float2bfloat16_rn(v);

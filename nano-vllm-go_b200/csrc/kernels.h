@@ -52,6 +52,9 @@ struct RouteOpts {
   const float* correction;
   int group_top2;
   const float* bias;  // [E] or null: added to the router's logits (choice and weights)
+  // > 0: the last `identity` of the E outputs are experts that return their input; the kernel that routes adds
+  // weight * input to x itself (norm kernel only), their slots keep an index past the real experts
+  int identity;
 };
 struct NormArgs {
   float* x;            // [*, H] residual stream, updated in place when p1/p2 given
@@ -83,7 +86,7 @@ struct NormArgs {
   // mixture-of-experts fusions (moe.cu holds the stand-alone kernels)
   //  * comb_rows != null: the first addend is the weighted combine of the expert outputs,
   //    sum_s comb_w[r, s] * p1[comb_rows[r, s], :] in slot order (moe.go:116-118), instead of a
-  //    split-K sum (S1 / stride1 unused)
+  //    split-K sum (S1 / stride1 unused); slots with comb_rows < 0 (identity experts) add nothing here
   const int* comb_rows;   // [*, comb_k] row of p1 holding (token r, slot s)
   const float* comb_w;    // [*, comb_k]
   int comb_k;
@@ -99,6 +102,10 @@ struct NormArgs {
   // always-on expert with a gate per token); gate_w [H] != null: gate_out[row] =
   // sigmoid(normed row . gate_w) for that expert's next run
   const float* xadd;
+  // instead of xadd: x += table[tokens[row]] * xadd_mult (0: 1), a row of the embedding (dtype ydt)
+  const void* xadd_table;
+  const int* xadd_tokens;
+  float xadd_mult;
   const float* row_m2;
   const float* gate_w;
   float* gate_out;
@@ -123,7 +130,7 @@ cudaError_t launch_norm(cudaStream_t st, const NormArgs& a);
 // SwiGLU: out[t,j] = silu(h[t,j]) * h[t,F+j]   (transformer.go:50-66, mamba2.go:360-367)
 // GELU:   out[t,j] = gelu_tanh(h[t,j] + b1[j]) (transformer.go:67-78, tensor.go:181-190)
 // glu_limit > 0 (with swiglu): the clamped gated unit g = min(gate, limit), u = clamp(up, +-limit),
-// out = g * sigmoid(1.702 g) * (u + 1)
+// out = g * sigmoid(1.702 g) * (u + 1); GLU_TANH_GELU: out = gelu_tanh(g) * u
 // swiglu == 2: out[t,j] = relu(h[t,j])^2
 cudaError_t launch_act(cudaStream_t st, int odt, int T, int F, const float* h, int S, size_t stride,
                        const float* bias, int swiglu, void* out, float glu_limit = 0.f);
@@ -243,7 +250,7 @@ struct GemvPre {
   int hld;
   const float* hbias;  // [K] (GELU branch) or null
   int swiglu;          // 0 tanh-GELU, 1 gated unit, 2 squared ReLU
-  float glu_limit;     // > 0 with swiglu: the clamped gated unit (see launch_act)
+  float glu_limit;     // with swiglu: which gated unit (see launch_act)
 };
 // split-K slices a skinny GEMV will produce for (M,N,K); workspace must hold S*M*N floats
 int gemv_splits(int M, int N, int K);
@@ -275,7 +282,7 @@ struct Tc5Args {
   void* epi_out;        // bf16 [M, epi_ld]
   int epi_ld;
   const float* epi_bias;  // [N] or null (GELU)
-  float glu_limit;        // TC5_EPI_SWIGLU: > 0 selects the clamped gated unit (see launch_act)
+  float glu_limit;        // TC5_EPI_SWIGLU: > 0 the clamped gated unit, GLU_TANH_GELU the tanh-GELU one (see launch_act)
   // ---- RMSNorm folded into the GEMMs (forward.cu "fold"): the producer of x writes
   // bf16(x * g) (g = norm weight), the row statistic is applied to the accumulator.
   // consumer side, rs_ssq != null: A holds bf16(x * g), not yet divided by the row's rms, and every
@@ -422,6 +429,10 @@ struct LatentArgs {
   void* pool;                        // [blocks * 256][R + rot] cache dtype
   void* cq;                          // [T, q_rank_p] act dtype (zero padded)
   float* gate;                       // [T, H] sigmoid of the head gates; null: the heads have none
+  float* out_gate;                   // [T, H vdim] sigmoid of the output gates (columns in place of the head gates'); null: none
+  const float* sink_w;               // [H]: one more term exp(sink_w[h]) of the softmax denominator, or null
+  // decode with key splits: the merge of the splits also expands and gates (launch_latent_expand's job) when exp_out is set
+  const void* exp_w; void* exp_out; int exp_ld;
   // folded query projection partials [S][T][q_ld] -> absorbed queries [T, H, R + rot] act dtype
   const float* q_p; int q_S; size_t q_stride; int q_ld;
   void* qabs;
@@ -443,6 +454,9 @@ cudaError_t launch_latent_q(cudaStream_t st, int qdt, const LatentArgs& a);
 cudaError_t launch_latent_fold(cudaStream_t st, int wdt, const void* w_uq, const void* w_uk, void* wq, const void* w_o,
                                const void* w_uv, void* wo, int W, int H, int dim, int rot, int vdim, int R,
                                int q_rank, int q_rank_p, int ov_p, int ovr_p);
+// out[t, h vdim + e] = out_gate[t, h vdim + e] (sigmoids) * sum_r W_uv[h vdim + e, r] * olat[t, h R + r] for layers whose output gate
+// sits between the value expansion and the output projection; out rows o_ld apart, padding columns written as zeros
+cudaError_t launch_latent_expand(cudaStream_t st, int qdt, const LatentArgs& a, const void* w_uv, void* out, int o_ld);
 int latent_attn_qtile();
 int latent_attn_splits(int n_seqs, int H, int max_len, int window, int sm_count);
 cudaError_t launch_latent_attn(cudaStream_t st, int qdt, int kvdt, const LatentArgs& a);
@@ -494,6 +508,11 @@ struct WinAttnArgs {
   // gate_head: `gate` holds one number per (token, head), gate[t * gate_ld + h]
   float slope_exp;
   const float* sink_w;          // [H]
+  // maps = 2 (0 or 1: one map): q and k rows hold two maps of dim entries per head, both over the same values;
+  // out = N(map 1 - diff_lambda * map 2) * out_mul, N divides a head's vdim entries by their root mean square.  q is
+  // then [T, H, 2, dim], the K pool [blocks][G][256][2 dim]; no gate, sink, cap or distance bias
+  int maps;
+  float diff_lambda, out_mul;
   int gate_head;
   // decode over long contexts: the keys of a (sequence, key / value head) are cut into n_split ranges, one CTA
   // each; their partial states meet in split_ws [n_seqs][G][n_split][16][vdim + 2] floats, merged by the CTA
@@ -524,7 +543,7 @@ struct ConvAttnPrep {
 cudaError_t launch_winattn_prep_conv(cudaStream_t st, int qdt, int kvdt, const WinAttnArgs& a, const ConvAttnPrep& c);
 cudaError_t launch_winattn(cudaStream_t st, int qdt, int kvdt, const WinAttnArgs& a);
 // queries per tile of the kernel launch_winattn picks for a prefill step (the host builds the tile list with it)
-int winattn_qtile(int qdt, int kvdt, int dim, int vdim);
+int winattn_qtile(int qdt, int kvdt, int dim, int vdim, int maps = 1);
 
 // ---------------------------------------------------------------- delta.cu
 // Gated delta rule between its two projections, ragged batch; state per slot in fp32.
@@ -554,6 +573,8 @@ cudaError_t launch_delta_out(cudaStream_t st, int odt, const DeltaArgs& a);
 //   gated linear attention   S <- diag(a_t) S + k_t v_t^T,  o_t = S^T q_t
 //   time mixing              o_t = (S + diag(u) k_t v_t^T)^T r_t,  then S <- diag(w_t) S + k_t v_t^T
 //   HGRN2                    S <- diag(f_t) S + (1 - f_t) v_t^T,  o_t = S^T silu(q_t),  f_t = l + (1 - l) sigmoid(z_t)
+//   mLSTM                    S <- a_t S + b_t k_t v_t^T,  n <- a_t n + b_t k_t,  o_t = S^T q_t / (max(|n . q_t|, c_t) + 1e-6)
+//                            a_t = exp(f_t + m_(t-1) - m_t), b_t = exp(i_t - m_t), c_t = exp(-m_t), m_t = max(f_t + m_(t-1), i_t)
 // between their projections.  A projection's result is a segment of split-K partials.
 struct LinSeg {
   const float* p;   // element (t, c) = sum_s p[s * stride + t * ld + c]
@@ -582,6 +603,14 @@ struct LinRecArgs {
   // instead of one per key entry
   int qk_div;
   const float* decay_p; int decay_ld;
+  // mLSTM (gi.p set): gi / gf [T, H] the gates' projections, + gi_b / gf_b, capped by cap tanh(z / cap).  gates: three
+  // arrays [T, H], a_t | b_t | c_t (the scan reads a_t as decay_p); nq [T, H] the scan's n . q.  n [H][dim] and m [H] of
+  // a sequence sit norm_off / max_off floats into its slot.  The read-out's gate is sigmoid(gate)
+  LinSeg gi, gf;
+  const float *gi_b, *gf_b;
+  float cap;
+  float *gates, *nq;
+  size_t norm_off, max_off;
   float* qkw;            // [T, 3 H dim]: q | k | decay
   float* vv;             // [T, H vdim]
   float* o;              // [T, H vdim] read-outs
@@ -590,6 +619,9 @@ struct LinRecArgs {
 cudaError_t launch_linrec_prep(cudaStream_t st, const LinRecArgs& a);
 // HGRN2's: qkw rows [silu(q) | 1 - f | f], vv = v's slices summed (not written when v is one slice)
 cudaError_t launch_hgrn_prep(cudaStream_t st, const LinRecArgs& a);
+// mLSTM's: the gates' logarithms, the running maximum over a sequence's tokens, gates[]; q, k, v slices summed unless
+// they are single ones
+cudaError_t launch_mlstm_prep(cudaStream_t st, const LinRecArgs& a);
 cudaError_t launch_linrec_scan(cudaStream_t st, const LinRecArgs& a);
 cudaError_t launch_linrec_out(cudaStream_t st, int odt, const LinRecArgs& a);
 // One row per sequence (T == n_seqs) and vdim <= 128: prep + scan + out as one launch (a CTA per sequence and head)

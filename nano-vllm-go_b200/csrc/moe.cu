@@ -43,7 +43,9 @@ moe_sort_kernel(const int* __restrict__ topk_idx, int n_pairs, int k, int E, Moe
   __shared__ int off[MOE_MAX_E + 1];
   for (int e = threadIdx.x; e < E; e += blockDim.x) cnt[e] = 0;
   __syncthreads();
-  for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) atomicAdd(&cnt[topk_idx[p]], 1);
+  // pairs of identity experts (index >= E) get no row: they stay out of the lists, pair_row = -1
+  for (int p = threadIdx.x; p < n_pairs; p += blockDim.x)
+    if (topk_idx[p] < E) atomicAdd(&cnt[topk_idx[p]], 1);
   __syncthreads();
   if (threadIdx.x == 0) {
     int run = 0, nt = 0;
@@ -68,11 +70,16 @@ moe_sort_kernel(const int* __restrict__ topk_idx, int n_pairs, int k, int E, Moe
   __syncthreads();
   for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) {
     const int e = topk_idx[p];
+    if (e >= E) {
+      b.pair_row[p] = -1;
+      continue;
+    }
     const int row = off[e] + atomicAdd(&cnt[e], 1);
     b.sorted_pair[row] = p;
     b.pair_row[p] = row;
     b.a_rows[row] = p / k;
   }
+  for (int r = off[E] + threadIdx.x; r < n_pairs; r += blockDim.x) b.a_rows[r] = 0;  // rows past the lists: a valid one
   TRACE_EXIT(tr);
 }
 
@@ -135,7 +142,8 @@ moe_sort_gather_kernel(const int* __restrict__ topk_idx, int n_pairs, int k, int
   if (tid < MOE_SG_MAX_E) s_cnt[tid] = s_base[tid] = 0;
   pdl_wait();
   __syncthreads();
-  for (int p = tid; p < n_pairs; p += 1024) atomicAdd(&s_cnt[topk_idx[p]], 1);
+  for (int p = tid; p < n_pairs; p += 1024)
+    if (topk_idx[p] < E) atomicAdd(&s_cnt[topk_idx[p]], 1);  // (others are identity experts: no row)
   __syncthreads();
   if (warp == 0) {
     // expert offsets and the tile list by warp scans (E <= 64: lane holds experts lane and
@@ -193,7 +201,11 @@ moe_sort_gather_kernel(const int* __restrict__ topk_idx, int n_pairs, int k, int
     for (int i = tid; i < 32 * MOE_SG_MAX_E; i += 1024) (&s_wcnt[0][0])[i] = 0;
     __syncthreads();
     const int p = c0 + tid;
-    const int e = p < n_pairs ? topk_idx[p] : -1;
+    int e = p < n_pairs ? topk_idx[p] : -1;
+    if (e >= E) {
+      e = -1;
+      if (blockIdx.x == 0) b.pair_row[p] = -1;
+    }
     const unsigned same = __match_any_sync(0xffffffffu, e);
     const int rank = __popc(same & ((1u << lane) - 1));
     if (e >= 0 && rank == 0) s_wcnt[warp][e] = __popc(same);
@@ -219,11 +231,12 @@ moe_sort_gather_kernel(const int* __restrict__ topk_idx, int n_pairs, int k, int
     }
     __syncthreads();
   }
-  const int rpc = (n_pairs + gridDim.x - 1) / gridDim.x;
+  const int n_rows = s_off[E];
+  const int rpc = (n_rows + gridDim.x - 1) / gridDim.x;
   const int r0 = blockIdx.x * rpc;
   for (int idx = tid; idx < rpc * vpr; idx += 1024) {
     const int r = r0 + idx / vpr, j = idx % vpr;
-    if (r < n_pairs) xs[(size_t)r * vpr + j] = x[(size_t)(s_inv[r] / k) * vpr + j];
+    if (r < n_rows) xs[(size_t)r * vpr + j] = x[(size_t)(s_inv[r] / k) * vpr + j];
   }
   TRACE_EXIT(tr);
 }
@@ -264,7 +277,7 @@ __global__ void moe_glu_kernel(size_t nvec, int I, const float* __restrict__ h,
     for (int i = 0; i < 8; i++) {
       const float a = i < 4 ? lo[2 * i] : hi[2 * i - 8];
       const float u = i < 4 ? lo[2 * i + 1] : hi[2 * i - 7];
-      if (glu_limit > 0.f) {
+      if (glu_limit != 0.f) {
         o[i] = glu_unit(a, u, glu_limit);
       } else {
         const float sig = 1.0f / (1.0f + expf(-a));

@@ -12,10 +12,11 @@ constexpr int MOE_MAX_E = 256;
 // (tensor.go:128-155), k rounds of first-max selection (ties -> lower index, which is what a
 // stable descending sort gives; the reference's sort.Slice is unstable, ties have measure zero
 // with random-init weights) and the renormalisation over the chosen k (moe.go:88-103).
-// probs, chs, gsc: shared scratch of E floats each, this warp's own.
+// probs, chs, gsc: shared scratch of E floats each, this warp's own.  identity_w (shared): receives the summed weight of
+// the chosen identity experts (RouteOpts::identity).
 __device__ __forceinline__ void moe_select_row(float* probs, float* chs, float* gsc, int E, int k, size_t t,
                                                int* __restrict__ topk_idx, float* __restrict__ topk_w,
-                                               RouteOpts ro) {
+                                               RouteOpts ro, float* identity_w = nullptr) {
   const int lane = threadIdx.x & 31;
   if (ro.sigmoid) {
     // every expert scores on its own
@@ -106,10 +107,16 @@ __device__ __forceinline__ void moe_select_row(float* probs, float* chs, float* 
     __syncwarp();
   }
   if (ro.sigmoid && !ro.raw) ksum += 1e-20f;
+  float id_w = 0.f;
   if (lane < k) {
     topk_idx[t * k + lane] = sel_i;
     const float wgt = ro.raw ? sel_p * ro.scale : sel_p / ksum;
     topk_w[t * k + lane] = ro.square ? wgt * wgt : wgt;
+    if (sel_i >= E - ro.identity) id_w = wgt;
+  }
+  if (identity_w) {
+    id_w = warp_sum(id_w);
+    if (lane == 0) *identity_w = id_w;
   }
 }
 
@@ -120,7 +127,7 @@ __device__ __forceinline__ void moe_route_row(const float* y, const float* __res
                                               int E, int k, float* probs, size_t t,
                                               int* __restrict__ topk_idx,
                                               float* __restrict__ topk_w,
-                                              RouteOpts ro = RouteOpts{}) {
+                                              RouteOpts ro = RouteOpts{}, float* identity_w = nullptr) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
   // Two experts per pass with the k loop unrolled four deep: up to 8 independent 32-byte loads
   // of R per lane in flight, so the E / nw passes cost one L2 round trip each instead of one
@@ -167,7 +174,7 @@ __device__ __forceinline__ void moe_route_row(const float* y, const float* __res
   __syncthreads();
   if (warp != 0) return;
   __shared__ float chs[MOE_MAX_E], gsc[MOE_MAX_E];
-  moe_select_row(probs, chs, gsc, E, k, t, topk_idx, topk_w, ro);
+  moe_select_row(probs, chs, gsc, E, k, t, topk_idx, topk_w, ro, identity_w);
 }
 
 }  // namespace nvllm
