@@ -28,7 +28,7 @@ void free_workspace(nvllm_handle* h) {
                   w.sort.counts, w.sort.offsets, w.sort.cursor, w.sort.sorted_pair, w.sort.pair_row,
                   w.sort.a_rows, w.sort.tile_expert, w.sort.tile_row0, w.sort.tile_rows,
                   w.sort.n_tiles, w.moe_Y, w.moe_y, w.moe_xs, w.lr_qkw, w.lr_v, w.lr_o, w.att_gate, w.sh_gate, w.mx_in,
-                  w.m2_xbc, w.m2_dtx, w.m2_decay, w.v_first, w.side_g, w.att_split, w.att_split_cnt};
+                  w.m2_xbc, w.m2_dtx, w.m2_decay, w.v_first, w.side_g, w.att_split, w.att_split_cnt, w.ml_gates, w.ml_nq};
   for (void* p : ptrs)
     if (p) cudaFree(p);
   for (auto& r : h->ropes) {
@@ -117,7 +117,7 @@ int ensure_workspace(nvllm_handle* h, int T, int n) {
     WS(w.dl_qkv, Tc * dch * 4);
     WS(w.dl_bg, Tc * 2 * dh * 4);
     WS(w.dl_o, Tc * dhv * 4);
-    size_t lhd = 0, lhv = 0, agate = 0, m2ch = 0, m2in = 0, m2h = 0, vfirst = 0, split_g = 0, split_v = 0;
+    size_t lhd = 0, lhv = 0, agate = 0, m2ch = 0, m2in = 0, m2h = 0, vfirst = 0, split_g = 0, split_v = 0, mlh = 0;
     bool tmix = false, shared = false;
     for (auto& y : h->ll) {
       const nvllm_layer_spec& s = y.s;
@@ -131,7 +131,10 @@ int ensure_workspace(nvllm_handle* h, int T, int n) {
         if (s.v_mix) vfirst = std::max(vfirst, (size_t)s.kv_heads * s.vdim);
         split_g = std::max(split_g, (size_t)s.kv_heads);
         split_v = std::max(split_v, (size_t)s.vdim);
-      } else if (s.mixer == NVLLM_MIXER_GLA || s.mixer == NVLLM_MIXER_HGRN2) {
+      } else if (s.mixer == NVLLM_MIXER_LATENT_ATTENTION) {
+        if (s.out_gate) agate = std::max(agate, (size_t)s.heads * s.vdim);
+      } else if (s.mixer == NVLLM_MIXER_GLA || s.mixer == NVLLM_MIXER_HGRN2 || s.mixer == NVLLM_MIXER_MLSTM) {
+        if (s.mixer == NVLLM_MIXER_MLSTM) mlh = std::max(mlh, (size_t)s.heads);
         lhd = std::max(lhd, (size_t)s.heads * s.dim);
         lhv = std::max(lhv, (size_t)s.heads * s.vdim);
       } else if (s.mixer == NVLLM_MIXER_ATTN_TMIX) {
@@ -146,6 +149,8 @@ int ensure_workspace(nvllm_handle* h, int T, int n) {
     WS(w.lr_v, Tc * lhv * 4);
     WS(w.lr_o, Tc * lhv * 4);
     WS(w.att_gate, Tc * agate * 4);
+    WS(w.ml_gates, Tc * 3 * mlh * 4);
+    WS(w.ml_nq, Tc * mlh * 4);
     WS(w.m2_xbc, Tc * m2ch * 4);
     WS(w.m2_dtx, Tc * m2in * 4);
     WS(w.m2_decay, Tc * m2h * 4);

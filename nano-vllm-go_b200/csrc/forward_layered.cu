@@ -18,15 +18,17 @@
 //     gate) beside time mixing with a token shift (linrec.cu), their outputs summed with two scales.
 //     Feed-forward: a mixture of squared-ReLU experts chosen by sigmoid scores, the weight on the
 //     expert's input, plus an always-on expert with a per-token gate.  Further mixers: attention with
-//     options, Mamba-2, HGRN2 (linrec.cu), latent attention (below; window, neighbouring pairs rotated, no
-//     gate); further feed-forwards: gated experts (+ a plain always-on one), a PolyNorm dense layer.  The
+//     options (also two score maps per head), Mamba-2, HGRN2 and mLSTM (linrec.cu), latent attention (below; window,
+//     neighbouring pairs rotated, a sink, no gate or one per entry of the heads' values); further feed-forwards: gated
+//     experts (+ an always-on one, plain or gated per token; some experts may be the identity), a PolyNorm or
+//     gated dense layer.  The passes of the repeated run may open with the embedding instead of a vector.  The
 //     norms may be LayerNorms with an additive term, and what a mixer or a feed-forward reads may pass a
 //     short causal convolution first: inside the norm kernel in steps with one row per sequence, as a launch
 //     of its own (which then also routes) otherwise.
 // Mixer "latent attention" (attention_latent.cu): one fused input projection [W_dq | W_dkv | W_g]
 // of h, RMS-normed latents, the query up projection with W_uk folded in, the absorbed-query
 // attention over the paged latent cache (per-head sigmoid gate applied to its result), the output
-// projection with W_uv folded in.  A layer with
+// projection with W_uv folded in (with a gate per entry W_uv stays apart: latent_expand).  A layer with
 // kv_from = j has no W_dkv and reads layer j's cache rows (written earlier in the same step).
 // Feed-forward: none, a dense clamped gated unit, or a group-limited top-k mixture of such
 // units (the routing runs inside the norm kernel, the expert GEMMs are the grouped ones the
@@ -56,6 +58,7 @@ void layered_free(nvllm_handle* h) {
     F(y.canon2_w); F(y.norm1_b); F(y.norm2_b); F(y.f_lower); F(y.route_bias); F(y.poly);
     F(y.sink_w); F(y.head_temp); F(y.vmix); F(y.conv_b); F(y.d_skip); F(y.route_corr); F(y.canon_w);
     F(y.side_gate); F(y.side_proj); F(y.side_norm);
+    F(y.diff_w); F(y.gate_b);
   }
   F(h->embed_norm_w);
   h->embed_norm_w = nullptr;
@@ -101,7 +104,7 @@ __global__ void add_const_kernel(float* p, size_t n, float c) {
 // layers of the sequential pre-norm blocks whose tensors follow one naming (see layered_set_weight)
 static bool option_block(const nvllm_handle* h, const nvllm_layer_spec& s) {
   return s.mixer == NVLLM_MIXER_ATTENTION || s.mixer == NVLLM_MIXER_MAMBA2 || s.mixer == NVLLM_MIXER_HGRN2 ||
-         (s.mixer == NVLLM_MIXER_LATENT_ATTENTION && h->block_style == NVLLM_LBLOCK_SEQUENTIAL_PRENORM);
+         s.mixer == NVLLM_MIXER_MLSTM || (s.mixer == NVLLM_MIXER_LATENT_ATTENTION && h->block_style == NVLLM_LBLOCK_SEQUENTIAL_PRENORM);
 }
 
 static bool parse_layer_name(const std::string& name, int* layer, std::string* rest) {
@@ -149,15 +152,15 @@ int layered_set_weight(nvllm_handle* h, const char* cname, int dtype, const void
     mat(h->loop_step, h->loop_times, W, W);
     d.ddt = DT_F32; d.p = h->loop_step;
   } else if (parse_layer_name(name, &l, &rest) && l < h->L && option_block(h, h->ll[l].s)) {
-    // sequential pre-norm blocks: attention with options / Mamba-2 / HGRN2 / latent attention, mixture of
-    // gated experts or PolyNorm dense layer, the convolutions on the sublayers' inputs, the per-layer token input
+    // sequential pre-norm blocks: attention with options / Mamba-2 / HGRN2 / mLSTM / latent attention, mixture of
+    // gated experts, PolyNorm or gated dense layer, the convolutions on the sublayers' inputs, the per-layer token input
     ListedLayer& y = h->ll[l];
     const nvllm_layer_spec& s = y.s;
     auto f32mat = [&](float* p, int64_t rows, int64_t cols) { mat(p, rows, cols, (int)cols); d.ddt = DT_F32; d.p = p; };
     const int hv = s.heads * s.vdim;
     auto taps = [&](float* p, int n) { mat(p, W, n, W); d.ddt = DT_F32; d.p = p; d.transposed = true; };
-    if (rest == "norm1") vec(y.post1_w, W);
-    else if (rest == "norm2" && s.mlp != NVLLM_MLP_NONE) vec(y.post2_w, W);
+    if (rest == "norm1") { vec(y.post1_w, W); d.add = noff; }
+    else if (rest == "norm2" && s.mlp != NVLLM_MLP_NONE) { vec(y.post2_w, W); d.add = noff; }
     else if (rest == "norm1.b" && y.norm1_b) vec(y.norm1_b, W);
     else if (rest == "norm2.b" && y.norm2_b) vec(y.norm2_b, W);
     else if (rest == "canon1" && y.canon_w) taps(y.canon_w, h->mixer_conv);
@@ -178,6 +181,21 @@ int layered_set_weight(nvllm_handle* h, const char* cname, int dtype, const void
       else if (rest == "mix.vmix" && s.v_mix) vec(y.vmix, 1);
       else if (rest == "mix.sink" && s.sink_learned) vec(y.sink_w, s.heads);
       else if (rest == "mix.temp" && s.head_temp) vec(y.head_temp, s.heads);
+      else if (rest == "mix.lq1" && s.diff_maps) vec(y.diff_w, s.dim);
+      else if (rest == "mix.lk1" && s.diff_maps) vec(y.diff_w + s.dim, s.dim);
+      else if (rest == "mix.lq2" && s.diff_maps) vec(y.diff_w + 2 * s.dim, s.dim);
+      else if (rest == "mix.lk2" && s.diff_maps) vec(y.diff_w + 3 * s.dim, s.dim);
+    } else if (s.mixer == NVLLM_MIXER_MLSTM) {
+      const int hd = s.heads * s.dim;
+      if (rest == "mix.q") mat(y.w_in, hd, W, W, 0);
+      else if (rest == "mix.k") mat(y.w_in, hd, W, W, hd);
+      else if (rest == "mix.v") mat(y.w_in, hv, W, W, 2 * hd);
+      else if (rest == "mix.g") mat(y.w_in, hv, W, W, 2 * hd + hv);
+      else if (rest == "mix.i") mat(y.w_in, s.heads, W, W, 2 * hd + 2 * hv);
+      else if (rest == "mix.f") mat(y.w_in, s.heads, W, W, 2 * hd + 2 * hv + s.heads);
+      else if (rest == "mix.i.b") vec(y.gate_b, s.heads);
+      else if (rest == "mix.f.b") vec(y.gate_b + s.heads, s.heads);
+      else if (rest == "mix.norm") vec(y.onorm_w, hv);
     } else if (s.mixer == NVLLM_MIXER_HGRN2) {
       const int hd = s.heads * s.dim;
       if (rest == "mix.q") mat(y.w_in, hd, W, W, 0);
@@ -190,7 +208,8 @@ int layered_set_weight(nvllm_handle* h, const char* cname, int dtype, const void
       const int own = s.kv_from < 0;
       if (rest == "mix.dq") mat(y.w_in, s.q_rank, W, W, 0);
       else if (rest == "mix.dkv" && own) mat(y.w_in, y.Dk, W, W, s.q_rank);
-      else if (rest == "mix.g" && y.lat_gate) mat(y.w_in, s.heads, W, W, s.q_rank + (own ? y.Dk : 0));
+      else if (rest == "mix.g" && (y.lat_gate || s.out_gate)) mat(y.w_in, s.out_gate ? hv : s.heads, W, W, s.q_rank + (own ? y.Dk : 0));
+      else if (rest == "mix.sink" && s.sink_learned) vec(y.sink_w, s.heads);
       else if (rest == "mix.dq.norm") vec(y.dq_norm, s.q_rank);
       else if (rest == "mix.dkv.norm" && own) vec(y.dkv_norm, s.kv_rank);
       else if (rest == "mix.uq") mat(y.w_uq, y.q_cols, s.q_rank, y.q_rank_p);
@@ -206,17 +225,22 @@ int layered_set_weight(nvllm_handle* h, const char* cname, int dtype, const void
       else if (rest == "mix.norm") vec(y.onorm_w, hv);
     }
     if (!d.p && s.mlp == NVLLM_MLP_DENSE) {
-      if (rest == "mlp.up") mat(y.w1, s.ff, W, W);
-      else if (rest == "mlp.down") mat(y.w2, W, s.ff, y.ff_p);
+      if (rest == "mlp.down") mat(y.w2, W, s.ff, y.ff_p);
+      else if (s.act == NVLLM_FFN_GEGLU) {
+        if (rest == "mlp.gate") mat(y.w1, s.ff, W, W, 0, 2, 0);
+        else if (rest == "mlp.up") mat(y.w1, s.ff, W, W, 0, 2, 1);
+      } else if (rest == "mlp.up") mat(y.w1, s.ff, W, W);
       else if (rest == "mlp.act") vec(y.poly, 4);
     }
     if (!d.p && s.mlp == NVLLM_MLP_MOE) {
-      if (rest == "mlp.router") f32mat(y.router, s.experts, W);
-      else if (rest == "mlp.router.b" && s.route_bias) vec(y.route_bias, s.experts);
+      const int outs = s.experts + s.route_identity;
+      if (rest == "mlp.router") f32mat(y.router, outs, W);
+      else if (rest == "mlp.router.b" && s.route_bias) vec(y.route_bias, outs);
+      else if (rest == "mlp.shared.sg" && y.sh_gate) f32mat(y.sh_gate, 1, W);
       else if (rest == "mlp.shared.gate" && s.shared_ff > 0) mat(y.w1, s.shared_ff, W, W, 0, 2, 0);
       else if (rest == "mlp.shared.up" && s.shared_ff > 0) mat(y.w1, s.shared_ff, W, W, 0, 2, 1);
       else if (rest == "mlp.shared.down" && s.shared_ff > 0) mat(y.w2, W, s.shared_ff, y.sff_p);
-      else if (rest == "mlp.correction" && s.route_correction) vec(y.route_corr, s.experts);
+      else if (rest == "mlp.correction" && s.route_correction) vec(y.route_corr, outs);
       else if (rest.compare(0, 5, "mlp.e") == 0) {
         size_t i = 5;
         int e = 0;
@@ -405,7 +429,10 @@ int layered_finalize(nvllm_handle* h) {
       } else if (s.mixer == NVLLM_MIXER_LATENT_ATTENTION) {
         for (const char* n : {"mix.dq", "mix.dq.norm", "mix.uq", "mix.uk", "mix.uv"}) need.push_back(p + n);
         if (s.kv_from < 0) { need.push_back(p + "mix.dkv"); need.push_back(p + "mix.dkv.norm"); }
-        if (h->ll[l].lat_gate) need.push_back(p + "mix.g");
+        if (h->ll[l].lat_gate || s.out_gate) need.push_back(p + "mix.g");
+        if (s.sink_learned) need.push_back(p + "mix.sink");
+      } else if (s.mixer == NVLLM_MIXER_MLSTM) {
+        for (const char* n : {"mix.q", "mix.k", "mix.v", "mix.g", "mix.i", "mix.i.b", "mix.f", "mix.f.b", "mix.norm"}) need.push_back(p + n);
       } else
       if (s.mixer == NVLLM_MIXER_ATTENTION) {
         for (const char* n : {"mix.q", "mix.k", "mix.v"}) need.push_back(p + n);
@@ -414,6 +441,8 @@ int layered_finalize(nvllm_handle* h) {
         if (s.sink_learned) need.push_back(p + "mix.sink");
         if (s.head_temp) need.push_back(p + "mix.temp");
         if (s.head_gate) need.push_back(p + "mix.g");
+        if (s.diff_maps)
+          for (const char* n : {"mix.lq1", "mix.lk1", "mix.lq2", "mix.lk2"}) need.push_back(p + n);
       } else {
         for (const char* n : {"mix.in", "mix.conv", "mix.conv.b", "mix.dt_bias", "mix.A_log", "mix.D", "mix.norm"})
           need.push_back(p + n);
@@ -427,11 +456,13 @@ int layered_finalize(nvllm_handle* h) {
         if (s.route_bias) need.push_back(p + "mlp.router.b");
         if (s.shared_ff > 0)
           for (const char* n : {"mlp.shared.gate", "mlp.shared.up", "mlp.shared.down"}) need.push_back(p + n);
+        if (h->ll[l].sh_gate) need.push_back(p + "mlp.shared.sg");
         if (s.route_correction) need.push_back(p + "mlp.correction");
         for (int e = 0; e < s.experts; e++)
           for (const char* n : {".gate", ".up", ".down"}) need.push_back(p + "mlp.e" + std::to_string(e) + n);
       } else if (s.mlp == NVLLM_MLP_DENSE) {
-        for (const char* n : {"norm2", "mlp.up", "mlp.down", "mlp.act"}) need.push_back(p + n);
+        for (const char* n : {"norm2", "mlp.up", "mlp.down"}) need.push_back(p + n);
+        need.push_back(p + (s.act == NVLLM_FFN_GEGLU ? "mlp.gate" : "mlp.act"));
       }
       continue;
     }
@@ -491,36 +522,51 @@ int layered_finalize(nvllm_handle* h) {
   }
   for (auto& n : need)
     if (!got(n)) return set_err(h, NVLLM_ERR_INVALID, "missing tensor %s", n.c_str());
+  // attention with two maps: the factor of the second one, in double from the loaded vectors
+  for (int l = 0; l < h->L; l++) {
+    ListedLayer& y = h->ll[l];
+    if (!y.diff_w) continue;
+    const int n = y.s.dim;
+    std::vector<float> v((size_t)4 * n);
+    NV_CHECK(h, cudaMemcpy(v.data(), y.diff_w, v.size() * 4, cudaMemcpyDeviceToHost));
+    double d1 = 0.0, d2 = 0.0;
+    for (int i = 0; i < n; i++) {
+      d1 += (double)v[i] * v[n + i];
+      d2 += (double)v[2 * n + i] * v[3 * n + i];
+    }
+    y.diff_lambda = (float)(exp(d1) - exp(d2) + (double)y.s.diff);
+  }
   // fold the per-head key / value up projections into the query and output projections
-  // (attention_latent.cu), then drop the four tensors as loaded
+  // (attention_latent.cu), then drop the four tensors as loaded (W_uv and W_o stay when a gate sits between them)
   for (int l = 0; l < h->L; l++) {
     ListedLayer& y = h->ll[l];
     const nvllm_layer_spec& s = y.s;
     if (s.mixer != NVLLM_MIXER_LATENT_ATTENTION) continue;
-    cudaError_t e = launch_latent_fold(h->stream, h->wdt, y.w_uq, y.w_uk, y.w_q, y.w_o, y.w_uv, y.w_ov, h->H, s.heads,
+    cudaError_t e = launch_latent_fold(h->stream, h->wdt, y.w_uq, y.w_uk, y.w_q, y.w_o, y.w_uv, s.out_gate ? nullptr : y.w_ov, h->H, s.heads,
                                        s.dim, s.rot_dim, s.vdim, s.kv_rank, s.q_rank, y.q_rank_p, y.ov_p, y.ovr_p);
     if (e == cudaSuccess) e = cudaStreamSynchronize(h->stream);
     if (e != cudaSuccess) return set_err(h, NVLLM_ERR_CUDA, "folding layer %d: %s", l, cudaGetErrorString(e));
     const size_t wsz = dt_size(h->wdt);
     const size_t freed = ((size_t)y.q_cols * y.q_rank_p + (size_t)s.heads * s.dim * s.kv_rank +
-                          (size_t)s.heads * s.vdim * s.kv_rank + (size_t)h->H * y.ov_p) * wsz;
+                          (s.out_gate ? 0 : (size_t)s.heads * s.vdim * s.kv_rank + (size_t)h->H * y.ov_p)) * wsz;
     for (void** p : {&y.w_uq, &y.w_uk, &y.w_uv, &y.w_o}) {
+      if (s.out_gate && (p == &y.w_uv || p == &y.w_o)) continue;
       cudaFree(*p);
       *p = nullptr;
     }
     h->weight_bytes -= std::min<uint64_t>(h->weight_bytes, freed);
   }
   // cache pools: one per layer with its own down projection, rows [c | rotated key part]
-  h->lat_pools.assign(h->L, nullptr);
-  // (pre-norm blocks: one K / V pool per EXECUTION of an attention layer, see LayerRun)
+  // (pre-norm blocks: one pool per EXECUTION of an attention layer, see LayerRun)
   const size_t n_pools = std::max((size_t)h->L, h->runs.size());
+  h->lat_pools.assign(n_pools, nullptr);
   h->win_kpools.assign(n_pools, nullptr);
   h->win_vpools.assign(n_pools, nullptr);
   for (size_t r = 0; r < h->runs.size(); r++) {
     const ListedLayer& y = h->ll[h->runs[r].layer];
     if (y.s.mixer != NVLLM_MIXER_ATTN_TMIX && y.s.mixer != NVLLM_MIXER_ATTENTION) continue;
     const size_t rows = (size_t)h->num_blocks * y.s.kv_heads * KV_BLOCK;
-    const size_t kb = rows * y.s.dim * dt_size(h->kvdt), vb = rows * y.s.vdim * dt_size(h->kvdt);
+    const size_t kb = rows * y.s.dim * (y.s.diff_maps ? 2 : 1) * dt_size(h->kvdt), vb = rows * y.s.vdim * dt_size(h->kvdt);
     cudaError_t e = cudaMalloc(&h->win_kpools[r], kb);
     if (e == cudaSuccess) e = cudaMalloc(&h->win_vpools[r], vb);
     if (e != cudaSuccess)
@@ -558,15 +604,15 @@ int layered_finalize(nvllm_handle* h) {
     NV_CHECK(h, cudaMalloc((void**)&h->pos_freq, (size_t)half * 8));
     NV_CHECK(h, cudaMemcpy(h->pos_freq, f.data(), (size_t)half * 8, cudaMemcpyHostToDevice));
   }
-  for (int l = 0; l < h->L; l++) {
-    ListedLayer& y = h->ll[l];
+  for (size_t r = 0; r < (h->runs.empty() ? (size_t)h->L : h->runs.size()); r++) {
+    ListedLayer& y = h->ll[h->runs.empty() ? (int)r : h->runs[r].layer];
     if (y.s.mixer != NVLLM_MIXER_LATENT_ATTENTION || y.s.kv_from >= 0) continue;
     const size_t bytes = (size_t)h->num_blocks * KV_BLOCK * y.Dk * dt_size(h->kvdt);
-    cudaError_t e = cudaMalloc(&h->lat_pools[l], bytes);
+    cudaError_t e = cudaMalloc(&h->lat_pools[r], bytes);
     if (e != cudaSuccess)
       return set_err(h, NVLLM_ERR_NOMEM, "latent cache of %d blocks does not fit: %s", h->num_blocks,
                      cudaGetErrorString(e));
-    NV_CHECK(h, cudaMemsetAsync(h->lat_pools[l], 0, bytes, h->stream));
+    NV_CHECK(h, cudaMemsetAsync(h->lat_pools[r], 0, bytes, h->stream));
     h->kv_bytes += bytes;
   }
   // rotation frequencies base^(-2i/dims), in double
@@ -758,10 +804,10 @@ static LinSeg seg_of(const Pending& p, int ld, int col) {
 template <typename Args>
 static void set_router(nvllm_handle* h, const ListedLayer& y, float* topk_w, Args* a) {
   const nvllm_layer_spec& s = y.s;
-  a->router = y.router; a->E = s.experts; a->topk = s.top;
+  a->router = y.router; a->E = s.experts + s.route_identity; a->topk = s.top;
   a->topk_idx = h->ws.topk_idx; a->topk_w = topk_w;
   a->route = RouteOpts{s.groups, s.keep_groups, s.route_norm ? 0 : 1, 1.f, s.route_sigmoid, s.weight_on_input,
-                       s.route_correction ? y.route_corr : nullptr, s.group_top2, y.route_bias};
+                       s.route_correction ? y.route_corr : nullptr, s.group_top2, y.route_bias, s.route_identity};
 }
 
 // A convolution between a norm and the sublayer that reads it
@@ -777,9 +823,10 @@ struct InputConv {
 // conv: the row passes a convolution first (and is routed after it).  In steps with one row per sequence
 // that happens in the norm kernel, the tail in the slot included; otherwise the normed rows stay in
 // conv->buf, *tail_job (n_jobs + 1) moves the tail once they have been read.  plain: no norm, xn = the updated x itself.
+// add_embed: the token's embedding (as it entered the first layer) joins x as well.
 static int run_prenorm(nvllm_handle* h, Pending* p1, Pending* p2, const float* row_m2, const float* xadd, const float* w,
                        const float* b, const ListedLayer* moe, float* topk_w, int T, const InputConv* conv = nullptr,
-                       TailJob* tail_job = nullptr, int* n_jobs = nullptr, bool plain = false) {
+                       TailJob* tail_job = nullptr, int* n_jobs = nullptr, bool plain = false, bool add_embed = false) {
   Workspace& ws = h->ws;
   const int32_t* d = h->lay.d;
   const bool fused = conv && T == h->lay.n;  // one row per sequence
@@ -801,6 +848,10 @@ static int run_prenorm(nvllm_handle* h, Pending* p1, Pending* p2, const float* r
     impl += (double)T * h->H * 4 * (p2->S - 1);
   }
   a.xadd = xadd;
+  if (add_embed) {
+    a.xadd_table = h->wte; a.xadd_tokens = d + h->lay.tokens; a.xadd_mult = h->cfg.embedding_multiplier;
+    bytes += (double)T * h->H * dt_size(h->wdt);
+  }
   a.w = w; a.b = b; a.eps = h->cfg.norm_eps; a.y = ws.xn; a.ydt = h->adt;
   if (fused) {
     a.conv_w = conv->w; a.conv_taps = conv->taps;
@@ -815,7 +866,7 @@ static int run_prenorm(nvllm_handle* h, Pending* p1, Pending* p2, const float* r
   if (moe && (fused || !conv)) {
     set_router(h, *moe, topk_w, &a);
     if (moe->sh_gate) { a.gate_w = moe->sh_gate; a.gate_out = ws.sh_gate; }
-    bytes += (double)moe->s.experts * h->H * 4;
+    bytes += (double)(moe->s.experts + moe->s.route_identity) * h->H * 4;
   }
   {
     ProfScope ps(h, NVLLM_K_NORM, bytes, 0, impl);
@@ -883,7 +934,9 @@ static int run_linrec(nvllm_handle* h, const LinRecArgs& a, double in_cols, int 
   {
     ProfScope ps(h, NVLLM_K_RECUR, (double)T * (in_cols * 4 + (3 * hd + hv) * 4) + hd * a.rank * 4, 2.0 * T * hd * a.rank,
                  (double)T * in_cols * 4 * (in_S - 1));
-    if (a.lower) {
+    if (a.gi.p) {
+      LAUNCH(h, launch_mlstm_prep(h->stream, a));
+    } else if (a.lower) {
       LAUNCH(h, launch_hgrn_prep(h->stream, a));
       sc.q = LinSeg{a.qkw, 1, 0, (int)(3 * hd)};
       sc.k = LinSeg{a.qkw + (size_t)hd, 1, 0, (int)(3 * hd)};
@@ -939,6 +992,30 @@ static int mixer_hgrn2(nvllm_handle* h, const ListedLayer& y, const LayerRun& r,
   a.q = seg_of(pin, y.n_in, 0); a.lr = seg_of(pin, y.n_in, hd); a.v = seg_of(pin, y.n_in, 2 * hd);
   a.w2b = y.lr_b; a.lower = y.f_lower;
   a.onorm_w = y.onorm_w;
+  a.o_ld = y.ov_p;
+  if ((rc = run_linrec(h, a, y.n_in, pin.S))) return rc;
+  return run_gemm(h, w.attn_out, y.ov_p, y.w_o, T, H, y.ov_p, 1.f, w.ws_b, w.ws_b_floats, H, out);
+}
+
+static int mixer_mlstm(nvllm_handle* h, const ListedLayer& y, const LayerRun& r, Pending* out) {
+  Workspace& w = h->ws;
+  const nvllm_layer_spec& s = y.s;
+  const int T = h->lay.T, H = h->H;
+  const int hd = s.heads * s.dim, hv = s.heads * s.vdim;
+  int rc;
+  Pending pin;
+  if ((rc = run_gemm(h, w.xn, H, y.w_in, T, y.n_in, H, 1.f, w.ws_a, w.ws_a_floats, y.n_in, &pin))) return rc;
+  LinRecArgs a{};
+  linrec_common(h, &a, r);
+  a.H = s.heads; a.dim = s.dim; a.vdim = s.vdim; a.tau = 1.f; a.qmul = 1.0f / sqrtf((float)s.dim);
+  a.q = seg_of(pin, y.n_in, 0); a.k = seg_of(pin, y.n_in, hd); a.v = seg_of(pin, y.n_in, 2 * hd);
+  a.gate = seg_of(pin, y.n_in, 2 * hd + hv);
+  a.gi = seg_of(pin, y.n_in, 2 * hd + 2 * hv); a.gf = seg_of(pin, y.n_in, 2 * hd + 2 * hv + s.heads);
+  a.gi_b = y.gate_b; a.gf_b = y.gate_b + s.heads; a.cap = s.gate_cap;
+  a.gates = w.ml_gates; a.nq = w.ml_nq;
+  a.decay_p = w.ml_gates; a.decay_ld = s.heads;
+  a.norm_off = r.norm_off; a.max_off = r.max_off;
+  a.onorm_w = y.onorm_w; a.onorm_ld = s.vdim;
   a.o_ld = y.ov_p;
   if ((rc = run_linrec(h, a, y.n_in, pin.S))) return rc;
   return run_gemm(h, w.attn_out, y.ov_p, y.w_o, T, H, y.ov_p, 1.f, w.ws_b, w.ws_b_floats, H, out);
@@ -1091,44 +1168,52 @@ static int ffn_poly(nvllm_handle* h, const ListedLayer& y, Pending* out) {
   return run_gemm(h, w.hbuf, ff, y.w2, T, H, ff, 1.f, w.ws_b, w.ws_b_floats, H, out);
 }
 
-// Mixture of gated experts: *p1 = the experts' outputs, combined by the next norm kernel; *p2 = the
-// always-on expert of the same form, if the layer has one
-static int ffn_moe_gated(nvllm_handle* h, const ListedLayer& y, float* topk_w, Pending* p1, Pending* p2) {
+// A gated unit W_down (act(W_gate h) * (W_up h)) of inner size ff: the unit rides in the up projection's epilogue (tcgen05,
+// no split-K), in the down projection's GEMV pre-stage (steps of <= 8 rows) or in its own kernel.  limit: see glu_unit
+static int ffn_glu(nvllm_handle* h, const ListedLayer& y, int ff, float limit, Pending* out) {
   Workspace& w = h->ws;
-  const nvllm_layer_spec& s = y.s;
   const int T = h->lay.T, H = h->H;
   const double asz = dt_size(h->adt);
-  int rc;
-  if ((rc = run_moe_ffn(h, T, w.xn, s.experts, s.top, y.ff_p, 0.f, y.moe_in, y.moe_out, topk_w, p1))) return rc;
-  if (s.shared_ff <= 0) return NVLLM_OK;
-  const int ff = y.sff_p;
   Pending h1;
-  if ((rc = run_gemm(h, w.xn, H, y.w1, T, 2 * ff, H, 1.f, w.ws_a, w.ws_a_floats, 2 * ff, &h1, TC5_EPI_SWIGLU, w.hbuf, ff, nullptr)))
-    return rc;
+  h->glu_limit_cur = limit;
+  const int rc = run_gemm(h, w.xn, H, y.w1, T, 2 * ff, H, 1.f, w.ws_a, w.ws_a_floats, 2 * ff, &h1, TC5_EPI_SWIGLU, w.hbuf, ff, nullptr);
+  h->glu_limit_cur = 0.f;
+  if (rc) return rc;
   // steps of <= 8 rows: the gated unit is built inside the down projection's GEMV (one launch less)
   const char* gpre_env = getenv("NVLLM_GEMV_PRE");
   if (h1.S > 0 && T <= 8 && !(gpre_env && atoi(gpre_env) == 0)) {
     GemvPre ga{};
-    ga.mode = 2; ga.hp = h1.p; ga.Sh = h1.S; ga.hstride = h1.stride; ga.hld = 2 * ff; ga.swiglu = 1;
-    return run_gemm(h, w.hbuf, ff, y.w2, T, H, ff, 1.f, w.ws_b, w.ws_b_floats, H, p2, 0, nullptr, 0, nullptr, nullptr, 0,
+    ga.mode = 2; ga.hp = h1.p; ga.Sh = h1.S; ga.hstride = h1.stride; ga.hld = 2 * ff; ga.swiglu = 1; ga.glu_limit = limit;
+    return run_gemm(h, w.hbuf, ff, y.w2, T, H, ff, 1.f, w.ws_b, w.ws_b_floats, H, out, 0, nullptr, 0, nullptr, nullptr, 0,
                     0.0, nullptr, nullptr, &ga);
   }
   if (h1.S > 0) {
     ProfScope ps(h, NVLLM_K_ACT, (double)T * ff * (8 + asz), 0, (double)T * 2 * ff * 4 * (h1.S - 1));
-    LAUNCH(h, launch_act(h->stream, h->adt, T, ff, h1.p, h1.S, h1.stride, nullptr, 1, w.hbuf));
+    LAUNCH(h, launch_act(h->stream, h->adt, T, ff, h1.p, h1.S, h1.stride, nullptr, 1, w.hbuf, limit));
   }
-  return run_gemm(h, w.hbuf, ff, y.w2, T, H, ff, 1.f, w.ws_b, w.ws_b_floats, H, p2);
+  return run_gemm(h, w.hbuf, ff, y.w2, T, H, ff, 1.f, w.ws_b, w.ws_b_floats, H, out);
+}
+
+// Mixture of gated experts: *p1 = the experts' outputs, combined by the next norm kernel; *p2 = the
+// always-on expert of the same form, if the layer has one (a gate per token is applied there too)
+static int ffn_moe_gated(nvllm_handle* h, const ListedLayer& y, float* topk_w, Pending* p1, Pending* p2) {
+  Workspace& w = h->ws;
+  const nvllm_layer_spec& s = y.s;
+  const int T = h->lay.T;
+  int rc;
+  if ((rc = run_moe_ffn(h, T, w.xn, s.experts, s.top, y.ff_p, 0.f, y.moe_in, y.moe_out, topk_w, p1))) return rc;
+  return s.shared_ff > 0 ? ffn_glu(h, y, y.sff_p, 0.f, p2) : NVLLM_OK;
 }
 
 // Prefill steps of an attention layer whose keys and values have one size, 64 or 128, in bf16, and whose scores are
-// neither capped nor biased by the distance (a sink and head gates are fine) run on the tcgen05 kernel
+// neither capped nor biased by the distance nor windowed nor two maps (a sink and head gates are fine) run on the tcgen05 kernel
 // (attention_tc5.cu, 128 queries per tile); everything else on the window kernels (attention_window.cu)
 static bool attention_on_tc5(const nvllm_handle* h, const nvllm_layer_spec& s) {
   return h->adt == DT_BF16 && h->kvdt == DT_BF16 && s.dim == s.vdim && (s.dim == 64 || s.dim == 128) &&
-         s.softcap == 0.f && s.dist_slope == 0.f && attn_prefill_tc5_enabled();
+         s.softcap == 0.f && s.dist_slope == 0.f && s.window == 0 && !s.diff_maps && attn_prefill_tc5_enabled();
 }
 
-// Grouped-query attention over the whole cached prefix with the options of the spec
+// Grouped-query attention over the cached prefix (or a window of it) with the options of the spec
 static int mixer_attention(nvllm_handle* h, const ListedLayer& y, int run_idx, Pending* out) {
   const StepLayout& L = h->lay;
   Workspace& w = h->ws;
@@ -1141,7 +1226,9 @@ static int mixer_attention(nvllm_handle* h, const ListedLayer& y, int run_idx, P
   if ((rc = run_gemm(h, w.xn, H, y.w_in, T, y.n_in, H, 1.f, w.ws_a, w.ws_a_floats, y.n_in, &pin))) return rc;
   WinAttnArgs a{};
   a.T = T; a.n_seqs = L.n; a.H = s.heads; a.G = s.kv_heads; a.dim = s.dim; a.vdim = s.vdim;
-  a.softcap = s.softcap; a.sink = s.sink; a.qk_norm = s.qk_norm; a.own_kv = 1;
+  a.window = s.window; a.softcap = s.softcap; a.sink = s.sink; a.qk_norm = s.qk_norm; a.own_kv = 1;
+  const int maps = s.diff_maps ? 2 : 1;
+  if (s.diff_maps) { a.maps = 2; a.diff_lambda = y.diff_lambda; a.out_mul = 1.f - s.diff; }
   a.eps = h->cfg.norm_eps; a.scale = s.scale;
   a.in_p = pin.p; a.in_S = pin.S; a.in_stride = pin.stride; a.in_ld = y.n_in;
   a.slots = d + L.slots;
@@ -1168,12 +1255,13 @@ static int mixer_attention(nvllm_handle* h, const ListedLayer& y, int run_idx, P
     a.tile_seq = d + L.tile_seq; a.tile_q0 = d + L.tile_q0; a.n_tiles = L.n_qtiles; a.qtile = h->attn_qtile;
   } else {
     a.n_tiles = L.n; a.qtile = 1;
-    // no window bounds the context: few sequences with long contexts would leave most SMs without a CTA, so the
+    // few sequences with long contexts (or wide windows) would leave most SMs without a CTA, so the
     // keys of a (sequence, key / value head) pair are cut into ranges.  The count depends on the number of
     // sequences only (a captured step replays with the same grid whatever the lengths have become)
     const int pairs = L.n * s.kv_heads;
     if (pairs <= w.att_split_pairs && pairs < 2 * h->sm_count) {
       a.n_split = std::min(WINATTN_MAX_SPLIT, std::max(1, 2 * h->sm_count / pairs));
+      if (s.window > 0) a.n_split = std::max(1, std::min(a.n_split, s.window / 256));  // (a range holds at least 256 keys)
       a.split_ws = w.att_split; a.split_cnt = w.att_split_cnt;
     }
   }
@@ -1184,10 +1272,12 @@ static int mixer_attention(nvllm_handle* h, const ListedLayer& y, int run_idx, P
     LAUNCH(h, launch_winattn_prep(h->stream, h->adt, h->kvdt, a));
   }
   {
-    // algorithmic: the K / V rows of every context once per step; flops over the visible pairs
+    // algorithmic: the K / V rows of every context (or window) once per step; flops over the visible pairs
+    const double win = s.window > 0 ? s.window : 1e30;
+    const double keys = std::min((double)L.sum_len, (double)L.n * (win - 1) + (double)T), pairs_seen = std::min(L.attn_pairs, (double)T * win);
     ProfScope ps(h, L.prefill ? NVLLM_K_ATTN_PREFILL : NVLLM_K_ATTN_DECODE,
-                 (double)L.sum_len * s.kv_heads * (s.dim + s.vdim) * kvsz, 2.0 * s.heads * (s.dim + s.vdim) * L.attn_pairs,
-                 (double)T * (s.heads * s.dim + y.ov_p) * asz);
+                 keys * s.kv_heads * (maps * s.dim + s.vdim) * kvsz, 2.0 * s.heads * maps * (s.dim + s.vdim) * pairs_seen,
+                 (double)T * (y.n_q + y.ov_p) * asz);
     if (L.prefill && h->attn_qtile == 128 && attention_on_tc5(h, s)) {
       AttnArgs t{};
       t.q = w.q; t.out = w.attn_out; t.qdt = h->adt; t.kvdt = h->kvdt;
@@ -1272,8 +1362,8 @@ static int mixer_mamba2(nvllm_handle* h, const ListedLayer& y, const LayerRun& r
   return run_gemm(h, w.attn_out, y.ov_p, y.w_o, T, H, y.ov_p, 1.f, w.ws_b, w.ws_b_floats, H, out);
 }
 
-// Latent attention on the normed rows in xn; its result stays pending in *out
-static int mixer_latent(nvllm_handle* h, const ListedLayer& y, Pending* out) {
+// Latent attention on the normed rows in xn over cache pool `pool`; its result stays pending in *out
+static int mixer_latent(nvllm_handle* h, const ListedLayer& y, int pool, Pending* out) {
   const StepLayout& L = h->lay;
   Workspace& w = h->ws;
   const nvllm_layer_spec& s = y.s;
@@ -1294,8 +1384,10 @@ static int mixer_latent(nvllm_handle* h, const ListedLayer& y, Pending* out) {
   a.dq_norm = y.dq_norm; a.dkv_norm = y.dkv_norm;
   a.cosT = rt.cosT; a.sinT = rt.sinT;
   a.slots = d + L.slots;
-  a.pool = h->lat_pools[y.pool];
+  a.pool = h->lat_pools[pool];
   a.cq = w.lat_cq; a.gate = y.lat_gate ? w.lat_gate : nullptr;
+  a.out_gate = s.out_gate ? w.att_gate : nullptr;
+  a.sink_w = s.sink_learned ? y.sink_w : nullptr;
   a.qabs = w.q;
   a.block_tables = d + L.block_tables; a.max_blocks = L.max_blocks;
   a.cu_q = d + L.cu_q; a.seq_start = d + L.seq_start; a.seq_len = d + L.seq_len;
@@ -1310,6 +1402,9 @@ static int mixer_latent(nvllm_handle* h, const ListedLayer& y, Pending* out) {
     a.n_splits = latent_attn_splits(n, s.heads, L.max_len, s.window, h->sm_count);
     while (a.n_splits > 1 && (size_t)T * s.heads * a.n_splits * (s.kv_rank + 2) > w.attn_ws_floats) a.n_splits--;
   }
+  // the gate sits between W_uv and W_o: with few rows and key splits their merge expands the values too
+  const bool expand_in_merge = s.out_gate && a.n_splits > 1 && T <= 16;
+  if (expand_in_merge) { a.exp_w = y.w_uv; a.exp_out = w.attn_out; a.exp_ld = y.ov_p; }
   {
     ProfScope ps(h, NVLLM_K_ROPE_KV, (double)T * y.n_in * 4 + (double)T * (y.q_rank_p * asz + own * y.Dk * kvsz), 0,
                  (double)T * y.n_in * 4 * (pin.S - 1));
@@ -1333,6 +1428,14 @@ static int mixer_latent(nvllm_handle* h, const ListedLayer& y, Pending* out) {
                  (double)T * (qn + y.ovr_p) * asz);
     LAUNCH(h, launch_latent_attn(st, h->adt, h->kvdt, a));
     if (a.n_splits > 1) h->launches++;
+  }
+  if (s.out_gate) {
+    if (!expand_in_merge) {
+      const double hv = (double)s.heads * s.vdim;
+      ProfScope ps(h, NVLLM_K_ATTN_PREFILL, hv * s.kv_rank * asz, 2.0 * T * hv * s.kv_rank, (double)T * (y.ovr_p * asz + hv * (4 + asz)));
+      LAUNCH(h, launch_latent_expand(st, h->adt, a, y.w_uv, w.attn_out, y.ov_p));
+    }
+    return run_gemm(h, w.attn_out, y.ov_p, y.w_o, T, H, y.ov_p, 1.f, w.ws_b, w.ws_b_floats, H, out);
   }
   return run_gemm(h, w.lat_o, y.ovr_p, y.w_ov, T, H, y.ovr_p, 1.f, w.ws_b, w.ws_b_floats, H, out);
 }
@@ -1368,11 +1471,12 @@ static int forward_layers_prenorm(nvllm_handle* h, Pending* p1, Pending* p2, con
   for (size_t ri = 0; ri < h->runs.size(); ri++) {
     const LayerRun& r = h->runs[ri];
     const ListedLayer& y = h->ll[r.layer];
-    const float* xadd = r.pass_start >= 0 ? h->loop_step + (size_t)r.pass_start * h->H : nullptr;
+    const float* xadd = r.pass_start >= 0 && h->loop_step ? h->loop_step + (size_t)r.pass_start * h->H : nullptr;
     TailJob jobs[TAIL_MAX_JOBS];
     int n_jobs = 0;
     const InputConv c1{y.canon_w, h->mixer_conv, r.canon_off, h->ws.xn_f32}, c2{y.canon2_w, h->ffn_conv, r.canon2_off, h->ws.xn2_f32};
-    if ((rc = run_prenorm(h, p1, p2, row_m2, xadd, y.post1_w, y.norm1_b, nullptr, nullptr, T, c1.w ? &c1 : nullptr, jobs, &n_jobs)))
+    if ((rc = run_prenorm(h, p1, p2, row_m2, xadd, y.post1_w, y.norm1_b, nullptr, nullptr, T, c1.w ? &c1 : nullptr, jobs, &n_jobs,
+                          false, h->loop_embed && r.pass_start > 0)))
       return rc;
     row_m2 = nullptr;
     Pending pa, pb, pin;
@@ -1380,7 +1484,8 @@ static int forward_layers_prenorm(nvllm_handle* h, Pending* p1, Pending* p2, con
     else if (y.s.mixer == NVLLM_MIXER_ATTENTION) rc = mixer_attention(h, y, (int)ri, &pa);
     else if (y.s.mixer == NVLLM_MIXER_MAMBA2) rc = mixer_mamba2(h, y, r, &pin, &pa);
     else if (y.s.mixer == NVLLM_MIXER_HGRN2) rc = mixer_hgrn2(h, y, r, &pa);
-    else if (y.s.mixer == NVLLM_MIXER_LATENT_ATTENTION) rc = mixer_latent(h, y, &pa);
+    else if (y.s.mixer == NVLLM_MIXER_MLSTM) rc = mixer_mlstm(h, y, r, &pa);
+    else if (y.s.mixer == NVLLM_MIXER_LATENT_ATTENTION) rc = mixer_latent(h, y, y.s.kv_from >= 0 ? y.pool : (int)ri, &pa);
     else rc = mixer_attn_tmix(h, y, r, (int)ri, &pa, &pb);
     if (rc) return rc;
     if (y.s.mixer == NVLLM_MIXER_MAMBA2 && y.s.conv > 1) {
@@ -1402,11 +1507,11 @@ static int forward_layers_prenorm(nvllm_handle* h, Pending* p1, Pending* p2, con
                             c2.w ? &c2 : nullptr, jobs, &n_jobs)))
         return rc;
       if ((rc = run_roll_tails(h, jobs, &n_jobs))) return rc;
-      if (!moe) rc = ffn_poly(h, y, p1);
+      if (!moe) rc = y.s.act == NVLLM_FFN_GEGLU ? ffn_glu(h, y, y.ff_p, GLU_TANH_GELU, p1) : ffn_poly(h, y, p1);
       else if (y.s.act == NVLLM_FFN_SWIGLU) rc = ffn_moe_gated(h, y, topk_w, p1, p2);
       else rc = ffn_moe_relu2(h, y, topk_w, p1, p2);
       if (rc) return rc;
-      row_m2 = moe && y.s.act == NVLLM_FFN_RELU2 && p2->p ? h->ws.sh_gate : nullptr;
+      row_m2 = moe && y.sh_gate && p2->p ? h->ws.sh_gate : nullptr;
     } else {
       *p1 = pa;
       *p2 = pb;
@@ -1471,7 +1576,7 @@ int forward_step_layered(nvllm_handle* h) {
                        s.mlp == NVLLM_MLP_MOE ? &ra : nullptr, true)))
       return rc;
     Pending pa;
-    if ((rc = mixer_latent(h, y, &pa))) return rc;
+    if ((rc = mixer_latent(h, y, y.pool, &pa))) return rc;
     // ---- feed-forward on the same normed input
     Pending pm;
     if (s.mlp == NVLLM_MLP_DENSE) {
@@ -1547,6 +1652,8 @@ static const char* latent_spec_error(const nvllm_layer_spec* layers, int l) {
   if (s.kv_rank > 512) return "kv_rank above 512";
   if (s.rot_dims < 2 || s.rot_dims > s.rot_dim || (s.rot_dims & 1)) return "rotated entries must be even and <= rot_dim";
   if (s.window < 0) return "negative window";
+  if (s.head_gate && s.out_gate) return "a gate per head or per entry, not both";
+  if (s.sink_learned && !s.sink) return "a learned sink needs sink = 1";
   if (s.kv_from >= 0) {
     if (s.kv_from >= l) return "kv_from must name an earlier layer";
     const nvllm_layer_spec& j = layers[s.kv_from];
@@ -1579,19 +1686,24 @@ extern "C" int nvllm_create_layered(const nvllm_layered_config* c, const nvllm_l
   if (c->mixer_conv < 0 || c->mixer_conv > INPUT_CONV_MAX_TAPS || c->ffn_conv < 0 || c->ffn_conv > INPUT_CONV_MAX_TAPS)
     return bad(-1, "convolution on a sublayer's input: at most 8 taps");
   if (c->side_dim < 0) return bad(-1, "negative side_dim");
+  if (c->loop_embed && (c->embed_norm || c->position == NVLLM_LPOS_SINUSOIDAL))
+    return bad(-1, "passes that open with the embedding need it to be the scaled table row");
   int vmix_first = -1;
   for (int l = 0; l < c->num_layers; l++) {
     const nvllm_layer_spec& s = layers[l];
     const bool seq_style = c->block_style == NVLLM_LBLOCK_SEQUENTIAL_POSTNORM;
     if (s.mixer == NVLLM_MIXER_ATTENTION || s.mixer == NVLLM_MIXER_MAMBA2 || s.mixer == NVLLM_MIXER_HGRN2 ||
-        (s.mixer == NVLLM_MIXER_LATENT_ATTENTION && pre_style)) {
-      if (!pre_style) return bad(l, "attention with options / Mamba-2 / HGRN2 need the sequential pre-norm block style");
+        s.mixer == NVLLM_MIXER_MLSTM || (s.mixer == NVLLM_MIXER_LATENT_ATTENTION && pre_style)) {
+      if (!pre_style) return bad(l, "attention with options / Mamba-2 / HGRN2 / mLSTM need the sequential pre-norm block style");
       if (s.heads <= 0 || s.vdim <= 0) return bad(l, "non-positive mixer size");
       if (s.mixer == NVLLM_MIXER_LATENT_ATTENTION) {
         if (const char* what = latent_spec_error(layers, l)) return bad(l, what);
-        if (has_loop) return bad(l, "latent attention has one cache per layer: no repeated run of layers");
+        if (has_loop && s.kv_from >= 0) return bad(l, "a repeated run of layers gives every pass a cache of its own: none to borrow");
       } else if (s.mixer == NVLLM_MIXER_HGRN2) {
         if (s.dim <= 0 || s.dim > LINREC_MAX_DIM) return bad(l, "HGRN2: 0 < dim <= 256");
+      } else if (s.mixer == NVLLM_MIXER_MLSTM) {
+        if (s.dim <= 0 || s.dim > LINREC_MAX_DIM) return bad(l, "mLSTM: 0 < dim <= 256");
+        if (!(s.gate_cap > 0.f)) return bad(l, "mLSTM: the gates' cap must be positive");
       } else if (s.mixer == NVLLM_MIXER_ATTENTION) {
         if (s.kv_heads <= 0 || s.dim <= 0 || s.heads % s.kv_heads) return bad(l, "heads must be a multiple of kv_heads");
         if (s.vdim > 512 || s.dim > 1024) return bad(l, "attention: dim <= 1024, vdim <= 512");
@@ -1600,6 +1712,9 @@ extern "C" int nvllm_create_layered(const nvllm_layered_config* c, const nvllm_l
         if (s.rot_piecewise && !(s.rot_factor > 0.f && s.rot_fast != s.rot_slow)) return bad(l, "piecewise frequency scaling: factor > 0, two different bounds");
         if (s.qtemp_coef > 0.f && s.qtemp_every <= 0) return bad(l, "query temperature: a positive step");
         if (s.sink_learned && !s.sink) return bad(l, "a learned sink needs sink = 1");
+        if (s.window < 0) return bad(l, "negative window");
+        if (s.diff_maps && (s.sink || s.head_gate || s.head_temp || s.softcap > 0.f || s.dist_slope > 0.f))
+          return bad(l, "two score maps have no sink, gate, temperature, cap or distance bias");
         if (s.v_mix) {
           if (vmix_first < 0) vmix_first = l;
           else if (layers[vmix_first].kv_heads != s.kv_heads || layers[vmix_first].vdim != s.vdim)
@@ -1613,15 +1728,20 @@ extern "C" int nvllm_create_layered(const nvllm_layered_config* c, const nvllm_l
         if (s.conv < 1 || s.conv > 8) return bad(l, "convolution taps 1..8");
       }
       if (s.mlp < NVLLM_MLP_NONE || s.mlp > NVLLM_MLP_MOE) return bad(l, "unknown feed-forward kind");
-      if (s.mlp == NVLLM_MLP_DENSE && (s.ff <= 0 || s.act != NVLLM_FFN_POLYNORM)) return bad(l, "pre-norm blocks: a dense feed-forward has ff > 0 and the PolyNorm activation");
-      if (s.mlp == NVLLM_MLP_DENSE && s.ff > 48 * 1024) return bad(l, "PolyNorm: ff <= 49152");
+      if (s.mlp == NVLLM_MLP_DENSE && (s.ff <= 0 || (s.act != NVLLM_FFN_POLYNORM && s.act != NVLLM_FFN_GEGLU)))
+        return bad(l, "pre-norm blocks: a dense feed-forward has ff > 0 and the PolyNorm or the tanh-GELU gated activation");
+      if (s.mlp == NVLLM_MLP_DENSE && s.act == NVLLM_FFN_POLYNORM && s.ff > 48 * 1024) return bad(l, "PolyNorm: ff <= 49152");
       if (s.mlp == NVLLM_MLP_MOE) {
         if (s.shared_ff < 0) return bad(l, "negative shared_ff");
         if (s.act != NVLLM_FFN_SWIGLU) return bad(l, "these blocks take gated experts W_down (silu(W_gate h) * W_up h)");
-        if (s.ff <= 0 || s.experts <= 0 || s.experts > 256 || s.top <= 0 || s.top > 32 || s.top > s.experts)
-          return bad(l, "ff > 0, experts 1..256, top 1..32");
+        const int outs = s.experts + s.route_identity;
+        if (s.ff <= 0 || s.experts <= 0 || s.route_identity < 0 || outs > 256 || s.top <= 0 || s.top > 32 || s.top > outs)
+          return bad(l, "ff > 0, experts 1..256 (identity ones included), top 1..32");
+        if (s.route_identity > 0 && (s.route_sigmoid || s.route_norm || s.groups > 1 || c->ffn_conv > 0))
+          return bad(l, "identity experts: softmax scores as they are, no groups, no convolution ahead of the feed-forward");
+        if (s.shared_gate && c->ffn_conv > 0) return bad(l, "an always-on expert with a gate: no convolution ahead of the feed-forward");
         const int g = s.groups > 0 ? s.groups : 1, keep = s.groups > 0 ? s.keep_groups : 1;
-        if (s.experts % g || keep <= 0 || keep > g || keep * (s.experts / g) < s.top)
+        if (outs % g || keep <= 0 || keep > g || keep * (outs / g) < s.top)
           return bad(l, "expert groups must divide the experts and the kept groups must hold `top` experts");
       }
       continue;
@@ -1677,7 +1797,8 @@ extern "C" int nvllm_create_layered(const nvllm_layered_config* c, const nvllm_l
     if (s.mixer != NVLLM_MIXER_LATENT_ATTENTION) return bad(l, "unknown mixer kind");
     if (seq_style) return bad(l, "latent attention needs the parallel pre-norm block style");
     if (const char* what = latent_spec_error(layers, l)) return bad(l, what);
-    if (s.window > 0 || s.rot_pairs) return bad(l, "latent attention in parallel blocks: no window, halves rotated");
+    if (s.window > 0 || s.rot_pairs || s.sink || s.out_gate || s.rot_factor > 0.f)
+      return bad(l, "latent attention in parallel blocks: no window, sink or entry-wise gate, halves rotated, plain frequencies");
     if (s.mlp < NVLLM_MLP_NONE || s.mlp > NVLLM_MLP_MOE) return bad(l, "unknown feed-forward kind");
     if (s.mlp != NVLLM_MLP_NONE && s.ff <= 0) return bad(l, "ff must be positive");
     if (s.mlp != NVLLM_MLP_NONE && !(s.limit > 0.f)) return bad(l, "limit must be positive");
@@ -1736,6 +1857,7 @@ extern "C" int nvllm_create_layered(const nvllm_layered_config* c, const nvllm_l
   h->mixer_conv = c->mixer_conv;
   h->ffn_conv = c->ffn_conv;
   h->layer_norm = c->layer_norm != 0;
+  h->loop_embed = c->loop_embed != 0;
   h->side_dim = c->side_dim;
   h->side_p = (int)up8((size_t)c->side_dim);
   h->logit_scale = c->logit_scale;
@@ -1790,19 +1912,22 @@ extern "C" int nvllm_create_layered(const nvllm_layered_config* c, const nvllm_l
     const nvllm_layer_spec& s = y.s;
     y.lat_gate = !pre_style || s.head_gate;
     y.Dk = s.kv_rank + s.rot_dim;
-    y.n_in = s.q_rank + (s.kv_from < 0 ? y.Dk : 0) + (y.lat_gate ? s.heads : 0);
+    y.n_in = s.q_rank + (s.kv_from < 0 ? y.Dk : 0) + (s.out_gate ? s.heads * s.vdim : y.lat_gate ? s.heads : 0);
     y.q_cols = s.heads * (s.dim + s.rot_dim);
     y.q_rank_p = (int)up8(s.q_rank);
     y.ovr_p = (int)up8((size_t)s.heads * s.kv_rank);
     y.pool = s.kv_from < 0 ? l : s.kv_from;
     for (size_t r = 0; r < h->ropes.size(); r++) {
       const RopeTable& t = h->ropes[r];
-      if (t.base == (double)s.rot_base && t.dims == s.rot_dims && t.factor == 0) y.rope = (int)r;
+      if (t.base == (double)s.rot_base && t.dims == s.rot_dims && t.factor == (double)s.rot_factor &&
+          t.original == (double)s.rot_original && t.fast == (double)s.rot_fast && t.slow == (double)s.rot_slow && !t.piecewise)
+        y.rope = (int)r;
     }
     if (y.rope < 0) {
       RopeTable rt;
       rt.base = s.rot_base;
       rt.dims = s.rot_dims;
+      rt.factor = s.rot_factor; rt.original = s.rot_original; rt.fast = s.rot_fast; rt.slow = s.rot_slow;
       y.rope = (int)h->ropes.size();
       h->ropes.push_back(rt);
     }
@@ -1813,9 +1938,10 @@ extern "C" int nvllm_create_layered(const nvllm_layered_config* c, const nvllm_l
     if (ce == cudaSuccess) ce = alloc(&y.w_uk, (size_t)s.heads * s.dim * s.kv_rank * wsz);
     if (ce == cudaSuccess) ce = alloc(&y.w_uv, (size_t)s.heads * s.vdim * s.kv_rank * wsz);
     if (ce == cudaSuccess) ce = alloc(&y.w_q, (size_t)s.heads * y.Dk * y.q_rank_p * wsz);
-    if (ce == cudaSuccess) ce = alloc(&y.w_ov, (size_t)W * y.ovr_p * wsz);
+    if (ce == cudaSuccess && !s.out_gate) ce = alloc(&y.w_ov, (size_t)W * y.ovr_p * wsz);
+    if (ce == cudaSuccess && s.sink_learned) ce = alloc((void**)&y.sink_w, (size_t)s.heads * 4);
     qkv_cols = std::max(qkv_cols, std::max(y.n_in, s.heads * y.Dk));
-    q_cols = std::max(q_cols, s.heads * y.Dk);
+    q_cols = std::max(q_cols, std::max(s.heads * y.Dk, s.out_gate ? y.ov_p : 0));
     h->nh = std::max(h->nh, s.heads);
     h->hd = std::max(h->hd, s.kv_rank);
     return ce;
@@ -1843,8 +1969,10 @@ extern "C" int nvllm_create_layered(const nvllm_layered_config* c, const nvllm_l
       y.ff_p = (int)up8((size_t)std::max(s.ff, 0));
       AL(y.post1_w, (size_t)W * 4);
       if (s.mixer == NVLLM_MIXER_ATTENTION) {
-        y.n_q = s.heads * s.dim; y.n_k = s.kv_heads * s.dim; y.n_v = s.kv_heads * s.vdim;
+        const int maps = s.diff_maps ? 2 : 1;
+        y.n_q = s.heads * maps * s.dim; y.n_k = s.kv_heads * maps * s.dim; y.n_v = s.kv_heads * s.vdim;
         y.n_in = y.n_q + y.n_k + y.n_v + (s.head_gate ? s.heads : 0);  // Q | K | V | head gates
+        if (s.diff_maps) AL(y.diff_w, (size_t)4 * s.dim * 4);
         AL(y.w_in, (size_t)y.n_in * W * wsz);
         if (s.qk_norm == 3) {
           AL(y.qnorm_w, (size_t)s.dim * 4);
@@ -1874,7 +2002,7 @@ extern "C" int nvllm_create_layered(const nvllm_layered_config* c, const nvllm_l
           }
         }
         // (a model whose attention layers all fit the tcgen05 kernel gets its tiles of 128 queries)
-        const int qt = attention_on_tc5(h, s) ? 128 : winattn_qtile(h->adt, h->kvdt, s.dim, s.vdim);
+        const int qt = attention_on_tc5(h, s) ? 128 : winattn_qtile(h->adt, h->kvdt, s.dim, s.vdim, maps);
         win_qtile = win_qtile ? std::min(win_qtile, qt) : qt;
         q_cols = std::max(q_cols, std::max(y.n_q, y.ov_p));
       } else if (s.mixer == NVLLM_MIXER_HGRN2) {
@@ -1883,6 +2011,13 @@ extern "C" int nvllm_create_layered(const nvllm_layered_config* c, const nvllm_l
         AL(y.lr_b, (size_t)s.heads * s.dim * 4);
         AL(y.f_lower, (size_t)s.heads * s.dim * 4);
         AL(y.onorm_w, (size_t)s.vdim * 4);
+        q_cols = std::max(q_cols, y.ov_p);
+      } else if (s.mixer == NVLLM_MIXER_MLSTM) {
+        // q | k | v | gate | i | f; padded, so that every row of the projection starts on a 16-byte boundary
+        y.n_in = (int)up8((size_t)2 * s.heads * s.dim + 2 * hv + 2 * s.heads);
+        AL(y.w_in, (size_t)y.n_in * W * wsz);
+        AL(y.gate_b, (size_t)2 * s.heads * 4);
+        AL(y.onorm_w, (size_t)hv * 4);
         q_cols = std::max(q_cols, y.ov_p);
       } else if (s.mixer == NVLLM_MIXER_LATENT_ATTENTION) {
         if ((e = alloc_latent(y, l)) != cudaSuccess) return fail(e, "cudaMalloc(weights)");
@@ -1902,24 +2037,27 @@ extern "C" int nvllm_create_layered(const nvllm_layered_config* c, const nvllm_l
       AL(y.w_o, (size_t)W * y.ov_p * wsz);
       if (s.mlp == NVLLM_MLP_DENSE) {
         AL(y.post2_w, (size_t)W * 4);
-        AL(y.w1, (size_t)y.ff_p * W * wsz);
+        const int cols = (s.act == NVLLM_FFN_GEGLU ? 2 : 1) * y.ff_p;  // gate / up rows interleaved, or up
+        AL(y.w1, (size_t)cols * W * wsz);
         AL(y.w2, (size_t)W * y.ff_p * wsz);
-        AL(y.poly, 4 * 4);
+        if (s.act == NVLLM_FFN_POLYNORM) AL(y.poly, 4 * 4);
         h->F = std::max(h->F, y.ff_p);
-        qkv_cols = std::max(qkv_cols, y.ff_p);
+        qkv_cols = std::max(qkv_cols, cols);
       }
       if (s.mlp == NVLLM_MLP_MOE) {
         AL(y.post2_w, (size_t)W * 4);
-        AL(y.router, (size_t)s.experts * W * 4);
-        if (s.route_bias) AL(y.route_bias, (size_t)s.experts * 4);
+        const int outs = s.experts + s.route_identity;
+        AL(y.router, (size_t)outs * W * 4);
+        if (s.route_bias) AL(y.route_bias, (size_t)outs * 4);
         if (s.shared_ff > 0) {
           y.sff_p = (int)up8((size_t)s.shared_ff);
           AL(y.w1, (size_t)2 * y.sff_p * W * wsz);
           AL(y.w2, (size_t)W * y.sff_p * wsz);
+          if (s.shared_gate) AL(y.sh_gate, (size_t)W * 4);
           h->F = std::max(h->F, y.sff_p);
           qkv_cols = std::max(qkv_cols, 2 * y.sff_p);
         }
-        if (s.route_correction) AL(y.route_corr, (size_t)s.experts * 4);
+        if (s.route_correction) AL(y.route_corr, (size_t)outs * 4);
         AL(y.moe_in, (size_t)s.experts * 2 * y.ff_p * W * wsz);
         AL(y.moe_out, (size_t)s.experts * W * y.ff_p * wsz);
         h->moe = true;
@@ -2103,6 +2241,10 @@ extern "C" int nvllm_create_layered(const nvllm_layered_config* c, const nvllm_l
         h->state_slot_floats = up4(r.tail_off + (size_t)(s.conv - 1) * h->ll[l].conv_ch);
       } else if (s.mixer == NVLLM_MIXER_GLA || s.mixer == NVLLM_MIXER_HGRN2) {
         h->state_slot_floats = up4(r.state_off + (size_t)s.heads * s.dim * s.vdim);
+      } else if (s.mixer == NVLLM_MIXER_MLSTM) {
+        r.norm_off = up4(r.state_off + (size_t)s.heads * s.dim * s.vdim);
+        r.max_off = up4(r.norm_off + (size_t)s.heads * s.dim);
+        h->state_slot_floats = up4(r.max_off + (size_t)s.heads);
       } else {
         r.tail_off = up4(r.state_off + (size_t)s.heads2 * s.dim2 * s.dim2);
         r.shift_off = up4(r.tail_off + (size_t)(s.conv - 1) * h->ll[l].conv_ch);
@@ -2116,7 +2258,7 @@ extern "C" int nvllm_create_layered(const nvllm_layered_config* c, const nvllm_l
     for (int t = 0; t < (loop ? h->loop_times : 0); t++)
       for (int l = a0; l < a1; l++) add_run(l, l == a0 ? t : -1);
     for (int l = a1; l < h->L; l++) add_run(l, -1);
-    if (loop) AL(h->loop_step, (size_t)h->loop_times * W * 4);
+    if (loop && !h->loop_embed) AL(h->loop_step, (size_t)h->loop_times * W * 4);
   }
 #undef AL
   h->attn_qtile = win_qtile ? win_qtile : latent_attn_qtile();

@@ -98,6 +98,11 @@ struct ListedLayer {
   float* route_bias = nullptr;      // [experts]: added to the router's logits
   float* poly = nullptr;            // [4]: coefficients of the PolyNorm activation
   int lat_gate = 0;                 // latent attention: the fused input projection holds gate rows
+  float diff_lambda = 0.f;          // attention with two maps: what the second map is multiplied by
+  float* diff_w = nullptr;          // [4][dim]: the vectors lq1 | lk1 | lq2 | lk2 it comes from (read at finalize)
+  // mLSTM: fused projection rows [q | k | v | gate | i | f | padding to 8] in w_in, the gates' additive terms [i | f] here,
+  // the norm weight [heads vdim] in onorm_w
+  float* gate_b = nullptr;
   void *side_gate = nullptr, *side_proj = nullptr;  // per-layer token input: [side_p, W], [W, side_p]
   float* side_norm = nullptr;       // [W]
 };
@@ -105,10 +110,12 @@ struct ListedLayer {
 // time with caches and state of its own.
 struct LayerRun {
   int layer = 0;
-  int pass_start = -1;   // >= 0: this run opens pass `pass_start` (the pass's vector is added to x first)
+  int pass_start = -1;   // >= 0: this run opens pass `pass_start` (the pass's vector, or from the second pass on the
+                         // embedding, is added to x first)
   size_t state_off = 0;  // recurrent state [heads][dim][vdim] (time mixing: [heads2][dim2][dim2]) inside a slot
   size_t tail_off = 0;   // attention side: convolution tail [taps - 1][n_q + n_k + n_v]
   size_t shift_off = 0;  // time mixing: the previous token's input [W]
+  size_t norm_off = 0, max_off = 0;      // mLSTM: the vector n [heads][dim] and the running maximum m [heads]
   size_t canon_off = 0, canon2_off = 0;  // tails [taps - 1][W] of the convolutions on the mixer's / the feed-forward's input
 };
 struct RopeTable {
@@ -188,6 +195,7 @@ struct Workspace {
   // time mixing's five shifted inputs [5][T][W] act dtype; attention output gates [T, max heads vdim] and
   // the always-on expert's gate [T] fp32
   float *lr_qkw = nullptr, *lr_v = nullptr, *lr_o = nullptr, *att_gate = nullptr, *sh_gate = nullptr;
+  float *ml_gates = nullptr, *ml_nq = nullptr;  // mLSTM: [3][T, max heads] gates, [T, max heads] n . q
   void* mx_in = nullptr;
   // Mamba-2 with state slots: activated convolution outputs [T, max channels], dt x [T, max inner], decays [T, max heads];
   // the values of the first value-mixing attention layer [T, kv_heads vdim] fp32; the per-layer token input's gated
@@ -257,13 +265,14 @@ struct nvllm_handle {
   // model given as a list of layers (nvllm_create_layered, forward_layered.cu)
   bool layered = false;
   std::vector<nvllm::ListedLayer> ll;
-  std::vector<void*> lat_pools;          // per cache-owning layer: [num_blocks * 256][Dk]
+  std::vector<void*> lat_pools;          // per cache-owning layer (pre-norm blocks: per execution): [num_blocks * 256][Dk]
   // window attention: per cache-owning layer K [num_blocks][kv_heads][256][dim], V [...][vdim]
   std::vector<void*> win_kpools, win_vpools;
   // sequential pre-norm blocks: the layer executions of a step in order (K / V pools above are
   // indexed by execution there), the vectors that open the passes of the repeated run [times][W]
   std::vector<nvllm::LayerRun> runs;
   float* loop_step = nullptr;
+  bool loop_embed = false;  // the passes after the first open with the embedding instead
   int loop_start = 0, loop_stop = 0, loop_times = 0;  // times >= 1 with stop > start: a repeated run exists
   // further options of the sequential pre-norm blocks (nvllm_layered_config)
   int norm_groups = 0, mixer_conv = 0, ffn_conv = 0, side_dim = 0, side_p = 0;

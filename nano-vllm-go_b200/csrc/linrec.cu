@@ -5,16 +5,22 @@
 //   gated linear attention   a_t = sigmoid(z_t)^(1 / tau),  S <- diag(a_t) S + k_t v_t^T,  o_t = S^T q_t
 //   time mixing              w_t = exp(-exp(z_t)),  o_t = (S + diag(u) k_t v_t^T)^T r_t,  S <- diag(w_t) S + k_t v_t^T
 //   HGRN2                    f_t = l + (1 - l) sigmoid(z_t),  S <- diag(f_t) S + (1 - f_t) v_t^T,  o_t = S^T silu(q_t)
+//   mLSTM                    S <- a_t S + b_t k_t v_t^T,  n <- a_t n + b_t k_t,  o_t = S^T q_t / (max(|n . q_t|, c_t) + 1e-6)
+//                            a_t = exp(f_t + m_(t-1) - m_t), b_t = exp(i_t - m_t), c_t = exp(-m_t), m_t = max(f_t + m_(t-1), i_t)
 // with z_t = W_2 f(W_1 x_t) + b per (head, key entry): f = identity / tanh.  The decay rows belong to
 // key entries.  (HGRN2: z_t = W_f x_t + b, one projection, and the
 // gate also is the key.)  The read-out of a head is divided by its root mean square, multiplied by a weight
-// and (HGRN2: not) by silu(gate) and goes to the output projection.
+// and (HGRN2: not) by silu(gate) and goes to the output projection.  mLSTM: one forget and one input gate per head,
+// given as logarithms f_t = log sigmoid(g(z)), i_t = g(z), g(z) = cap tanh(z / cap); S and n are kept relative to the
+// running maximum m_t (0 before the first token); weight per entry of all heads, sigmoid(gate).
 //
 //   linrec_prep_kernel   per tile of tokens: split-K sums of the projections, q scaled, the second step of
 //                        the decay's projection (fp32 FMA, the inner size is small) and the decay itself —
 //                        logarithms, exponentials and sigmoids in fp32 (log-sigmoid form, no overflow).
 //   hgrn_prep_kernel     HGRN2's epilogue: silu(q), the bounded gate and its complement (neither by a
 //                        subtraction from one: both sides of the sigmoid come from one exponential).
+//   mlstm_prep_kernel    mLSTM's: the gates' logarithms and the running maximum, which is a scan over the tokens (the
+//                        pairs (sum of f, maximum) compose associatively: no long sums of f are subtracted), a | b | c.
 //   linrec_scan_kernel   CTA = (sequence, head, range of value columns).  The state sits in registers, a tile of
 //                        8 rows by CN columns per lane, updated with packed fp32 instructions.  Token inputs are
 //                        staged through shared memory in chunks, the next chunk's loads in flight (cp.async)
@@ -250,6 +256,88 @@ cudaError_t launch_hgrn_prep(cudaStream_t st, const LinRecArgs& a) {
   return cudaGetLastError();
 }
 
+// ---- mLSTM
+__device__ __forceinline__ void mlstm_log_gates(float zi, float zf, float cap, float* gi, float* gf) {
+  *gi = cap * tanhf(zi / cap);
+  const float x = cap * tanhf(zf / cap);
+  *gf = fminf(x, 0.f) - log1pf(expf(-fabsf(x)));  // log sigmoid(x)
+}
+// The first n_seqs * H CTAs: one (sequence, head) each, 256 tokens at a time.  Token t takes the running maximum m to
+// max(m + F, I) with (F, I) = (f_t, i_t), and two such steps compose to (F1 + F2, max(I1 + F2, I2)): a warp scans its 32
+// tokens by shuffles, the warps' totals meet in shared memory.  The others sum q, k and v's slices (none when direct).
+constexpr int MP_NT = 256;
+__global__ void __launch_bounds__(MP_NT) mlstm_prep_kernel(LinRecArgs a, Trace tr) {
+  TRACE_ENTRY(tr);
+  pdl_launch_dependents();
+  pdl_wait();
+  const int n_gate = a.n_seqs * a.H;
+  if ((int)blockIdx.x >= n_gate) {
+    const int hd = a.H * a.dim, hv = a.H * a.vdim;
+    for (int t = blockIdx.x - n_gate; t < a.T; t += gridDim.x - n_gate) {
+      float* qkw = a.qkw + (size_t)t * 3 * hd;
+      for (int c = threadIdx.x; c < hd; c += MP_NT) {
+        qkw[c] = seg_at(a.q, t, c);
+        qkw[hd + c] = seg_at(a.k, t, c);
+      }
+      for (int c = threadIdx.x; c < hv; c += MP_NT) a.vv[(size_t)t * hv + c] = seg_at(a.v, t, c);
+    }
+    TRACE_EXIT(tr);
+    return;
+  }
+  __shared__ float sF[MP_NT / 32], sI[MP_NT / 32], s_last;
+  const int seq = blockIdx.x / a.H, head = blockIdx.x % a.H;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int r0 = a.cu_q[seq], n_new = a.cu_q[seq + 1] - r0;
+  if (n_new <= 0) return;
+  float* top = a.state_pool + (size_t)a.state_slots[seq] * a.slot_floats + a.max_off + head;
+  float m0 = a.positions[r0] > 0 ? *top : 0.f;
+  const size_t plane = (size_t)a.T * a.H;
+  for (int t0 = 0; t0 < n_new; t0 += MP_NT) {
+    const int t = t0 + threadIdx.x;
+    const bool ok = t < n_new;
+    float gi = -INFINITY, gf = 0.f;
+    if (ok) mlstm_log_gates(seg_at(a.gi, r0 + t, head) + a.gi_b[head], seg_at(a.gf, r0 + t, head) + a.gf_b[head], a.cap, &gi, &gf);
+    float F = gf, I = gi;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float F1 = __shfl_up_sync(0xffffffffu, F, o), I1 = __shfl_up_sync(0xffffffffu, I, o);
+      if (lane >= o) {
+        I = fmaxf(I1 + F, I);
+        F += F1;
+      }
+    }
+    if (lane == 31) {
+      sF[warp] = F;
+      sI[warp] = I;
+    }
+    __syncthreads();
+    float base = m0;  // the maximum before the warp's first token
+    for (int w = 0; w < warp; w++) base = fmaxf(base + sF[w], sI[w]);
+    const float m = fmaxf(base + F, I);
+    float prev = __shfl_up_sync(0xffffffffu, m, 1);
+    if (lane == 0) prev = base;
+    if (ok) {
+      float* g = a.gates + (size_t)(r0 + t) * a.H + head;
+      g[0] = expf(gf + prev - m);
+      g[plane] = expf(gi - m);
+      g[2 * plane] = expf(-m);
+    }
+    if (threadIdx.x == MP_NT - 1) s_last = m;  // (tokens past the end leave the maximum as it is)
+    __syncthreads();
+    m0 = s_last;
+  }
+  if (threadIdx.x == 0) *top = m0;
+  TRACE_EXIT(tr);
+}
+
+cudaError_t launch_mlstm_prep(cudaStream_t st, const LinRecArgs& a) {
+  if (a.T <= 0) return cudaSuccess;
+  if (!a.gi.p || !a.gf.p || !a.gates || !(a.cap > 0.f)) return cudaErrorInvalidValue;
+  const int sums = linrec_direct(a) ? 0 : std::min(a.T, 148 * 8);
+  (void)launch_k(mlstm_prep_kernel, dim3(a.n_seqs * a.H + sums), dim3(MP_NT), 0, st, a, next_trace(40));
+  return cudaGetLastError();
+}
+
 // ------------------------------------------------------------------ scan over tokens
 // A lane holds a tile of the state, 8 rows (four packed pairs of neighbouring rows) by CN value columns, in
 // registers; a warp covers 8 RG rows by (32 / RG) CN columns, a CTA's WR warps the rows of the head.  Per token a
@@ -277,8 +365,9 @@ __device__ __forceinline__ void unpack2(unsigned long long v, float& lo, float& 
 }
 
 // DP: rows of the state, padded (RG * 8 * WR); TMIX: read before the update, with a bonus; SD: one decay per
-// (token, head) instead of one per row
-template <int RG, int WR, int CN, bool TMIX, bool SD>
+// (token, head) instead of one per row; NRM (with SD): mLSTM — keys are scaled by the token's input gate, and the CTAs of
+// the first column range carry the vector n beside the state (every column group of lanes holds its 8 entries)
+template <int RG, int WR, int CN, bool TMIX, bool SD, bool NRM>
 __global__ void __launch_bounds__(32 * WR) linrec_scan_kernel(LinRecArgs a, int vec16, Trace tr) {
   TRACE_ENTRY(tr);
   pdl_launch_dependents();
@@ -288,6 +377,7 @@ __global__ void __launch_bounds__(32 * WR) linrec_scan_kernel(LinRecArgs a, int 
   constexpr int NO = CN >= RG ? CN / RG : 1;                   // columns a lane holds after the shuffles
   __shared__ __align__(16) float stage[2][TC][ROW];
   __shared__ float part[WR][TC][VC];
+  __shared__ float part_n[NRM ? WR : 1][TC];
   const int seq = blockIdx.x, head = blockIdx.y, col0 = blockIdx.z * VC;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int rg = lane / CG, cg = lane % CG;
@@ -338,8 +428,11 @@ __global__ void __launch_bounds__(32 * WR) linrec_scan_kernel(LinRecArgs a, int 
       }
     }
     if (SD)
-      for (int tt = tid; tt < TC; tt += NT)
-        lr_cp_async4(smem_addr(&stage[buf][tt][2 * DP]), part_p[2] + (size_t)(r0 + t0 + (tt < nt ? tt : 0)) * part_ld[2], tt < nt);
+      for (int tt = tid; tt < TC; tt += NT) {
+        const size_t t = r0 + t0 + (tt < nt ? tt : 0);
+        lr_cp_async4(smem_addr(&stage[buf][tt][2 * DP]), part_p[2] + t * part_ld[2], tt < nt);
+        if (NRM) lr_cp_async4(smem_addr(&stage[buf][tt][2 * DP + 1]), a.gates + ((size_t)a.T + t) * a.H + head, tt < nt);
+      }
   };
   load_chunk(0, 0);
   cp_async_commit();
@@ -362,6 +455,16 @@ __global__ void __launch_bounds__(32 * WR) linrec_scan_kernel(LinRecArgs a, int 
       U[p] = pack2(r < dim ? a.bonus[head * dim + r] : 0.f, r + 1 < dim ? a.bonus[head * dim + r + 1] : 0.f);
     }
   }
+
+  const bool with_n = NRM && blockIdx.z == 0;
+  float* nvec = NRM ? a.state_pool + (size_t)a.state_slots[seq] * a.slot_floats + a.norm_off + (size_t)head * dim : nullptr;
+  unsigned long long N[NRM ? 4 : 1];
+  if (NRM)
+#pragma unroll
+    for (int p = 0; p < 4; p++) {
+      const int r = row0 + 2 * p;
+      N[NRM ? p : 0] = pack2(with_n && has_prev && r < dim ? nvec[r] : 0.f, with_n && has_prev && r + 1 < dim ? nvec[r + 1] : 0.f);
+    }
 
   const int n_chunks = (n_new + TC - 1) / TC;
   for (int ch = 0; ch < n_chunks; ch++) {
@@ -390,6 +493,26 @@ __global__ void __launch_bounds__(32 * WR) linrec_scan_kernel(LinRecArgs a, int 
       if (SD) {
         const float d = row[2 * DP];
         w[0] = w[1] = w[2] = w[3] = pack2(d, d);
+      }
+      if (NRM) {
+        const float b = row[2 * DP + 1];
+        const unsigned long long bb = pack2(b, b);
+#pragma unroll
+        for (int p = 0; p < 4; p++) k[p] = mul2(k[p], bb);
+        if (with_n) {
+          unsigned long long ac = 0ull;
+#pragma unroll
+          for (int p = 0; p < 4; p++) {
+            N[NRM ? p : 0] = fma2(w[p], N[NRM ? p : 0], k[p]);
+            ac = fma2(q[p], N[NRM ? p : 0], ac);
+          }
+          float lo, hi;
+          unpack2(ac, lo, hi);
+          float s = lo + hi;
+#pragma unroll
+          for (int off = 16; off >= CG; off >>= 1) s += __shfl_xor_sync(0xffffffffu, s, off);
+          if (lane == 0) part_n[NRM ? warp : 0][tt] = s;
+        }
       }
       const float* vr = row + 3 * DP + cg * CN;
       if constexpr (CN >= 4) {
@@ -455,8 +578,24 @@ __global__ void __launch_bounds__(32 * WR) linrec_scan_kernel(LinRecArgs a, int 
       for (int w = 0; w < WR; w++) t += part[w][tt][c];
       if (col0 + c < vdim) a.o[(size_t)(r0 + ch * TC + tt) * hv + head * vdim + col0 + c] = t * a.qmul;
     }
+    if (with_n)
+      for (int tt = tid; tt < nt; tt += NT) {
+        float t = 0.f;
+#pragma unroll
+        for (int w = 0; w < WR; w++) t += part_n[NRM ? w : 0][tt];
+        a.nq[(size_t)(r0 + ch * TC + tt) * a.H + head] = t * a.qmul;
+      }
   }
   cp_async_wait<0>();
+  if (with_n && cg == 0)
+#pragma unroll
+    for (int p = 0; p < 4; p++) {
+      float lo, hi;
+      unpack2(N[NRM ? p : 0], lo, hi);
+      const int r = row0 + 2 * p;
+      if (r < dim) nvec[r] = lo;
+      if (r + 1 < dim) nvec[r + 1] = hi;
+    }
 #pragma unroll
   for (int p = 0; p < 4; p++)
 #pragma unroll
@@ -480,9 +619,10 @@ static cudaError_t linrec_scan_launch_cn(cudaStream_t st, const LinRecArgs& a) {
   else vec = vec && ok(a.qkw, 3 * (size_t)hd) && ok(a.vv, (size_t)a.H * a.vdim);
   if (!a.decay_p) vec = vec && ok(a.qkw, 3 * (size_t)hd);
   const int v16 = vec ? 1 : 0;
-  if (a.tmix) (void)launch_k(linrec_scan_kernel<RG, WR, CN, true, false>, grid, dim3(32 * WR), 0, st, a, v16, next_trace(41));
-  else if (a.decay_p) (void)launch_k(linrec_scan_kernel<RG, WR, CN, false, true>, grid, dim3(32 * WR), 0, st, a, v16, next_trace(41));
-  else (void)launch_k(linrec_scan_kernel<RG, WR, CN, false, false>, grid, dim3(32 * WR), 0, st, a, v16, next_trace(41));
+  if (a.gi.p) (void)launch_k(linrec_scan_kernel<RG, WR, CN, false, true, true>, grid, dim3(32 * WR), 0, st, a, v16, next_trace(41));
+  else if (a.tmix) (void)launch_k(linrec_scan_kernel<RG, WR, CN, true, false, false>, grid, dim3(32 * WR), 0, st, a, v16, next_trace(41));
+  else if (a.decay_p) (void)launch_k(linrec_scan_kernel<RG, WR, CN, false, true, false>, grid, dim3(32 * WR), 0, st, a, v16, next_trace(41));
+  else (void)launch_k(linrec_scan_kernel<RG, WR, CN, false, false, false>, grid, dim3(32 * WR), 0, st, a, v16, next_trace(41));
   return cudaGetLastError();
 }
 template <int RG, int WR>
@@ -497,7 +637,7 @@ static cudaError_t linrec_scan_launch(cudaStream_t st, const LinRecArgs& a) {
 
 cudaError_t launch_linrec_scan(cudaStream_t st, const LinRecArgs& a) {
   if (a.T <= 0 || a.n_seqs <= 0) return cudaSuccess;
-  if (a.dim > LINREC_MAX_DIM || (a.tmix && !a.bonus)) return cudaErrorInvalidValue;
+  if (a.dim > LINREC_MAX_DIM || (a.tmix && !a.bonus) || (a.gi.p && (!a.decay_p || !a.gates || !a.nq))) return cudaErrorInvalidValue;
   if (a.dim <= 16) return linrec_scan_launch<2, 1>(st, a);
   if (a.dim <= 32) return linrec_scan_launch<4, 1>(st, a);
   if (a.dim <= 64) return linrec_scan_launch<4, 2>(st, a);
@@ -511,7 +651,7 @@ cudaError_t launch_linrec_scan(cudaStream_t st, const LinRecArgs& a) {
 // decay), the state update with its read-out, the head's RMS norm, weight and gate run as ONE
 // launch per layer instead of three.  CTA = (sequence, head); the state slice of a thread is as
 // in linrec_scan_kernel and its loads are in flight while the row's inputs are prepared.
-// KIND: 0 gated linear attention, 1 time mixing, 2 HGRN2
+// KIND: 0 gated linear attention, 1 time mixing, 2 HGRN2, 3 mLSTM
 template <int RPL, int NW, int CC, int KIND>
 __global__ void __launch_bounds__(32 * NW) linrec_decode_kernel(LinRecArgs a, int out_bf16, Trace tr) {
   TRACE_ENTRY(tr);
@@ -526,6 +666,7 @@ __global__ void __launch_bounds__(32 * NW) linrec_decode_kernel(LinRecArgs a, in
   float* part = sv + VC;          // [NW][VC]
   float* slr = part + NW * VC;    // [rank]
   __shared__ float red[32];
+  __shared__ float s_gate[3];     // mLSTM: a | b | c
   const int t = blockIdx.x, head = blockIdx.y;
   const int tid = threadIdx.x, l = tid >> 5, lane = tid & 31;
   const int dim = a.dim, vdim = a.vdim;
@@ -550,11 +691,35 @@ __global__ void __launch_bounds__(32 * NW) linrec_decode_kernel(LinRecArgs a, in
     slr[r] = a.tmix ? tanhf(x) : x;
   }
   for (int c = tid; c < VC; c += NT) sv[c] = c < vdim ? seg_at(a.v, t, head * vdim + c) : 0.f;
+  float* slot = a.state_pool + (size_t)a.state_slots[t] * a.slot_floats;
+  if (KIND == 3 && tid == 0) {
+    float gi, gf;
+    mlstm_log_gates(seg_at(a.gi, t, head) + a.gi_b[head], seg_at(a.gf, t, head) + a.gf_b[head], a.cap, &gi, &gf);
+    float* top = slot + a.max_off + head;
+    const float prev = has_prev ? *top : 0.f, m = fmaxf(gf + prev, gi);
+    *top = m;
+    s_gate[0] = expf(gf + prev - m);
+    s_gate[1] = expf(gi - m);
+    s_gate[2] = expf(-m);
+  }
   __syncthreads();
   const float inv_tau = 1.0f / a.tau;
+  float nq = 0.f;
   for (int i = tid; i < DP; i += NT) {
     float q = 0.f, k = 0.f, decay = 0.f;
-    if (KIND == 2) {
+    if (KIND == 3) {
+      if (i < dim) {
+        const int c = head * dim + i;
+        float* nvec = slot + a.norm_off + c;
+        const float n0 = has_prev ? *nvec : 0.f;
+        q = seg_at(a.q, t, c);
+        k = seg_at(a.k, t, c) * s_gate[1];
+        decay = s_gate[0];
+        const float n1 = fmaf(decay, n0, k);
+        *nvec = n1;
+        nq = fmaf(n1, q, nq);
+      }
+    } else if (KIND == 2) {
       if (i < dim) {
         const int c = head * dim + i;
         bounded_gate(seg_at(a.lr, t, c) + a.w2b[c], a.lower[c], &decay, &k);
@@ -644,8 +809,9 @@ __global__ void __launch_bounds__(32 * NW) linrec_decode_kernel(LinRecArgs a, in
     if (KIND != 2) gt = seg_at(a.gate, t, head * vdim + tid);
     wn = a.onorm_w[(size_t)head * a.onorm_ld + tid];
   }
+  if (KIND == 3) o /= fmaxf(fabsf(block_sum(nq, red) * a.qmul), s_gate[2]) + 1e-6f;
   const float inv = 1.0f / sqrtf(block_sum(o * o, red) / (float)vdim + a.eps);
-  const float res = KIND == 2 ? o * inv * wn : o * inv * wn * silu(gt);
+  const float res = KIND == 2 ? o * inv * wn : o * inv * wn * (KIND == 3 ? 1.0f / (1.0f + expf(-gt)) : silu(gt));
   if (out_bf16) {
     bf16* out = (bf16*)a.out + (size_t)t * a.o_ld;
     if (mine) out[head * vdim + tid] = __float2bfloat16_rn(res);
@@ -670,7 +836,8 @@ static cudaError_t linrec_decode_launch_cc(cudaStream_t st, int odt, const LinRe
       cudaFuncSetAttribute(linrec_decode_kernel<RPL, NW, CC, KIND_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
     (void)launch_k(linrec_decode_kernel<RPL, NW, CC, KIND_>, dim3(a.T, a.H), dim3(32 * NW), smem, st, a, bf, next_trace(45)); \
   } while (0)
-  if (a.lower) LD(2);
+  if (a.gi.p) LD(3);
+  else if (a.lower) LD(2);
   else if (a.tmix) LD(1);
   else LD(0);
 #undef LD
@@ -707,8 +874,11 @@ __device__ __forceinline__ void store4(bf16* p, const float (&v)[4]) {
   reinterpret_cast<__nv_bfloat162*>(&u)[1] = __floats2bfloat162_rn(v[2], v[3]);
   *reinterpret_cast<uint2*>(p) = u;
 }
-// MJ: 16-byte pieces per lane (vdim <= 128 MJ)
-template <typename OT, int MJ, bool GATED>
+// MJ: 16-byte pieces per lane (vdim <= 128 MJ); GATED: 0 no gate, 1 silu(gate), 2 mLSTM: the read-out is first divided by
+// max(|n . q|, c) + 1e-6, sigmoid(gate)
+template <int GATED>
+__device__ __forceinline__ float out_gate(float z) { return GATED == 2 ? 1.0f / (1.0f + expf(-z)) : silu(z); }
+template <typename OT, int MJ, int GATED>
 __global__ void __launch_bounds__(256) linrec_out_kernel(LinRecArgs a, Trace tr) {
   TRACE_ENTRY(tr);
   pdl_launch_dependents();
@@ -722,6 +892,8 @@ __global__ void __launch_bounds__(256) linrec_out_kernel(LinRecArgs a, Trace tr)
                    (reinterpret_cast<size_t>(a.gate.p) % 16) == 0 && (a.onorm_ld % 4) == 0;
   for (int h = blockIdx.y * nw + warp; h < a.H; h += gridDim.y * nw) {
     const float* o = a.o + (size_t)t * a.H * vdim + (size_t)h * vdim;
+    float od = 1.f;  // what the read-out is divided by
+    if (GATED == 2) od = fmaxf(fabsf(a.nq[(size_t)t * a.H + h]), a.gates[((size_t)2 * a.T + t) * a.H + h]) + 1e-6f;
     if (vec) {
       // four neighbouring columns per lane, all loads (read-outs, gate slices, weights) before the arithmetic
       float4 ov[MJ], gv[GATED ? MJ : 1];
@@ -731,6 +903,7 @@ __global__ void __launch_bounds__(256) linrec_out_kernel(LinRecArgs a, Trace tr)
         const int i = lane * 4 + 128 * j;
         if (i < vdim) {
           ov[j] = *reinterpret_cast<const float4*>(o + i);
+          if constexpr (GATED == 2) { ov[j].x /= od; ov[j].y /= od; ov[j].z /= od; ov[j].w /= od; }
           ss += ov[j].x * ov[j].x + ov[j].y * ov[j].y + ov[j].z * ov[j].z + ov[j].w * ov[j].w;
           if constexpr (GATED) {
             const float* gp = a.gate.p + (size_t)t * a.gate.ld + h * vdim + i;
@@ -751,7 +924,8 @@ __global__ void __launch_bounds__(256) linrec_out_kernel(LinRecArgs a, Trace tr)
           const float4 w4 = *reinterpret_cast<const float4*>(w + i);
           float r[4] = {ov[j].x * inv * w4.x, ov[j].y * inv * w4.y, ov[j].z * inv * w4.z, ov[j].w * inv * w4.w};
           if constexpr (GATED) {
-            r[0] *= silu(gv[j].x); r[1] *= silu(gv[j].y); r[2] *= silu(gv[j].z); r[3] *= silu(gv[j].w);
+            r[0] *= out_gate<GATED>(gv[j].x); r[1] *= out_gate<GATED>(gv[j].y);
+            r[2] *= out_gate<GATED>(gv[j].z); r[3] *= out_gate<GATED>(gv[j].w);
           }
           store4(out + h * vdim + i, r);
         }
@@ -759,12 +933,12 @@ __global__ void __launch_bounds__(256) linrec_out_kernel(LinRecArgs a, Trace tr)
       continue;
     }
     float ss = 0.f;
-    for (int i = lane; i < vdim; i += 32) ss += o[i] * o[i];
+    for (int i = lane; i < vdim; i += 32) ss += (o[i] / od) * (o[i] / od);
     const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)vdim + a.eps);
     const float* w = a.onorm_w + (size_t)h * a.onorm_ld;
     for (int i = lane; i < vdim; i += 32) {
-      const float r = o[i] * inv * w[i];
-      out[h * vdim + i] = from_f32<OT>(GATED ? r * silu(seg_at(a.gate, t, h * vdim + i)) : r);
+      const float r = o[i] / od * inv * w[i];
+      out[h * vdim + i] = from_f32<OT>(GATED ? r * out_gate<GATED>(seg_at(a.gate, t, h * vdim + i)) : r);
     }
   }
   if (blockIdx.y == 0)
@@ -777,8 +951,9 @@ cudaError_t launch_linrec_out(cudaStream_t st, int odt, const LinRecArgs& a) {
   const dim3 grid(a.T, a.T >= 1024 ? 1 : ceil_div(a.H, 8));
 #define LO(OT_, MJ_)                                                                                           \
   do {                                                                                                         \
-    if (a.gate.p) (void)launch_k(linrec_out_kernel<OT_, MJ_, true>, grid, dim3(256), 0, st, a, next_trace(42)); \
-    else (void)launch_k(linrec_out_kernel<OT_, MJ_, false>, grid, dim3(256), 0, st, a, next_trace(42));         \
+    if (a.gi.p) (void)launch_k(linrec_out_kernel<OT_, MJ_, 2>, grid, dim3(256), 0, st, a, next_trace(42));         \
+    else if (a.gate.p) (void)launch_k(linrec_out_kernel<OT_, MJ_, 1>, grid, dim3(256), 0, st, a, next_trace(42));  \
+    else (void)launch_k(linrec_out_kernel<OT_, MJ_, 0>, grid, dim3(256), 0, st, a, next_trace(42));         \
   } while (0)
   if (odt == DT_F32) {
     if (a.vdim <= 128) LO(float, 1); else LO(float, 4);
