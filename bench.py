@@ -756,6 +756,71 @@ SOZURAX_SIZES = {
 }
 
 
+def defilorn_cfg(width, n_layers, vocab, m_heads, m_dim, m_vdim, l_heads, l_dim, l_rot, l_vdim, kv_rank, q_rank, a_heads, a_kv, a_dim, a_vdim,
+                 window, experts, identity, top, ff, shared, dense_ff, loop=None):
+    """mLSTM layers alternate with attention layers, which are latent and differential (windowed) in turn; a
+    tanh-GELU gated dense feed-forward in the first layer, gated experts with identity experts and a gated
+    always-on one in the others; loop = (start, stop, times) repeats a run of layers."""
+    layers = []
+    for l in range(n_layers):
+        if l % 2 == 0:
+            kw = dict(mixer=C.MIXER_MLSTM, heads=m_heads, dim=m_dim, vdim=m_vdim, gate_cap=15.0)
+        elif l % 4 == 1:
+            kw = dict(mixer=C.MIXER_LATENT_ATTENTION, heads=l_heads, dim=l_dim, rot_dim=l_rot, vdim=l_vdim, kv_rank=kv_rank, q_rank=q_rank,
+                      rot_base=20000.0, rot_dims=l_rot, rot_pairs=1, rot_factor=4.0, rot_original=4096.0, rot_fast=32.0, rot_slow=1.0,
+                      scale=float((l_dim + l_rot) ** -0.5), sink=1, sink_learned=1, out_gate=1)
+        else:
+            kw = dict(mixer=C.MIXER_ATTENTION, heads=a_heads, kv_heads=a_kv, dim=a_dim, vdim=a_vdim, scale=float(a_dim ** -0.5), qk_norm=3,
+                      window=window, diff_maps=1, diff=0.5)
+        if l == 0:
+            kw.update(mlp=C.MLP_DENSE, act=C.FFN_GEGLU, ff=dense_ff)
+        else:
+            kw.update(mlp=C.MLP_MOE, act=C.FFN_SWIGLU, ff=ff, experts=experts, top=top, route_identity=identity, route_correction=1,
+                      route_raw=1, shared_ff=shared, shared_gate=1)
+        layers.append(C.LayerSpec(**kw))
+    start, stop, times = loop or (0, 0, 0)
+    return C.ListedModelConfig("defilorn", vocab, width, tuple(layers), 1e-5, arch=C.ARCH_DEFILORN,
+                               block_style=C.LBLOCK_SEQUENTIAL_PRENORM, norm_offset=1.0, loop_start=start, loop_stop=stop,
+                               loop_times=times, loop_embed=True)
+
+
+def defilorn_device_weights(cfg, device, seed=1234):
+    import torch
+    g = torch.Generator(device=f"cuda:{device}")
+    for i, (name, shape) in enumerate(cfg.tensor_shapes().items()):
+        g.manual_seed(seed * 1000003 + i)
+        t = torch.empty(shape, dtype=torch.float32, device=f"cuda:{device}")
+        if name.endswith(".f.b"):
+            t.uniform_(2.0, 5.0, generator=g)
+        elif name.endswith((".norm1", ".norm2", "final.norm")) or name.endswith((".i.b", ".correction", ".sink")):
+            t.normal_(0.0, 0.02, generator=g)
+        elif name.endswith((".lq1", ".lk1", ".lq2", ".lk2")):
+            t.normal_(0.0, 0.1, generator=g)
+        elif len(shape) == 1:
+            t.normal_(1.0, 0.02, generator=g)
+        else:
+            t.normal_(0.0, 0.02 if name == "embed" else shape[1] ** -0.5, generator=g)
+        yield name, t.to(torch.bfloat16).view(torch.int16).cpu().numpy().view(np.uint16)
+        del t
+
+
+# width 1024, 24 layers like Granite-MoE-1B: 12 mLSTM layers (8 heads of 64 x 128 state, as so-1b's recurrences), 6
+# latent-attention layers (so-1b's sizes, no window), 6 differential-attention layers (8 heads of two maps of 64 and
+# values of 128, 4 key / value heads, window 1024); 32 gated experts of 512 and 4 identity experts, 8 per token,
+# beside an always-on expert of 1024.
+def _de(loop=None, n_layers=24):
+    return lambda: defilorn_cfg(1024, n_layers, 49155, 8, 64, 128, 16, 64, 32, 64, 128, 384, 8, 4, 64, 128, 1024, 32, 4, 8, 512, 1024, 4096, loop)
+
+
+DEFILORN_SIZES = {
+    "de-1b": (_de(), "granite-moe-1b", 128, 128, 128),
+    "de-1b-long": (_de(), "granite-moe-1b", 16, 4096, 64),
+    "de-1b-batch": (_de(), "granite-moe-1b", 64, 512, 128),
+    # 16 layers of which eight run twice: 24 executions
+    "de-1b-loop": (_de((4, 12, 2), 16), "granite-moe-1b", 64, 512, 128),
+}
+
+
 def dugopel_moe_width():
     """The other latent-attention design at the width, depth, expert and attention sizes of the sizes above."""
     return dugopel_cfg(1024, 24, 16, 64, 32, 64, 128, 384, 512, 49155, moe=(32, 8, 8, 4))
@@ -783,15 +848,17 @@ def design_bench(args):
     peaks = load_peaks()
     R = nvllm_pkg.sub("runner")
     design = args.design
-    sizes = {"zozonex": ZOZONEX_SIZES, "lazovik": LAZOVIK_SIZES, "sutuvik": SUTUVIK_SIZES, "sozurax": SOZURAX_SIZES}.get(design, DESIGN_SIZES)
+    sizes = {"zozonex": ZOZONEX_SIZES, "lazovik": LAZOVIK_SIZES, "sutuvik": SUTUVIK_SIZES, "sozurax": SOZURAX_SIZES,
+             "defilorn": DEFILORN_SIZES}.get(design, DESIGN_SIZES)
     gen = {"zozonex": zozonex_device_weights, "lazovik": lazovik_device_weights,
-           "sutuvik": sutuvik_device_weights, "sozurax": sozurax_device_weights}.get(design, dugopel_device_weights)
+           "sutuvik": sutuvik_device_weights, "sozurax": sozurax_device_weights,
+           "defilorn": defilorn_device_weights}.get(design, dugopel_device_weights)
     # further baselines: uniform models (configuration) and layer-listed ones (configuration, weights)
     uniform = {"hybrid-mamba2-1b": hybrid_1b, "hybrid-mamba2-w1024": hybrid_moe_width}
     listed = {"zozonex-1b": (zozonex_moe_width, zozonex_device_weights), "lazovik-w1024": (_lz(24), lazovik_device_weights),
-              "dugopel-w1024": (dugopel_moe_width, dugopel_device_weights)}
+              "dugopel-w1024": (dugopel_moe_width, dugopel_device_weights), "sozurax-w1024": (_so, sozurax_device_weights)}
     second = {"zozonex": ("hybrid-mamba2-1b",), "lazovik": ("zozonex-1b",), "sutuvik": ("hybrid-mamba2-w1024",),
-              "sozurax": ("lazovik-w1024", "dugopel-w1024")}.get(design, ())
+              "sozurax": ("lazovik-w1024", "dugopel-w1024"), "defilorn": ("sozurax-w1024", "zozonex-1b")}.get(design, ())
     out = {"design": design, "dtype": "bf16", "data": "synthetic (random-init weights, random prompts)",
            "steps": args.steps, "warmup": args.warmup, "peaks": peaks, "sizes": {}}
     names = [n for n in sizes if args.design_size in (None, n)]
@@ -892,14 +959,14 @@ def main():
     ap.add_argument("--no-profile", action="store_true")
     ap.add_argument("--no-tp", action="store_true",
                     help="skip the Falcon-7B tensor-parallel leg (configs[3] at tp = --gpus)")
-    ap.add_argument("--design", default=None, choices=["dugopel", "zozonex", "lazovik", "sutuvik", "sozurax"],
+    ap.add_argument("--design", default=None, choices=["dugopel", "zozonex", "lazovik", "sutuvik", "sozurax", "defilorn"],
                     help="instead of the default workload: the layer-listed design beside the closest "
                          "uniform model at equal size (prefill and decode, per-kernel roofline)")
     ap.add_argument("--no-hybrid", action="store_true",
-                    help="--design zozonex / lazovik / sutuvik / sozurax: only the closest uniform model as a baseline (no Mamba2 "
+                    help="--design zozonex / lazovik / sutuvik / sozurax / defilorn: only the closest uniform model as a baseline (no Mamba2 "
                          "hybrid / other layer-listed design at equal width)")
     ap.add_argument("--design-size", default=None, choices=sorted(DESIGN_SIZES) + sorted(ZOZONEX_SIZES) + sorted(LAZOVIK_SIZES) + sorted(SUTUVIK_SIZES) +
-                    sorted(SOZURAX_SIZES))
+                    sorted(SOZURAX_SIZES) + sorted(DEFILORN_SIZES))
     args = ap.parse_args()
     if args.design:
         return design_bench(args)
