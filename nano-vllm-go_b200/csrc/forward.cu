@@ -27,7 +27,7 @@ void free_workspace(nvllm_handle* h) {
                   w.xb, w.ssq, w.chain_ctr, w.lat_cq, w.lat_gate, w.lat_o, w.dl_qkv, w.dl_bg, w.dl_o, w.m_xbc, w.m_dt, w.m_y, w.m_yn, w.logits_p, w.logits, w.attn_ws, w.out_tokens, w.amax, w.amax_ticket, w.topk_idx, w.topk_w,
                   w.sort.counts, w.sort.offsets, w.sort.cursor, w.sort.sorted_pair, w.sort.pair_row,
                   w.sort.a_rows, w.sort.tile_expert, w.sort.tile_row0, w.sort.tile_rows,
-                  w.sort.n_tiles, w.moe_Y, w.moe_y, w.moe_xs, w.lr_qkw, w.lr_v, w.lr_o, w.att_gate, w.sh_gate, w.mx_in,
+                  w.sort.n_tiles, w.sort.part, w.moe_Y, w.moe_y, w.moe_xs, w.lr_qkw, w.lr_v, w.lr_o, w.att_gate, w.sh_gate, w.mx_in,
                   w.m2_xbc, w.m2_dtx, w.m2_decay, w.v_first, w.side_g, w.att_split, w.att_split_cnt, w.ml_gates, w.ml_nq};
   for (void* p : ptrs)
     if (p) cudaFree(p);
@@ -206,6 +206,7 @@ int ensure_workspace(nvllm_handle* h, int T, int n) {
     WS(w.sort.tile_row0, w.max_tiles * 4);
     WS(w.sort.tile_rows, w.max_tiles * 4);
     WS(w.sort.n_tiles, 4);
+    WS(w.sort.part, (size_t)MOE_SORT_CTAS * h->E * 4);
     WS(w.moe_Y, P * H * 4);
     if (h->adt == DT_BF16) WS(w.moe_xs, P * H * 2);
     WS(w.moe_y, Tc * H * 4);

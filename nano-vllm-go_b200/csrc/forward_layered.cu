@@ -870,7 +870,7 @@ static int run_prenorm(nvllm_handle* h, Pending* p1, Pending* p2, const float* r
   }
   {
     ProfScope ps(h, NVLLM_K_NORM, bytes, 0, impl);
-    LAUNCH(h, launch_norm(h->stream, a));
+    if (const int rc = launch_norm_routed(h, a)) return rc;
   }
   *p1 = Pending();
   *p2 = Pending();

@@ -212,6 +212,20 @@ static bool resid_gemm_ok(const nvllm_handle* h, int M, int N, int K, int lda) {
   return ce && atoi(ce) != 0;
 }
 
+// Norm kernel of a routed layer: steps of many rows route in a kernel of their own (launch_moe_route_rows)
+static int launch_norm_routed(nvllm_handle* h, NormArgs a) {
+  if (a.router && !a.row_idx && !a.y_f32 && h->ws.xn_f32 && moe_route_rows_fits(a.n_rows, a.H, a.E)) {
+    NormArgs n = a;
+    n.router = nullptr;
+    n.y_f32 = h->ws.xn_f32;
+    LAUNCH(h, launch_norm(h->stream, n));
+    LAUNCH(h, launch_moe_route_rows(h->stream, a, h->ws.xn_f32));
+    return NVLLM_OK;
+  }
+  LAUNCH(h, launch_norm(h->stream, a));
+  return NVLLM_OK;
+}
+
 static int run_norm(nvllm_handle* h, float* x, Pending* p1, Pending* p2, const float* w,
                     const float* b, void* y, float* y_f32, const int* row_idx, int n_rows,
                     const RouterArgs* route = nullptr, bool centered = false, const float* row_m2 = nullptr) {
@@ -245,7 +259,7 @@ static int run_norm(nvllm_handle* h, float* x, Pending* p1, Pending* p2, const f
   a.row_bias = row_idx ? h->view_r0 : 0;  // row_idx holds rows of the whole step
   a.groups = h->norm_groups;  // > 1: RMS norm in equal parts of the row (layered pre-norm models)
   ProfScope ps(h, NVLLM_K_NORM, bytes, 0, impl);
-  LAUNCH(h, launch_norm(h->stream, a));
+  if (const int rc = launch_norm_routed(h, a)) return rc;
   if (p1) *p1 = Pending();
   if (p2) *p2 = Pending();
   return NVLLM_OK;

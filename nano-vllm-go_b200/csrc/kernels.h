@@ -126,6 +126,11 @@ struct NormArgs {
   size_t conv_slot_floats, conv_tail_off;
 };
 cudaError_t launch_norm(cudaStream_t st, const NormArgs& a);
+// A routed norm of many rows (prefill) is better split in two: the norm kernel leaves its fp32 rows in scratch (y_f32,
+// router = null), and this kernel routes eight rows at a time (and adds the identity experts' share to x).  a: the
+// arguments of the routed norm; rows: those fp32 rows.
+bool moe_route_rows_fits(int n_rows, int H, int E);
+cudaError_t launch_moe_route_rows(cudaStream_t st, const NormArgs& a, const float* rows);
 
 // SwiGLU: out[t,j] = silu(h[t,j]) * h[t,F+j]   (transformer.go:50-66, mamba2.go:360-367)
 // GELU:   out[t,j] = gelu_tanh(h[t,j] + b1[j]) (transformer.go:67-78, tensor.go:181-190)
@@ -728,7 +733,9 @@ struct MoeSortBufs {
   int* tile_row0;
   int* tile_rows;
   int* n_tiles;      // [1]
+  int* part;         // [MOE_SORT_CTAS][E] expert counts of the CTAs' shares (prefill-sized sorts)
 };
+constexpr int MOE_SORT_CTAS = 148;
 cudaError_t launch_moe_sort(cudaStream_t st, const int* topk_idx, int T, int k, int E,
                             const MoeSortBufs& b, int max_tiles, int tile);
 // sort + gather in one launch for decode-sized batches (moe_sort_gather_fits)

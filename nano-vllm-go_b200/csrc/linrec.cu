@@ -1099,17 +1099,15 @@ __global__ void __launch_bounds__(512) input_conv_kernel(InputConvArgs a, Trace 
 }
 
 // The same for steps of many rows with a router: a CTA takes TT tokens, their convolved rows stay in
-// shared memory, and a warp accumulates four experts against all of them — a router row crosses L2 once per TT tokens
-// instead of once per token.
+// shared memory and are routed together (moe_route_tile).
 template <typename AT, int TAPS, int TT>
 __global__ void __launch_bounds__(256) input_conv_route_kernel(InputConvArgs a, Trace tr) {
   TRACE_ENTRY(tr);
   pdl_launch_dependents();
   extern __shared__ __align__(16) float rows[];  // [TT][W], then probs | chs | gsc [TT][E] each
   __shared__ int s_seq[TT];
-  constexpr int EB = 4;
   const int W = a.W, E = a.E, t0 = blockIdx.x * TT, nt = min(TT, a.T - t0), keep = a.taps - 1;
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  const int warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
   for (int i = threadIdx.x; i < a.n_seqs; i += blockDim.x) {
     const int lo = max(a.cu_q[i], t0), hi = min(a.cu_q[i + 1], t0 + nt);
     for (int t = lo; t < hi; t++) s_seq[t - t0] = i;
@@ -1145,37 +1143,7 @@ __global__ void __launch_bounds__(256) input_conv_route_kernel(InputConvArgs a, 
   }
   __syncthreads();
   float* probs = rows + (size_t)TT * W;
-  for (int e0 = warp * EB; e0 < E; e0 += nw * EB) {
-    float acc[EB][TT];
-#pragma unroll
-    for (int q = 0; q < EB; q++)
-#pragma unroll
-      for (int tt = 0; tt < TT; tt++) acc[q][tt] = 0.f;
-#pragma unroll 2
-    for (int i = lane * 4; i < W; i += 128) {  // neighbouring lanes, neighbouring 16-byte pieces: no bank conflicts
-      float4 r[EB];
-#pragma unroll
-      for (int q = 0; q < EB; q++) r[q] = *reinterpret_cast<const float4*>(a.router + (size_t)min(e0 + q, E - 1) * W + i);
-#pragma unroll
-      for (int tt = 0; tt < TT; tt++) {
-        const float4 y = *reinterpret_cast<const float4*>(rows + (size_t)tt * W + i);
-#pragma unroll
-        for (int q = 0; q < EB; q++) {
-          acc[q][tt] = fmaf(y.x, r[q].x, acc[q][tt]);
-          acc[q][tt] = fmaf(y.y, r[q].y, acc[q][tt]);
-          acc[q][tt] = fmaf(y.z, r[q].z, acc[q][tt]);
-          acc[q][tt] = fmaf(y.w, r[q].w, acc[q][tt]);
-        }
-      }
-    }
-#pragma unroll
-    for (int q = 0; q < EB; q++)
-#pragma unroll
-      for (int tt = 0; tt < TT; tt++) {
-        const float z = warp_sum(acc[q][tt]);
-        if (lane == 0 && e0 + q < E) probs[tt * E + e0 + q] = a.route.bias ? z + a.route.bias[e0 + q] : z;
-      }
-  }
+  moe_route_tile<TT>(rows, W, a.router, E, a.route.bias, probs);
   __syncthreads();
   for (int tt = warp; tt < nt; tt += nw)
     moe_select_row(probs + tt * E, probs + (size_t)(TT + tt) * E, probs + (size_t)(2 * TT + tt) * E, E, a.topk, (size_t)(t0 + tt),

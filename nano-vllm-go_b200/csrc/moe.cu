@@ -30,6 +30,166 @@ cudaError_t launch_moe_router(cudaStream_t st, const float* x, const float* R, i
   return cudaGetLastError();
 }
 
+// ------------------------------------------------------------------ routing of many rows
+constexpr int MRR_TT = 8;                // rows per CTA
+constexpr int MRR_MAX_WARPS = 12;
+constexpr size_t MRR_SMEM = 96 * 1024;   // as long as they fit (two CTAs per SM)
+
+__global__ void __launch_bounds__(32 * MRR_MAX_WARPS, 2) moe_route_rows_kernel(NormArgs a, const float* __restrict__ src, Trace tr) {
+  TRACE_ENTRY(tr);
+  pdl_launch_dependents();
+  extern __shared__ __align__(16) float rows[];  // [TT][H], then probs | chs | gsc [TT][E] each
+  __shared__ float id_w[MRR_TT];
+  const int H = a.H, E = a.E, t0 = blockIdx.x * MRR_TT, nt = min(MRR_TT, a.n_rows - t0), vpr = H / 4;
+  const int warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  pdl_wait();
+  for (int i = threadIdx.x; i < MRR_TT * vpr; i += blockDim.x)
+    reinterpret_cast<float4*>(rows)[i] = i < nt * vpr ? reinterpret_cast<const float4*>(src + (size_t)t0 * H)[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+  __syncthreads();
+  float* probs = rows + (size_t)MRR_TT * H;
+  moe_route_tile<MRR_TT>(rows, H, a.router, E, a.route.bias, probs);
+  __syncthreads();
+  for (int tt = warp; tt < nt; tt += nw)
+    moe_select_row(probs + tt * E, probs + (size_t)(MRR_TT + tt) * E, probs + (size_t)(2 * MRR_TT + tt) * E, E, a.topk,
+                   (size_t)(t0 + tt), a.topk_idx, a.topk_w, a.route, a.route.identity > 0 ? &id_w[tt] : nullptr);
+  if (a.route.identity > 0) {  // the chosen identity experts return the row itself
+    __syncthreads();
+    for (int i = threadIdx.x; i < nt * vpr; i += blockDim.x) {
+      const float w = id_w[i / vpr];
+      if (w == 0.f) continue;
+      float4* xp = reinterpret_cast<float4*>(a.x + (size_t)t0 * H) + i;
+      const float4 y = reinterpret_cast<const float4*>(rows)[i];
+      float4 v = *xp;
+      v.x = fmaf(w, y.x, v.x); v.y = fmaf(w, y.y, v.y); v.z = fmaf(w, y.z, v.z); v.w = fmaf(w, y.w, v.w);
+      *xp = v;
+    }
+  }
+  TRACE_EXIT(tr);
+}
+
+static size_t moe_route_rows_smem(int H, int E) { return ((size_t)MRR_TT * H + 3 * (size_t)MRR_TT * E) * sizeof(float); }
+bool moe_route_rows_fits(int n_rows, int H, int E) { return n_rows >= 1024 && (H % 8) == 0 && moe_route_rows_smem(H, E) <= MRR_SMEM; }
+cudaError_t launch_moe_route_rows(cudaStream_t st, const NormArgs& a, const float* rows) {
+  if (a.n_rows <= 0) return cudaSuccess;
+  if (!a.router || a.row_idx || !moe_route_rows_fits(a.n_rows, a.H, a.E)) return cudaErrorInvalidValue;
+  const size_t smem = moe_route_rows_smem(a.H, a.E);
+  if (smem > 48 * 1024) cudaFuncSetAttribute(moe_route_rows_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  // a warp takes four experts at a time: as few rounds as possible, with as few warps as that needs
+  const int groups = (a.E + 3) / 4;
+  int nw = 8;
+  for (int n = 9; n <= MRR_MAX_WARPS; n++)
+    if ((groups + n - 1) / n < (groups + nw - 1) / nw) nw = n;
+  (void)launch_k(moe_route_rows_kernel, dim3((a.n_rows + MRR_TT - 1) / MRR_TT), dim3(32 * nw), smem, st, a, rows, next_trace(18));
+  return cudaGetLastError();
+}
+
+// ------------------------------------------------------------------ sort of many pairs
+// Two launches of MOE_SORT_CTAS CTAs with a contiguous share of the pairs each: counts per share and expert, then
+// every CTA adds up the table (its own first row per expert = expert's offset + earlier shares' counts) and hands out
+// its rows; CTA 0 publishes the lists.
+__global__ void __launch_bounds__(1024) moe_count_kernel(const int* __restrict__ topk_idx, int n_pairs, int E, MoeSortBufs b, Trace tr) {
+  TRACE_ENTRY(tr);
+  pdl_launch_dependents();
+  __shared__ int cnt[MOE_MAX_E];
+  for (int e = threadIdx.x; e < E; e += blockDim.x) cnt[e] = 0;
+  pdl_wait();
+  __syncthreads();
+  const int per = (n_pairs + gridDim.x - 1) / gridDim.x, lo = blockIdx.x * per, hi = min(n_pairs, lo + per);
+  for (int p = lo + threadIdx.x; p < hi; p += blockDim.x) {
+    const int e = topk_idx[p];
+    if (e < E) atomicAdd(&cnt[e], 1);  // (others are identity experts: no row)
+  }
+  __syncthreads();
+  for (int e = threadIdx.x; e < E; e += blockDim.x) b.part[(size_t)blockIdx.x * E + e] = cnt[e];
+  TRACE_EXIT(tr);
+}
+__global__ void __launch_bounds__(1024) moe_place_kernel(const int* __restrict__ topk_idx, int n_pairs, int k, int E, MoeSortBufs b,
+                                                         int max_tiles, int tile, Trace tr) {
+  TRACE_ENTRY(tr);
+  pdl_launch_dependents();
+  __shared__ int tot[MOE_MAX_E], cur[MOE_MAX_E], off[MOE_MAX_E + 1], toff[MOE_MAX_E + 1];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  pdl_wait();
+  for (int e = warp; e < E; e += nw) {  // a warp per expert, its lanes over the shares
+    int mine = 0, all = 0;
+    for (int g = lane; g < (int)gridDim.x; g += 32) {
+      const int c = b.part[(size_t)g * E + e];
+      all += c;
+      if (g < (int)blockIdx.x) mine += c;
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      mine += __shfl_xor_sync(0xffffffffu, mine, o);
+      all += __shfl_xor_sync(0xffffffffu, all, o);
+    }
+    if (lane == 0) {
+      tot[e] = all;
+      cur[e] = mine;
+    }
+  }
+  __syncthreads();
+  if (warp == 0) {  // exclusive sums of rows and tiles over the experts
+    int run = 0, trun = 0;
+    for (int e0 = 0; e0 < E; e0 += 32) {
+      const int e = e0 + lane, c = e < E ? tot[e] : 0, t = (c + tile - 1) / tile;
+      int ic = c, it = t;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int x = __shfl_up_sync(0xffffffffu, ic, o), y = __shfl_up_sync(0xffffffffu, it, o);
+        if (lane >= o) {
+          ic += x;
+          it += y;
+        }
+      }
+      if (e < E) {
+        off[e] = run + ic - c;
+        toff[e] = trun + it - t;
+        cur[e] += run + ic - c;
+      }
+      run += __shfl_sync(0xffffffffu, ic, 31);
+      trun += __shfl_sync(0xffffffffu, it, 31);
+    }
+    if (lane == 0) {
+      off[E] = run;
+      toff[E] = trun;
+    }
+  }
+  __syncthreads();
+  if (blockIdx.x == 0) {
+    for (int e = warp; e < E; e += nw) {
+      const int c = tot[e], nt = (c + tile - 1) / tile;
+      for (int r = lane; r < nt && toff[e] + r < max_tiles; r += 32) {
+        b.tile_expert[toff[e] + r] = e;
+        b.tile_row0[toff[e] + r] = off[e] + r * tile;
+        b.tile_rows[toff[e] + r] = min(tile, c - r * tile);
+      }
+      if (lane == 0) {
+        b.counts[e] = c;
+        b.offsets[e] = off[e];
+      }
+    }
+    if (threadIdx.x == 0) {
+      b.offsets[E] = off[E];
+      *b.n_tiles = min(toff[E], max_tiles);
+    }
+  }
+  const int per = (n_pairs + gridDim.x - 1) / gridDim.x, lo = blockIdx.x * per, hi = min(n_pairs, lo + per);
+  for (int p = lo + threadIdx.x; p < hi; p += blockDim.x) {
+    const int e = topk_idx[p];
+    if (e >= E) {
+      b.pair_row[p] = -1;
+      continue;
+    }
+    const int row = atomicAdd(&cur[e], 1);
+    b.sorted_pair[row] = p;
+    b.pair_row[p] = row;
+    b.a_rows[row] = p / k;
+  }
+  // rows past the lists (as many as there are identity pairs): a valid one
+  for (int r = off[E] + blockIdx.x * blockDim.x + threadIdx.x; r < n_pairs; r += gridDim.x * blockDim.x) b.a_rows[r] = 0;
+  TRACE_EXIT(tr);
+}
+
 // Single-CTA counting sort of the T*k pairs by expert + tile list.  Rows inside an expert are
 // in arbitrary order; every consumer addresses them through pair_row / a_rows, so results do
 // not depend on it.
@@ -87,6 +247,11 @@ cudaError_t launch_moe_sort(cudaStream_t st, const int* topk_idx, int T, int k, 
                             const MoeSortBufs& b, int max_tiles, int tile) {
   if (T <= 0) return cudaSuccess;
   if (E > MOE_MAX_E || tile <= 0) return cudaErrorInvalidValue;
+  if (b.part && (long)T * k > 8192) {
+    (void)launch_k(moe_count_kernel, dim3(MOE_SORT_CTAS), dim3(1024), 0, st, topk_idx, T * k, E, b, next_trace(15));
+    (void)launch_k(moe_place_kernel, dim3(MOE_SORT_CTAS), dim3(1024), 0, st, topk_idx, T * k, k, E, b, max_tiles, tile, next_trace(15));
+    return cudaGetLastError();
+  }
   (void)launch_k(moe_sort_kernel, dim3(1), dim3(1024), 0, st, topk_idx, T * k, k, E, b, max_tiles,
                  tile, next_trace(15));
   return cudaGetLastError();

@@ -177,4 +177,44 @@ __device__ __forceinline__ void moe_route_row(const float* y, const float* __res
   moe_select_row(probs, chs, gsc, E, k, t, topk_idx, topk_w, ro, identity_w);
 }
 
+// Router logits of TT rows that sit in shared memory (rows [TT][W], W a multiple of 4): a warp accumulates four experts
+// against all of them — a router row crosses L2 once per TT tokens instead of once per token.  probs [TT][E].
+template <int TT>
+__device__ __forceinline__ void moe_route_tile(const float* rows, int W, const float* __restrict__ R, int E,
+                                               const float* __restrict__ bias, float* probs) {
+  constexpr int EB = 4;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  for (int e0 = warp * EB; e0 < E; e0 += nw * EB) {
+    float acc[EB][TT];
+#pragma unroll
+    for (int q = 0; q < EB; q++)
+#pragma unroll
+      for (int tt = 0; tt < TT; tt++) acc[q][tt] = 0.f;
+#pragma unroll 2
+    for (int i = lane * 4; i < W; i += 128) {  // neighbouring lanes, neighbouring 16-byte pieces: no bank conflicts
+      float4 r[EB];
+#pragma unroll
+      for (int q = 0; q < EB; q++) r[q] = *reinterpret_cast<const float4*>(R + (size_t)min(e0 + q, E - 1) * W + i);
+#pragma unroll
+      for (int tt = 0; tt < TT; tt++) {
+        const float4 y = *reinterpret_cast<const float4*>(rows + (size_t)tt * W + i);
+#pragma unroll
+        for (int q = 0; q < EB; q++) {
+          acc[q][tt] = fmaf(y.x, r[q].x, acc[q][tt]);
+          acc[q][tt] = fmaf(y.y, r[q].y, acc[q][tt]);
+          acc[q][tt] = fmaf(y.z, r[q].z, acc[q][tt]);
+          acc[q][tt] = fmaf(y.w, r[q].w, acc[q][tt]);
+        }
+      }
+    }
+#pragma unroll
+    for (int q = 0; q < EB; q++)
+#pragma unroll
+      for (int tt = 0; tt < TT; tt++) {
+        const float z = warp_sum(acc[q][tt]);
+        if (lane == 0 && e0 + q < E) probs[tt * E + e0 + q] = bias ? z + bias[e0 + q] : z;
+      }
+  }
+}
+
 }  // namespace nvllm
