@@ -189,9 +189,76 @@ __global__ void __launch_bounds__(256) winattn_prep_kernel(WinAttnArgs a, Trace 
   TRACE_EXIT(tr);
 }
 
+// The same for rows without rotation, value mixing and head gates whose heads are 4 LPH entries: a thread takes four
+// neighbouring entries (16-byte loads), LPH neighbouring lanes hold a head.  grid (T, Y).
+template <typename QT, typename KT, int LPH>
+__global__ void __launch_bounds__(256) winattn_prep_vec_kernel(WinAttnArgs a, Trace tr) {
+  TRACE_ENTRY(tr);
+  pdl_launch_dependents();
+  pdl_wait();
+  constexpr int DIM = 4 * LPH;
+  const int t = blockIdx.x;
+  const int maps = max(1, a.maps), HQ = a.H * maps, GK = a.own_kv ? a.G * maps : 0;
+  const int qk4 = (HQ + GK) * LPH, total4 = qk4 + (a.own_kv ? a.G * a.vdim / 4 : 0);
+  const float* row = a.in_p + (size_t)t * a.in_ld;
+  const int slot = a.slots[t];
+  const int blk = slot / KV_BLOCK, off = slot % KV_BLOCK;
+  float qmul = 1.f;
+  if (a.qtemp_coef > 0.f && a.qtemp_every > 0)
+    qmul = 1.0f + a.qtemp_coef * logf((float)((a.positions[t] + 1) / a.qtemp_every) + 1.0f);
+  for (int i0 = blockIdx.y * blockDim.x; i0 < total4; i0 += gridDim.y * blockDim.x) {
+    const int i = i0 + threadIdx.x, col = 4 * i;
+    const bool ok = i < total4;
+    float v[4] = {0.f, 0.f, 0.f, 0.f};
+    if (ok)
+      for (int sl = 0; sl < a.in_S; sl++) {
+        const float4 x = *reinterpret_cast<const float4*>(row + (size_t)sl * a.in_stride + col);
+        v[0] += x.x; v[1] += x.y; v[2] += x.z; v[3] += x.w;
+      }
+    float ss = v[0] * v[0] + v[1] * v[1] + v[2] * v[2] + v[3] * v[3];
+#pragma unroll
+    for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (!ok) continue;
+    if (i >= qk4) {
+      const int c = col - 4 * qk4, g = c / a.vdim;
+      store4((KT*)a.vpool + (((size_t)blk * a.G + g) * KV_BLOCK + off) * a.vdim + (c - g * a.vdim), v);
+      continue;
+    }
+    const int head = i / LPH, d = col % DIM;
+    const bool isq = head < HQ;
+    float m = a.qk_norm ? 1.0f / sqrtf(ss / (float)DIM + a.eps) : 1.f;
+    if (isq) m *= qmul * (a.head_scale ? a.head_scale[head] : 1.f);
+    float4 w = make_float4(1.f, 1.f, 1.f, 1.f);
+    if (a.qk_norm == 3) w = *reinterpret_cast<const float4*>((isq ? a.qnorm_w : a.knorm_w) + d);
+    v[0] *= m * w.x; v[1] *= m * w.y; v[2] *= m * w.z; v[3] *= m * w.w;
+    if (isq) {
+      store4((QT*)a.q + (size_t)t * HQ * DIM + col, v);
+    } else {
+      const int kh = head - HQ;
+      store4((KT*)a.kpool + ((((size_t)blk * a.G + kh / maps) * KV_BLOCK + off) * maps + kh % maps) * DIM + d, v);
+    }
+  }
+  TRACE_EXIT(tr);
+}
+template <typename QT, typename KT>
+static bool winattn_prep_vec(cudaStream_t st, const WinAttnArgs& a) {
+  if (a.rot_half || a.vfirst || a.gate_out || a.vdim % 4 || a.in_ld % 4 || a.in_stride % 4 || reinterpret_cast<size_t>(a.in_p) % 16)
+    return false;
+  const int maps = std::max(1, a.maps);
+  const int total4 = (a.H * maps * a.dim + (a.own_kv ? a.G * (maps * a.dim + a.vdim) : 0)) / 4;
+  const dim3 grid(a.T, a.T >= 1024 ? 1 : ceil_div(total4, 256));
+  if (a.dim == 32) (void)launch_k(winattn_prep_vec_kernel<QT, KT, 8>, grid, dim3(256), 0, st, a, next_trace(30));
+  else if (a.dim == 64) (void)launch_k(winattn_prep_vec_kernel<QT, KT, 16>, grid, dim3(256), 0, st, a, next_trace(30));
+  else if (a.dim == 128) (void)launch_k(winattn_prep_vec_kernel<QT, KT, 32>, grid, dim3(256), 0, st, a, next_trace(30));
+  else return false;
+  return true;
+}
+
 cudaError_t launch_winattn_prep(cudaStream_t st, int qdt, int kvdt, const WinAttnArgs& a) {
   if (a.T <= 0) return cudaSuccess;
   if (2 * a.rot_half > a.dim || (a.vfirst && !a.own_kv)) return cudaErrorInvalidValue;
+  if (qdt == DT_F32 && kvdt == DT_F32 && winattn_prep_vec<float, float>(st, a)) return cudaGetLastError();
+  if (qdt == DT_BF16 && kvdt == DT_BF16 && winattn_prep_vec<bf16, bf16>(st, a)) return cudaGetLastError();
   // few rows (decode): the heads of a row spread over several CTAs
   const int maps = std::max(1, a.maps);
   const int n_items = a.H * maps + (a.own_kv ? a.G * (maps + 1) : 0) + (a.gate_out ? 1 : 0);

@@ -27,6 +27,14 @@ template <typename T> __device__ __forceinline__ T from_f32(float v);
 template <> __device__ __forceinline__ float from_f32<float>(float v) { return v; }
 template <> __device__ __forceinline__ bf16 from_f32<bf16>(float v) { return __float2bfloat16_rn(v); }
 
+// four neighbouring entries (16 bytes of fp32, 8 of bf16)
+__device__ __forceinline__ void store4(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void store4(bf16* p, const float (&v)[4]) {
+  uint2 u;
+  reinterpret_cast<__nv_bfloat162*>(&u)[0] = __floats2bfloat162_rn(v[0], v[1]);
+  reinterpret_cast<__nv_bfloat162*>(&u)[1] = __floats2bfloat162_rn(v[2], v[3]);
+  *reinterpret_cast<uint2*>(p) = u;
+}
 // 8 consecutive elements -> fp32 registers (16 B load for bf16, 2x16 B for fp32)
 __device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
   float4 a = *reinterpret_cast<const float4*>(p);

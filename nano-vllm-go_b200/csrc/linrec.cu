@@ -867,13 +867,6 @@ cudaError_t launch_linrec_decode(cudaStream_t st, int odt, const LinRecArgs& a) 
 }
 
 // ------------------------------------------------------------------ gated norm of the read-out
-__device__ __forceinline__ void store4(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
-__device__ __forceinline__ void store4(bf16* p, const float (&v)[4]) {
-  uint2 u;
-  reinterpret_cast<__nv_bfloat162*>(&u)[0] = __floats2bfloat162_rn(v[0], v[1]);
-  reinterpret_cast<__nv_bfloat162*>(&u)[1] = __floats2bfloat162_rn(v[2], v[3]);
-  *reinterpret_cast<uint2*>(p) = u;
-}
 // MJ: 16-byte pieces per lane (vdim <= 128 MJ); GATED: 0 no gate, 1 silu(gate), 2 mLSTM: the read-out is first divided by
 // max(|n . q|, c) + 1e-6, sigmoid(gate)
 template <int GATED>
