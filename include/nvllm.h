@@ -191,8 +191,8 @@ int nvllm_create(const nvllm_config* cfg, const uint8_t* tp_id, nvllm_handle** o
  *   NVLLM_LBLOCK_SEQUENTIAL_PRENORM   x += mixer(RMSNorm(x)), then x += feed_forward(RMSNorm(x)); a run of
  *                                   layers may repeat with the same weights (loop_*), every pass with caches and
  *                                   state of its own and a learned vector added to x at its start (Lazovik, Sutuvik);
- *                                   with layer_norm = 1 LayerNorm (weight and additive term) instead (Sozurax); with loop_embed = 1 the
- *                                   passes after the first open with the embedding instead (Defilorn)
+ *                                   with layer_norm = 1 LayerNorm (weight and additive term) instead (Sozurax);
+ *                                   with loop_embed = 1 the passes after the first open with the embedding instead (Defilorn)
  * Tensors are handed in by checkpoint name (nvllm_set_named_weight, or nvllm_load_safetensors
  * with NVLLM_ARCH_DUGOPEL / NVLLM_ARCH_ZOZONEX / NVLLM_ARCH_LAZOVIK / NVLLM_ARCH_SUTUVIK / NVLLM_ARCH_SOZURAX /
  * NVLLM_ARCH_DEFILORN). */
@@ -204,8 +204,8 @@ enum nvllm_mixer_kind {
   NVLLM_MIXER_ATTN_TMIX = 5,        /* two mixers on one input, their outputs summed with two scales: grouped-query
                                        attention (short convolution, whole-row q / k norm, rotation, score cap, chunked
                                        mask, output gate) and time mixing with a token shift (heads2 x dim2) */
-  NVLLM_MIXER_ATTENTION = 6,        /* grouped-query attention over the whole cached prefix, every option a field of the
-                                       spec: per-head q / k norm (qk_norm 1 / 3), partial rotation of interleaved pairs with
+  NVLLM_MIXER_ATTENTION = 6,        /* grouped-query attention over the whole cached prefix or a window of it, every option a field of
+                                       the spec: one or two score maps per head, per-head q / k norm (qk_norm 1 / 3), partial rotation of interleaved pairs with
                                        piecewise frequency scaling, a query multiplier that grows with the position, a
                                        multiplier per head, score cap, a bias linear in the distance, a sink of score 0 or a
                                        learned one per head, values mixed with an earlier layer's, a gate per head */
